@@ -11,6 +11,7 @@
 // (areal/experimental/models/archon/qwen3/model/model.py:103-293).
 #include "common/gemm_core.cuh"
 #include "common/host_utils.h"
+#include "common/io.cuh"
 
 namespace b200 {
 
@@ -348,6 +349,94 @@ __global__ void splitk_reduce_rmsnorm_kernel(const float* __restrict__ ws, const
   }
 }
 
+// ------------------------------------------ projection + scaled residual add + Dynamic Tanh --
+// Epilogue of a block's output projection in decoders with an fp32 residual stream, a per-column scale on the
+// sublayer's result and an element-wise norm in front of the next sublayer:
+//   res[r, c] += scale[c] * acc;   y[r, c] = tanh(alpha * res[r, c]) * w[c] + b[c]
+// No row statistics are needed, so it runs on the accumulator tile; every element of res belongs to one thread.
+struct DytTail {
+  float* res;
+  const __nv_bfloat16 *scale, *alpha, *w, *b;
+  __nv_bfloat16* y;
+  int N;
+
+  __device__ __forceinline__ void apply4(float al, long long row, int c, float4 acc) const {
+    const float4 s = ld4(scale + c), ww = ld4(w + c), bb = ld4(b + c);
+    float4 h = ld4(res + row * N + c);
+    h.x = fmaf(s.x, acc.x, h.x); h.y = fmaf(s.y, acc.y, h.y);
+    h.z = fmaf(s.z, acc.z, h.z); h.w = fmaf(s.w, acc.w, h.w);
+    st4(res + row * N + c, h);
+    st4(y + row * N + c, make_float4(fmaf(tanhf(al * h.x), ww.x, bb.x), fmaf(tanhf(al * h.y), ww.y, bb.y),
+                                     fmaf(tanhf(al * h.z), ww.z, bb.z), fmaf(tanhf(al * h.w), ww.w, bb.w)));
+  }
+};
+
+struct DytEpi {
+  DytTail t;
+  int M;
+  struct State { float al; };
+
+  __device__ __forceinline__ bool tile(int cta, int ncta, int it, int tiles_m, int tiles_n, int& m_blk,
+                                       int& n_blk) const {
+    return default_tile(cta, ncta, it, tiles_m, tiles_n, m_blk, n_blk);
+  }
+  __device__ __forceinline__ bool gate(int, int, volatile int*, int*) const { return true; }
+  __device__ __forceinline__ void begin(State& s, int, int, int) const { s.al = __bfloat162float(*t.alpha); }
+  __device__ __forceinline__ void end(State&, int, int, int) const {}
+  __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
+    if (row >= M) return;
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (col0 + 4 * i < t.N)  // N % 4 == 0
+        t.apply4(s.al, row, col0 + 4 * i, make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]));
+  }
+};
+
+__global__ void splitk_reduce_dyt_kernel(const float* __restrict__ ws, DytTail t, int M, int S, long long slice_stride) {
+  const int nq = t.N >> 2;
+  const float al = __bfloat162float(*t.alpha);
+  const long long total = static_cast<long long>(M) * nq;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int row = static_cast<int>(i / nq), c = static_cast<int>(i % nq) * 4;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < S; ++s) {
+      const float4 v = ld4(ws + s * slice_stride + static_cast<long long>(row) * t.N + c);
+      acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
+    }
+    t.apply4(al, row, c, acc);
+  }
+}
+
+// --------------------------------------------------------------------- one product per head --
+// C[r, h * ldc_head + n] = sum_k A[r, h * a_head + k] * W_h(n, k): the same rows against H stacked weights, every head
+// with its own column slice of A and C. Row block h * tiles_m + m is row block m of head h.
+struct HeadsEpi {
+  StoreEpi st;  // M, N of one head; C and ldc of the whole output
+  int tiles_m_real, a_head, c_head, w_rows;  // w_rows: rows of the stacked weight that belong to one head
+  using State = StoreEpi::State;
+
+  __device__ __forceinline__ bool tile(int cta, int ncta, int it, int tiles_m, int tiles_n, int& m_blk,
+                                       int& n_blk) const {
+    return default_tile(cta, ncta, it, tiles_m, tiles_n, m_blk, n_blk);
+  }
+  __device__ __forceinline__ bool gate(int, int, volatile int*, int*) const { return true; }
+  __device__ __forceinline__ int a_m0(int mv) const { return (mv % tiles_m_real) * kBM; }
+  __device__ __forceinline__ int b_offset(int mv) const { return (mv / tiles_m_real) * w_rows; }
+  __device__ __forceinline__ bool k_load(int mv, int kb, int& ax, int& ay, int& bx, volatile int*, int*) const {
+    ax = (mv / tiles_m_real) * a_head + kb * kBK;
+    return true;
+  }
+  __device__ __forceinline__ void begin(State&, int, int, int) const {}
+  __device__ __forceinline__ void end(State&, int, int, int) const {}
+  __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
+    const int mv = row / kBM, h = mv / tiles_m_real;
+    StoreEpi e = st;
+    e.C = static_cast<__nv_bfloat16*>(st.C) + static_cast<long long>(h) * c_head;
+    e.chunk(s, row - h * tiles_m_real * kBM, col0, v);
+  }
+};
+
 }  // namespace b200
 
 extern "C" {
@@ -510,6 +599,85 @@ int b200_gemm_bf16_splitk_rmsnorm(const void* A, const void* B, const void* bias
   else if (nv <= 16) B200_LAUNCH_RN(16);
   else B200_LAUNCH_RN(32);
 #undef B200_LAUNCH_RN
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// A [M, K] . B [N, K]^T with the DytEpi tail: res [M, N] fp32 (in place), y [M, N] bf16, N % 4 == 0. splits > 1: split-K
+// into `workspace` (fp32 [splits * ceil(M/128)*128 * N]) with the tail in the reduction kernel.
+int b200_gemm_bf16_dyt(const void* A, const void* B, float* workspace, int M, int N, int K, long long lda,
+                       long long ldb, int splits, const void* scale, float* res, const void* alpha, const void* w,
+                       const void* b, void* y, cudaStream_t stream) {
+  using namespace b200;
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((lda & 7) || (ldb & 7) || (N & 3)) return -100;
+  using bf = __nv_bfloat16;
+  const DytTail tail{res, (const bf*)scale, (const bf*)alpha, (const bf*)w, (const bf*)b, (bf*)y, N};
+  if (splits > 1) {
+    int S = 0;
+    long long stride = 0;
+    const int rc = launch_splitk_partials(A, B, workspace, M, N, K, lda, ldb, splits, &S, &stride, stream);
+    if (rc) return rc;
+    long long rg = (static_cast<long long>(M) * (N >> 2) + 255) / 256;
+    const long long maxg = static_cast<long long>(sm_count()) * 8;
+    if (rg > maxg) rg = maxg;
+    splitk_reduce_dyt_kernel<<<(unsigned)rg, 256, 0, stream>>>(workspace, tail, M, S, stride);
+    B200_CHECK(cudaGetLastError());
+    return 0;
+  }
+  constexpr int BN = 128;
+  using Cfg = GemmCfg<BN>;
+  CUtensorMap tmA, tmB;
+  int rc = make_tmap_2d(&tmA, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, K, lda * 2, kBM, 64);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tmB, B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, N, K, ldb * 2, BN, 64);
+  if (rc) return rc;
+  auto kern = gemm_tcgen05_kernel<BN, false, false, DytEpi>;
+  static bool attr_set = false;
+  if (!attr_set) {
+    B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
+    attr_set = true;
+  }
+  const long long tiles = static_cast<long long>((M + kBM - 1) / kBM) * ((N + BN - 1) / BN);
+  const int grid = static_cast<int>(tiles < sm_count() ? tiles : sm_count());
+  int* status = device_status_word();
+  if (!status) return -3;
+  kern<<<grid, kGemmThreads, Cfg::kSmemBytes, stream>>>(tmA, tmB, M, N, K, DytEpi{tail, M}, status);
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// Per-head products (HeadsEpi). A: [M][lda], head h reads columns [h * a_head, h * a_head + K). W is stacked:
+// b_mn 0: [H * N, K] (K contiguous); b_mn 1: [H * K, N] (N contiguous; K % 64 == 0, else a tile's last reduction block
+// would run into the next head). C: [M][ldc], head h writes columns [h * c_head, h * c_head + N).
+int b200_gemm_heads(const void* A, long long lda, int a_head, const void* W, long long ldw, int b_mn, void* C,
+                    long long ldc, int c_head, int H, int M, int N, int K, cudaStream_t stream) {
+  using namespace b200;
+  if (M <= 0 || N <= 0 || K <= 0 || H <= 0) return 0;
+  if ((lda & 7) || (ldw & 7) || (a_head & 7) || (c_head & 7) || (ldc & 7) || (K & 7) || (b_mn && (K % kBK)))
+    return -100;
+  constexpr int BN = 128;
+  using Cfg = GemmCfg<BN>;
+  const int tiles_m = (M + kBM - 1) / kBM;
+  CUtensorMap tmA, tmB;
+  // A's extent ends with the last head's columns
+  int rc = make_tmap_2d(&tmA, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, static_cast<uint64_t>(H - 1) * a_head + K,
+                        lda * 2, kBM, 64);
+  if (rc) return rc;
+  if (b_mn)
+    rc = make_tmap_2d(&tmB, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, static_cast<uint64_t>(H) * K, N, ldw * 2, 64, 64);
+  else
+    rc = make_tmap_2d(&tmB, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, static_cast<uint64_t>(H) * N, K, ldw * 2, BN, 64);
+  if (rc) return rc;
+  HeadsEpi epi{StoreEpi{C, nullptr, ldc, M, N, 0, 0}, tiles_m, a_head, c_head, b_mn ? K : N};
+  const int Mv = H * tiles_m * kBM;
+  const long long tiles = static_cast<long long>(H) * tiles_m * ((N + BN - 1) / BN);
+  const int grid = static_cast<int>(tiles < sm_count() ? tiles : sm_count());
+  int* status = device_status_word();
+  if (!status) return -3;
+#define B200_GH(MN_)                                                                                                  {                                                                                                                     auto kern = gemm_tcgen05_kernel<BN, false, MN_, HeadsEpi>;                                                          static bool attr_set = false;                                                                                       if (!attr_set) {                                                                                                      B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));               attr_set = true;                                                                                                  }                                                                                                                   kern<<<grid, kGemmThreads, Cfg::kSmemBytes, stream>>>(tmA, tmB, Mv, N, K, epi, status);                           }
+  if (b_mn) B200_GH(true) else B200_GH(false)
+#undef B200_GH
   B200_CHECK(cudaGetLastError());
   return 0;
 }

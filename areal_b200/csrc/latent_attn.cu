@@ -1,0 +1,261 @@
+// Latent attention with a compressed paged cache: per token the normed latent c [rank] followed by one rotated key
+// part [rot] shared by all heads (one "kv head" of width rank + rot).
+//
+//   latent_prep   splits the down projection's row [q_rank | rank | rot]: RMS norm of the query latent, RMS norm of
+//                 the key / value latent, rotation of the shared key part, write of (latent | rotated part) into the
+//                 cache page of the token
+//   rope_pairs    rotates neighbouring pairs (2i, 2i+1) inside a slice of every head, in place
+//   attend        softmax attention of any widths, fp32 throughout: one warp per (query, head). Keys come in two
+//                 parts (per head, shared) and from rows of a packed batch (prefill) or from pages (decode, where the
+//                 per-head part is the latent itself, shared by the heads too, and the queries carry the key
+//                 up-projection). The tensor-core kernels cover the widths of real models; this one covers the rest
+//                 and fp32.
+#include "common/host_utils.h"
+#include "common/io.cuh"
+
+namespace b200 {
+
+template <class T>
+__global__ void latent_prep_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ wq,
+                                   const T* __restrict__ wc, const float* __restrict__ cosT,
+                                   const float* __restrict__ sinT, const int* __restrict__ pos, int max_pos,
+                                   const long long* __restrict__ slot_mapping, T* __restrict__ cq, T* __restrict__ c,
+                                   T* __restrict__ kr, T* __restrict__ cache, long long cache_rows, int q_rank,
+                                   int rank, int rot, float eps) {
+  __shared__ float red[33];
+  const long long t = blockIdx.x;
+  const T* row = x + t * ldx;
+  float s = 0.f;
+  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = ld1(row + i); s = fmaf(v, v, s); }
+  s = block_sum(s, red);
+  const float kq = 1.f / sqrtf(s / q_rank + eps);
+  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) st1(cq + t * q_rank + i, ld1(row + i) * kq * ld1(wq + i));
+  row += q_rank;
+  s = 0.f;
+  for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = ld1(row + i); s = fmaf(v, v, s); }
+  s = block_sum(s, red);
+  const float kc = 1.f / sqrtf(s / rank + eps);
+  long long slot = slot_mapping ? slot_mapping[t] : -1;
+  if (slot >= cache_rows) slot = -1;
+  T* dst = slot >= 0 ? cache + slot * (rank + rot) : nullptr;
+  for (int i = threadIdx.x; i < rank; i += blockDim.x) {
+    const float v = ld1(row + i) * kc * ld1(wc + i);
+    if (c) st1(c + t * rank + i, v);
+    if (dst) st1(dst + i, v);
+  }
+  row += rank;
+  const int p = min(max(pos[t], 0), max_pos - 1);
+  for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
+    const float cs = cosT[static_cast<long long>(p) * (rot / 2) + i], sn = sinT[static_cast<long long>(p) * (rot / 2) + i];
+    const float u = ld1(row + 2 * i), v = ld1(row + 2 * i + 1);
+    const float a = u * cs - v * sn, b = v * cs + u * sn;
+    if (kr) { st1(kr + t * rot + 2 * i, a); st1(kr + t * rot + 2 * i + 1, b); }
+    if (dst) { st1(dst + rank + 2 * i, a); st1(dst + rank + 2 * i + 1, b); }
+  }
+}
+
+template <class T>
+__global__ void rope_pairs_kernel(T* __restrict__ x, long long ldx, int H, int head_stride, int offset, int half,
+                                  const float* __restrict__ cosT, const float* __restrict__ sinT,
+                                  const int* __restrict__ pos, int max_pos, long long rows) {
+  const long long total = rows * H * half;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int e = static_cast<int>(i % half);
+    const int h = static_cast<int>((i / half) % H);
+    const long long t = i / (static_cast<long long>(half) * H);
+    const int p = min(max(pos[t], 0), max_pos - 1);
+    const float cs = cosT[static_cast<long long>(p) * half + e], sn = sinT[static_cast<long long>(p) * half + e];
+    T* q = x + t * ldx + static_cast<long long>(h) * head_stride + offset + 2 * e;
+    const float u = ld1(q), v = ld1(q + 1);
+    st1(q, u * cs - v * sn);
+    st1(q + 1, v * cs + u * sn);
+  }
+}
+
+struct AttendArgs {
+  const void *qa, *qb;             // query parts: [rows][ld] + h * head stride
+  long long ldqa, ldqb;
+  int hqa, hqb;
+  const void *ka, *kb, *v;         // key parts and values: [rows][ld] + h * head stride (0: shared by the heads)
+  long long ldka, ldkb, ldv;
+  int hka, hkb, hv;
+  int da, db, dv;                  // widths
+  const int* seq_start;            // packed: first row of the query's sequence per query row [n]; paged: null
+  const int* kv_len;               // visible keys per query row [n]
+  const int* block_table;          // paged: [n, max_blocks]; else null
+  int max_blocks, block_size;
+  float* o_part;                   // [n, H, nsplit, dv] when nsplit > 1
+  float* ml_part;                  // [n, H, nsplit, 2]
+  void* out;                       // [n][ldo] + h * dv
+  long long ldo;
+  int H, nsplit;
+  float scale;
+};
+
+// grid (n query rows, ceil(H / warps), nsplit)
+template <class T>
+__global__ void attend_kernel(AttendArgs a) {
+  extern __shared__ float sm[];
+  const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.y * nw + warp;
+  const int dq = a.da + a.db;
+  float* q = sm + warp * (dq + a.dv);  // this warp's query and accumulator
+  float* acc = q + dq;
+  if (h >= a.H) return;                // whole warp; no block-wide barrier follows
+  const long long r = blockIdx.x;
+  const int L = a.kv_len[r];
+  const int per = (L + a.nsplit - 1) / a.nsplit;
+  const int k0 = blockIdx.z * per, k1 = min(L, k0 + per);
+  for (int i = lane; i < a.da; i += 32) q[i] = ld1(static_cast<const T*>(a.qa) + r * a.ldqa + h * a.hqa + i);
+  for (int i = lane; i < a.db; i += 32) q[a.da + i] = ld1(static_cast<const T*>(a.qb) + r * a.ldqb + h * a.hqb + i);
+  for (int i = lane; i < a.dv; i += 32) acc[i] = 0.f;
+  __syncwarp();
+  const long long first = a.seq_start ? a.seq_start[r] : 0;
+  const int* bt = a.block_table ? a.block_table + r * a.max_blocks : nullptr;
+  float m = -INFINITY, l = 0.f;
+  for (int kb = k0; kb < k1; kb += 32) {
+    const int j = kb + lane;
+    long long row = 0;
+    float s = -INFINITY;
+    if (j < k1) {
+      row = bt ? static_cast<long long>(bt[j / a.block_size]) * a.block_size + j % a.block_size : first + j;
+      const T* ka = static_cast<const T*>(a.ka) + row * a.ldka + h * a.hka;
+      const T* kp = static_cast<const T*>(a.kb) + row * a.ldkb + h * a.hkb;
+      float d = 0.f;
+      for (int i = 0; i < a.da; ++i) d = fmaf(q[i], ld1(ka + i), d);
+      for (int i = 0; i < a.db; ++i) d = fmaf(q[a.da + i], ld1(kp + i), d);
+      s = d * a.scale;
+    }
+    float mx = s;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    const float mn = fmaxf(m, mx);
+    const float sc = m == -INFINITY ? 0.f : expf(m - mn);
+    const float p = j < k1 ? expf(s - mn) : 0.f;
+    l = l * sc + warp_sum(p);
+    m = mn;
+    const int n = min(32, k1 - kb);
+    for (int i0 = 0; i0 < a.dv; i0 += 32) {
+      const int i = i0 + lane;
+      float t = 0.f;
+      for (int e = 0; e < n; ++e) {
+        const long long rr = __shfl_sync(0xffffffffu, row, e);
+        const float pe = __shfl_sync(0xffffffffu, p, e);
+        if (i < a.dv) t = fmaf(pe, ld1(static_cast<const T*>(a.v) + rr * a.ldv + h * a.hv + i), t);
+      }
+      if (i < a.dv) acc[i] = fmaf(acc[i], sc, t);
+    }
+  }
+  if (a.nsplit == 1) {
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    for (int i = lane; i < a.dv; i += 32)
+      st1(static_cast<T*>(a.out) + r * a.ldo + static_cast<long long>(h) * a.dv + i, acc[i] * inv);
+  } else {
+    const long long u = (r * a.H + h) * a.nsplit + blockIdx.z;
+    for (int i = lane; i < a.dv; i += 32) a.o_part[u * a.dv + i] = acc[i];
+    if (lane == 0) { a.ml_part[2 * u] = m; a.ml_part[2 * u + 1] = l; }
+  }
+}
+
+// Merge of split partials. m in natural-log units when LOG2 is false, in log2 units else.
+template <class T, bool LOG2>
+__global__ void attend_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ ml, T* __restrict__ out,
+                                    long long ldo, int H, int nsplit, int dv) {
+  const long long u = blockIdx.x;
+  const long long r = u / H;
+  const int h = static_cast<int>(u % H);
+  float m = -INFINITY;
+  for (int s = 0; s < nsplit; ++s) m = fmaxf(m, ml[(u * nsplit + s) * 2]);
+  float l = 0.f;
+  for (int s = 0; s < nsplit; ++s) {
+    const float ms = ml[(u * nsplit + s) * 2];
+    if (ms != -INFINITY) l += ml[(u * nsplit + s) * 2 + 1] * (LOG2 ? exp2f(ms - m) : expf(ms - m));
+  }
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  for (int i = threadIdx.x; i < dv; i += blockDim.x) {
+    float t = 0.f;
+    for (int s = 0; s < nsplit; ++s) {
+      const float ms = ml[(u * nsplit + s) * 2];
+      if (ms != -INFINITY) t = fmaf(o_part[(u * nsplit + s) * dv + i], LOG2 ? exp2f(ms - m) : expf(ms - m), t);
+    }
+    st1(out + r * ldo + static_cast<long long>(h) * dv + i, t * inv);
+  }
+}
+
+}  // namespace b200
+
+extern "C" {
+
+// x [T][ldx]: [q_rank | rank | rot]. Tables [max_pos, rot / 2]. c, kr, slot_mapping + cache may be null.
+int b200_latent_prep(const void* x, long long ldx, const void* wq, const void* wc, const float* cosT, const float* sinT,
+                     const int* pos, int max_pos, const long long* slot_mapping, void* cq, void* c, void* kr,
+                     void* cache, long long cache_rows, int T, int q_rank, int rank, int rot, float eps, int fp32,
+                     cudaStream_t stream) {
+  using namespace b200;
+  if (T <= 0) return 0;
+  if (rot & 1) return -100;
+  const int widest = q_rank > rank ? q_rank : rank;
+  int block = 64;
+  while (block < 512 && block * 2 < widest) block <<= 1;
+#define B200_LP(T_)                                                                                                 \
+  latent_prep_kernel<T_><<<T, block, 0, stream>>>((const T_*)x, ldx, (const T_*)wq, (const T_*)wc, cosT, sinT, pos, \
+                                                  max_pos, slot_mapping, (T_*)cq, (T_*)c, (T_*)kr, (T_*)cache,      \
+                                                  cache_rows, q_rank, rank, rot, eps)
+  if (fp32) B200_LP(float);
+  else B200_LP(__nv_bfloat16);
+#undef B200_LP
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// Rotates columns [offset, offset + dims) of every head of x [rows][ldx] in place; tables [max_pos, dims / 2].
+int b200_rope_pairs(void* x, long long ldx, int H, int head_stride, int offset, int dims, const float* cosT,
+                    const float* sinT, const int* pos, int max_pos, long long rows, int fp32, cudaStream_t stream) {
+  using namespace b200;
+  if (rows <= 0 || dims <= 0) return 0;
+  if (dims & 1) return -100;
+  const long long total = rows * H * (dims / 2);
+  long long grid = (total + 255) / 256;
+  const long long cap = static_cast<long long>(sm_count()) * 16;
+  if (grid > cap) grid = cap;
+  if (fp32)
+    rope_pairs_kernel<float><<<(unsigned)grid, 256, 0, stream>>>((float*)x, ldx, H, head_stride, offset, dims / 2, cosT,
+                                                                 sinT, pos, max_pos, rows);
+  else
+    rope_pairs_kernel<__nv_bfloat16><<<(unsigned)grid, 256, 0, stream>>>((__nv_bfloat16*)x, ldx, H, head_stride, offset,
+                                                                         dims / 2, cosT, sinT, pos, max_pos, rows);
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// General softmax attention; see AttendArgs for the meaning of every operand. n query rows.
+int b200_attend(const void* qa, long long ldqa, int hqa, const void* qb, long long ldqb, int hqb, const void* ka,
+                long long ldka, int hka, const void* kb, long long ldkb, int hkb, const void* v, long long ldv, int hv,
+                int da, int db, int dv, const int* seq_start, const int* kv_len, const int* block_table, int max_blocks,
+                int block_size, float* o_part, float* ml_part, void* out, long long ldo, int n, int H, int nsplit,
+                float scale, int fp32, cudaStream_t stream) {
+  using namespace b200;
+  if (n <= 0) return 0;
+  AttendArgs a{qa, qb, ldqa, ldqb, hqa, hqb, ka, kb, v, ldka, ldkb, ldv, hka, hkb, hv, da, db, dv, seq_start, kv_len,
+               block_table, max_blocks, block_size, o_part, ml_part, out, ldo, H, nsplit, scale};
+  int nw = H < 4 ? H : 4;
+  const size_t per_warp = static_cast<size_t>(da + db + dv) * sizeof(float);
+  while (nw > 1 && per_warp * nw > 48 * 1024) nw >>= 1;
+  const size_t smem = per_warp * nw;
+  if (smem > 48 * 1024) return -100;
+  dim3 grid(n, (H + nw - 1) / nw, nsplit);
+  if (fp32) attend_kernel<float><<<grid, nw * 32, smem, stream>>>(a);
+  else attend_kernel<__nv_bfloat16><<<grid, nw * 32, smem, stream>>>(a);
+  B200_CHECK(cudaGetLastError());
+  if (nsplit > 1) {
+    if (fp32) attend_merge_kernel<float, false><<<n * H, 128, 0, stream>>>(o_part, ml_part, (float*)out, ldo, H, nsplit, dv);
+    else
+      attend_merge_kernel<__nv_bfloat16, false><<<n * H, 128, 0, stream>>>(o_part, ml_part, (__nv_bfloat16*)out, ldo, H,
+                                                                          nsplit, dv);
+    B200_CHECK(cudaGetLastError());
+  }
+  return 0;
+}
+
+}  // extern "C"

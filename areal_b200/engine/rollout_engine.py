@@ -162,30 +162,36 @@ class _DecodeGraphs:
         self.bt = torch.zeros((maxb, mb), dtype=torch.int32, device=dev)
         self.temp = torch.ones(maxb, dtype=torch.float32, device=dev)
         self.u = torch.zeros(maxb, dtype=torch.float32, device=dev)
+        # slots of the sequences' recurrent states (negative: padding row); models without such state ignore them
+        self.state_slots = torch.full((maxb,), -1, dtype=torch.int32, device=dev)
         pctx = getattr(engine.model, "pctx", None)
         self.fused_sampling = bool(getattr(engine.ncfg, "fused_sampling", True)) and \
-            (pctx is None or pctx.tp_size == 1) and engine.model_config.hidden_size % 8 == 0
+            (pctx is None or pctx.tp_size == 1) and engine.model_config.hidden_size % 8 == 0 and \
+            next(engine.model.parameters()).dtype == torch.bfloat16
         self.rng_state = new_sampling_rng(engine.ncfg.seed, dev)
         pin = dict(pin_memory=True)
         self.h_pad_slots = torch.full((maxb,), -1, dtype=torch.int64, **pin)
         self.h_pad_lens = torch.zeros(maxb, dtype=torch.int32, **pin)
         self.h_temp = torch.ones(maxb, dtype=torch.float32, **pin)
+        self.h_state = torch.full((maxb,), -1, dtype=torch.int32, **pin)
         self.h_tok = torch.zeros(maxb, dtype=torch.int32, **pin)
         self.h_lp = torch.zeros(maxb, dtype=torch.float32, **pin)
-        self.graphs: dict[int, tuple[torch.cuda.CUDAGraph, torch.Tensor, torch.Tensor]] = {}
+        # batch size -> (graph, tokens, logprobs, final hidden states)
+        self.graphs: dict[int, tuple[torch.cuda.CUDAGraph, torch.Tensor, torch.Tensor, torch.Tensor]] = {}
         self.pool = None
         self.prev_n = 0
         self._last_temps = None
 
     def _forward(self, b: int):
         e = self.e
+        extra = dict(hybrid_state=e.hybrid_state, state_slots=self.state_slots[:b]) if e.hybrid_state is not None else {}
         hidden = e.model.decode(self.ids[:b], self.pos[:b], e.kv_caches, self.bt[:b], self.seq_lens[:b],
-                                self.slots[:b], max_seq_len=e.ncfg.context_length)
+                                self.slots[:b], max_seq_len=e.ncfg.context_length, **extra)
         if self.fused_sampling:
             # the token is drawn in the LM-head GEMM's epilogue: no [B, V] logits, no separate sampler pass
-            return lm_head_sample(hidden, e.model.output_weight(), self.temp[:b], self.rng_state)
+            return (*lm_head_sample(hidden, e.model.output_weight(), self.temp[:b], self.rng_state), hidden)
         logits = e.model.logits(hidden, out_dtype=torch.float32)
-        return sample(logits, self.temp[:b], None, None, self.u[:b])
+        return (*sample(logits, self.temp[:b], None, None, self.u[:b]), hidden)
 
     def capture_all(self, stream):
         with torch.cuda.stream(stream), torch.no_grad():
@@ -194,10 +200,10 @@ class _DecodeGraphs:
                 torch.cuda.synchronize()
                 g = torch.cuda.CUDAGraph()
                 with torch.cuda.graph(g, pool=self.pool, stream=stream, capture_error_mode="thread_local"):
-                    toks, lps = self._forward(b)
+                    toks, lps, hidden = self._forward(b)
                 if self.pool is None:
                     self.pool = g.pool()
-                self.graphs[b] = (g, toks, lps)
+                self.graphs[b] = (g, toks, lps, hidden)
             torch.cuda.synchronize()
 
     def bucket(self, n: int) -> int | None:
@@ -206,7 +212,8 @@ class _DecodeGraphs:
                 return b if b in self.graphs else None
         return None
 
-    def run(self, n: int, b: int, sched: "PagedScheduler", temps: list[float], rng) -> tuple[np.ndarray, np.ndarray]:
+    def run(self, n: int, b: int, sched: "PagedScheduler", temps: list[float], rng,
+            state_slots: list[int] | None = None) -> tuple[np.ndarray, np.ndarray]:
         ts0 = time.perf_counter()
         mb = sched.max_blocks_per_seq
         # inputs go to the device straight from the scheduler's pinned plan arrays
@@ -218,6 +225,11 @@ class _DecodeGraphs:
         if self.prev_n > n:  # rows used by the previous step but not by this one become padding
             self.slots[n:self.prev_n].copy_(self.h_pad_slots[n:self.prev_n], non_blocking=True)
             self.seq_lens[n:self.prev_n].copy_(self.h_pad_lens[n:self.prev_n], non_blocking=True)
+        if state_slots is not None:
+            m = max(n, self.prev_n)
+            self.h_state[:n] = torch.tensor(state_slots, dtype=torch.int32)
+            self.h_state[n:m] = -1
+            self.state_slots[:m].copy_(self.h_state[:m], non_blocking=True)
         if temps != self._last_temps:
             self.h_temp[:n] = torch.tensor(temps, dtype=torch.float32)
             self.temp[:n].copy_(self.h_temp[:n], non_blocking=True)
@@ -225,7 +237,7 @@ class _DecodeGraphs:
         if not self.fused_sampling:
             self.u[:b].uniform_(generator=rng)
         self.prev_n = n
-        g, toks, lps = self.graphs[b]
+        g, toks, lps, _ = self.graphs[b]
         g.replay()
         self.h_tok[:n].copy_(toks[:n], non_blocking=True)
         self.h_lp[:n].copy_(lps[:n], non_blocking=True)
@@ -301,7 +313,8 @@ class NativeRolloutEngine(InferenceEngine):
 
     # ------------------------------------------------------------------ setup
     def initialize(self, engine_id: str | None = None, train_data_parallel_size: int | None = None,
-                   device=None, model=None, **kwargs):
+                   device=None, model=None, start_loop: bool = True, **kwargs):
+        """``start_loop=False``: no background thread; the caller drives the steps itself (``engine/trace_replay.py``)."""
         ncfg = self.ncfg
         use_cuda = torch.cuda.is_available()
         self.device = torch.device(device) if device is not None else (
@@ -316,12 +329,16 @@ class NativeRolloutEngine(InferenceEngine):
             setattr(mc, k, v)
         self.model_config = mc
         dtype = torch.float32 if self.device.type == "cpu" else getattr(torch, ncfg.dtype)
+        if dtype == torch.float32 and self.device.type == "cuda":
+            torch.backends.cuda.matmul.allow_tf32 = False  # a 32-bit model is served in true 32-bit
         self.model = build_model(mc, dtype=dtype, device=self.device, seed=ncfg.seed)
         if ncfg.model_path:
             from ..utils.hf_io import load_hf_weights
 
             load_hf_weights(self.model, ncfg.model_path)
         self.model.eval()
+        if hasattr(self.model, "reserve_positions"):
+            self.model.reserve_positions(ncfg.context_length)
         for p in self.model.parameters():
             p.requires_grad_(False)
         # weights live in one flat buffer with the trainer's layout: weight sync is a flat copy
@@ -334,7 +351,7 @@ class NativeRolloutEngine(InferenceEngine):
                                     max_blocks_per_seq)
         # Hybrid models: per-sequence state of the linear-attention layers, addressed by a slot that a
         # request keeps from its first prefill until it finishes. Prompts are not shared (a shared page
-        # says nothing about the recurrent state) and decode steps run eagerly.
+        # says nothing about the recurrent state).
         self.hybrid_state = None
         self._state_slot: dict[int, int] = {}
         self._free_state_slots: list[int] = []
@@ -342,7 +359,7 @@ class NativeRolloutEngine(InferenceEngine):
             if mc.is_hybrid:
                 from ..models.qwen3_5 import HybridState as State
             else:
-                from ..models.lightning import LightningState as State
+                from ..models.lightning import RecurrentState as State
 
             self.hybrid_state = State(mc, ncfg.max_num_seqs, dtype, self.device)
             self._free_state_slots = list(range(ncfg.max_num_seqs - 1, -1, -1))
@@ -360,10 +377,11 @@ class NativeRolloutEngine(InferenceEngine):
         self._rng = torch.Generator(device=self.device).manual_seed(ncfg.seed)
         self._graphs = None
         self.launches_per_decode = 0
-        if (self.device.type == "cuda" and ncfg.cuda_graph and not mc.has_recurrent_state and not mc.is_vl
-                and not mc.is_mla
-                and _lib.use_cuda_kernels(next(self.model.parameters()))):
+        if self._graphs_supported():
             self._capture_graphs()
+        if not start_loop:
+            logger.info(f"rollout engine ready on {self.device} (stepped by the caller): {nblocks} KV pages of {bs} tokens")
+            return self
         self._thread = threading.Thread(target=self._loop, name="rollout-engine", daemon=True)
         self._thread.start()
         from ..infra.workflow_executor import WorkflowExecutor
@@ -373,13 +391,22 @@ class NativeRolloutEngine(InferenceEngine):
         logger.info(f"rollout engine ready on {self.device}: {nblocks} KV pages of {bs} tokens")
         return self
 
+    def _graphs_supported(self) -> bool:
+        return (self.device.type == "cuda" and self.ncfg.cuda_graph and self.model_config.graph_decode
+                and _lib.use_cuda_kernels(next(self.model.parameters())))
+
     def _alloc_kv(self, nblocks: int, dtype):
-        """Paged K/V caches, one pair per layer (None for linear-attention layers of a hybrid model)."""
+        """Paged caches ``[pages, heads, page size, width]``, a tuple per layer (keys and values, or the one latent cache
+        of compressed latent attention; None for layers that keep a recurrent state instead)."""
         mc, bs = self.model_config, self.ncfg.kv_block_size
-        mk = lambda: torch.zeros(nblocks, mc.num_key_value_heads, bs, mc.head_dim, dtype=dtype, device=self.device)
-        return [(mk(), mk()) if mc.layer_type(i) == "full_attention" else None for i in range(mc.num_hidden_layers)]
+        mk = lambda h, d: torch.zeros(nblocks, h, bs, d, dtype=dtype, device=self.device)
+        return [tuple(mk(h, d) for h, d in mc.cache_shapes(i)) or None for i in range(mc.num_hidden_layers)]
 
     def _state_slots_of(self, seq_ids: list[int]):
+        """Slots of these requests in the hybrid state, as a device tensor."""
+        return torch.tensor(self._state_slot_list(seq_ids), dtype=torch.long, device=self.device)
+
+    def _state_slot_list(self, seq_ids: list[int]) -> list[int]:
         """Slots of these requests in the hybrid state (assigned on first sight, freed when they finish)."""
         out = []
         for r in seq_ids:
@@ -387,7 +414,7 @@ class NativeRolloutEngine(InferenceEngine):
             if slot is None:
                 slot = self._state_slot[r] = self._free_state_slots.pop()
             out.append(slot)
-        return torch.tensor(out, dtype=torch.long, device=self.device)
+        return out
 
     def _capture_graphs(self):
         t0 = time.perf_counter()
@@ -404,7 +431,7 @@ class NativeRolloutEngine(InferenceEngine):
                     f"({self.launches_per_decode} kernels per step)")
 
     def _auto_num_blocks(self, mc: ModelConfig, dtype, bs: int) -> int:
-        per_block = 2 * mc.num_hidden_layers * bs * mc.num_key_value_heads * mc.head_dim * \
+        per_block = bs * sum(h * d for i in range(mc.num_hidden_layers) for h, d in mc.cache_shapes(i)) * \
             torch.empty((), dtype=dtype).element_size()
         if self.device.type == "cuda":
             free, total = torch.cuda.mem_get_info(self.device)
@@ -412,7 +439,7 @@ class NativeRolloutEngine(InferenceEngine):
         else:
             budget = 256 << 20
         need = self.ncfg.max_num_seqs * ((self.ncfg.context_length + bs - 1) // bs)
-        return max(16, min(budget // per_block, need))
+        return max(16, min(budget // max(per_block, 1), need))  # (purely recurrent models cache nothing per token)
 
     def destroy(self):
         self._stop.set()
@@ -486,7 +513,7 @@ class NativeRolloutEngine(InferenceEngine):
             b = self._graphs.bucket(n)
             if b is not None and not any(p[1] > 0 or p[2] < 1.0 or p[3] for p in pr):
                 t1 = time.perf_counter()
-                toks, lps = self._graphs.run(n, b, s, [p[0] for p in pr], self._rng)
+                toks, lps = self._graphs.run(n, b, s, [p[0] for p in pr], self._rng, self._graph_slots(seq_ids))
                 t2 = time.perf_counter()
                 s.commit(toks, lps)
                 self._gen_tokens += n
@@ -499,35 +526,11 @@ class NativeRolloutEngine(InferenceEngine):
                 tm["commit_deliver"] += t3 - t2
                 return True
         t_slow = time.perf_counter()
-        ids = torch.from_numpy(s.tokens[:T].copy()).to(dev, non_blocking=True)
-        pos = torch.from_numpy(s.positions[:T].copy()).to(dev, non_blocking=True)
-        slots = torch.from_numpy(s.slots[:T].copy()).to(dev, non_blocking=True)
         seq_ids = s.seq_ids[:n].tolist()
+        hidden = self._forward_plan(kind)
         if kind == 1:
-            cu = s.cu[: n + 1].copy()
-            meta = VarlenMeta(cu.tolist(), dev)
-            extra = dict(hybrid_state=self.hybrid_state, state_slots=self._state_slots_of(seq_ids)) \
-                if self.hybrid_state is not None else {}
-            if self.model_config.is_vl:
-                extra.update(self._vision_prefill_inputs(ids, seq_ids, cu))
-                pos = torch.arange(T, dtype=torch.int32, device=dev) if "rope" in extra else pos
-            hidden = self.model.prefill(ids, pos, meta, self.kv_caches, slots, **extra)
-            last = torch.from_numpy((cu[1:] - 1).astype(np.int64)).to(dev)
+            last = torch.from_numpy((s.cu[1:n + 1] - 1).astype(np.int64)).to(dev)
             hidden = hidden.index_select(0, last)
-        else:
-            seq_lens = torch.from_numpy(s.seq_lens[:n].copy()).to(dev, non_blocking=True)
-            bt = torch.from_numpy(s.block_table[: n * s.max_blocks_per_seq].copy()).view(n, -1)
-            nb = (int(s.hdr.max_seq_len) + self.ncfg.kv_block_size - 1) // self.ncfg.kv_block_size
-            bt = bt[:, :max(nb, 1)].contiguous().to(dev, non_blocking=True)
-            extra = dict(hybrid_state=self.hybrid_state, state_slots=self._state_slots_of(seq_ids)) \
-                if self.hybrid_state is not None else {}
-            if self._mm:
-                # text after an image continues from the largest grid coordinate, not from the token count
-                with self._lock:
-                    delta = [self._mm[r]["delta"] if r in self._mm else 0 for r in seq_ids]
-                pos = pos + torch.tensor(delta, dtype=pos.dtype, device=dev)
-            hidden = self.model.decode(ids, pos, self.kv_caches, bt, seq_lens, slots,
-                                       max_seq_len=int(s.hdr.max_seq_len), **extra)
         logits = self.model.logits(hidden, out_dtype=torch.float32)
         with self._lock:
             pr = [self._params.get(r, (1.0, 0, 1.0, 0.0)) for r in seq_ids]
@@ -562,6 +565,44 @@ class NativeRolloutEngine(InferenceEngine):
         else:
             self._phase_s["run"] += time.perf_counter() - t_slow  # an eager decode step (no graph for this batch)
         return True
+
+    def _graph_slots(self, seq_ids: list[int]) -> list[int] | None:
+        return self._state_slot_list(seq_ids) if self.hybrid_state is not None else None
+
+    @torch.no_grad()
+    def _forward_plan(self, kind: int) -> torch.Tensor:
+        """Runs the model on the scheduler's current plan (prefill or decode, without a captured graph): final hidden
+        states of every token of the plan, in plan order."""
+        s, dev = self.sched, self.device
+        n, T = s.hdr.n_seqs, s.hdr.n_tokens
+        ids = torch.from_numpy(s.tokens[:T].copy()).to(dev, non_blocking=True)
+        pos = torch.from_numpy(s.positions[:T].copy()).to(dev, non_blocking=True)
+        slots = torch.from_numpy(s.slots[:T].copy()).to(dev, non_blocking=True)
+        seq_ids = s.seq_ids[:n].tolist()
+        if kind == 1:
+            cu = s.cu[: n + 1].copy()
+            meta = VarlenMeta(cu.tolist(), dev)
+            extra = dict(hybrid_state=self.hybrid_state, state_slots=self._state_slots_of(seq_ids)) \
+                if self.hybrid_state is not None else {}
+            if self.model_config.is_vl:
+                extra.update(self._vision_prefill_inputs(ids, seq_ids, cu))
+                pos = torch.arange(T, dtype=torch.int32, device=dev) if "rope" in extra else pos
+            hidden = self.model.prefill(ids, pos, meta, self.kv_caches, slots, **extra)
+        else:
+            seq_lens = torch.from_numpy(s.seq_lens[:n].copy()).to(dev, non_blocking=True)
+            bt = torch.from_numpy(s.block_table[: n * s.max_blocks_per_seq].copy()).view(n, -1)
+            nb = (int(s.hdr.max_seq_len) + self.ncfg.kv_block_size - 1) // self.ncfg.kv_block_size
+            bt = bt[:, :max(nb, 1)].contiguous().to(dev, non_blocking=True)
+            extra = dict(hybrid_state=self.hybrid_state, state_slots=self._state_slots_of(seq_ids)) \
+                if self.hybrid_state is not None else {}
+            if self._mm:
+                # text after an image continues from the largest grid coordinate, not from the token count
+                with self._lock:
+                    delta = [self._mm[r]["delta"] if r in self._mm else 0 for r in seq_ids]
+                pos = pos + torch.tensor(delta, dtype=pos.dtype, device=dev)
+            hidden = self.model.decode(ids, pos, self.kv_caches, bt, seq_lens, slots,
+                                       max_seq_len=int(s.hdr.max_seq_len), **extra)
+        return hidden
 
     def _vision_prefill_inputs(self, ids: torch.Tensor, seq_ids: list[int], cu: np.ndarray) -> dict[str, Any]:
         """Embeddings with image features and the per-token rotary table of a prefill plan; empty when no
@@ -644,12 +685,9 @@ class NativeRolloutEngine(InferenceEngine):
         """Private copies of the page holding a shared prompt's last positions (prompt forks)."""
         idx = torch.from_numpy(pairs.reshape(-1, 2).astype(np.int64)).to(self.device)
         src, dst = idx[:, 0], idx[:, 1]
-        for pair in self.kv_caches:
-            if pair is None:
-                continue
-            kc, vc = pair
-            kc.index_copy_(0, dst, kc.index_select(0, src))
-            vc.index_copy_(0, dst, vc.index_select(0, src))
+        for layer in self.kv_caches:
+            for cache in layer or ():
+                cache.index_copy_(0, dst, cache.index_select(0, src))
 
     def _deliver(self):
         while True:
@@ -883,9 +921,7 @@ class NativeRolloutEngine(InferenceEngine):
             dtype = next(self.model.parameters()).dtype
             nblocks = self.sched.stats()["free_blocks"]
             self.kv_caches = self._alloc_kv(nblocks, dtype)
-            if (self.device.type == "cuda" and self.ncfg.cuda_graph and not self.model_config.has_recurrent_state
-                    and not self.model_config.is_vl and not self.model_config.is_mla
-                    and _lib.use_cuda_kernels(next(self.model.parameters()))):
+            if self._graphs_supported():
                 self._capture_graphs()
         self.continue_generation()
 

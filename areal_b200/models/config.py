@@ -84,6 +84,9 @@ class ModelConfig:
     lightning_group_size: int = 0
     lightning_head_dim: int = 128
     lightning_norm_groups: int = 1
+    # decoders given as an explicit list of layers (`models/layered.py`): every entry names the mixer's type and sizes
+    # and the feed-forward's (None: the layer has none); the sizes above then only summarise the list
+    layer_specs: list[dict] = field(default_factory=list)
     moe_group_score_top: int = 2  # a group's score: the sum of its this many best experts
     decoder_sparse_step: int = 1
     mlp_only_layers: list[int] = field(default_factory=list)
@@ -118,9 +121,41 @@ class ModelConfig:
     @property
     def has_recurrent_state(self) -> bool:
         """Some layers carry a per-sequence recurrent state through generation (linear-attention layers)."""
-        return self.is_hybrid or self.lightning_group_size > 1
+        return (self.is_hybrid or self.lightning_group_size > 1
+                or any(self.recurrent_shape(i) is not None for i in range(len(self.layer_specs))))
+
+    @property
+    def is_layered(self) -> bool:
+        return bool(self.layer_specs)
+
+    def cache_shapes(self, i: int) -> list[tuple[int, int]]:
+        """Paged-cache tensors of layer ``i`` as ``(heads, width)`` per token; empty for layers without a cache."""
+        if self.is_layered:
+            m = self.layer_specs[i]["mixer"]
+            return [(1, m["kv_rank"] + m["rot_dim"])] if self.layer_type(i) == "latent_attention" else []
+        if self.layer_type(i) != "full_attention":
+            return []
+        return [(self.num_key_value_heads, self.head_dim)] * 2
+
+    def recurrent_shape(self, i: int) -> tuple[int, int, int] | None:
+        """State of layer ``i`` per sequence ``(heads, key width, value width)``, None for layers without one. Covers
+        the families whose state is one matrix per head (the Qwen3.5 hybrid also keeps convolution inputs)."""
+        if self.is_layered:
+            m = self.layer_specs[i]["mixer"]
+            return (m["heads"], m["dim"], m["vdim"]) if self.layer_type(i) in ("hgrn2", "lightning") else None
+        if self.layer_is_lightning(i):
+            return (self.num_attention_heads, self.lightning_head_dim, self.lightning_head_dim)
+        return None
+
+    @property
+    def graph_decode(self) -> bool:
+        """A decode step of this family can be captured as a CUDA graph: every per-sequence input (page table, lengths,
+        state slots) is read on the device."""
+        return self.is_layered or not (self.has_recurrent_state or self.is_vl or self.is_mla)
 
     def layer_type(self, i: int) -> str:
+        if self.is_layered:
+            return self.layer_specs[i]["type"]
         if self.layer_is_lightning(i):
             return "lightning_attention"
         return self.layer_types[i] if self.layer_types else "full_attention"
@@ -161,8 +196,26 @@ class ModelConfig:
     def kv_size(self) -> int:
         return self.num_key_value_heads * self.head_dim
 
+    def _layered_params(self, i: int) -> int:
+        h, spec = self.hidden_size, self.layer_specs[i]
+        m, t = spec["mixer"], spec["type"]
+        H, D, Dv = m["heads"], m["dim"], m["vdim"]
+        if t == "latent_attention":
+            n = (h * (m["q_rank"] + m["kv_rank"] + m["rot_dim"]) + m["q_rank"] * (1 + H * (D + m["rot_dim"]))
+                 + m["kv_rank"] * (1 + H * (D + Dv)))
+        elif t == "hgrn2":
+            n = h * H * (2 * D + Dv) + 2 * H * D + Dv
+        else:
+            n = h * H * (2 * D + 2 * Dv) + H * Dv
+        n += h * H * Dv + 3 * h + 1
+        if spec["mlp"] is not None:
+            n += 2 * h * spec["mlp"]["ff"] + 4 + 3 * h + 1
+        return n
+
     def num_params(self) -> int:
         h, L = self.hidden_size, self.num_hidden_layers
+        if self.is_layered:
+            return 2 * self.vocab_size * h + 2 * h + 1 + sum(self._layered_params(i) for i in range(L))
         attn = self.attn_params()
         if self.attention_bias:
             attn += self.q_size + 2 * self.kv_size
@@ -204,6 +257,16 @@ class ModelConfig:
     def flops_per_token(self, seq_len: int, backward: bool = True) -> float:
         """Model FLOPs per token for a sequence of ``seq_len`` (causal attention)."""
         h, L = self.hidden_size, self.num_hidden_layers
+        if self.is_layered:
+            total = 2 * h * self.vocab_size
+            for i, spec in enumerate(self.layer_specs):
+                m = spec["mixer"]
+                total += 2 * self._layered_params(i)
+                if spec["type"] == "latent_attention":
+                    total += 2 * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"]) * (seq_len / 2)
+                else:
+                    total += 4 * m["heads"] * m["dim"] * m["vdim"]
+            return total * (3 if backward else 1)
         lin = self.attn_params()
         act_mlp = (3 * h * self.moe_intermediate_size * self.num_experts_per_tok
                    if self.is_moe else 3 * h * self.intermediate_size)
@@ -220,6 +283,8 @@ class ModelConfig:
             p = p / "config.json" if p.is_dir() else p
             cfg = json.loads(p.read_text())
         top = cfg
+        if cfg.get("architecture") == "Fofosun":
+            return cls._from_fofosun(cfg, overrides)
         if "text_config" in cfg:  # composite (vision-language) checkpoints nest the decoder's config
             cfg = cfg["text_config"]
         mt = cfg.get("model_type", "qwen3")
@@ -352,7 +417,41 @@ class ModelConfig:
             setattr(out, k, v)
         return out
 
+    @classmethod
+    def _from_fofosun(cls, cfg: dict, overrides: dict) -> "ModelConfig":
+        """``config.json`` of a Fofosun checkpoint: ``layers`` lists mixers (``type``, sizes in ``mixer``) and
+        feed-forwards (``mlp``, null for none)."""
+        keys = {"latent_attention": ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "scale", "rot"),
+                "hgrn2": ("heads", "dim", "vdim"), "lightning": ("heads", "dim", "vdim", "decay")}
+        specs = []
+        for i, layer in enumerate(cfg["layers"]):
+            t, m, mlp = layer["type"], layer["mixer"], layer.get("mlp")
+            if t not in keys:
+                raise NotImplementedError(f"layer {i}: mixer {t!r}; supported are {sorted(keys)}")
+            spec = {k: m[k] for k in keys[t]}
+            if t == "latent_attention":
+                spec["rot"] = {"base": float(m["rot"]["base"]), "dims": int(m["rot"]["dims"])}
+                if spec["rot"]["dims"] != spec["rot_dim"] or spec["rot_dim"] % 2:
+                    raise NotImplementedError(f"layer {i}: the rotated part must be rotated whole, in pairs")
+            if t == "lightning" and len(spec["decay"]) != spec["heads"]:
+                raise ValueError(f"layer {i}: {len(spec['decay'])} decays for {spec['heads']} heads")
+            if mlp is not None and mlp.get("kind", "dense") != "dense":
+                raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']!r}; supported is 'dense'")
+            specs.append({"type": t, "mixer": spec, "mlp": None if mlp is None else {"kind": "dense", "ff": mlp["ff"]}})
+        heads = max((s["mixer"]["heads"] for s in specs), default=1)
+        out = cls(model_type="fofosun", vocab_size=cfg["vocab"], hidden_size=cfg["width"], layer_specs=specs,
+                  num_hidden_layers=len(specs), rms_norm_eps=cfg["norm"]["eps"],
+                  intermediate_size=max((s["mlp"]["ff"] for s in specs if s["mlp"]), default=0),
+                  num_attention_heads=heads, num_key_value_heads=heads,
+                  head_dim=max((s["mixer"]["dim"] for s in specs), default=1), tie_word_embeddings=False, qk_norm=False)
+        for k, v in overrides.items():
+            setattr(out, k, v)
+        return out
+
     def to_hf_config(self) -> dict:
+        if self.model_type == "fofosun":
+            return {"architecture": "Fofosun", "layers": self.layer_specs, "norm": {"eps": self.rms_norm_eps},
+                    "vocab": self.vocab_size, "width": self.hidden_size}
         if self.is_vl:
             return self._to_hf_config_vl()
         arch = {"qwen2": "Qwen2ForCausalLM", "qwen3": "Qwen3ForCausalLM",
@@ -586,6 +685,15 @@ PRESETS: dict[str, ModelConfig] = {
                                        qk_nope_head_dim=32, qk_rope_head_dim=16, v_head_dim=32, rope_interleave=True,
                                        lightning_group_size=2, lightning_head_dim=32, lightning_norm_groups=2,
                                        partial_rotary_factor=0.5, max_position_embeddings=32768),
+    # Fofosun at test size: both recurrent mixers and latent attention, layers with and without a feed-forward
+    "tiny-fofosun": ModelConfig._from_fofosun({
+        "vocab": 1024, "width": 192, "norm": {"eps": 1e-6}, "layers": [
+            {"type": "hgrn2", "mixer": {"heads": 3, "dim": 32, "vdim": 16}, "mlp": {"kind": "dense", "ff": 256}},
+            {"type": "latent_attention", "mixer": {"heads": 4, "dim": 32, "rot_dim": 16, "vdim": 32, "q_rank": 64,
+                                                   "kv_rank": 80, "scale": 0.15, "rot": {"base": 1e4, "dims": 16}},
+             "mlp": None},
+            {"type": "lightning", "mixer": {"heads": 2, "dim": 48, "vdim": 64, "decay": [0.7, 0.99]},
+             "mlp": {"kind": "dense", "ff": 320}}]}, {}),
     # DeepSeek-V2-Lite: latent attention without the query bottleneck, softmax routing, two shared experts
     "deepseek-v2-lite": ModelConfig(model_type="deepseek_v2", vocab_size=102400, hidden_size=2048,
                                     intermediate_size=10944, num_hidden_layers=27, num_attention_heads=16,

@@ -17,7 +17,7 @@ q / k / v are rotated on the rank that holds the tokens, exchanged tokens → he
 sp`` heads over the whole packed stream with their slice of the decays), and the outputs are exchanged back.
 
 Generation: the rollout engine keeps the state ``S [heads, head_dim, head_dim]`` (fp32) of every running sequence
-per lightning layer (:class:`LightningState`); a prefill leaves the state after the prompt's last token there, a decode
+per lightning layer (:class:`RecurrentState`); a prefill leaves the state after the prompt's last token there, a decode
 step reads, advances and writes it back.
 
 Checkpoint names: ``attention.{query_key_value,query_layernorm,key_layernorm,g_proj,g_norm,dense}``.
@@ -75,13 +75,14 @@ def _rope_partial(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, rot: in
     return torch.cat((out, x[..., rot:]), dim=-1) if rot < x.shape[-1] else out
 
 
-class LightningState:
-    """``rec[i] [slots, heads, head_dim, head_dim]`` fp32 for lightning layer ``i``, ``None`` for the others."""
+class RecurrentState:
+    """``rec[i] [slots, heads, key width, value width]`` fp32 for every layer with a matrix state per head
+    (``ModelConfig.recurrent_shape``), ``None`` for the others."""
 
     def __init__(self, cfg: ModelConfig, max_slots: int, dtype, device):
-        D = cfg.lightning_head_dim
-        self.rec = [torch.zeros(max_slots, cfg.num_attention_heads, D, D, dtype=torch.float32, device=device)
-                    if cfg.layer_is_lightning(i) else None for i in range(cfg.num_hidden_layers)]
+        shapes = [cfg.recurrent_shape(i) for i in range(cfg.num_hidden_layers)]
+        self.rec = [None if s is None else torch.zeros(max_slots, *s, dtype=torch.float32, device=device)
+                    for s in shapes]
 
 
 class LightningAttention(nn.Module):
@@ -184,3 +185,40 @@ class LightningAttention(nn.Module):
         yield p + "attention.g_proj.weight", self.gate
         yield p + "attention.g_norm.weight", self.g_norm
         yield p + "attention.dense.weight", self.o
+
+
+class ConstantDecayLightning(nn.Module):
+    """Lightning attention with decays given by the configuration, one per head, and SiLU on all three projections
+    (no q / k norms, no rotation, no scale; key and value widths may differ):
+
+        q, k, v = silu(split(W x));   S_t = decay_h S_{t-1} + k_t v_t^T;   o_t = S_t^T q_t
+        result  = rmsnorm(o, all heads together) * sigmoid(W_g x), to be projected by ``o``
+
+    A mixer of the layered decoder (``models/layered.py``): ``hidden`` returns the activations in front of the output
+    projection."""
+
+    def __init__(self, hidden: int, spec: dict, eps: float, dtype, device):
+        super().__init__()
+        self.H, self.D, self.Dv, self.eps = spec["heads"], spec["dim"], spec["vdim"], eps
+        mk = lambda *shape: nn.Parameter(torch.empty(*shape, dtype=dtype, device=device))
+        self.in_proj = mk(self.H * (2 * self.D + 2 * self.Dv), hidden)  # q | k | v | gate
+        self.norm = nn.Parameter(torch.ones(self.H * self.Dv, dtype=dtype, device=device))
+        self.o = mk(hidden, self.H * self.Dv)
+        self.register_buffer("decay", torch.tensor(spec["decay"], dtype=torch.float32, device=device), persistent=False)
+
+    def hidden(self, y, ctx, cache=None, rec=None):
+        from ..ops.dyt import group_rms
+        from ..ops.gated_scan import ScanSpec, scan_prefill, scan_step
+
+        x = linear(y, self.in_proj)
+        spec = ScanSpec("lightning", self.H, self.D, self.Dv, decay=self.decay)
+        o = scan_step(x, spec, rec, ctx.state_slots) if ctx.decode else \
+            scan_prefill(x, spec, ctx.meta, rec, ctx.state_slots)
+        return group_rms(o, self.norm, 1, self.eps, gate=spec.gate(x))
+
+    def tensors(self, p: str):
+        a, b = self.H * self.D, self.H * self.Dv
+        for name, lo, hi in (("q", 0, a), ("k", a, 2 * a), ("v", 2 * a, 2 * a + b), ("g", 2 * a + b, 2 * a + 2 * b)):
+            yield p + name, self.in_proj[lo:hi]
+        yield p + "norm", self.norm
+        yield p + "o", self.o

@@ -170,3 +170,54 @@ class MLAttention(nn.Module):
         yield p + "kv_a_layernorm.weight", self.kv_a_norm
         yield p + "kv_b_proj.weight", self.kv_b
         yield p + ("dense.weight" if bailing else "o_proj.weight"), self.o
+
+
+class LatentAttention(nn.Module):
+    """Latent attention served from a compressed cache: a token leaves its normed latent and one rotated key part
+    shared by all heads (``rank + rot`` numbers) instead of every head's keys and values.
+
+        c_q = rmsnorm(W_dq x);  q = W_uq c_q          per head [unrotated | rotated]
+        c, r = split(W_dkv x);  c = rmsnorm(c)        latent, shared rotated key part
+        k_h = [W_uk,h c | rope(r)],  v_h = W_uv,h c;  softmax(q k^T * scale) v, causal
+
+    Rotation turns neighbouring pairs and keeps the layout. A mixer of the layered decoder (``models/layered.py``):
+    ``hidden`` returns the concatenated heads in front of the output projection. Prefills expand keys and values
+    (``ops/latent_attn.py::latent_attention``); decode steps stay in the latent space (``latent_decode``)."""
+
+    def __init__(self, hidden: int, spec: dict, eps: float, dtype, device):
+        super().__init__()
+        self.H, self.D, self.R, self.Dv = spec["heads"], spec["dim"], spec["rot_dim"], spec["vdim"]
+        self.q_rank, self.rank, self.scale, self.eps = spec["q_rank"], spec["kv_rank"], float(spec["scale"]), eps
+        self.rot_base = float(spec["rot"]["base"])
+        mk = lambda *shape: nn.Parameter(torch.empty(*shape, dtype=dtype, device=device))
+        ones = lambda n: nn.Parameter(torch.ones(n, dtype=dtype, device=device))
+        self.down = mk(self.q_rank + self.rank + self.R, hidden)        # dq | dkv (latent, rotated part)
+        self.q_norm, self.c_norm = ones(self.q_rank), ones(self.rank)
+        self.uq = mk(self.H * (self.D + self.R), self.q_rank)
+        self.ukv = mk(self.H * (self.D + self.Dv), self.rank)           # uk | uv
+        self.o = mk(hidden, self.H * self.Dv)
+
+    def hidden(self, y, ctx, cache=None, rec=None):
+        from ..ops import latent_attn as la
+
+        H, D, R = self.H, self.D, self.R
+        cos, sin = ctx.rotary(R, self.rot_base)
+        cq, c, kr = la.latent_prep(linear(y, self.down), self.q_norm, self.c_norm, self.rank, R, self.eps, cos, sin,
+                                   ctx.pos, cache, ctx.slot_mapping, want_rows=not ctx.decode)
+        q = la.rope_pairs_(linear(cq, self.uq), H, D, R, cos, sin, ctx.pos)
+        if not ctx.decode:
+            return la.latent_attention(q, linear(c, self.ukv), kr, ctx.meta, H, D, R, self.Dv, self.scale)
+        qa = la.heads_matmul(q, H, D, self.ukv[:H * D], transposed=True)
+        ol = la.latent_decode(qa, q, cache, ctx.block_table, ctx.seq_lens, H, D, R, self.rank, self.scale,
+                              ctx.max_seq_len)
+        return la.heads_matmul(ol, H, self.rank, self.ukv[H * D:], transposed=False)
+
+    def tensors(self, p: str):
+        yield p + "dq", self.down[:self.q_rank]
+        yield p + "dkv", self.down[self.q_rank:]
+        yield p + "dq.norm", self.q_norm
+        yield p + "dkv.norm", self.c_norm
+        yield p + "uq", self.uq
+        yield p + "uk", self.ukv[:self.H * self.D]
+        yield p + "uv", self.ukv[self.H * self.D:]
+        yield p + "o", self.o

@@ -968,6 +968,10 @@ def build_model(cfg: ModelConfig, dtype=torch.bfloat16, device="cpu", seed: int 
         from .qwen_vl import QwenVLModel
 
         m = QwenVLModel(cfg, dtype=dtype, device=device, pctx=pctx)
+    elif cfg.is_layered:
+        from .layered import LayeredModel
+
+        m = LayeredModel(cfg, dtype=dtype, device=device, pctx=pctx)
     else:
         m = QwenModel(cfg, dtype=dtype, device=device, pctx=pctx)
     if seed is not None:
