@@ -100,6 +100,7 @@ sample_kernel(const float* __restrict__ logits, long long ld, int V,
     if (tid == 0) {
       int best = 0x7fffffff;
       for (int w = 0; w < kSampThreads / 32; ++w) best = min(best, s_cand[w]);
+      if (best >= V) best = 0;  // a row without any maximum (all NaN): the NaN log-probability tells
       tokens[row] = best;
       logprobs[row] = x[best] * inv_t - logZ;
     }

@@ -319,6 +319,8 @@ class NativeRolloutEngine(InferenceEngine):
         use_cuda = torch.cuda.is_available()
         self.device = torch.device(device) if device is not None else (
             torch.device("cuda", torch.cuda.current_device()) if use_cuda else torch.device("cpu"))
+        if self.device.type == "cuda" and self.device.index is None:  # the loop thread selects the device by its index
+            self.device = torch.device("cuda", torch.cuda.current_device())
         if ncfg.model_path:
             mc = ModelConfig.from_hf_config(ncfg.model_path)
         elif ncfg.model_preset:
