@@ -1,0 +1,311 @@
+// Decode attention over the compressed latent cache on tensor cores: one query token per sequence, all heads of it
+// against the same cached rows [rank | rot] (see latent_attn.cu). A cached row is read once for 16 heads and serves as
+// key (all of it) and value (its first `rank` numbers), so the kernel is bound by the cache stream.
+//
+// One CTA per (sequence, group of 16 heads, split): 4 warps, tiles of 32 tokens in a ring of stages. The rows of a tile
+// arrive by bulk copies (one per token, rows are padded to an odd number of 16-byte units so that ldmatrix is free of
+// bank conflicts). Warp w computes the scores of tokens 8w..8w+7; the [16, 32] scores meet in shared memory, every warp
+// takes the softmax of all of them (max, sum and weights in fp32) and multiplies its share of the value columns. The
+// weights enter the product as two bf16 terms (hi + lo), so they keep fp32-like precision.
+#include "common/host_utils.h"
+#include "common/io.cuh"
+#include "common/mma16.cuh"
+#include "common/ptx.cuh"
+
+namespace b200 {
+
+constexpr int kLdTok = 32;     // tokens per tile
+constexpr int kLdWarps = 4;
+constexpr int kLdSPitch = 40;  // floats per score row
+constexpr int kLdMaxStages = 4;
+
+struct LatentDecodeArgs {
+  const __nv_bfloat16 *qa, *q, *cache;
+  long long ldqa, ldq;
+  int q_stride, q_off;  // rotated query part of head h: q + h * q_stride + q_off
+  const int *block_table, *seq_lens;
+  __nv_bfloat16* out;   // [B, H * rank]
+  float *o_part, *ml_part;
+  int H, rank, rot, block_size, max_blocks, nsplit, stages, pitch;  // pitch: bytes of a row in shared memory
+  float scale_log2;
+};
+
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                   smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+}
+
+// NP: pairs of value column tiles (16 columns) per warp
+template <int NP>
+__global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentDecodeArgs a, int* status) {
+  extern __shared__ __align__(128) uint8_t sm[];
+  const int W = a.rank + a.rot, pitch = a.pitch;
+  uint64_t* full = reinterpret_cast<uint64_t*>(sm);                        // [stages]
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + 64);
+  float* sS = reinterpret_cast<float*>(sm + 128);                          // [2][16][kLdSPitch]
+  uint8_t* sQ = sm + 128 + 2 * 16 * kLdSPitch * 4;                         // [16][pitch]
+  uint8_t* ring = sQ + 16 * pitch;                                         // [stages][32][pitch]
+  const int b = blockIdx.x, h0 = blockIdx.y * 16, split = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int L = a.seq_lens[b];
+  const int tiles = (L + kLdTok - 1) / kLdTok, per = (tiles + a.nsplit - 1) / a.nsplit;
+  const int j0 = split * per, n = max(0, min(tiles, j0 + per) - j0);
+  const int* bt = a.block_table + static_cast<long long>(b) * a.max_blocks;
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < a.stages; ++i) mbar_init(&full[i], 1);
+    *abort_flag = 0;
+    fence_mbar_init();
+  }
+  // queries: 16 rows of W, zero for heads past the last
+  for (int i = threadIdx.x; i < 16 * (W / 8); i += blockDim.x) {
+    const int r = i / (W / 8), c = (i % (W / 8)) * 8, h = h0 + r;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (h < a.H)
+      v = c < a.rank ? *reinterpret_cast<const uint4*>(a.qa + b * a.ldqa + static_cast<long long>(h) * a.rank + c)
+                     : *reinterpret_cast<const uint4*>(a.q + b * a.ldq + static_cast<long long>(h) * a.q_stride + a.q_off + c - a.rank);
+    *reinterpret_cast<uint4*>(sQ + r * pitch + c * 2) = v;
+  }
+  __syncthreads();
+
+  // warp 0 fills a stage: lane = token of the tile; rows past the end are zeroed (a weight of 0 must meet a number)
+  auto fill = [&](int j) {
+    uint64_t* bar = &full[j % a.stages];
+    const int tok = (j0 + j) * kLdTok + lane;
+    uint8_t* dst = ring + ((j % a.stages) * kLdTok + lane) * pitch;
+    const int valid = min(kLdTok, L - (j0 + j) * kLdTok);
+    if (lane >= valid)
+      for (int i = 0; i < W / 8; ++i) *reinterpret_cast<uint4*>(dst + i * 16) = make_uint4(0, 0, 0, 0);
+    __syncwarp();
+    if (lane == 0) mbar_arrive_expect_tx(bar, valid * W * 2);
+    __syncwarp();
+    if (lane < valid) {
+      const long long row = static_cast<long long>(bt[tok / a.block_size]) * a.block_size + tok % a.block_size;
+      bulk_load(dst, a.cache + row * W, W * 2, bar);
+    }
+  };
+  if (warp == 0)
+    for (int j = 0; j < a.stages && j < n; ++j) fill(j);
+
+  float o[2 * NP][4];
+#pragma unroll
+  for (int i = 0; i < 2 * NP; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) o[i][c] = 0.f;
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;  // rows g and g + 8
+  const int g = lane >> 2, t = lane & 3;
+  const int pairs = a.rank >> 4;
+  const uint32_t qrow = smem_u32(sQ) + (lane & 15) * pitch + (lane >> 4) * 16;
+  bool ok = true;
+  for (int j = 0; j < n; ++j) {
+    const int st = j % a.stages;
+    if (!mbar_wait(&full[st], (j / a.stages) & 1, abort_flag)) {
+      ok = false;
+      *abort_flag = 1;
+    }
+    const uint32_t base = smem_u32(ring + st * kLdTok * pitch);
+    float s[4] = {0.f, 0.f, 0.f, 0.f};
+    if (ok) {
+      // scores of this warp's 8 tokens: two key blocks of 16 per ldmatrix
+      const uint32_t krow = base + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 16;
+      float s2[4] = {0.f, 0.f, 0.f, 0.f};  // a second chain hides the tensor-core latency
+      const int kt = W >> 4;
+      int k = 0;
+      for (; k + 2 <= kt; k += 2) {
+        uint32_t kb[4], qf[4];
+        ldm_x4(krow + k * 32, kb);
+        ldm_x4(qrow + k * 32, qf);
+        mma_bf16(s, qf, kb[0], kb[1]);
+        ldm_x4(qrow + k * 32 + 32, qf);
+        mma_bf16(s2, qf, kb[2], kb[3]);
+      }
+      if (k < kt) {
+        uint32_t kb[2], qf[4];
+        ldm_x2(base + (warp * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 16 + k * 32, kb);
+        ldm_x4(qrow + k * 32, qf);
+        mma_bf16(s, qf, kb[0], kb[1]);
+      }
+#pragma unroll
+      for (int c = 0; c < 4; ++c) s[c] += s2[c];
+    }
+    float* S = sS + (j & 1) * 16 * kLdSPitch;
+    *reinterpret_cast<float2*>(S + g * kLdSPitch + warp * 8 + 2 * t) = make_float2(s[0], s[1]);
+    *reinterpret_cast<float2*>(S + (g + 8) * kLdSPitch + warp * 8 + 2 * t) = make_float2(s[2], s[3]);
+    __syncthreads();  // scores complete; every warp has left tile j - 1
+    if (*abort_flag) { ok = false; break; }
+    if (warp == 0 && j >= 1 && j - 1 + a.stages < n) {
+      fence_proxy_async_smem();  // the stage was read through the generic proxy
+      fill(j - 1 + a.stages);
+    }
+    // softmax of the 16 x 32 scores; fragment order: [k block][row half][8-column half][2]
+    float p[2][2][2][2];
+    float x0 = -INFINITY, x1 = -INFINITY;
+    const int tok = (j0 + j) * kLdTok + 2 * t;
+#pragma unroll
+    for (int kb = 0; kb < 2; ++kb)
+#pragma unroll
+      for (int ch = 0; ch < 2; ++ch) {
+        const float2 u = *reinterpret_cast<const float2*>(S + g * kLdSPitch + kb * 16 + ch * 8 + 2 * t);
+        const float2 v = *reinterpret_cast<const float2*>(S + (g + 8) * kLdSPitch + kb * 16 + ch * 8 + 2 * t);
+        const bool a0 = tok + kb * 16 + ch * 8 < L, a1 = tok + kb * 16 + ch * 8 + 1 < L;
+        p[kb][0][ch][0] = a0 ? u.x * a.scale_log2 : -INFINITY;
+        p[kb][0][ch][1] = a1 ? u.y * a.scale_log2 : -INFINITY;
+        p[kb][1][ch][0] = a0 ? v.x * a.scale_log2 : -INFINITY;
+        p[kb][1][ch][1] = a1 ? v.y * a.scale_log2 : -INFINITY;
+        x0 = fmaxf(x0, fmaxf(p[kb][0][ch][0], p[kb][0][ch][1]));
+        x1 = fmaxf(x1, fmaxf(p[kb][1][ch][0], p[kb][1][ch][1]));
+      }
+    x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
+    x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
+    // the running maximum is raised only when a score passes it by 2^8 (every tile holds at least one token)
+    const bool up0 = x0 > m0 + 8.f, up1 = x1 > m1 + 8.f;
+    if (__any_sync(0xffffffffu, up0 || up1)) {
+      const float n0 = up0 ? x0 : m0, n1 = up1 ? x1 : m1;
+      const float c0 = m0 == -INFINITY ? 0.f : exp2f(m0 - n0), c1 = m1 == -INFINITY ? 0.f : exp2f(m1 - n1);
+      l0 *= c0; l1 *= c1; m0 = n0; m1 = n1;
+#pragma unroll
+      for (int i = 0; i < 2 * NP; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+    }
+    uint32_t hi[2][4], lo[2][4];
+#pragma unroll
+    for (int kb = 0; kb < 2; ++kb)
+#pragma unroll
+      for (int ch = 0; ch < 2; ++ch) {
+        const float p00 = exp2f(p[kb][0][ch][0] - m0), p01 = exp2f(p[kb][0][ch][1] - m0);
+        const float p10 = exp2f(p[kb][1][ch][0] - m1), p11 = exp2f(p[kb][1][ch][1] - m1);
+        l0 += p00 + p01;
+        l1 += p10 + p11;
+        hi[kb][ch * 2] = split2(p00, p01, lo[kb][ch * 2]);
+        hi[kb][ch * 2 + 1] = split2(p10, p11, lo[kb][ch * 2 + 1]);
+      }
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      const int pr = warp + i * kLdWarps;
+      if (pr < pairs) {
+#pragma unroll
+        for (int kb = 0; kb < 2; ++kb) {
+          uint32_t v[4];  // tokens 0-7 / 8-15 of the block x columns 0-7, then columns 8-15
+          ldm_x4_t(base + (kb * 16 + (lane & 15)) * pitch + (pr * 16 + (lane >> 4) * 8) * 2, v);
+          mma_bf16(o[2 * i], hi[kb], v[0], v[1]);
+          mma_bf16(o[2 * i + 1], hi[kb], v[2], v[3]);
+          mma_bf16(o[2 * i], lo[kb], v[0], v[1]);
+          mma_bf16(o[2 * i + 1], lo[kb], v[2], v[3]);
+        }
+      }
+    }
+  }
+  if (!ok) {
+    if (threadIdx.x == 0) {
+      atomicCAS(status, 0, kErrMbarTimeoutEpilogue);
+      const unsigned long long t0 = globaltimer_ns();  // copies in flight land before the CTA retires
+      while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
+    }
+    return;
+  }
+  l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
+  l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  const bool direct = a.nsplit == 1;
+  const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int h = h0 + g + half * 8;
+    if (h >= a.H) continue;
+    const long long u = (static_cast<long long>(b) * a.H + h);
+    const float inv = half ? i1 : i0;
+#pragma unroll
+    for (int i = 0; i < 2 * NP; ++i) {
+      const int pr = warp + (i >> 1) * kLdWarps;
+      if (pr >= pairs) continue;
+      const int c = pr * 16 + (i & 1) * 8 + 2 * t;
+      const float v0 = o[i][half * 2], v1 = o[i][half * 2 + 1];
+      if (direct)
+        *reinterpret_cast<uint32_t*>(a.out + u * a.rank + c) = pack2(v0 * inv, v1 * inv);
+      else
+        *reinterpret_cast<float2*>(a.o_part + (u * a.nsplit + split) * a.rank + c) = make_float2(v0, v1);
+    }
+    if (!direct && warp == 0 && t == 0) {
+      a.ml_part[(u * a.nsplit + split) * 2] = half ? m1 : m0;
+      a.ml_part[(u * a.nsplit + split) * 2 + 1] = half ? l1 : l0;
+    }
+  }
+}
+
+// One block per (sequence, head); threads over the columns, two at a time.
+__global__ void latent_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ ml,
+                                    __nv_bfloat16* __restrict__ out, int nsplit, int rank) {
+  __shared__ float w[64];
+  const long long u = blockIdx.x;
+  float m = -INFINITY, l = 0.f;
+  for (int s = 0; s < nsplit; ++s) m = fmaxf(m, ml[(u * nsplit + s) * 2]);
+  for (int s = 0; s < nsplit; ++s) {
+    const float ms = ml[(u * nsplit + s) * 2];
+    const float e = ms == -INFINITY ? 0.f : exp2f(ms - m);
+    l += ml[(u * nsplit + s) * 2 + 1] * e;
+    if (threadIdx.x == 0) w[s] = e;
+  }
+  __syncthreads();
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  for (int c = threadIdx.x * 2; c < rank; c += blockDim.x * 2) {
+    float x = 0.f, y = 0.f;
+    for (int s = 0; s < nsplit; ++s) {
+      if (w[s] == 0.f) continue;  // an empty split
+      const float2 v = *reinterpret_cast<const float2*>(o_part + (u * nsplit + s) * rank + c);
+      x = fmaf(v.x, w[s], x);
+      y = fmaf(v.y, w[s], y);
+    }
+    *reinterpret_cast<uint32_t*>(out + u * rank + c) = pack2(x * inv, y * inv);
+  }
+}
+
+}  // namespace b200
+
+extern "C" {
+
+// 0 when the kernel takes these widths (bf16), negative otherwise.
+int b200_latent_decode_ok(int rank, int rot) {
+  using namespace b200;
+  return (rank % 16 == 0 && rot % 16 == 0 && rank >= 16 && rank <= 512 && rot <= 128) ? 0 : -100;
+}
+
+// qa [B][ldqa]: head h at h * rank; q [B][ldq]: rotated part of head h at h * q_stride + q_off. All bf16, 16-byte
+// aligned, pitches and strides multiples of 8. cache rows are rank + rot wide. nsplit <= 64.
+int b200_latent_decode(const void* qa, long long ldqa, const void* q, long long ldq, int q_stride, int q_off,
+                       const void* cache, const int* block_table, int max_blocks, int block_size, const int* seq_lens,
+                       void* out, float* o_part, float* ml_part, int B, int H, int rank, int rot, int nsplit,
+                       float scale, cudaStream_t stream) {
+  using namespace b200;
+  if (B <= 0) return 0;
+  if (b200_latent_decode_ok(rank, rot) || (ldqa & 7) || (ldq & 7) || (q_stride & 7) || (q_off & 7) || nsplit < 1 || nsplit > 64)
+    return -100;
+  using bf = __nv_bfloat16;
+  const int W = rank + rot, pitch = ((W / 8) | 1) * 16;
+  const int fixed = 128 + 2 * 16 * kLdSPitch * 4 + 16 * pitch, stage = kLdTok * pitch;
+  int stages = (112 * 1024 - fixed) / stage;
+  stages = stages < 2 ? 2 : stages > kLdMaxStages ? kLdMaxStages : stages;
+  const int smem = fixed + stages * stage;
+  LatentDecodeArgs a{(const bf*)qa, (const bf*)q, (const bf*)cache, ldqa, ldq, q_stride, q_off, block_table, seq_lens,
+                     (bf*)out, o_part, ml_part, H, rank, rot, block_size, max_blocks, nsplit, stages, pitch,
+                     scale * 1.4426950408889634f};
+  int* status = device_status_word();
+  if (!status) return -3;
+  dim3 grid(B, (H + 15) / 16, nsplit);
+  const int np = (rank / 16 + kLdWarps - 1) / kLdWarps;
+#define B200_LD(NP_)                                                                                                \
+  {                                                                                                                 \
+    B200_CHECK(cudaFuncSetAttribute(latent_decode_kernel<NP_>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)); \
+    latent_decode_kernel<NP_><<<grid, kLdWarps * 32, smem, stream>>>(a, status);                                    \
+  }
+  if (np <= 1) B200_LD(1)
+  else if (np <= 2) B200_LD(2)
+  else if (np <= 4) B200_LD(4)
+  else if (np <= 6) B200_LD(6)
+  else B200_LD(8)
+#undef B200_LD
+  B200_CHECK(cudaGetLastError());
+  if (nsplit > 1) {
+    latent_merge_kernel<<<B * H, rank >= 256 ? 256 : 128, 0, stream>>>(o_part, ml_part, (bf*)out, nsplit, rank);
+    B200_CHECK(cudaGetLastError());
+  }
+  return 0;
+}
+
+}  // extern "C"

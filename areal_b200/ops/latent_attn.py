@@ -1,4 +1,5 @@
-"""Latent attention over a compressed cache (``csrc/latent_attn.cu``): what a token leaves behind is its normed latent
+"""Latent attention over a compressed cache (``csrc/latent_attn.cu``,
+``csrc/latent_decode.cu``): what a token leaves behind is its normed latent
 and one rotated key part shared by all heads, ``rank + rot`` numbers in a paged cache ``[blocks, 1, block_size, rank +
 rot]``.
 
@@ -179,6 +180,27 @@ def latent_decode_ref(qa, q, cache, block_table, seq_lens, H, D, rot, rank, scal
     return out.reshape(B, H * rank).to(q.dtype)
 
 
+def _latent_decode_mma(qa, q, cache, block_table, seq_lens, H, D, rot, rank, scale, max_seq_len):
+    B = q.shape[0]
+    ctas = B * -(-H // 16)
+    # two CTAs per SM and a few waves of them; a split keeps at least 128 tokens
+    nsplit = max(1, min(64, 1184 // ctas, max_seq_len // 128))
+    c, ll = ctypes.c_int, ctypes.c_longlong
+    out = torch.empty((B, H * rank), dtype=q.dtype, device=q.device)
+    o_part = ml = None
+    if nsplit > 1:
+        o_part = torch.empty((B, H, nsplit, rank), dtype=torch.float32, device=q.device)
+        ml = torch.empty((B, H, nsplit, 2), dtype=torch.float32, device=q.device)
+    rc = _lib.kernels().b200_latent_decode(
+        _lib.ptr(qa), ll(qa.stride(0)), _lib.ptr(q), ll(q.stride(0)), c(D + rot), c(D), _lib.ptr(cache),
+        _lib.ptr(block_table), c(block_table.shape[1]), c(cache.shape[2]), _lib.ptr(seq_lens), _lib.ptr(out),
+        _lib.ptr(o_part), _lib.ptr(ml), c(B), c(H), c(rank), c(rot), c(nsplit), ctypes.c_float(scale),
+        _lib.stream_ptr())
+    _lib.check(rc, "b200_latent_decode")
+    _lib.count_launch(2 if nsplit > 1 else 1)
+    return out
+
+
 def latent_decode(qa, q, cache, block_table, seq_lens, H: int, D: int, rot: int, rank: int, scale: float,
                   max_seq_len: int | None = None):
     """One query token per sequence against its pages: ``qa [B, H * rank]`` are the queries in latent space, the rotated
@@ -194,6 +216,10 @@ def latent_decode(qa, q, cache, block_table, seq_lens, H: int, D: int, rot: int,
         used = torch.arange(block_table.shape[1], device=q.device)[None, :] < ((lens + bs - 1) // bs)[:, None]
         _lib.check_index("latent_decode.block_table", block_table[:B], cache.shape[0], where=used)
     rows = cache.view(-1, rank + rot)
+    if (q.dtype == torch.bfloat16 and _lib.kernels().b200_latent_decode_ok(ctypes.c_int(rank), ctypes.c_int(rot)) == 0
+            and D % 8 == 0 and cache.is_contiguous() and all(t.is_contiguous() and t.data_ptr() % 16 == 0
+                                                             for t in (qa, q, cache))):
+        return _latent_decode_mma(qa, q, cache, block_table, seq_lens, H, D, rot, rank, scale, max_seq_len)
     nsplit = 1
     while B * -(-H // 4) * nsplit < 1184 and nsplit < 64 and max_seq_len // (nsplit * 2) >= 64:
         nsplit *= 2
