@@ -14,44 +14,9 @@
 // token with bf16 inputs that were activated beforehand.
 #include "common/host_utils.h"
 #include "common/io.cuh"
+#include "common/scan_inputs.cuh"
 
 namespace b200 {
-
-struct ScanArgs {
-  const void* x;       // [T, row] projections, pitch ldx
-  long long ldx;
-  const void* bias;    // mode 0: [H * D] gate bias (model dtype)
-  const void* lower;   // mode 0: [H * D] lower bound of the gate (model dtype)
-  const float* decay;  // mode 1: [H]
-  const int* cu;       // prefill: [n_seq + 1]
-  const int* slots;    // [n_seq] state slot of every sequence (negative: keep nothing)
-  float* state;        // [n_slots, H, D, Dv]
-  float* o;            // [T, H, Dv] fp32
-  int H, D, Dv, mode;
-};
-
-// q, f and k of one channel of one token.
-template <class T>
-__device__ __forceinline__ void scan_channel(const ScanArgs& a, const T* row, int h, int d, float& q, float& f,
-                                             float& k) {
-  const int hd = h * a.D + d;
-  q = silu_acc(ld1(row + hd));
-  const float u = ld1(row + a.H * a.D + hd);
-  if (a.mode == 0) {
-    const float z = u + ld1(static_cast<const T*>(a.bias) + hd), l = ld1(static_cast<const T*>(a.lower) + hd);
-    // 1 - f as (1 - l) sigmoid(-z): no cancellation when the gate is nearly open
-    k = (1.f - l) * sigmoid_f(-z);
-    f = fmaf(1.f - l, sigmoid_f(z), l);
-  } else {
-    k = silu_acc(u);
-    f = a.decay[h];
-  }
-}
-template <class T>
-__device__ __forceinline__ float scan_value(const ScanArgs& a, const T* row, int h, int j) {
-  const float v = ld1(row + 2 * a.H * a.D + h * a.Dv + j);
-  return a.mode == 0 ? v : silu_acc(v);
-}
 
 // Token-by-token form for any D and Dv: one block per (sequence, head, 32 value columns). Lane = column, the warps
 // split the rows; the state slice [D][32] stays in shared memory. Tokens come in groups of kGrp whose activations are

@@ -14,7 +14,6 @@ from __future__ import annotations
 import torch
 import torch.nn as nn
 
-from ..ops.dyt import group_rms
 from ..ops.gated_scan import ScanSpec, scan_prefill, scan_step
 from ..ops.gemm import linear
 
@@ -33,9 +32,9 @@ class HGRN2(nn.Module):
     def hidden(self, y, ctx, cache=None, rec=None):
         x = linear(y, self.in_proj)
         spec = ScanSpec("hgrn2", self.H, self.D, self.Dv, bias=self.f_bias, lower=self.lower)
-        if ctx.decode:  # the head's norm runs in the step kernel
+        if ctx.decode:  # the heads' norm runs in the recurrence kernels
             return scan_step(x, spec, rec, ctx.state_slots, self.norm, self.eps)
-        return group_rms(scan_prefill(x, spec, ctx.meta, rec, ctx.state_slots), self.norm, self.H, self.eps)
+        return scan_prefill(x, spec, ctx.meta, rec, ctx.state_slots, self.norm, self.eps)
 
     def tensors(self, p: str):
         a = self.H * self.D

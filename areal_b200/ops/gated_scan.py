@@ -1,4 +1,5 @@
-"""Gated linear recurrences on fused input projections (``csrc/gated_scan.cu``):
+"""Gated linear recurrences on fused input projections (``csrc/gated_scan.cu``, prefills of
+bf16 models: ``csrc/gated_scan_chunk.cu``):
 
     S_t = diag(f_t) S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t        per head, fp32 state [D, Dv]
 
@@ -21,7 +22,7 @@ import torch
 import torch.nn.functional as F
 
 from . import _lib
-from .dyt import fp32_flag, kernel_ok
+from .dyt import fp32_flag, group_rms, group_rms_ref, kernel_ok
 
 
 @dataclass
@@ -51,7 +52,7 @@ class ScanSpec:
             k = ((1 - low) * torch.sigmoid(-z)).view(T, H, D)
             return q, f, k, v
         f = self.decay.view(1, H, 1).expand(T, H, D)
-        return q, f, F.silu(u).view(T, H, D), F.silu(v)
+        return q, f, F.silu(u).view(T, H, D), F.silu(v).to(x.dtype).float()  # values have the model's precision
 
     def gate(self, x: torch.Tensor):
         """The output gate's columns of ``x`` (lightning)."""
@@ -84,20 +85,72 @@ def scan_ref(x, spec: ScanSpec, cu, state=None, slots=None):
 
 
 def scan_prefill(x: torch.Tensor, spec: ScanSpec, meta, state: torch.Tensor | None = None,
-                 slots: torch.Tensor | None = None):
+                 slots: torch.Tensor | None = None, norm_w: torch.Tensor | None = None, eps: float = 0.0):
+    """With ``norm_w`` (``[Dv]``) every head's output is RMS-normed and returned in the model's dtype."""
     if not kernel_ok(x, spec.bias, spec.lower):
-        return scan_ref(x, spec, meta.cu_cpu, state, slots)
+        o = scan_ref(x, spec, meta.cu_cpu, state, slots)
+        return o if norm_w is None else group_rms_ref(o, norm_w, spec.heads, eps)
     x = x if x.stride(1) == 1 else x.contiguous()
     T, n_seq = x.shape[0], meta.cu_seqlens.numel() - 1
-    o = torch.empty((T, spec.heads * spec.vdim), dtype=torch.float32, device=x.device)
     slots = slots.to(torch.int32).contiguous() if state is not None else None
     _check_state(spec, state, slots)
+    if x.dtype == torch.bfloat16 and _lib.kernels().b200_scan_chunk_ok(ctypes.c_int(spec.dim), ctypes.c_int(spec.vdim)) == 0:
+        fuse = norm_w is not None and spec.vdim <= 128
+        o = _scan_chunk(x, spec, meta, state, slots, norm_w if fuse else None, eps)
+        return o if fuse or norm_w is None else group_rms(o, norm_w, spec.heads, eps)
+    o = torch.empty((T, spec.heads * spec.vdim), dtype=torch.float32, device=x.device)
     rc = _lib.kernels().b200_scan_tokens(_lib.ptr(x), ctypes.c_longlong(x.stride(0)), *_args(spec),
                                          _lib.ptr(meta.cu_seqlens), _lib.ptr(slots), _lib.ptr(state), _lib.ptr(o),
                                          ctypes.c_int(n_seq), *_dims(spec), fp32_flag(x), _lib.stream_ptr())
     _lib.check(rc, "b200_scan_tokens")
     _lib.count_launch()
-    return o
+    return o if norm_w is None else group_rms(o, norm_w, spec.heads, eps)
+
+
+def segment_length(lens: list[int], units: int, slots: int = 296) -> int:
+    """Tokens per segment for sequences of these lengths with ``units`` independent CTAs (heads x column blocks) each, 0
+    for whole sequences. The walk along a sequence is serial: cut when the longest one would take much longer than the
+    work spread evenly over ``slots`` CTAs (two per SM). A cut costs a second, cheaper pass over the inputs."""
+    even = sum(lens) * units / slots
+    longest = max(lens, default=0)
+    if longest <= 2 * even + 256:
+        return 0
+    return max(128, -(-int(even) // 16) * 16)
+
+
+def _segments(meta, units: int):
+    """Device tables of a packed batch: ``(segments [n, 4], first segment of every sequence, any sequence cut)``."""
+    cu = [int(c) for c in meta.cu_cpu]
+    L = segment_length([b - a for a, b in zip(cu[:-1], cu[1:])], units)
+    cache = meta.__dict__.setdefault("_scan_segments", {})
+    if L not in cache:
+        segs, first = [], [0]
+        for n, (a, b) in enumerate(zip(cu[:-1], cu[1:])):
+            step = L or max(b - a, 1)
+            for t in range(a, b, step):
+                segs.append((t, min(step, b - t), n, int(t + step >= b)))
+            first.append(len(segs))
+        dev = meta.cu_seqlens.device
+        cache[L] = (torch.tensor(segs, dtype=torch.int32).reshape(-1, 4).to(dev),
+                    torch.tensor(first, dtype=torch.int32).to(dev), len(segs) > len(cu) - 1)
+    return cache[L]
+
+
+def _scan_chunk(x, spec: ScanSpec, meta, state, slots, norm_w, eps):
+    H, D, Dv = spec.heads, spec.dim, spec.vdim
+    segs, first, cut = _segments(meta, H * -(-Dv // 128))
+    n = segs.shape[0]
+    new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=x.device)
+    seg_state, seg_decay = (new(n, H, D, Dv), new(n, H, D)) if cut else (None, None)
+    out = torch.empty((x.shape[0], H * Dv), dtype=torch.float32 if norm_w is None else x.dtype, device=x.device)
+    rc = _lib.kernels().b200_scan_chunk(
+        _lib.ptr(x), ctypes.c_longlong(x.stride(0)), *_args(spec), _lib.ptr(segs), ctypes.c_int(n), _lib.ptr(first),
+        ctypes.c_int(first.numel() - 1), _lib.ptr(slots), _lib.ptr(state), _lib.ptr(seg_state), _lib.ptr(seg_decay),
+        _lib.ptr(out if norm_w is None else None), _lib.ptr(norm_w), _lib.ptr(None if norm_w is None else out),
+        ctypes.c_float(eps), *_dims(spec), _lib.stream_ptr())
+    _lib.check(rc, "b200_scan_chunk")
+    _lib.count_launch(3 if cut else 1)
+    return out
 
 
 def _check_state(spec: ScanSpec, state, slots):
@@ -129,8 +182,6 @@ def scan_step(x: torch.Tensor, spec: ScanSpec, state: torch.Tensor, slots: torch
         o = scan_step_ref(x, spec, state, slots)
         if norm_w is None:
             return o
-        from .dyt import group_rms_ref
-
         return group_rms_ref(o, norm_w, spec.heads, eps)
     x = x if x.stride(1) == 1 else x.contiguous()
     B = x.shape[0]

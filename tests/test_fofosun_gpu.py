@@ -111,6 +111,8 @@ def _scan_case(mode, H, D, Dv, T, dt, seed=0):
 
 def _scan_oracle(x, spec, lens):
     q, f, k, v = (t.double().cpu() for t in spec.inputs(x.double()))
+    if spec.mode == "lightning" and x.dtype == torch.bfloat16:
+        v = v.to(torch.bfloat16).double()   # an activated value has the model's precision
     outs, states, s0 = [], [], 0
     for n in lens:
         o, S = oracle.gated_scan(q[s0:s0 + n], f[s0:s0 + n], k[s0:s0 + n], v[s0:s0 + n])
@@ -155,6 +157,32 @@ def test_scan_prefill_and_steps(dt, mode, H, D, Dv):
         _close(state[s], S, tol)
     untouched = [i for i in range(20) if i not in slots.tolist()]
     assert bool((state[untouched] == 7.0).all())
+
+
+@pytest.mark.parametrize("mode", ["hgrn2", "lightning"])
+@pytest.mark.parametrize("D,Dv", [(64, 64), (128, 128), (24, 40)])
+def test_scan_cut_into_segments(mode, D, Dv):
+    """One long sequence beside short ones: it is cut into segments whose states are chained, and the result is that of
+    the uncut walk. With the heads' norm fused."""
+    from areal_b200.ops.attention import VarlenMeta
+    from areal_b200.ops.gated_scan import _segments, scan_prefill
+
+    lens = [1100, 3, 130, 16]
+    spec, x = _scan_case(mode, 2, D, Dv, sum(lens), torch.bfloat16)
+    if mode == "hgrn2":
+        spec.bias.add_(4.0)
+    meta = VarlenMeta([0] + np.cumsum(lens).tolist(), "cuda")
+    assert _segments(meta, 2)[2] and _segments(meta, 2)[0].shape[0] > 8
+    want, states = _scan_oracle(x, spec, lens)
+    state = torch.zeros(4, 2, D, Dv, device="cuda")
+    o = scan_prefill(x, spec, meta, state, torch.arange(4, device="cuda"))
+    _close(o, want, 3e-5)
+    for i in range(4):
+        _close(state[i], states[i], 3e-5)
+    w = _rand(Dv, dt=torch.bfloat16, seed=8)
+    y = scan_prefill(x, spec, meta, state, torch.arange(4, device="cuda"), w, 1e-5)
+    assert y.dtype == torch.bfloat16
+    _close(y, (oracle.rms_norm(want.view(-1, 2, Dv), 1e-5) * w.double().cpu()).reshape(-1, 2 * Dv), 4e-3)
 
 
 def test_scan_of_a_long_sequence_keeps_what_the_first_token_wrote():
