@@ -1,5 +1,5 @@
 """Latent attention over a compressed cache (``csrc/latent_attn.cu``,
-``csrc/latent_decode.cu``): what a token leaves behind is its normed latent
+``csrc/latent_prefill.cu``, ``csrc/latent_decode.cu``): what a token leaves behind is its normed latent
 and one rotated key part shared by all heads, ``rank + rot`` numbers in a paged cache ``[blocks, 1, block_size, rank +
 rot]``.
 
@@ -162,6 +162,16 @@ def latent_attention(q, kv, kr, meta, H: int, D: int, rot: int, Dv: int, scale: 
     [T, rot]``. Returns ``[T, H * Dv]``."""
     if not kernel_ok(q, kv, kr):
         return latent_attention_ref(q, kv, kr, meta.cu_cpu, H, D, rot, Dv, scale)
+    if (q.dtype == torch.bfloat16 and _lib.kernels().b200_latent_prefill_ok(ctypes.c_int(D), ctypes.c_int(rot), ctypes.c_int(Dv)) == 0
+            and all(t.is_contiguous() and t.data_ptr() % 16 == 0 for t in (q, kv, kr))):
+        c = ctypes.c_int
+        out = torch.empty((q.shape[0], H * Dv), dtype=q.dtype, device=q.device)
+        rc = _lib.kernels().b200_latent_prefill(
+            _lib.ptr(q), _lib.ptr(kv), _lib.ptr(kr), _lib.ptr(out), _lib.ptr(meta.fwd_tiles), c(meta.n_fwd), c(q.shape[0]),
+            c(H), c(D), c(rot), c(Dv), ctypes.c_float(scale), _lib.stream_ptr())
+        _lib.check(rc, "b200_latent_prefill")
+        _lib.count_launch()
+        return out
     start, length = _query_rows(meta)
     w = D + rot
     return _attend(q, w, q[:, D:], w, kv, D, kr, 0, kv[:, H * D:], Dv, D, rot, Dv, start, length, None, 1, H, 1, scale)
