@@ -1,0 +1,144 @@
+"""Serving throughput of a layered (Fofosun) model beside the closest other family, the Bailing hybrid, at equal sizes,
+and the new kernels one by one beside their counterparts.
+
+    python bench.py --serving [--serving-sizes s,m,l] [--serving-kernels]
+
+Models: 8 layers of the given width with random weights, 6 recurrent and 2 latent-attention layers, a feed-forward of the
+same width on each. Both run through the rollout engine's scheduler and step functions (captured decode graphs where the
+family has them). Prefill: 8 prompts of 2048 tokens in one step. Decode: 64 sequences at a context of 2048 tokens.
+Times are CUDA events on the launching stream; weights, caches and states exceed the L2. Kernel timings flush the L2
+between iterations; fractions are of the measured peaks.
+"""
+
+from __future__ import annotations
+
+import dataclasses
+import json
+import statistics
+import time
+
+import numpy as np
+import torch
+
+from ..models.config import ModelConfig
+
+SIZES = {  # width, heads, query latent, latent, feed-forward
+    "s": dict(width=1024, heads=8, q_rank=384, kv_rank=256, ff=3072),
+    "m": dict(width=2048, heads=16, q_rank=768, kv_rank=512, ff=6144),
+    "l": dict(width=4096, heads=32, q_rank=1536, kv_rank=512, ff=12288),
+}
+VOCAB, LAYERS = 32000, 8
+
+
+def fofosun_config(width, heads, q_rank, kv_rank, ff) -> ModelConfig:
+    mlp = {"kind": "dense", "ff": ff}
+    lat = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": q_rank, "kv_rank": kv_rank,
+        "scale": 192 ** -0.5, "rot": {"base": 1e4, "dims": 64}}}
+    hg = {"type": "hgrn2", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "vdim": 128}}
+    li = {"type": "lightning", "mlp": mlp, "mixer": {
+        "heads": heads, "dim": 128, "vdim": 128, "decay": np.linspace(0.8, 0.999, heads).tolist()}}
+    return ModelConfig.from_hf_config({"architecture": "Fofosun", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6},
+                                       "layers": [hg, hg, li, lat] * (LAYERS // 4)})
+
+
+def bailing_config(width, heads, q_rank, kv_rank, ff) -> ModelConfig:
+    return ModelConfig(model_type="bailing_hybrid", vocab_size=VOCAB, hidden_size=width, intermediate_size=ff,
+                       num_hidden_layers=LAYERS, num_attention_heads=heads, num_key_value_heads=heads, head_dim=192,
+                       rope_theta=1e4, tie_word_embeddings=False, qk_norm=False, q_lora_rank=q_rank,
+                       kv_lora_rank=kv_rank, qk_nope_head_dim=128, qk_rope_head_dim=64, v_head_dim=128,
+                       rope_interleave=True, lightning_group_size=4, lightning_head_dim=128, lightning_norm_groups=1,
+                       partial_rotary_factor=0.5, max_position_embeddings=8192)
+
+
+def _engine(cfg: ModelConfig, seqs: int, context: int, tokens: int):
+    from ..api.cli_args import InferenceEngineConfig, NativeRolloutConfig
+    from ..engine.rollout_engine import NativeRolloutEngine
+
+    over = {f.name: getattr(cfg, f.name) for f in dataclasses.fields(cfg)}
+    native = NativeRolloutConfig(model_preset="tiny-fofosun", model_overrides=over, context_length=context,
+                                 max_num_seqs=seqs, max_num_batched_tokens=tokens, kv_block_size=16,
+                                 num_kv_blocks=seqs * (context // 16 + 1), cuda_graph_batch_sizes=[seqs])
+    return NativeRolloutEngine(InferenceEngineConfig(backend="native:d1", native=native)).initialize(start_loop=False)
+
+
+def _timed(fn, iters: int, warmup: int = 3) -> float:
+    """Median milliseconds of ``fn`` between two events."""
+    out = []
+    for i in range(warmup + iters):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        if i >= warmup:
+            out.append(a.elapsed_time(b))
+    return statistics.median(out)
+
+
+def serve(cfg: ModelConfig, prompts=8, length=2048, batch=64, steps=20) -> dict:
+    """Prefill and decode tokens per second through the engine."""
+    from ..engine.trace_replay import TraceEntry, TraceReplay
+    from ..ops import _lib
+
+    eng = _engine(cfg, batch, length + 64, prompts * length)
+    g = np.random.default_rng(0)
+    rand = lambda n: g.integers(0, VOCAB, n).tolist()
+    r = TraceReplay(eng)
+    toks = {f"p{i}": rand(length) for i in range(prompts)}
+
+    def prefill():
+        r.step([TraceEntry(k, v) for k, v in toks.items()], list(toks))
+
+    _lib.reset_launch_count()
+    pre_ms = _timed(prefill, 5, 2)
+    # decode: the requests enter in groups that fit one prefill step, then all of them step together
+    s = eng.sched
+    ids = []
+    for i in range(0, batch, prompts):
+        for j in range(i, min(i + prompts, batch)):
+            ids.append(s.add(rand(length), 1 << 30, 0, [], True))
+        assert s.plan() == 1
+        eng._forward_plan(1)
+        s.commit(np.zeros(s.hdr.n_seqs, np.int32), np.zeros(s.hdr.n_seqs, np.float32))
+
+    def step():
+        assert s.plan() == 2
+        n = s.hdr.n_seqs
+        order = s.seq_ids[:n].tolist()
+        if eng._graphs is not None:
+            eng._graphs.run(n, eng._graphs.bucket(n), s, [0.0] * n, eng._rng, eng._graph_slots(order))
+        else:
+            from ..ops.rollout_ops import sample
+
+            h = eng._forward_plan(2)
+            sample(eng.model.logits(h), torch.zeros(n, device=h.device), None, None, torch.rand(n, device=h.device))
+        s.commit(np.zeros(n, np.int32), np.zeros(n, np.float32))
+
+    # eager families pay host time per launch and per sequence: fewer steps are enough
+    dec_ms = _timed(step, steps if eng._graphs is not None else 5, 3)
+    out = dict(params_m=round(cfg.num_params() / 1e6), prefill_ms=round(pre_ms, 3),
+               prefill_tok_s=round(prompts * length / pre_ms * 1e3), decode_ms=round(dec_ms, 3),
+               decode_tok_s=round(batch / dec_ms * 1e3), graph=eng._graphs is not None,
+               launches=_lib.launch_count(), fallbacks=sorted(_lib.fallback_counts()))
+    eng.destroy()
+    eng.flat = eng.hybrid_state = eng._graphs = None
+    return out
+
+
+def main(sizes: list[str], kernels: bool) -> int:
+    t0 = time.time()
+    res: dict = {"benchmark": "serving", "layers": LAYERS, "dtype": "bf16", "data": "random tokens, random weights",
+                 "prefill": "8 x 2048 tokens", "decode": "64 sequences at 2048 tokens", "models": {}}
+    for name in sizes:
+        for fam, make in (("fofosun", fofosun_config), ("bailing_hybrid", bailing_config)):
+            res["models"][f"{fam}-{name}"] = serve(make(**SIZES[name]))
+            torch.cuda.empty_cache()
+    if kernels:
+        from .bench_serving_kernels import run
+
+        res["kernels"] = run()
+    res["seconds"] = round(time.time() - t0)
+    print(json.dumps(res), flush=True)
+    return 0

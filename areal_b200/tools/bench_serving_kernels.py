@@ -1,0 +1,119 @@
+"""Kernels of the layered decoder beside their counterparts in the other families: time, roofline time (the slower of
+algorithmic FLOPs over the measured bf16 peak and algorithmic bytes over the measured copy bandwidth) and the ratio."""
+
+from __future__ import annotations
+
+import numpy as np
+import torch
+
+from ..ops import dyt, fused, latent_attn as la
+from ..ops.attention import VarlenMeta, varlen_attention
+from ..ops.gated_scan import ScanSpec, scan_prefill, scan_step
+from ..ops.gemm import linear_rmsnorm
+from ..ops.linear_attn import linear_attn_prefill, linear_attn_step
+from ..ops.microbench import peaks, timeit
+from ..ops.rollout_ops import paged_decode
+
+BF, F32 = torch.bfloat16, torch.float32
+
+
+def _rand(*shape, dt=BF, s=1.0):
+    return torch.randn(*shape, device="cuda", dtype=dt) * s
+
+
+def _row(name, fn, nbytes=0.0, flops=0.0, iters=10, flush=True):
+    pk = peaks()
+    ms = timeit(fn, iters, flush=flush)
+    roof = max(nbytes / pk["hbm_gbs"] / 1e6, flops / pk["bf16_tflops"] / 1e9)
+    return dict(kernel=name, us=round(ms * 1e3, 1), roofline_us=round(roof * 1e3, 1), times_roofline=round(ms / roof, 2))
+
+
+@torch.no_grad()
+def run() -> list[dict]:
+    out = []
+    H, D, n, L = 16, 128, 8, 2048
+    T = n * L
+    meta = VarlenMeta([L * i for i in range(n + 1)], "cuda")
+    one = VarlenMeta([0, T], "cuda")
+    slots = torch.arange(n, device="cuda", dtype=torch.int32)
+    # --- recurrences, prefill: inputs and outputs once (bf16), final states
+    hg = ScanSpec("hgrn2", H, D, D, bias=_rand(H * D) + 2, lower=torch.rand(H * D, device="cuda").to(BF))
+    li = ScanSpec("lightning", H, D, D, decay=torch.linspace(0.8, 0.999, H, device="cuda"))
+    xh, xl = _rand(T, hg.row), _rand(T, li.row)
+    st = torch.zeros(64, H, D, D, device="cuda")
+    w = _rand(D)
+    io = T * H * D * 2
+    fl = T * H * D * D * 4
+    out.append(_row("scan_prefill hgrn2 8x2048 (norm fused)", lambda: scan_prefill(xh, hg, meta, st, slots, w, 1e-6), 4 * io, fl))
+    out.append(_row("scan_prefill hgrn2 1x16384 (norm fused)", lambda: scan_prefill(xh, hg, one, st, slots[:1], w, 1e-6), 4 * io, fl))
+    out.append(_row("scan_prefill lightning 8x2048", lambda: scan_prefill(xl, li, meta, st, slots), 5 * io, fl))
+    q, k, v = _rand(T, H, D), _rand(T, H, D), _rand(T, H, D)
+    a = torch.rand(T, H, device="cuda")
+    out.append(_row("[bailing] linear_attn_prefill 8x2048", lambda: linear_attn_prefill(q, k, v, a, None, meta.cu_seqlens, 1.0, "simple_gla"), 4 * io, fl, 3))
+    o32, gate, wl = _rand(T, H * D, dt=F32), xl[:, -H * D:], _rand(H * D)
+    out.append(_row("group_rms + gate (lightning) 16384 tokens", lambda: dyt.group_rms(o32, wl, 1, 1e-6, gate), 4 * io))
+    # --- recurrences, one decode step: the state twice
+    B = 64
+    sb = torch.arange(B, device="cuda", dtype=torch.int32)
+    stb = B * H * D * D * 4 * 2
+    out.append(_row("scan_step hgrn2 batch 64 (norm fused)", lambda: scan_step(xh[:B], hg, st, sb, w, 1e-6), stb))
+    out.append(_row("scan_step lightning batch 64", lambda: scan_step(xl[:B], li, st, sb), stb))
+    out.append(_row("[bailing] linear_attn_step batch 64", lambda: linear_attn_step(q[:B], k[:B], v[:B], a[:B], None, st, 1.0, "simple_gla"), stb))
+    # --- latent attention, prefill: causal FLOPs
+    R, rank = 64, 512
+    ql, kv, kr = _rand(T, H * (D + R)), _rand(T, H * 2 * D), _rand(T, R)
+    afl = n * H * L * L / 2 * 2 * (D + R + D)
+    out.append(_row("latent_prefill 8x2048, 16 heads of 128+64 / 128", lambda: la.latent_attention(ql, kv, kr, meta, H, D, R, D, 0.07), 0, afl))
+    q192 = _rand(T, H, D + R)
+    out.append(_row("[bailing] varlen_attention 8x2048, heads of 192", lambda: varlen_attention(q192, q192, q192, meta), 0, afl, 3))
+    out.append(_row("[qwen3] attn_fwd 8x2048, 16 heads of 128", lambda: varlen_attention(q, k, v, meta), 0, n * H * L * L / 2 * 4 * D))
+    # --- latent attention, decode: the cached rows once
+    ctx, bs = 2048, 16
+    nb = B * ctx // bs
+    bt = torch.randperm(nb, device="cuda").view(B, -1).int()
+    lens = torch.full((B,), ctx, device="cuda", dtype=torch.int32)
+    cache = _rand(nb, 1, bs, rank + R)
+    for heads in (16, 32):
+        qa, qr = _rand(B, heads * rank, s=0.1), _rand(B, heads * (D + R))
+        out.append(_row(f"latent_decode batch 64 x 2048, {heads} heads, 512 + 64",
+                        lambda: la.latent_decode(qa, qr, cache, bt, lens, heads, D, R, rank, 0.07, ctx), B * ctx * (rank + R) * 2))
+    kc, vc = _rand(nb, H, bs, D + R), _rand(nb, H, bs, D + R)
+    qd = _rand(B, H, D + R)
+    out.append(_row("[bailing] paged_decode batch 64 x 2048, expanded 16 heads of 192", lambda: paged_decode(qd, kc, vc, bt, lens, max_seq_len=ctx),
+                    2 * B * ctx * H * (D + R) * 2, iters=2))
+    kc, vc = _rand(nb, 8, bs, D), _rand(nb, 8, bs, D)
+    qd = _rand(B, H, D)
+    out.append(_row("[qwen3] paged_decode batch 64 x 2048, 16 / 8 heads of 128", lambda: paged_decode(qd, kc, vc, bt, lens, max_seq_len=ctx),
+                    2 * B * ctx * 8 * D * 2))
+    wuk = _rand(H * D, rank)
+    qq = _rand(B, H * (D + R))
+    out.append(_row("heads_matmul (query to latent) batch 64", lambda: la.heads_matmul(qq, H, D, wuk, True),
+                    H * D * rank * 2 + B * H * (D + R + rank) * 2, iters=20))
+    wuv = _rand(H * D, rank)
+    ol = _rand(B, H * rank)
+    out.append(_row("heads_matmul (latent to value) batch 64", lambda: la.heads_matmul(ol, H, rank, wuv, False),
+                    H * D * rank * 2 + B * H * (D + rank) * 2, iters=20))
+    # --- row kernels
+    W, F = 2048, 6144
+    norm = (torch.tensor(0.5, device="cuda", dtype=BF), _rand(W), _rand(W))
+    sc, res = _rand(W), _rand(T, W, dt=F32)
+    z, act = _rand(T, F), _rand(4)
+    out.append(_row("polynorm 16384 x 6144", lambda: dyt.polynorm(z, act, 1e-6), T * F * 4))
+    gu = _rand(T, 2 * F)
+    out.append(_row("[bailing] swiglu 16384 x 6144", lambda: fused.swiglu(gu), T * F * 6))
+    cos, sin = la.rotary_tables(L, R, 1e4, "cuda")
+    pos = torch.arange(L, device="cuda", dtype=torch.int32).repeat(n)
+    xd, w1, w2 = _rand(T, 768 + rank + R), _rand(768), _rand(rank)
+    out.append(_row("latent_prep 16384 x (768 | 512 | 64)", lambda: la.latent_prep(xd, w1, w2, rank, R, 1e-6, cos, sin, pos), T * (768 + rank + R) * 4))
+    out.append(_row("rope_pairs 16384 x 16 heads x 64", lambda: la.rope_pairs_(ql, H, D, R, cos, sin, pos), T * H * R * 4))
+    aw, ww = _rand(T, W), _rand(W, W, s=W ** -0.5)
+    out.append(_row("linear_residual_dyt 16384 x 2048 x 2048", lambda: dyt.linear_residual_dyt(aw, ww, sc, res, norm), T * W * 12, 2.0 * T * W * W))
+    resb, wn = _rand(T, W), _rand(W)
+    out.append(_row("[bailing] linear + rmsnorm 16384 x 2048 x 2048", lambda: linear_rmsnorm(aw, ww, wn, 1e-6, resb), T * W * 10, 2.0 * T * W * W))
+    out.append(_row("linear_residual_dyt 64 x 2048 x 2048", lambda: dyt.linear_residual_dyt(aw[:B], ww, sc, res[:B], norm), W * W * 2, iters=20))
+    out.append(_row("[bailing] linear_rmsnorm 64 x 2048 x 2048", lambda: linear_rmsnorm(aw[:B], ww, wn, 1e-6, resb[:B]), W * W * 2, iters=20))
+    out.append(_row("residual_dyt 16384 x 2048", lambda: dyt.residual_dyt(aw, sc, res, norm), T * W * 12))
+    ids = torch.from_numpy(np.random.default_rng(0).integers(0, 32000, T)).to("cuda")
+    table = _rand(32000, W)
+    out.append(_row("embed_dyt 16384 x 2048", lambda: dyt.embed_dyt(ids, table, norm), T * W * 8))
+    return out
