@@ -45,7 +45,14 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return t;
 }
 
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float silu_acc(float x) { return x / (1.f + expf(-x)); }
+// tanh for results in the given dtype: fp32 gets the library function; for bf16 results 1 - 2 / (1 + e^2x), whose absolute
+// error (about 1e-7 of the range) is far below the result's rounding.
+__device__ __forceinline__ float tanh_as(float x, const float*) { return tanhf(x); }
+__device__ __forceinline__ float tanh_as(float x, const __nv_bfloat16*) {
+  return 1.f - __fdividef(2.f, 1.f + __expf(2.f * x));
+}
+
+__device__ __forceinline__ float sigmoid_as(float x, const float*) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_as(float x, const __nv_bfloat16*) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
 }  // namespace b200

@@ -28,9 +28,15 @@ __device__ __forceinline__ void scan_activate(int mode, float u0, float u1, floa
   if (mode == 0) {
     const float z = u1 + bias, e = __expf(-fabsf(z));
     const float big = __fdividef(1.f, 1.f + e), small = e * big;  // sigmoid(|z|), sigmoid(-|z|)
-    // 1 - f as (1 - l) sigmoid(-z): no cancellation when the gate is nearly open
-    k = (1.f - low) * (z >= 0.f ? small : big);
-    f = fmaf(1.f - low, z >= 0.f ? big : small, low);
+    // the smaller of f and 1 - f comes from the small sigmoid and the other by subtraction where needed: gates that
+    // are nearly open keep their distance from 1 to full precision over long products
+    if (z >= 0.f) {
+      k = (1.f - low) * small;
+      f = 1.f - k;
+    } else {
+      k = (1.f - low) * big;
+      f = fmaf(1.f - low, small, low);
+    }
   } else {
     k = silu_fast(u1);
     f = decay;

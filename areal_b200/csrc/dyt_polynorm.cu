@@ -31,35 +31,47 @@ __global__ void residual_dyt_kernel(const D* __restrict__ delta, long long ld_de
       float4 h = ld4(rp);
       h.x = fmaf(s.x, d.x, h.x); h.y = fmaf(s.y, d.y, h.y); h.z = fmaf(s.z, d.z, h.z); h.w = fmaf(s.w, d.w, h.w);
       st4(rp, h);
-      st4(y + r * W + c, make_float4(fmaf(tanhf(al * h.x), ww.x, bb.x), fmaf(tanhf(al * h.y), ww.y, bb.y),
-                                     fmaf(tanhf(al * h.z), ww.z, bb.z), fmaf(tanhf(al * h.w), ww.w, bb.w)));
+      st4(y + r * W + c, make_float4(fmaf(tanh_as(al * h.x, y), ww.x, bb.x), fmaf(tanh_as(al * h.y, y), ww.y, bb.y),
+                                     fmaf(tanh_as(al * h.z, y), ww.z, bb.z), fmaf(tanh_as(al * h.w, y), ww.w, bb.w)));
     } else {
       const float h = fmaf(ld1(scale + c), ld1(delta + r * ld_delta + c), *rp);
       *rp = h;
-      st1(y + r * W + c, fmaf(tanhf(al * h), ld1(w + c), ld1(b + c)));
+      st1(y + r * W + c, fmaf(tanh_as(al * h, y), ld1(w + c), ld1(b + c)));
     }
   }
 }
 
 // ids outside [0, vocab) give a zero row (as the plain embedding kernel does)
-template <class T>
+template <class T, int V>
 __global__ void embed_dyt_kernel(const int* __restrict__ ids, const T* __restrict__ table, long long vocab,
                                  float* __restrict__ res, const T* __restrict__ alpha, const T* __restrict__ w,
                                  const T* __restrict__ b, T* __restrict__ y, long long rows, int W) {
   const float al = ld1(alpha);
-  const long long total = rows * W;
+  const int nv = W / V;
+  const long long total = rows * nv;
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const long long r = i / W;
-    const int c = static_cast<int>(i % W);
+    const long long r = i / nv;
+    const int c = static_cast<int>(i % nv) * V;
     const long long id = ids[r];
-    const float h = (id >= 0 && id < vocab) ? ld1(table + id * W + c) : 0.f;
-    res[i] = h;
-    st1(y + i, fmaf(tanhf(al * h), ld1(w + c), ld1(b + c)));
+    const bool in = id >= 0 && id < vocab;
+    if (V == 4) {
+      const float4 h = in ? ld4(table + id * W + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 ww = ld4(w + c), bb = ld4(b + c);
+      st4(res + r * W + c, h);
+      st4(y + r * W + c, make_float4(fmaf(tanh_as(al * h.x, y), ww.x, bb.x), fmaf(tanh_as(al * h.y, y), ww.y, bb.y),
+                                     fmaf(tanh_as(al * h.z, y), ww.z, bb.z), fmaf(tanh_as(al * h.w, y), ww.w, bb.w)));
+    } else {
+      const float h = in ? ld1(table + id * W + c) : 0.f;
+      res[r * W + c] = h;
+      st1(y + r * W + c, fmaf(tanh_as(al * h, y), ld1(w + c), ld1(b + c)));
+    }
   }
 }
 
-// One block per row; the row is read twice, the second time from L1 / L2.
+// One block per row. Up to kPnKeep vectors per thread stay in registers between the two passes; what does not fit is read
+// again (from L1 / L2).
+constexpr int kPnKeep = 4;
 template <class T, int V>
 __global__ void polynorm_kernel(const T* __restrict__ z, long long ldz, const T* __restrict__ coef, T* __restrict__ y,
                                 int F, float eps) {
@@ -74,13 +86,18 @@ __global__ void polynorm_kernel(const T* __restrict__ z, long long ldz, const T*
     s2 = fmaf(u2, u2, s2);
     s3 = fmaf(u3, u3, s3);
   };
-  for (int c = threadIdx.x * V; c < F; c += blockDim.x * V) {
-    if (V == 4) {
-      const float4 v = ld4(zr + c);
-      acc(v.x); acc(v.y); acc(v.z); acc(v.w);
-    } else {
-      acc(ld1(zr + c));
-    }
+  auto load = [&](int c) { return V == 4 ? ld4(zr + c) : make_float4(ld1(zr + c), 0.f, 0.f, 0.f); };
+  const int step = blockDim.x * V;
+  float4 keep[kPnKeep];
+#pragma unroll
+  for (int i = 0; i < kPnKeep; ++i) {
+    const int c = threadIdx.x * V + i * step;
+    keep[i] = c < F ? load(c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    acc(keep[i].x); acc(keep[i].y); acc(keep[i].z); acc(keep[i].w);
+  }
+  for (int c = threadIdx.x * V + kPnKeep * step; c < F; c += step) {
+    const float4 v = load(c);
+    acc(v.x); acc(v.y); acc(v.z); acc(v.w);
   }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   s1 = warp_sum(s1); s2 = warp_sum(s2); s3 = warp_sum(s3);
@@ -91,19 +108,21 @@ __global__ void polynorm_kernel(const T* __restrict__ z, long long ldz, const T*
   const float k1 = ld1(coef) / sqrtf(s1 / F + eps), k2 = ld1(coef + 1) / sqrtf(s2 / F + eps),
               k3 = ld1(coef + 2) / sqrtf(s3 / F + eps), e = ld1(coef + 3);
   auto out = [&](float u) { return fmaf(fmaf(fmaf(k3, u, k2), u, k1), u, e); };
-  for (int c = threadIdx.x * V; c < F; c += blockDim.x * V) {
-    if (V == 4) {
-      const float4 v = ld4(zr + c);
-      st4(yr + c, make_float4(out(v.x), out(v.y), out(v.z), out(v.w)));
-    } else {
-      st1(yr + c, out(ld1(zr + c)));
-    }
+  auto store = [&](int c, float4 v) {
+    if (V == 4) st4(yr + c, make_float4(out(v.x), out(v.y), out(v.z), out(v.w)));
+    else st1(yr + c, out(v.x));
+  };
+#pragma unroll
+  for (int i = 0; i < kPnKeep; ++i) {
+    const int c = threadIdx.x * V + i * step;
+    if (c < F) store(c, keep[i]);
   }
+  for (int c = threadIdx.x * V + kPnKeep * step; c < F; c += step) store(c, load(c));
 }
 
 // o [rows, groups * n] fp32. One warp per (row, group) when a group is narrow, one block per (row, group) else.
 // w: [n] shared by the groups (w_per_group 0) or [groups * n]. gate: null or [rows, groups * n] with pitch ld_gate.
-template <class T, bool WARP>
+template <class T, bool WARP, int V>
 __global__ void group_rms_kernel(const float* __restrict__ o, const T* __restrict__ w, int w_per_group,
                                  const T* __restrict__ gate, long long ld_gate, T* __restrict__ y, long long rows,
                                  int groups, int n, float eps) {
@@ -114,15 +133,36 @@ __global__ void group_rms_kernel(const float* __restrict__ o, const T* __restric
   if (unit >= rows * groups) return;  // whole warps (or no thread) leave
   const long long r = unit / groups;
   const int g = static_cast<int>(unit % groups);
-  const long long base = r * groups * n + static_cast<long long>(g) * n;
+  const float* ob = o + r * groups * n + static_cast<long long>(g) * n;
+  T* yb = y + r * groups * n + static_cast<long long>(g) * n;
+  const T* wb = w + (w_per_group ? g * n : 0);
+  const T* gb = gate ? gate + r * ld_gate + static_cast<long long>(g) * n : nullptr;
   float s = 0.f;
-  for (int c = tid; c < n; c += nthr) s = fmaf(o[base + c], o[base + c], s);
+  for (int c = tid * V; c < n; c += nthr * V) {
+    if (V == 4) {
+      const float4 v = ld4(ob + c);
+      s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+    } else {
+      s = fmaf(ob[c], ob[c], s);
+    }
+  }
   s = WARP ? warp_sum(s) : block_sum(s, red);
   const float k = 1.f / sqrtf(s / n + eps);
-  for (int c = tid; c < n; c += nthr) {
-    float v = o[base + c] * k * ld1(w + (w_per_group ? g * n + c : c));
-    if (gate) v *= sigmoid_f(ld1(gate + r * ld_gate + static_cast<long long>(g) * n + c));
-    st1(y + base + c, v);
+  for (int c = tid * V; c < n; c += nthr * V) {
+    if (V == 4) {
+      float4 v = ld4(ob + c);
+      const float4 ww = ld4(wb + c);
+      v.x *= k * ww.x; v.y *= k * ww.y; v.z *= k * ww.z; v.w *= k * ww.w;
+      if (gb) {
+        const float4 u = ld4(gb + c);
+        v.x *= sigmoid_as(u.x, y); v.y *= sigmoid_as(u.y, y); v.z *= sigmoid_as(u.z, y); v.w *= sigmoid_as(u.w, y);
+      }
+      st4(yb + c, v);
+    } else {
+      float v = ob[c] * k * ld1(wb + c);
+      if (gb) v *= sigmoid_as(ld1(gb + c), y);
+      st1(yb + c, v);
+    }
   }
 }
 
@@ -168,14 +208,14 @@ int b200_embed_dyt(const int* ids, const void* table, long long vocab, float* re
                    const void* b, void* y, long long rows, int W, int fp32, cudaStream_t stream) {
   using namespace b200;
   if (rows <= 0 || W <= 0) return 0;
-  const unsigned grid = grid_for(rows * W, 256, 16);
-  if (fp32)
-    embed_dyt_kernel<float><<<grid, 256, 0, stream>>>(ids, (const float*)table, vocab, res, (const float*)alpha,
-                                                      (const float*)w, (const float*)b, (float*)y, rows, W);
-  else
-    embed_dyt_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(
-        ids, (const __nv_bfloat16*)table, vocab, res, (const __nv_bfloat16*)alpha, (const __nv_bfloat16*)w,
-        (const __nv_bfloat16*)b, (__nv_bfloat16*)y, rows, W);
+  const bool v4 = W % 4 == 0;
+  const unsigned grid = grid_for(rows * (v4 ? W / 4 : W), 256, 16);
+#define B200_ED(T_, V_)                                                                                             \
+  embed_dyt_kernel<T_, V_><<<grid, 256, 0, stream>>>(ids, (const T_*)table, vocab, res, (const T_*)alpha,           \
+                                                     (const T_*)w, (const T_*)b, (T_*)y, rows, W)
+  if (fp32) { if (v4) B200_ED(float, 4); else B200_ED(float, 1); }
+  else { if (v4) B200_ED(__nv_bfloat16, 4); else B200_ED(__nv_bfloat16, 1); }
+#undef B200_ED
   B200_CHECK(cudaGetLastError());
   return 0;
 }
@@ -185,9 +225,10 @@ int b200_polynorm(const void* z, long long ldz, const void* coef, void* y, long 
   using namespace b200;
   if (rows <= 0 || F <= 0) return 0;
   const bool v4 = (F % 4 == 0) && (ldz % 4 == 0);
-  int block = 1024;
-  while (block > 32 && block / 2 * (v4 ? 4 : 1) >= F) block >>= 1;
-  if (block > 512 && rows >= 4LL * sm_count()) block = 512;
+  // three or four vectors per thread when there are rows enough to fill the GPU, one otherwise
+  const int vecs = v4 ? F / 4 : F, per = rows >= 4LL * sm_count() ? 3 : 1;
+  int block = ((vecs + per - 1) / per + 31) / 32 * 32;
+  if (block > 1024) block = 1024;
   using bf = __nv_bfloat16;
   const unsigned grid = static_cast<unsigned>(rows);
   if (fp32) {
@@ -207,15 +248,19 @@ int b200_group_rms(const float* o, const void* w, int w_per_group, const void* g
   if (rows <= 0 || groups <= 0 || n <= 0) return 0;
   using bf = __nv_bfloat16;
   const bool warp = n <= 512;
+  const bool v4 = n % 4 == 0 && (!gate || (ld_gate % 4 == 0 && reinterpret_cast<uintptr_t>(gate) % (fp32 ? 16 : 8) == 0));
   int block = 256;
-  if (!warp) while (block < 1024 && block * 4 < n) block <<= 1;
+  if (!warp) while (block < 1024 && block * 8 < n) block <<= 1;
   const long long units = rows * groups;
   const unsigned grid = static_cast<unsigned>(warp ? (units + 7) / 8 : units);
-#define B200_GR(T_, W_)                                                                                             \
-  group_rms_kernel<T_, W_><<<grid, block, 0, stream>>>(o, (const T_*)w, w_per_group, (const T_*)gate, ld_gate,      \
-                                                       (T_*)y, rows, groups, n, eps)
-  if (fp32) { if (warp) B200_GR(float, true); else B200_GR(float, false); }
-  else { if (warp) B200_GR(bf, true); else B200_GR(bf, false); }
+#define B200_GR(T_, W_, V_)                                                                                         \
+  group_rms_kernel<T_, W_, V_><<<grid, block, 0, stream>>>(o, (const T_*)w, w_per_group, (const T_*)gate, ld_gate,  \
+                                                           (T_*)y, rows, groups, n, eps)
+#define B200_GRV(T_)                                                                                                \
+  if (warp) { if (v4) B200_GR(T_, true, 4); else B200_GR(T_, true, 1); }                                            \
+  else { if (v4) B200_GR(T_, false, 4); else B200_GR(T_, false, 1); }
+  if (fp32) { B200_GRV(float) } else { B200_GRV(bf) }
+#undef B200_GRV
 #undef B200_GR
   B200_CHECK(cudaGetLastError());
   return 0;

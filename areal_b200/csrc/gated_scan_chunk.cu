@@ -10,7 +10,8 @@
 //
 // Products of gates only ever run forward (no quotients, no logarithms), so nothing overflows or loses precision when
 // gates close. fp32 operands enter the bf16 products as two terms (hi + lo, three products where both sides have two);
-// values are bf16 numbers and enter exactly. A is computed in fp32 on the CUDA cores with running products.
+// values are bf16 numbers and enter exactly. A is computed in fp32 on the CUDA
+// cores: inside a half block with running products held in registers, between the halves as plain products.
 //
 // Few long sequences would leave most SMs idle: they are cut into segments. A first pass computes every segment's state
 // from zero and its gate product, a scan over a sequence's segments turns them into the states the segments start
@@ -40,11 +41,44 @@ struct ScanSmem {
   static constexpr int DP = ND * 16, PB = (DP + 8) * 2;  // padded channels, bytes of a bf16 row
   __nv_bfloat16 q[2][16 * (DP + 8)], k[2][16 * (DP + 8)];  // hi, lo
   __nv_bfloat16 v[16 * 136];
-  __nv_bfloat16 A[2][16 * 24];
-  float fq[16 * DP], fk[16 * DP], ff[16 * DP];
+  float A[4][16 * 16];        // partial sums over 32 channels each; the part above the diagonal stays zero
+  float qx[8 * 128], kx[8 * 128];  // second half's q and first half's k with the gates of their own half
   float tot[2][DP], F[DP];
   float o[16 * 132];
 };
+
+// Sums 16 per-lane values over the warp: every lane ends with the total of value (lane >> 1). Halves the values while
+// doubling the lanes that share one.
+__device__ __forceinline__ float warp_sum16(float (&v)[16], int lane) {
+#pragma unroll
+  for (int s = 8; s >= 1; s >>= 1) {
+    const bool up = lane & (2 * s);
+#pragma unroll
+    for (int r = 0; r < s; ++r) {
+      const float give = up ? v[r] : v[r + s];
+      const float keep = up ? v[r + s] : v[r];
+      v[r] = keep + __shfl_xor_sync(0xffffffffu, give, 2 * s);
+    }
+  }
+  return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
+}
+// The 36 entries (i, j), j <= i < 8, of a half block's triangle in three batches of whole columns: columns 0, 1, 7; then
+// 2, 3, 5, 6; then 4. Entry e of a batch as i * 16 + j.
+__device__ __forceinline__ int tri_entry(int batch, int e) {
+  if (batch == 0) return e < 8 ? e * 16 : e < 15 ? (e - 7) * 16 + 1 : 7 * 16 + 7;
+  if (batch == 1) return e < 6 ? (e + 2) * 16 + 2 : e < 11 ? (e - 3) * 16 + 3 : e < 14 ? (e - 6) * 16 + 5 : (e - 8) * 16 + 6;
+  return (e + 4) * 16 + 4;
+}
+// One column j of the triangle: q_i k_j prod_{j < t <= i} f_t for i = j..7 into v[at..]
+template <int J>
+__device__ __forceinline__ void tri_column(const float (&q)[8], const float (&f)[8], const float (&k)[8], float (&v)[16], int at) {
+  float w = k[J];
+#pragma unroll
+  for (int i = J; i < 8; ++i) {
+    if (i > J) w *= f[i];
+    v[at + i - J] = q[i] * w;
+  }
+}
 
 // STATE_ONLY: pass 1 (no outputs; starts from zero; writes seg_state and seg_decay)
 template <int ND, bool STATE_ONLY>
@@ -92,6 +126,10 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
         if (p.x < D && p.y < Dv) S[i][c] = a.seg_state[seg_base + static_cast<long long>(p.x) * Dv + p.y];
       }
   }
+  const bool warp_live = (warp & 3) * 32 < DP;  // this warp has channels
+  if (!STATE_ONLY)
+    for (int i = tid; i < 4 * 256; i += kScThreads) (&sm.A[0][0])[i] = 0.f;
+  __syncthreads();
   float seg_f = 1.f;  // product of all gates of the segment (threads of half 0)
 
   __nv_bfloat16 rq[8], rf[8], rv[8];
@@ -109,7 +147,7 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
   };
   load(0);
   for (int t0 = 0; t0 < seg.y; t0 += 16) {
-    // ---- activations, running products of the gates inside this half block
+    // ---- activations; the triangle of A inside this half; running products of the gates inside the half
     float q[8], f[8], k[8];
     float run = 1.f;
 #pragma unroll
@@ -118,11 +156,33 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
       q[i] = 0.f; k[i] = 0.f; f[i] = 1.f;
       if (dch && t0 + tok < seg.y)
         scan_activate(mode, __bfloat162float(rq[i]), __bfloat162float(rf[i]), bias, low, decay, q[i], f[i], k[i]);
-      if (!STATE_ONLY && d < DP) {
-        sm.fq[tok * DP + d] = q[i];
-        sm.fk[tok * DP + d] = k[i];
-        sm.ff[tok * DP + d] = f[i];
+    }
+    if (!STATE_ONLY && warp_live) {
+      float* A = sm.A[warp & 3] + half * (8 * 16 + 8);
+#pragma unroll
+      for (int batch = 0; batch < 3; ++batch) {
+        float v[16];
+#pragma unroll
+        for (int e = 0; e < 16; ++e) v[e] = 0.f;
+        if (batch == 0) {
+          tri_column<0>(q, f, k, v, 0);
+          tri_column<1>(q, f, k, v, 8);
+          tri_column<7>(q, f, k, v, 15);
+        } else if (batch == 1) {
+          tri_column<2>(q, f, k, v, 0);
+          tri_column<3>(q, f, k, v, 6);
+          tri_column<5>(q, f, k, v, 11);
+          tri_column<6>(q, f, k, v, 14);
+        } else {
+          tri_column<4>(q, f, k, v, 0);
+        }
+        const float sum = warp_sum16(v, lane);
+        const int e = lane >> 1;
+        if (!(lane & 1) && (batch < 2 || e < 4)) A[tri_entry(batch, e)] = sum;
       }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
       run *= f[i];
       if (!STATE_ONLY) q[i] *= run;  // q_i P_i, still without the gates of the first half
     }
@@ -139,6 +199,13 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
       sm.v[(half * 8 + i) * 136 + d] = d < nv ? __float2bfloat16(v) : zero;
     }
     if (d < DP) sm.tot[half][d] = run;
+    if (!STATE_ONLY) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        if (half) sm.qx[i * 128 + d] = q[i];
+        else sm.kx[i * 128 + d] = k[i];
+      }
+    }
     __syncthreads();
     if (t0 + 16 < seg.y) load(t0 + 16);
     // ---- operands: the other half's gates, then two bf16 terms
@@ -163,43 +230,24 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
         seg_f *= run * other;
       }
     }
-    // ---- A: warp w takes keys w and 15 - w (17 products in all)
-    if (!STATE_ONLY) {
-#pragma unroll 1
+    // ---- A between the halves: q_i of the second against k_j of the first; half h of the threads takes i = 8 + 4h ..
+    if (!STATE_ONLY && warp_live) {
+      float kj[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) kj[j] = sm.kx[j * 128 + d];
+      float* A = sm.A[warp & 3] + (8 + half * 4) * 16;
+#pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int j = e ? 15 - warp : warp;
-        float acc[16];
+        const float q0 = sm.qx[(half * 4 + e * 2) * 128 + d], q1 = sm.qx[(half * 4 + e * 2 + 1) * 128 + d];
+        float v[16];
 #pragma unroll
-        for (int i = 0; i < 16; ++i) acc[i] = 0.f;
-#pragma unroll 1
-        for (int c = lane; c < DP; c += 32) {
-          float w = sm.fk[j * DP + c];
-#pragma unroll
-          for (int i = 0; i < 16; ++i)
-            if (i >= j) {  // the same for the whole warp
-              if (i > j) w *= sm.ff[i * DP + c];
-              acc[i] = fmaf(sm.fq[i * DP + c], w, acc[i]);
-            }
+        for (int j = 0; j < 8; ++j) {
+          v[j] = q0 * kj[j];
+          v[8 + j] = q1 * kj[j];
         }
-        // 16 sums over 32 lanes: halve the values while doubling the lanes that share one
-#pragma unroll
-        for (int s = 8; s >= 1; s >>= 1) {
-          const bool up = lane & (2 * s);
-#pragma unroll
-          for (int r = 0; r < s; ++r) {
-            const float give = up ? acc[r] : acc[r + s];
-            const float keep = up ? acc[r + s] : acc[r];
-            acc[r] = keep + __shfl_xor_sync(0xffffffffu, give, 2 * s);
-          }
-        }
-        const float v = acc[0] + __shfl_xor_sync(0xffffffffu, acc[0], 1);
-        if (!(lane & 1)) {
-          const int i = lane >> 1;
-          const float av = i >= j ? v : 0.f;
-          const __nv_bfloat16 hi = __float2bfloat16(av);
-          sm.A[0][i * 24 + j] = hi;
-          sm.A[1][i * 24 + j] = __float2bfloat16(av - __bfloat162float(hi));
-        }
+        const float sum = warp_sum16(v, lane);
+        const int x = lane >> 1;
+        if (!(lane & 1)) A[(e * 2 + (x >> 3)) * 16 + (x & 7)] = sum;
       }
     }
     __syncthreads();
@@ -215,8 +263,19 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
 #pragma unroll
           for (int c = 0; c < 4; ++c) o[n][c] = 0.f;
         uint32_t ah[4], al[4];
-        ldm_x4(s32(sm.A[0] + r8 * 24 + c8), ah);
-        ldm_x4(s32(sm.A[1] + r8 * 24 + c8), al);
+        // A as the second operand: entries (i = g + 8n, j = 2t + 8c, +1) of the channel groups' partial sums
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int at = (g + (e >> 1) * 8) * 16 + 2 * t + (e & 1) * 8;
+          float2 sum = *reinterpret_cast<const float2*>(&sm.A[0][at]);
+#pragma unroll
+          for (int c = 1; c < (ND * 16 + 31) / 32; ++c) {
+            const float2 p = *reinterpret_cast<const float2*>(&sm.A[c][at]);
+            sum.x += p.x;
+            sum.y += p.y;
+          }
+          ah[e] = split2(sum.x, sum.y, al[e]);
+        }
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
           mma_bf16(o[n], vt, ah[2 * n], ah[2 * n + 1]);

@@ -366,8 +366,8 @@ struct DytTail {
     h.x = fmaf(s.x, acc.x, h.x); h.y = fmaf(s.y, acc.y, h.y);
     h.z = fmaf(s.z, acc.z, h.z); h.w = fmaf(s.w, acc.w, h.w);
     st4(res + row * N + c, h);
-    st4(y + row * N + c, make_float4(fmaf(tanhf(al * h.x), ww.x, bb.x), fmaf(tanhf(al * h.y), ww.y, bb.y),
-                                     fmaf(tanhf(al * h.z), ww.z, bb.z), fmaf(tanhf(al * h.w), ww.w, bb.w)));
+    st4(y + row * N + c, make_float4(fmaf(tanh_as(al * h.x, y), ww.x, bb.x), fmaf(tanh_as(al * h.y, y), ww.y, bb.y),
+                                     fmaf(tanh_as(al * h.z, y), ww.z, bb.z), fmaf(tanh_as(al * h.w, y), ww.w, bb.w)));
   }
 };
 

@@ -15,37 +15,56 @@
 
 namespace b200 {
 
-template <class T>
+// One warp per token; V: elements per load (4 when every part's width and the pitch allow it).
+template <class T, int V>
 __global__ void latent_prep_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ wq,
                                    const T* __restrict__ wc, const float* __restrict__ cosT,
                                    const float* __restrict__ sinT, const int* __restrict__ pos, int max_pos,
                                    const long long* __restrict__ slot_mapping, T* __restrict__ cq, T* __restrict__ c,
-                                   T* __restrict__ kr, T* __restrict__ cache, long long cache_rows, int q_rank,
+                                   T* __restrict__ kr, T* __restrict__ cache, long long cache_rows, int T_, int q_rank,
                                    int rank, int rot, float eps) {
-  __shared__ float red[33];
-  const long long t = blockIdx.x;
+  const int lane = threadIdx.x & 31;
+  const long long t = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (t >= T_) return;
   const T* row = x + t * ldx;
-  float s = 0.f;
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = ld1(row + i); s = fmaf(v, v, s); }
-  s = block_sum(s, red);
-  const float kq = 1.f / sqrtf(s / q_rank + eps);
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) st1(cq + t * q_rank + i, ld1(row + i) * kq * ld1(wq + i));
-  row += q_rank;
-  s = 0.f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = ld1(row + i); s = fmaf(v, v, s); }
-  s = block_sum(s, red);
-  const float kc = 1.f / sqrtf(s / rank + eps);
   long long slot = slot_mapping ? slot_mapping[t] : -1;
   if (slot >= cache_rows) slot = -1;
   T* dst = slot >= 0 ? cache + slot * (rank + rot) : nullptr;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-    const float v = ld1(row + i) * kc * ld1(wc + i);
-    if (c) st1(c + t * rank + i, v);
-    if (dst) st1(dst + i, v);
+  auto sumsq = [&](const T* p, int n) {
+    float s = 0.f;
+    for (int i = lane * V; i < n; i += 32 * V) {
+      if (V == 4) {
+        const float4 v = ld4(p + i);
+        s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+      } else {
+        s = fmaf(ld1(p + i), ld1(p + i), s);
+      }
+    }
+    return warp_sum(s);
+  };
+  auto scaled = [&](const T* p, const T* w, float k, int i) {
+    if (V == 4) {
+      const float4 v = ld4(p + i), ww = ld4(w + i);
+      return make_float4(v.x * k * ww.x, v.y * k * ww.y, v.z * k * ww.z, v.w * k * ww.w);
+    }
+    return make_float4(ld1(p + i) * k * ld1(w + i), 0.f, 0.f, 0.f);
+  };
+  auto put = [&](T* p, float4 v) {
+    if (V == 4) st4(p, v);
+    else st1(p, v.x);
+  };
+  const float sq = sumsq(row, q_rank), sc = sumsq(row + q_rank, rank);
+  const float kq = 1.f / sqrtf(sq / q_rank + eps), kc = 1.f / sqrtf(sc / rank + eps);
+  for (int i = lane * V; i < q_rank; i += 32 * V) put(cq + t * q_rank + i, scaled(row, wq, kq, i));
+  row += q_rank;
+  for (int i = lane * V; i < rank; i += 32 * V) {
+    const float4 v = scaled(row, wc, kc, i);
+    if (c) put(c + t * rank + i, v);
+    if (dst) put(dst + i, v);
   }
   row += rank;
   const int p = min(max(pos[t], 0), max_pos - 1);
-  for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
+  for (int i = lane; i < rot / 2; i += 32) {
     const float cs = cosT[static_cast<long long>(p) * (rot / 2) + i], sn = sinT[static_cast<long long>(p) * (rot / 2) + i];
     const float u = ld1(row + 2 * i), v = ld1(row + 2 * i + 1);
     const float a = u * cs - v * sn, b = v * cs + u * sn;
@@ -54,22 +73,36 @@ __global__ void latent_prep_kernel(const T* __restrict__ x, long long ldx, const
   }
 }
 
-template <class T>
+__device__ __forceinline__ float2 ld_pair(const float* p) { return make_float2(p[0], p[1]); }
+__device__ __forceinline__ float2 ld_pair(const __nv_bfloat16* p) {  // 4-byte aligned
+  return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+}
+__device__ __forceinline__ void st_pair(float* p, float a, float b) { p[0] = a; p[1] = b; }
+__device__ __forceinline__ void st_pair(__nv_bfloat16* p, float a, float b) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+}
+
+// One block per token; PAIR: pairs are aligned to their size (even pitch, head stride and offset).
+template <class T, bool PAIR>
 __global__ void rope_pairs_kernel(T* __restrict__ x, long long ldx, int H, int head_stride, int offset, int half,
                                   const float* __restrict__ cosT, const float* __restrict__ sinT,
-                                  const int* __restrict__ pos, int max_pos, long long rows) {
-  const long long total = rows * H * half;
-  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
-       i += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const int e = static_cast<int>(i % half);
-    const int h = static_cast<int>((i / half) % H);
-    const long long t = i / (static_cast<long long>(half) * H);
-    const int p = min(max(pos[t], 0), max_pos - 1);
-    const float cs = cosT[static_cast<long long>(p) * half + e], sn = sinT[static_cast<long long>(p) * half + e];
-    T* q = x + t * ldx + static_cast<long long>(h) * head_stride + offset + 2 * e;
-    const float u = ld1(q), v = ld1(q + 1);
-    st1(q, u * cs - v * sn);
-    st1(q + 1, v * cs + u * sn);
+                                  const int* __restrict__ pos, int max_pos) {
+  const long long t = blockIdx.x;
+  const int p = min(max(pos[t], 0), max_pos - 1);
+  const float* cr = cosT + static_cast<long long>(p) * half;
+  const float* sr = sinT + static_cast<long long>(p) * half;
+  T* row = x + t * ldx + offset;
+  for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
+    const int h = i / half, e = i - h * half;
+    T* q = row + static_cast<long long>(h) * head_stride + 2 * e;
+    const float2 uv = PAIR ? ld_pair(q) : make_float2(ld1(q), ld1(q + 1));
+    const float a = uv.x * cr[e] - uv.y * sr[e], b = uv.y * cr[e] + uv.x * sr[e];
+    if (PAIR) {
+      st_pair(q, a, b);
+    } else {
+      st1(q, a);
+      st1(q + 1, b);
+    }
   }
 }
 
@@ -195,15 +228,14 @@ int b200_latent_prep(const void* x, long long ldx, const void* wq, const void* w
   using namespace b200;
   if (T <= 0) return 0;
   if (rot & 1) return -100;
-  const int widest = q_rank > rank ? q_rank : rank;
-  int block = 64;
-  while (block < 512 && block * 2 < widest) block <<= 1;
-#define B200_LP(T_)                                                                                                 \
-  latent_prep_kernel<T_><<<T, block, 0, stream>>>((const T_*)x, ldx, (const T_*)wq, (const T_*)wc, cosT, sinT, pos, \
-                                                  max_pos, slot_mapping, (T_*)cq, (T_*)c, (T_*)kr, (T_*)cache,      \
-                                                  cache_rows, q_rank, rank, rot, eps)
-  if (fp32) B200_LP(float);
-  else B200_LP(__nv_bfloat16);
+  const bool v4 = q_rank % 4 == 0 && rank % 4 == 0 && rot % 4 == 0 && ldx % 4 == 0;
+  const unsigned grid = (T + 7) / 8;
+#define B200_LP(T_, V_)                                                                                             \
+  latent_prep_kernel<T_, V_><<<grid, 256, 0, stream>>>((const T_*)x, ldx, (const T_*)wq, (const T_*)wc, cosT, sinT, \
+                                                       pos, max_pos, slot_mapping, (T_*)cq, (T_*)c, (T_*)kr,        \
+                                                       (T_*)cache, cache_rows, T, q_rank, rank, rot, eps)
+  if (fp32) { if (v4) B200_LP(float, 4); else B200_LP(float, 1); }
+  else { if (v4) B200_LP(__nv_bfloat16, 4); else B200_LP(__nv_bfloat16, 1); }
 #undef B200_LP
   B200_CHECK(cudaGetLastError());
   return 0;
@@ -215,16 +247,15 @@ int b200_rope_pairs(void* x, long long ldx, int H, int head_stride, int offset, 
   using namespace b200;
   if (rows <= 0 || dims <= 0) return 0;
   if (dims & 1) return -100;
-  const long long total = rows * H * (dims / 2);
-  long long grid = (total + 255) / 256;
-  const long long cap = static_cast<long long>(sm_count()) * 16;
-  if (grid > cap) grid = cap;
-  if (fp32)
-    rope_pairs_kernel<float><<<(unsigned)grid, 256, 0, stream>>>((float*)x, ldx, H, head_stride, offset, dims / 2, cosT,
-                                                                 sinT, pos, max_pos, rows);
-  else
-    rope_pairs_kernel<__nv_bfloat16><<<(unsigned)grid, 256, 0, stream>>>((__nv_bfloat16*)x, ldx, H, head_stride, offset,
-                                                                         dims / 2, cosT, sinT, pos, max_pos, rows);
+  const bool pair = !((ldx | head_stride | offset) & 1);
+  int block = 64;
+  while (block < 256 && block < H * (dims / 2)) block <<= 1;
+#define B200_RP(T_, P_)                                                                                             \
+  rope_pairs_kernel<T_, P_><<<(unsigned)rows, block, 0, stream>>>((T_*)x, ldx, H, head_stride, offset, dims / 2,    \
+                                                                  cosT, sinT, pos, max_pos)
+  if (fp32) { if (pair) B200_RP(float, true); else B200_RP(float, false); }
+  else { if (pair) B200_RP(__nv_bfloat16, true); else B200_RP(__nv_bfloat16, false); }
+#undef B200_RP
   B200_CHECK(cudaGetLastError());
   return 0;
 }

@@ -113,9 +113,13 @@ def segment_length(lens: list[int], units: int, slots: int = 296) -> int:
     work spread evenly over ``slots`` CTAs (two per SM). A cut costs a second, cheaper pass over the inputs."""
     even = sum(lens) * units / slots
     longest = max(lens, default=0)
-    if longest <= 2 * even + 256:
+    if longest <= 3 * even + 256:
         return 0
-    return max(128, -(-int(even) // 16) * 16)
+    L = max(128, -(-int(even) // 16) * 16)
+    if len(lens) * units <= slots // 2:  # few sequences: all segments fit at once
+        while L < longest and sum(-(-n // L) for n in lens) * units > slots:
+            L += 16
+    return L
 
 
 def _segments(meta, units: int):

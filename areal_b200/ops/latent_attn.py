@@ -193,8 +193,8 @@ def latent_decode_ref(qa, q, cache, block_table, seq_lens, H, D, rot, rank, scal
 def _latent_decode_mma(qa, q, cache, block_table, seq_lens, H, D, rot, rank, scale, max_seq_len):
     B = q.shape[0]
     ctas = B * -(-H // 16)
-    # two CTAs per SM and a few waves of them; a split keeps at least 128 tokens
-    nsplit = max(1, min(64, 1184 // ctas, max_seq_len // 128))
+    # one wave of two CTAs per SM; a split keeps at least 128 tokens
+    nsplit = max(1, min(64, 296 // ctas, max_seq_len // 128))
     c, ll = ctypes.c_int, ctypes.c_longlong
     out = torch.empty((B, H * rank), dtype=q.dtype, device=q.device)
     o_part = ml = None
