@@ -8,10 +8,10 @@
 //   O^T = S^T (q_i P_i)^T + V^T A^T,   A_ij = sum_d q_id k_jd prod_{j < t <= i} f_td  (j <= i)
 //   S^T <- S^T diag(F) + V^T (k_j R_j)
 //
-// Products of gates only ever run forward (no quotients, no logarithms), so nothing overflows or loses precision when
-// gates close. fp32 operands enter the bf16 products as two terms (hi + lo, three products where both sides have two);
-// values are bf16 numbers and enter exactly. A is computed in fp32 on the CUDA
-// cores: inside a half block with running products held in registers, between the halves as plain products.
+// fp32 operands enter the bf16 products as two terms (hi + lo, three products where both sides have two); values are bf16
+// numbers and enter exactly. A is a product of (q_i P_i / F) with (k_j R_j): every term has the size of the true weight,
+// only the factors need range, so this holds as long as F stays inside the exponent range. A block in which some channel
+// forgets more than that (F < 2^-90) takes a slow path that multiplies the gates up pair by pair, in fp32.
 //
 // Few long sequences would leave most SMs idle: they are cut into segments. A first pass computes every segment's state
 // from zero and its gate product, a scan over a sequence's segments turns them into the states the segments start
@@ -39,45 +39,21 @@ __device__ __forceinline__ uint32_t s32(const void* p) { return static_cast<uint
 template <int ND>
 struct ScanSmem {
   static constexpr int DP = ND * 16, PB = (DP + 8) * 2;  // padded channels, bytes of a bf16 row
-  __nv_bfloat16 q[2][16 * (DP + 8)], k[2][16 * (DP + 8)];  // hi, lo
+  __nv_bfloat16 raw[2][3][16 * 128];                     // double-buffered projections: q, f / k, v
+  __nv_bfloat16 q[2][16 * (DP + 8)], k[2][16 * (DP + 8)], s[2][16 * (DP + 8)];  // hi, lo of q P, k R, q P / F
   __nv_bfloat16 v[16 * 136];
-  float A[4][16 * 16];        // partial sums over 32 channels each; the part above the diagonal stays zero
-  float qx[8 * 128], kx[8 * 128];  // second half's q and first half's k with the gates of their own half
+  float A[4][16 * 16];  // partial sums over channels
   float tot[2][DP], F[DP];
   float o[16 * 132];
 };
 
-// Sums 16 per-lane values over the warp: every lane ends with the total of value (lane >> 1). Halves the values while
-// doubling the lanes that share one.
-__device__ __forceinline__ float warp_sum16(float (&v)[16], int lane) {
-#pragma unroll
-  for (int s = 8; s >= 1; s >>= 1) {
-    const bool up = lane & (2 * s);
-#pragma unroll
-    for (int r = 0; r < s; ++r) {
-      const float give = up ? v[r] : v[r + s];
-      const float keep = up ? v[r + s] : v[r];
-      v[r] = keep + __shfl_xor_sync(0xffffffffu, give, 2 * s);
-    }
-  }
-  return v[0] + __shfl_xor_sync(0xffffffffu, v[0], 1);
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, int bytes) {  // bytes < 16: the rest is zero
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(s32(dst)), "l"(src), "r"(bytes) : "memory");
 }
-// The 36 entries (i, j), j <= i < 8, of a half block's triangle in three batches of whole columns: columns 0, 1, 7; then
-// 2, 3, 5, 6; then 4. Entry e of a batch as i * 16 + j.
-__device__ __forceinline__ int tri_entry(int batch, int e) {
-  if (batch == 0) return e < 8 ? e * 16 : e < 15 ? (e - 7) * 16 + 1 : 7 * 16 + 7;
-  if (batch == 1) return e < 6 ? (e + 2) * 16 + 2 : e < 11 ? (e - 3) * 16 + 3 : e < 14 ? (e - 6) * 16 + 5 : (e - 8) * 16 + 6;
-  return (e + 4) * 16 + 4;
-}
-// One column j of the triangle: q_i k_j prod_{j < t <= i} f_t for i = j..7 into v[at..]
-template <int J>
-__device__ __forceinline__ void tri_column(const float (&q)[8], const float (&f)[8], const float (&k)[8], float (&v)[16], int at) {
-  float w = k[J];
-#pragma unroll
-  for (int i = J; i < 8; ++i) {
-    if (i > J) w *= f[i];
-    v[at + i - J] = q[i] * w;
-  }
+__device__ __forceinline__ void put_split(__nv_bfloat16* hi, __nv_bfloat16* lo, int at, float v) {
+  const __nv_bfloat16 h = __float2bfloat16(v);
+  hi[at] = h;
+  lo[at] = __float2bfloat16(v - __bfloat162float(h));
 }
 
 // STATE_ONLY: pass 1 (no outputs; starts from zero; writes seg_state and seg_decay)
@@ -100,12 +76,13 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
   const int d = tid & 127, half = tid >> 7;
   const bool dch = d < D;
   float bias = 0.f, low = 0.f, decay = 0.f;
+  const float decay_h = mode == 0 ? 0.f : a.s.decay[h];
   if (dch) {
     if (mode == 0) {
       bias = ld1(static_cast<const __nv_bfloat16*>(a.s.bias) + h * D + d);
       low = ld1(static_cast<const __nv_bfloat16*>(a.s.lower) + h * D + d);
     } else {
-      decay = a.s.decay[h];
+      decay = decay_h;
     }
   }
   float S[2 * ND][4];
@@ -126,65 +103,52 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
         if (p.x < D && p.y < Dv) S[i][c] = a.seg_state[seg_base + static_cast<long long>(p.x) * Dv + p.y];
       }
   }
-  const bool warp_live = (warp & 3) * 32 < DP;  // this warp has channels
-  if (!STATE_ONLY)
-    for (int i = tid; i < 4 * 256; i += kScThreads) (&sm.A[0][0])[i] = 0.f;
-  __syncthreads();
   float seg_f = 1.f;  // product of all gates of the segment (threads of half 0)
-
-  __nv_bfloat16 rq[8], rf[8], rv[8];
-  const __nv_bfloat16 zero = __float2bfloat16(0.f);
-  auto load = [&](int t0) {  // raw projections of the block that starts at token t0 of the segment
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int tok = t0 + half * 8 + i;
-      const __nv_bfloat16* row = x + (static_cast<long long>(seg.x) + tok) * a.s.ldx + h * D + d;
-      const bool in = tok < seg.y;
-      rq[i] = in && dch ? row[0] : zero;
-      rf[i] = in && dch ? row[H * D] : zero;
-      rv[i] = in && d < nv ? x[(static_cast<long long>(seg.x) + tok) * a.s.ldx + 2 * H * D + h * Dv + vb + d] : zero;
+  float nw[4] = {0.f, 0.f, 0.f, 0.f};  // the norm's weights of the columns this lane writes
+  if (!STATE_ONLY && a.norm_w)
+    for (int c = 0; c < 4; ++c)
+      if (lane * 4 + c < nv) nw[c] = ld1(a.norm_w + lane * 4 + c);
+  // projections of 16 tokens into a stage; tokens past the end become zeros
+  const bool wide = !((D | Dv | a.s.ldx) & 7) && !(reinterpret_cast<uintptr_t>(x) & 15);
+  auto load = [&](int t0, int st) {
+    if (wide) {
+      for (int i = tid; i < 3 * 16 * 16; i += kScThreads) {
+        const int part = i >> 8, tok = (i >> 4) & 15, c = (i & 15) * 8;
+        if (c < (part == 2 ? nv : D)) {
+          const long long row = static_cast<long long>(seg.x) + min(t0 + tok, seg.y - 1);
+          const int col = part == 2 ? 2 * H * D + h * Dv + vb + c : part * H * D + h * D + c;
+          cp_async16(&sm.raw[st][part][tok * 128 + c], x + row * a.s.ldx + col, t0 + tok < seg.y ? 16 : 0);
+        }
+      }
+    } else {
+      for (int i = tid; i < 3 * 16 * 128; i += kScThreads) {
+        const int part = i >> 11, tok = (i >> 7) & 15, c = i & 127;
+        if (c < (part == 2 ? nv : D)) {
+          const long long row = static_cast<long long>(seg.x) + t0 + tok;
+          const int col = part == 2 ? 2 * H * D + h * Dv + vb + c : part * H * D + h * D + c;
+          sm.raw[st][part][tok * 128 + c] = t0 + tok < seg.y ? x[row * a.s.ldx + col] : __float2bfloat16(0.f);
+        }
+      }
     }
+    asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  load(0);
-  for (int t0 = 0; t0 < seg.y; t0 += 16) {
-    // ---- activations; the triangle of A inside this half; running products of the gates inside the half
-    float q[8], f[8], k[8];
-    float run = 1.f;
+  load(0, 0);
+  int st = 0;
+  for (int t0 = 0; t0 < seg.y; t0 += 16, st ^= 1) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();  // this block's projections are here; every warp has left the block before
+    if (t0 + 16 < seg.y) load(t0 + 16, st ^ 1);
+    // ---- activations, running products of the gates inside this half
+    float q[8], k[8], f[8], run = 1.f;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       const int tok = half * 8 + i;
       q[i] = 0.f; k[i] = 0.f; f[i] = 1.f;
       if (dch && t0 + tok < seg.y)
-        scan_activate(mode, __bfloat162float(rq[i]), __bfloat162float(rf[i]), bias, low, decay, q[i], f[i], k[i]);
-    }
-    if (!STATE_ONLY && warp_live) {
-      float* A = sm.A[warp & 3] + half * (8 * 16 + 8);
-#pragma unroll
-      for (int batch = 0; batch < 3; ++batch) {
-        float v[16];
-#pragma unroll
-        for (int e = 0; e < 16; ++e) v[e] = 0.f;
-        if (batch == 0) {
-          tri_column<0>(q, f, k, v, 0);
-          tri_column<1>(q, f, k, v, 8);
-          tri_column<7>(q, f, k, v, 15);
-        } else if (batch == 1) {
-          tri_column<2>(q, f, k, v, 0);
-          tri_column<3>(q, f, k, v, 6);
-          tri_column<5>(q, f, k, v, 11);
-          tri_column<6>(q, f, k, v, 14);
-        } else {
-          tri_column<4>(q, f, k, v, 0);
-        }
-        const float sum = warp_sum16(v, lane);
-        const int e = lane >> 1;
-        if (!(lane & 1) && (batch < 2 || e < 4)) A[tri_entry(batch, e)] = sum;
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
+        scan_activate(mode, __bfloat162float(sm.raw[st][0][tok * 128 + d]), __bfloat162float(sm.raw[st][1][tok * 128 + d]),
+                      bias, low, decay, q[i], f[i], k[i]);
       run *= f[i];
-      if (!STATE_ONLY) q[i] *= run;  // q_i P_i, still without the gates of the first half
+      q[i] *= run;  // q_i P_i, still without the gates of the first half
     }
     float suf = 1.f;
 #pragma unroll
@@ -194,93 +158,100 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
     }
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      float v = __bfloat162float(rv[i]);
-      if (mode != 0) v = silu_fast(v);
-      sm.v[(half * 8 + i) * 136 + d] = d < nv ? __float2bfloat16(v) : zero;
+      const int tok = half * 8 + i;
+      __nv_bfloat16 v = __float2bfloat16(0.f);
+      if (d < nv) {
+        v = sm.raw[st][2][tok * 128 + d];
+        if (mode != 0) v = __float2bfloat16(silu_fast(__bfloat162float(v)));
+      }
+      sm.v[tok * 136 + d] = v;
     }
     if (d < DP) sm.tot[half][d] = run;
-    if (!STATE_ONLY) {
-#pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        if (half) sm.qx[i * 128 + d] = q[i];
-        else sm.kx[i * 128 + d] = k[i];
-      }
-    }
     __syncthreads();
-    if (t0 + 16 < seg.y) load(t0 + 16);
     // ---- operands: the other half's gates, then two bf16 terms
+    bool far = false;
     if (d < DP) {
-      const float other = sm.tot[half ^ 1][d];
+      const float other = sm.tot[half ^ 1][d], F = run * other;
+      far = F < 0x1p-90f;
+      const float inv = far ? 0.f : __fdividef(1.f, F);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const int at = (half * 8 + i) * (DP + 8) + d;
         if (!STATE_ONLY) {
           const float qq = half ? q[i] * other : q[i];
-          const __nv_bfloat16 hi = __float2bfloat16(qq);
-          sm.q[0][at] = hi;
-          sm.q[1][at] = __float2bfloat16(qq - __bfloat162float(hi));
+          put_split(sm.q[0], sm.q[1], at, qq);
+          put_split(sm.s[0], sm.s[1], at, qq * inv);
         }
-        const float kk = half ? k[i] : k[i] * other;
-        const __nv_bfloat16 hi = __float2bfloat16(kk);
-        sm.k[0][at] = hi;
-        sm.k[1][at] = __float2bfloat16(kk - __bfloat162float(hi));
+        put_split(sm.k[0], sm.k[1], at, half ? k[i] : k[i] * other);
       }
       if (half == 0) {
-        sm.F[d] = run * other;
-        seg_f *= run * other;
+        sm.F[d] = F;
+        seg_f *= F;
       }
     }
-    // ---- A between the halves: q_i of the second against k_j of the first; half h of the threads takes i = 8 + 4h ..
-    if (!STATE_ONLY && warp_live) {
-      float kj[8];
+    bool slow = false;
+    if (STATE_ONLY) __syncthreads();
+    else slow = __syncthreads_or(far);
+    const int r8 = (lane & 7) + ((lane >> 4) << 3), c8 = ((lane >> 3) & 1) * 8;
+    float o[2][4];
+    if (!STATE_ONLY) {
+      if (!slow) {
+        // ---- A: warp w computes keys 8 (w & 1) .. over channels 32 (w >> 1) ..
+        if ((warp >> 1) * 32 < DP) {
+          float acc[4] = {0.f, 0.f, 0.f, 0.f};
+          const uint32_t sh = s32(sm.s[0]) + (lane & 15) * PB + (lane >> 4) * 16, sl = s32(sm.s[1]) + (lane & 15) * PB + (lane >> 4) * 16;
+          const int kr = ((warp & 1) * 8 + (lane & 7)) * PB + (lane >> 3) * 16;
+          uint32_t bh[4], bl[4], ah[4], al[4];
+          const int c0 = (warp >> 1) * 64;  // bytes: two reduction blocks of 16 channels
+          ldm_x4(s32(sm.k[0]) + kr + c0, bh);
+          ldm_x4(s32(sm.k[1]) + kr + c0, bl);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) kj[j] = sm.kx[j * 128 + d];
-      float* A = sm.A[warp & 3] + (8 + half * 4) * 16;
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const float q0 = sm.qx[(half * 4 + e * 2) * 128 + d], q1 = sm.qx[(half * 4 + e * 2 + 1) * 128 + d];
-        float v[16];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          v[j] = q0 * kj[j];
-          v[8 + j] = q1 * kj[j];
-        }
-        const float sum = warp_sum16(v, lane);
-        const int x = lane >> 1;
-        if (!(lane & 1)) A[(e * 2 + (x >> 3)) * 16 + (x & 7)] = sum;
-      }
-    }
-    __syncthreads();
-    // ---- products
-    if (mma) {
-      const int r8 = (lane & 7) + ((lane >> 4) << 3), c8 = ((lane >> 3) & 1) * 8;
-      uint32_t vt[4];
-      ldm_x4_t(s32(sm.v + r8 * 136 + warp * 16 + c8), vt);
-      if (!STATE_ONLY) {
-        float o[2][4];
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-          for (int c = 0; c < 4; ++c) o[n][c] = 0.f;
-        uint32_t ah[4], al[4];
-        // A as the second operand: entries (i = g + 8n, j = 2t + 8c, +1) of the channel groups' partial sums
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int at = (g + (e >> 1) * 8) * 16 + 2 * t + (e & 1) * 8;
-          float2 sum = *reinterpret_cast<const float2*>(&sm.A[0][at]);
-#pragma unroll
-          for (int c = 1; c < (ND * 16 + 31) / 32; ++c) {
-            const float2 p = *reinterpret_cast<const float2*>(&sm.A[c][at]);
-            sum.x += p.x;
-            sum.y += p.y;
+          for (int e = 0; e < 2; ++e) {
+            ldm_x4(sh + c0 + e * 32, ah);
+            ldm_x4(sl + c0 + e * 32, al);
+            mma_bf16(acc, ah, bh[2 * e], bh[2 * e + 1]);
+            mma_bf16(acc, al, bh[2 * e], bh[2 * e + 1]);
+            mma_bf16(acc, ah, bl[2 * e], bl[2 * e + 1]);
           }
-          ah[e] = split2(sum.x, sum.y, al[e]);
+          float* A = sm.A[warp >> 1] + (warp & 1) * 8 + 2 * t;
+          *reinterpret_cast<float2*>(A + g * 16) = make_float2(acc[0], acc[1]);
+          *reinterpret_cast<float2*>(A + (g + 8) * 16) = make_float2(acc[2], acc[3]);
         }
+      } else {
+        // some channel forgets everything inside the block: pair by pair, lanes over channels
+        for (int j = warp; j < 16; j += 8) {
+          float w[4], acc = 0.f;
+          for (int i = j; i < 16; ++i) {
+            acc = 0.f;
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          mma_bf16(o[n], vt, ah[2 * n], ah[2 * n + 1]);
-          mma_bf16(o[n], vt, al[2 * n], al[2 * n + 1]);
+            for (int e = 0; e < 4; ++e) {
+              const int c = lane + 32 * e;
+              if (c < D && t0 + i < seg.y) {
+                float qq, ff, kk;
+                const bool gated = mode == 0;
+                const int hd = h * D + c;
+                scan_activate(mode, __bfloat162float(sm.raw[st][0][i * 128 + c]), __bfloat162float(sm.raw[st][1][i * 128 + c]),
+                              gated ? ld1(static_cast<const __nv_bfloat16*>(a.s.bias) + hd) : 0.f,
+                              gated ? ld1(static_cast<const __nv_bfloat16*>(a.s.lower) + hd) : 0.f, decay_h, qq, ff, kk);
+                w[e] = i == j ? kk : w[e] * ff;
+                acc = fmaf(qq, w[e], acc);
+              }
+            }
+            acc = warp_sum(acc);
+            if (lane == 0) {
+              sm.A[0][i * 16 + j] = acc;
+#pragma unroll
+              for (int c = 1; c < 4; ++c) sm.A[c][i * 16 + j] = 0.f;
+            }
+          }
         }
+      }
+      // ---- outputs from the state at the block's start
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) o[n][c] = 0.f;
+      if (mma) {
         const uint32_t qh = s32(sm.q[0]) + r8 * PB + c8 * 2, ql = s32(sm.q[1]) + r8 * PB + c8 * 2;
 #pragma unroll
         for (int kt = 0; kt < ND; ++kt) {
@@ -298,11 +269,38 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
             mma_bf16(o[n], hi, bl[2 * n], bl[2 * n + 1]);
           }
         }
+      }
+      __syncthreads();
+    }
+    if (mma) {
+      uint32_t vt[4];
+      ldm_x4_t(s32(sm.v + r8 * 136 + warp * 16 + c8), vt);
+      if (!STATE_ONLY) {
+        // ---- outputs from the block itself: A as the second operand, entries (i = g + 8n, j = 2t + 8c, +1), j <= i
+        uint32_t ah[4], al[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = g + (e >> 1) * 8, j = 2 * t + (e & 1) * 8;
+          float2 sum = *reinterpret_cast<const float2*>(&sm.A[0][i * 16 + j]);
+#pragma unroll
+          for (int c = 1; c < (DP + 31) / 32; ++c) {
+            const float2 p = *reinterpret_cast<const float2*>(&sm.A[c][i * 16 + j]);
+            sum.x += p.x;
+            sum.y += p.y;
+          }
+          ah[e] = split2(j <= i ? sum.x : 0.f, j + 1 <= i ? sum.y : 0.f, al[e]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          mma_bf16(o[n], vt, ah[2 * n], ah[2 * n + 1]);
+          mma_bf16(o[n], vt, al[2 * n], al[2 * n + 1]);
+        }
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int c = 0; c < 4; ++c) sm.o[(n * 8 + 2 * t + (c & 1)) * 132 + warp * 16 + g + (c >> 1) * 8] = o[n][c];
       }
+      // ---- the state at the block's end
       const uint32_t kh = s32(sm.k[0]) + (lane & 15) * PB + (lane >> 4) * 16,
                      kl = s32(sm.k[1]) + (lane & 15) * PB + (lane >> 4) * 16;
 #pragma unroll
@@ -320,21 +318,34 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
         }
       }
     }
-    __syncthreads();
-    // ---- outputs: warp w writes tokens w and w + 8
     if (!STATE_ONLY) {
+      __syncthreads();
+      // ---- warp w writes tokens w and w + 8, a lane four columns
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int i = warp + 8 * e;
+        const int i = warp + 8 * e, c = lane * 4;
         if (t0 + i < seg.y) {
-          const long long at = ((static_cast<long long>(seg.x) + t0 + i) * H + h) * Dv + vb;
+          const long long at = ((static_cast<long long>(seg.x) + t0 + i) * H + h) * Dv + vb + c;
+          float4 v = *reinterpret_cast<const float4*>(&sm.o[i * 132 + c]);
+          if (c >= nv) v.x = 0.f;
+          if (c + 1 >= nv) v.y = 0.f;
+          if (c + 2 >= nv) v.z = 0.f;
+          if (c + 3 >= nv) v.w = 0.f;
           if (a.norm_w) {
-            float ss = 0.f;
-            for (int c = lane; c < nv; c += 32) ss = fmaf(sm.o[i * 132 + c], sm.o[i * 132 + c], ss);
-            const float r = rsqrtf(warp_sum(ss) / nv + a.eps);
-            for (int c = lane; c < nv; c += 32) a.y[at + c] = __float2bfloat16(sm.o[i * 132 + c] * r * ld1(a.norm_w + c));
+            const float r = rsqrtf(warp_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)))) / nv + a.eps);
+            v.x *= r * nw[0]; v.y *= r * nw[1]; v.z *= r * nw[2]; v.w *= r * nw[3];
+          }
+          if (!(Dv & 3)) {
+            if (c < nv) {
+              if (a.norm_w) st4(a.y + at, v);
+              else st4(a.s.o + at, v);
+            }
           } else {
-            for (int c = lane; c < nv; c += 32) a.s.o[at + c] = sm.o[i * 132 + c];
+            const float u[4] = {v.x, v.y, v.z, v.w};
+            for (int n = 0; n < 4 && c + n < nv; ++n) {
+              if (a.norm_w) st1(a.y + at + n, u[n]);
+              else a.s.o[at + n] = u[n];
+            }
           }
         }
       }
