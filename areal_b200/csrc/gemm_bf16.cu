@@ -360,9 +360,9 @@ struct DytTail {
   __nv_bfloat16* y;
   int N;
 
-  __device__ __forceinline__ void apply4(float al, long long row, int c, float4 acc) const {
+  // h: the residual's four elements at (row, c), loaded by the caller (ahead of any store, so that loads overlap)
+  __device__ __forceinline__ void apply4(float al, long long row, int c, float4 acc, float4 h) const {
     const float4 s = ld4(scale + c), ww = ld4(w + c), bb = ld4(b + c);
-    float4 h = ld4(res + row * N + c);
     h.x = fmaf(s.x, acc.x, h.x); h.y = fmaf(s.y, acc.y, h.y);
     h.z = fmaf(s.z, acc.z, h.z); h.w = fmaf(s.w, acc.w, h.w);
     st4(res + row * N + c, h);
@@ -385,10 +385,14 @@ struct DytEpi {
   __device__ __forceinline__ void end(State&, int, int, int) const {}
   __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
     if (row >= M) return;
+    float4 h[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      h[i] = col0 + 4 * i < t.N ? ld4(t.res + static_cast<long long>(row) * t.N + col0 + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < 8; ++i)
       if (col0 + 4 * i < t.N)  // N % 4 == 0
-        t.apply4(s.al, row, col0 + 4 * i, make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]));
+        t.apply4(s.al, row, col0 + 4 * i, make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]), h[i]);
   }
 };
 
@@ -399,12 +403,13 @@ __global__ void splitk_reduce_dyt_kernel(const float* __restrict__ ws, DytTail t
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
     const int row = static_cast<int>(i / nq), c = static_cast<int>(i % nq) * 4;
+    const float4 h = ld4(t.res + static_cast<long long>(row) * t.N + c);
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int s = 0; s < S; ++s) {
       const float4 v = ld4(ws + s * slice_stride + static_cast<long long>(row) * t.N + c);
       acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
     }
-    t.apply4(al, row, c, acc);
+    t.apply4(al, row, c, acc, h);
   }
 }
 

@@ -2,22 +2,20 @@
 // against the same cached rows [rank | rot] (see latent_attn.cu). A cached row is read once for 16 heads and serves as
 // key (all of it) and value (its first `rank` numbers), so the kernel is bound by the cache stream.
 //
-// One CTA per (sequence, group of 16 heads, split): 4 warps, tiles of 32 tokens in a ring of stages. The rows of a tile
-// arrive by bulk copies (one per token, rows are padded to an odd number of 16-byte units so that ldmatrix is free of
-// bank conflicts). Warp w computes the scores of tokens 8w..8w+7; the [16, 32] scores meet in shared memory, every warp
-// takes the softmax of all of them (max, sum and weights in fp32) and multiplies its share of the value columns. The
-// weights enter the product as two bf16 terms (hi + lo), so they keep fp32-like precision.
+// One CTA per (sequence, group of 16 heads, split): 8 warps, tiles of 32 tokens in a ring of stages filled by cp.async
+// (rows are padded to an odd number of 16-byte units so that ldmatrix is free of bank conflicts). A warp computes the
+// scores of 8 tokens over half of the width; the [16, 32] scores meet in shared memory, every warp takes the softmax of
+// all of them (max, sum and weights in fp32) and multiplies its share of the value columns. The weights enter the product as two bf16 terms
+// (hi + lo), so they keep fp32-like precision.
 #include "common/host_utils.h"
 #include "common/io.cuh"
 #include "common/mma16.cuh"
-#include "common/ptx.cuh"
 
 namespace b200 {
 
 constexpr int kLdTok = 32;     // tokens per tile
-constexpr int kLdWarps = 4;
+constexpr int kLdWarps = 8;
 constexpr int kLdSPitch = 40;  // floats per score row
-constexpr int kLdMaxStages = 4;
 
 struct LatentDecodeArgs {
   const __nv_bfloat16 *qa, *q, *cache;
@@ -26,36 +24,26 @@ struct LatentDecodeArgs {
   const int *block_table, *seq_lens;
   __nv_bfloat16* out;   // [B, H * rank]
   float *o_part, *ml_part;
-  int H, rank, rot, block_size, max_blocks, nsplit, stages, pitch;  // pitch: bytes of a row in shared memory
+  int H, rank, rot, block_size, max_blocks, nsplit, pitch;  // pitch: bytes of a row in shared memory
   float scale_log2;
 };
 
-__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
-                   smem_u32(dst)), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
-}
+__device__ __forceinline__ uint32_t sa32(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
 
-// NP: pairs of value column tiles (16 columns) per warp
-template <int NP>
-__global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentDecodeArgs a, int* status) {
+// NP: pairs of value column tiles (16 columns) per warp; ST: stages
+template <int NP, int ST>
+__global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentDecodeArgs a) {
   extern __shared__ __align__(128) uint8_t sm[];
   const int W = a.rank + a.rot, pitch = a.pitch;
-  uint64_t* full = reinterpret_cast<uint64_t*>(sm);                        // [stages]
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + 64);
-  float* sS = reinterpret_cast<float*>(sm + 128);                          // [2][16][kLdSPitch]
-  uint8_t* sQ = sm + 128 + 2 * 16 * kLdSPitch * 4;                         // [16][pitch]
-  uint8_t* ring = sQ + 16 * pitch;                                         // [stages][32][pitch]
+  float* sS = reinterpret_cast<float*>(sm);             // [2][width half][16][kLdSPitch]
+  uint8_t* sQ = sm + 4 * 16 * kLdSPitch * 4;            // [16][pitch]
+  uint8_t* ring = sQ + 16 * pitch;                      // [ST][32][pitch]
   const int b = blockIdx.x, h0 = blockIdx.y * 16, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int L = a.seq_lens[b];
   const int tiles = (L + kLdTok - 1) / kLdTok, per = (tiles + a.nsplit - 1) / a.nsplit;
   const int j0 = split * per, n = max(0, min(tiles, j0 + per) - j0);
   const int* bt = a.block_table + static_cast<long long>(b) * a.max_blocks;
-  if (threadIdx.x == 0) {
-    for (int i = 0; i < a.stages; ++i) mbar_init(&full[i], 1);
-    *abort_flag = 0;
-    fence_mbar_init();
-  }
   // queries: 16 rows of W, zero for heads past the last
   for (int i = threadIdx.x; i < 16 * (W / 8); i += blockDim.x) {
     const int r = i / (W / 8), c = (i % (W / 8)) * 8, h = h0 + r;
@@ -65,26 +53,25 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
                      : *reinterpret_cast<const uint4*>(a.q + b * a.ldq + static_cast<long long>(h) * a.q_stride + a.q_off + c - a.rank);
     *reinterpret_cast<uint4*>(sQ + r * pitch + c * 2) = v;
   }
-  __syncthreads();
 
-  // warp 0 fills a stage: lane = token of the tile; rows past the end are zeroed (a weight of 0 must meet a number)
+  // eight threads per row; rows past the end become zeros (a weight of 0 must meet a number)
+  const int fr = threadIdx.x >> 3, fc = threadIdx.x & 7;
   auto fill = [&](int j) {
-    uint64_t* bar = &full[j % a.stages];
-    const int tok = (j0 + j) * kLdTok + lane;
-    uint8_t* dst = ring + ((j % a.stages) * kLdTok + lane) * pitch;
-    const int valid = min(kLdTok, L - (j0 + j) * kLdTok);
-    if (lane >= valid)
-      for (int i = 0; i < W / 8; ++i) *reinterpret_cast<uint4*>(dst + i * 16) = make_uint4(0, 0, 0, 0);
-    __syncwarp();
-    if (lane == 0) mbar_arrive_expect_tx(bar, valid * W * 2);
-    __syncwarp();
-    if (lane < valid) {
-      const long long row = static_cast<long long>(bt[tok / a.block_size]) * a.block_size + tok % a.block_size;
-      bulk_load(dst, a.cache + row * W, W * 2, bar);
+    if (j < n) {
+      const int tok = (j0 + j) * kLdTok + fr;
+      const bool in = tok < L;
+      const int tk = in ? tok : L - 1;
+      const __nv_bfloat16* src = a.cache + (static_cast<long long>(bt[tk / a.block_size]) * a.block_size + tk % a.block_size) * W;
+      const uint32_t dst = sa32(ring + ((j % ST) * kLdTok + fr) * pitch);
+#pragma unroll 4
+      for (int c = fc; c < W / 8; c += 8)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + c * 16), "l"(src + c * 8), "r"(in ? 16 : 0)
+                     : "memory");
     }
+    asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  if (warp == 0)
-    for (int j = 0; j < a.stages && j < n; ++j) fill(j);
+#pragma unroll
+  for (int j = 0; j < ST - 1; ++j) fill(j);
 
   float o[2 * NP][4];
 #pragma unroll
@@ -94,48 +81,41 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;  // rows g and g + 8
   const int g = lane >> 2, t = lane & 3;
   const int pairs = a.rank >> 4;
-  const uint32_t qrow = smem_u32(sQ) + (lane & 15) * pitch + (lane >> 4) * 16;
-  bool ok = true;
+  const uint32_t qrow = sa32(sQ) + (lane & 15) * pitch + (lane >> 4) * 16;
   for (int j = 0; j < n; ++j) {
-    const int st = j % a.stages;
-    if (!mbar_wait(&full[st], (j / a.stages) & 1, abort_flag)) {
-      ok = false;
-      *abort_flag = 1;
+    asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");
+    __syncthreads();  // tile j is here for everyone; every warp has left tile j - 1
+    fill(j + ST - 1);
+    const uint32_t base = sa32(ring + (j % ST) * kLdTok * pitch);
+    // scores of this warp's 8 tokens over its half of the width: two blocks of 16 per ldmatrix, two chains against the
+    // tensor-core latency
+    float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
+    const int tg = warp & 3, wh = warp >> 2;
+    const uint32_t krow = base + (tg * 8 + (lane & 7)) * pitch + (lane >> 3) * 16;
+    const int mid = (((W >> 4) + 3) >> 2) * 2, kt = wh ? W >> 4 : min(mid, W >> 4);
+    int k = wh ? min(mid, W >> 4) : 0;
+#pragma unroll 4
+    for (; k + 2 <= kt; k += 2) {
+      uint32_t kb[4], q0[4], q1[4];
+      ldm_x4(krow + k * 32, kb);
+      ldm_x4(qrow + k * 32, q0);
+      ldm_x4(qrow + k * 32 + 32, q1);
+      mma_bf16(s, q0, kb[0], kb[1]);
+      mma_bf16(s2, q1, kb[2], kb[3]);
     }
-    const uint32_t base = smem_u32(ring + st * kLdTok * pitch);
-    float s[4] = {0.f, 0.f, 0.f, 0.f};
-    if (ok) {
-      // scores of this warp's 8 tokens: two key blocks of 16 per ldmatrix
-      const uint32_t krow = base + (warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 16;
-      float s2[4] = {0.f, 0.f, 0.f, 0.f};  // a second chain hides the tensor-core latency
-      const int kt = W >> 4;
-      int k = 0;
-      for (; k + 2 <= kt; k += 2) {
-        uint32_t kb[4], qf[4];
-        ldm_x4(krow + k * 32, kb);
-        ldm_x4(qrow + k * 32, qf);
-        mma_bf16(s, qf, kb[0], kb[1]);
-        ldm_x4(qrow + k * 32 + 32, qf);
-        mma_bf16(s2, qf, kb[2], kb[3]);
-      }
-      if (k < kt) {
-        uint32_t kb[2], qf[4];
-        ldm_x2(base + (warp * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 16 + k * 32, kb);
-        ldm_x4(qrow + k * 32, qf);
-        mma_bf16(s, qf, kb[0], kb[1]);
-      }
+    if (k < kt) {
+      uint32_t kb[2], q0[4];
+      ldm_x2(base + (tg * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 16 + k * 32, kb);
+      ldm_x4(qrow + k * 32, q0);
+      mma_bf16(s, q0, kb[0], kb[1]);
+    }
 #pragma unroll
-      for (int c = 0; c < 4; ++c) s[c] += s2[c];
-    }
-    float* S = sS + (j & 1) * 16 * kLdSPitch;
-    *reinterpret_cast<float2*>(S + g * kLdSPitch + warp * 8 + 2 * t) = make_float2(s[0], s[1]);
-    *reinterpret_cast<float2*>(S + (g + 8) * kLdSPitch + warp * 8 + 2 * t) = make_float2(s[2], s[3]);
-    __syncthreads();  // scores complete; every warp has left tile j - 1
-    if (*abort_flag) { ok = false; break; }
-    if (warp == 0 && j >= 1 && j - 1 + a.stages < n) {
-      fence_proxy_async_smem();  // the stage was read through the generic proxy
-      fill(j - 1 + a.stages);
-    }
+    for (int c = 0; c < 4; ++c) s[c] += s2[c];
+    constexpr int kHalf = 16 * kLdSPitch;
+    float* S = sS + (j & 1) * 2 * kHalf;
+    *reinterpret_cast<float2*>(S + wh * kHalf + g * kLdSPitch + tg * 8 + 2 * t) = make_float2(s[0], s[1]);
+    *reinterpret_cast<float2*>(S + wh * kHalf + (g + 8) * kLdSPitch + tg * 8 + 2 * t) = make_float2(s[2], s[3]);
+    __syncthreads();  // scores complete
     // softmax of the 16 x 32 scores; fragment order: [k block][row half][8-column half][2]
     float p[2][2][2][2];
     float x0 = -INFINITY, x1 = -INFINITY;
@@ -144,8 +124,10 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
     for (int kb = 0; kb < 2; ++kb)
 #pragma unroll
       for (int ch = 0; ch < 2; ++ch) {
-        const float2 u = *reinterpret_cast<const float2*>(S + g * kLdSPitch + kb * 16 + ch * 8 + 2 * t);
-        const float2 v = *reinterpret_cast<const float2*>(S + (g + 8) * kLdSPitch + kb * 16 + ch * 8 + 2 * t);
+        const float* at = S + g * kLdSPitch + kb * 16 + ch * 8 + 2 * t;
+        float2 u = *reinterpret_cast<const float2*>(at), v = *reinterpret_cast<const float2*>(at + 8 * kLdSPitch);
+        const float2 u1 = *reinterpret_cast<const float2*>(at + kHalf), v1 = *reinterpret_cast<const float2*>(at + kHalf + 8 * kLdSPitch);
+        u.x += u1.x; u.y += u1.y; v.x += v1.x; v.y += v1.y;
         const bool a0 = tok + kb * 16 + ch * 8 < L, a1 = tok + kb * 16 + ch * 8 + 1 < L;
         p[kb][0][ch][0] = a0 ? u.x * a.scale_log2 : -INFINITY;
         p[kb][0][ch][1] = a1 ? u.y * a.scale_log2 : -INFINITY;
@@ -192,14 +174,6 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
         }
       }
     }
-  }
-  if (!ok) {
-    if (threadIdx.x == 0) {
-      atomicCAS(status, 0, kErrMbarTimeoutEpilogue);
-      const unsigned long long t0 = globaltimer_ns();  // copies in flight land before the CTA retires
-      while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
-    }
-    return;
   }
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
@@ -278,28 +252,27 @@ int b200_latent_decode(const void* qa, long long ldqa, const void* q, long long 
     return -100;
   using bf = __nv_bfloat16;
   const int W = rank + rot, pitch = ((W / 8) | 1) * 16;
-  const int fixed = 128 + 2 * 16 * kLdSPitch * 4 + 16 * pitch, stage = kLdTok * pitch;
-  int stages = (112 * 1024 - fixed) / stage;
-  stages = stages < 2 ? 2 : stages > kLdMaxStages ? kLdMaxStages : stages;
+  const int fixed = 4 * 16 * kLdSPitch * 4 + 16 * pitch, stage = kLdTok * pitch;
+  const int stages = fixed + 3 * stage <= 113 * 1024 ? 3 : 2;
   const int smem = fixed + stages * stage;
   LatentDecodeArgs a{(const bf*)qa, (const bf*)q, (const bf*)cache, ldqa, ldq, q_stride, q_off, block_table, seq_lens,
-                     (bf*)out, o_part, ml_part, H, rank, rot, block_size, max_blocks, nsplit, stages, pitch,
+                     (bf*)out, o_part, ml_part, H, rank, rot, block_size, max_blocks, nsplit, pitch,
                      scale * 1.4426950408889634f};
-  int* status = device_status_word();
-  if (!status) return -3;
   dim3 grid(B, (H + 15) / 16, nsplit);
   const int np = (rank / 16 + kLdWarps - 1) / kLdWarps;
-#define B200_LD(NP_)                                                                                                \
+#define B200_LDS(NP_, ST_)                                                                                          \
   {                                                                                                                 \
-    B200_CHECK(cudaFuncSetAttribute(latent_decode_kernel<NP_>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)); \
-    latent_decode_kernel<NP_><<<grid, kLdWarps * 32, smem, stream>>>(a, status);                                    \
+    B200_CHECK(cudaFuncSetAttribute(latent_decode_kernel<NP_, ST_>, cudaFuncAttributeMaxDynamicSharedMemorySize,    \
+                                    smem));                                                                         \
+    latent_decode_kernel<NP_, ST_><<<grid, kLdWarps * 32, smem, stream>>>(a);                                       \
   }
-  if (np <= 1) B200_LD(1)
-  else if (np <= 2) B200_LD(2)
-  else if (np <= 4) B200_LD(4)
-  else if (np <= 6) B200_LD(6)
-  else B200_LD(8)
+#define B200_LD(NP_)                                                                                                \
+  if (stages == 3) B200_LDS(NP_, 3) else B200_LDS(NP_, 2)
+  if (np <= 1) { B200_LD(1) }
+  else if (np <= 2) { B200_LD(2) }
+  else { B200_LD(4) }
 #undef B200_LD
+#undef B200_LDS
   B200_CHECK(cudaGetLastError());
   if (nsplit > 1) {
     latent_merge_kernel<<<B * H, rank >= 256 ? 256 : 128, 0, stream>>>(o_part, ml_part, (bf*)out, nsplit, rank);
