@@ -4,8 +4,9 @@
 //
 // One CTA per (sequence, group of 16 heads, split): 8 warps, tiles of 32 tokens in a ring of stages filled by cp.async
 // (rows are padded to an odd number of 16-byte units so that ldmatrix is free of bank conflicts). A warp computes the
-// scores of 8 tokens over half of the width; the [16, 32] scores meet in shared memory, every warp takes the softmax of
-// all of them (max, sum and weights in fp32) and multiplies its share of the value columns. The weights enter the product as two bf16 terms
+// scores of 8 tokens over half of the width; the [16, 32] scores meet in shared memory, every warp takes the softmax of two
+// heads (max, sum and weights in fp32, a lane per token) and, with all heads' weights, multiplies its share of the value
+// columns. The weights enter the product as two bf16 terms
 // (hi + lo), so they keep fp32-like precision.
 #include "common/host_utils.h"
 #include "common/io.cuh"
@@ -16,6 +17,9 @@ namespace b200 {
 constexpr int kLdTok = 32;     // tokens per tile
 constexpr int kLdWarps = 8;
 constexpr int kLdSPitch = 40;  // floats per score row
+constexpr int kLdPPitch = 80;  // bytes per row of weights (32 bf16 and padding)
+// shared memory ahead of the queries: scores of both width halves, weights (hi, lo), correction factors, row statistics
+constexpr int kLdFixed = 2 * 16 * kLdSPitch * 4 + 2 * 16 * kLdPPitch + 16 * 4 + 32 * 4 + 64;
 
 struct LatentDecodeArgs {
   const __nv_bfloat16 *qa, *q, *cache;
@@ -35,8 +39,11 @@ template <int NP, int ST>
 __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentDecodeArgs a) {
   extern __shared__ __align__(128) uint8_t sm[];
   const int W = a.rank + a.rot, pitch = a.pitch;
-  float* sS = reinterpret_cast<float*>(sm);             // [2][width half][16][kLdSPitch]
-  uint8_t* sQ = sm + 4 * 16 * kLdSPitch * 4;            // [16][pitch]
+  float* sS = reinterpret_cast<float*>(sm);             // [width half][16][kLdSPitch]
+  uint8_t* sP = sm + 2 * 16 * kLdSPitch * 4;            // [hi, lo][16][kLdPPitch]
+  float* sC = reinterpret_cast<float*>(sP + 2 * 16 * kLdPPitch);  // [16] factor for what a head has accumulated
+  float* sML = sC + 16;                                 // [16][2] maximum and sum at the end
+  uint8_t* sQ = sm + kLdFixed;                          // [16][pitch]
   uint8_t* ring = sQ + 16 * pitch;                      // [ST][32][pitch]
   const int b = blockIdx.x, h0 = blockIdx.y * 16, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -56,12 +63,17 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
 
   // eight threads per row; rows past the end become zeros (a weight of 0 must meet a number)
   const int fr = threadIdx.x >> 3, fc = threadIdx.x & 7;
+  auto page_of = [&](int j) {  // page of this thread's row of tile j (any page past the end: the row is zeroed)
+    return j < n ? __ldg(bt + min((j0 + j) * kLdTok + fr, L - 1) / a.block_size) : 0;
+  };
+  int page = page_of(0);  // looked up one tile ahead: its latency would delay every copy
   auto fill = [&](int j) {
     if (j < n) {
       const int tok = (j0 + j) * kLdTok + fr;
       const bool in = tok < L;
       const int tk = in ? tok : L - 1;
-      const __nv_bfloat16* src = a.cache + (static_cast<long long>(bt[tk / a.block_size]) * a.block_size + tk % a.block_size) * W;
+      const __nv_bfloat16* src = a.cache + (static_cast<long long>(page) * a.block_size + tk % a.block_size) * W;
+      page = page_of(j + 1);
       const uint32_t dst = sa32(ring + ((j % ST) * kLdTok + fr) * pitch);
 #pragma unroll 4
       for (int c = fc; c < W / 8; c += 8)
@@ -78,7 +90,7 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
   for (int i = 0; i < 2 * NP; ++i)
 #pragma unroll
     for (int c = 0; c < 4; ++c) o[i][c] = 0.f;
-  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;  // rows g and g + 8
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};  // heads 2 * warp and 2 * warp + 1; l: this lane's tokens
   const int g = lane >> 2, t = lane & 3;
   const int pairs = a.rank >> 4;
   const uint32_t qrow = sa32(sQ) + (lane & 15) * pitch + (lane >> 4) * 16;
@@ -112,53 +124,43 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
 #pragma unroll
     for (int c = 0; c < 4; ++c) s[c] += s2[c];
     constexpr int kHalf = 16 * kLdSPitch;
-    float* S = sS + (j & 1) * 2 * kHalf;
-    *reinterpret_cast<float2*>(S + wh * kHalf + g * kLdSPitch + tg * 8 + 2 * t) = make_float2(s[0], s[1]);
-    *reinterpret_cast<float2*>(S + wh * kHalf + (g + 8) * kLdSPitch + tg * 8 + 2 * t) = make_float2(s[2], s[3]);
+    *reinterpret_cast<float2*>(sS + wh * kHalf + g * kLdSPitch + tg * 8 + 2 * t) = make_float2(s[0], s[1]);
+    *reinterpret_cast<float2*>(sS + wh * kHalf + (g + 8) * kLdSPitch + tg * 8 + 2 * t) = make_float2(s[2], s[3]);
     __syncthreads();  // scores complete
-    // softmax of the 16 x 32 scores; fragment order: [k block][row half][8-column half][2]
-    float p[2][2][2][2];
-    float x0 = -INFINITY, x1 = -INFINITY;
-    const int tok = (j0 + j) * kLdTok + 2 * t;
 #pragma unroll
-    for (int kb = 0; kb < 2; ++kb)
+    for (int e = 0; e < 2; ++e) {
+      const int r = 2 * warp + e;
+      const bool in = (j0 + j) * kLdTok + lane < L;
+      const float x = in ? (sS[r * kLdSPitch + lane] + sS[kHalf + r * kLdSPitch + lane]) * a.scale_log2 : -INFINITY;
+      float mx = x;
 #pragma unroll
-      for (int ch = 0; ch < 2; ++ch) {
-        const float* at = S + g * kLdSPitch + kb * 16 + ch * 8 + 2 * t;
-        float2 u = *reinterpret_cast<const float2*>(at), v = *reinterpret_cast<const float2*>(at + 8 * kLdSPitch);
-        const float2 u1 = *reinterpret_cast<const float2*>(at + kHalf), v1 = *reinterpret_cast<const float2*>(at + kHalf + 8 * kLdSPitch);
-        u.x += u1.x; u.y += u1.y; v.x += v1.x; v.y += v1.y;
-        const bool a0 = tok + kb * 16 + ch * 8 < L, a1 = tok + kb * 16 + ch * 8 + 1 < L;
-        p[kb][0][ch][0] = a0 ? u.x * a.scale_log2 : -INFINITY;
-        p[kb][0][ch][1] = a1 ? u.y * a.scale_log2 : -INFINITY;
-        p[kb][1][ch][0] = a0 ? v.x * a.scale_log2 : -INFINITY;
-        p[kb][1][ch][1] = a1 ? v.y * a.scale_log2 : -INFINITY;
-        x0 = fmaxf(x0, fmaxf(p[kb][0][ch][0], p[kb][0][ch][1]));
-        x1 = fmaxf(x1, fmaxf(p[kb][1][ch][0], p[kb][1][ch][1]));
+      for (int d = 16; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+      // the running maximum is raised only when a score passes it by 2^8 (every tile holds at least one token)
+      float corr = 1.f;
+      if (mx > m[e] + 8.f) {
+        corr = m[e] == -INFINITY ? 0.f : exp2f(m[e] - mx);
+        m[e] = mx;
       }
-    x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
-    x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
-    // the running maximum is raised only when a score passes it by 2^8 (every tile holds at least one token)
-    const bool up0 = x0 > m0 + 8.f, up1 = x1 > m1 + 8.f;
-    if (__any_sync(0xffffffffu, up0 || up1)) {
-      const float n0 = up0 ? x0 : m0, n1 = up1 ? x1 : m1;
-      const float c0 = m0 == -INFINITY ? 0.f : exp2f(m0 - n0), c1 = m1 == -INFINITY ? 0.f : exp2f(m1 - n1);
-      l0 *= c0; l1 *= c1; m0 = n0; m1 = n1;
+      const float w = exp2f(x - m[e]);
+      l[e] = l[e] * corr + w;
+      const __nv_bfloat16 hi = __float2bfloat16(w);
+      reinterpret_cast<__nv_bfloat16*>(sP + r * kLdPPitch)[lane] = hi;
+      reinterpret_cast<__nv_bfloat16*>(sP + (16 + r) * kLdPPitch)[lane] = __float2bfloat16(w - __bfloat162float(hi));
+      if (lane == 0) sC[r] = corr;
+    }
+    __syncthreads();  // weights complete
+    const float c0 = sC[g], c1 = sC[g + 8];
+    if (__any_sync(0xffffffffu, c0 != 1.f || c1 != 1.f)) {
 #pragma unroll
       for (int i = 0; i < 2 * NP; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
     }
     uint32_t hi[2][4], lo[2][4];
+    const uint32_t prow = sa32(sP) + (lane & 15) * kLdPPitch + (lane >> 4) * 16;
 #pragma unroll
-    for (int kb = 0; kb < 2; ++kb)
-#pragma unroll
-      for (int ch = 0; ch < 2; ++ch) {
-        const float p00 = exp2f(p[kb][0][ch][0] - m0), p01 = exp2f(p[kb][0][ch][1] - m0);
-        const float p10 = exp2f(p[kb][1][ch][0] - m1), p11 = exp2f(p[kb][1][ch][1] - m1);
-        l0 += p00 + p01;
-        l1 += p10 + p11;
-        hi[kb][ch * 2] = split2(p00, p01, lo[kb][ch * 2]);
-        hi[kb][ch * 2 + 1] = split2(p10, p11, lo[kb][ch * 2 + 1]);
-      }
+    for (int kb = 0; kb < 2; ++kb) {
+      ldm_x4(prow + kb * 32, hi[kb]);
+      ldm_x4(prow + 16 * kLdPPitch + kb * 32, lo[kb]);
+    }
 #pragma unroll
     for (int i = 0; i < NP; ++i) {
       const int pr = warp + i * kLdWarps;
@@ -175,16 +177,22 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
       }
     }
   }
-  l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
-  l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const float sum = warp_sum(l[e]);
+    if (lane == 0) {
+      sML[(2 * warp + e) * 2] = m[e];
+      sML[(2 * warp + e) * 2 + 1] = sum;
+    }
+  }
+  __syncthreads();
   const bool direct = a.nsplit == 1;
-  const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int h = h0 + g + half * 8;
     if (h >= a.H) continue;
     const long long u = (static_cast<long long>(b) * a.H + h);
-    const float inv = half ? i1 : i0;
+    const float sum = sML[(g + half * 8) * 2 + 1], inv = sum > 0.f ? 1.f / sum : 0.f;
 #pragma unroll
     for (int i = 0; i < 2 * NP; ++i) {
       const int pr = warp + (i >> 1) * kLdWarps;
@@ -197,8 +205,8 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
         *reinterpret_cast<float2*>(a.o_part + (u * a.nsplit + split) * a.rank + c) = make_float2(v0, v1);
     }
     if (!direct && warp == 0 && t == 0) {
-      a.ml_part[(u * a.nsplit + split) * 2] = half ? m1 : m0;
-      a.ml_part[(u * a.nsplit + split) * 2 + 1] = half ? l1 : l0;
+      a.ml_part[(u * a.nsplit + split) * 2] = sML[(g + half * 8) * 2];
+      a.ml_part[(u * a.nsplit + split) * 2 + 1] = sum;
     }
   }
 }
@@ -252,7 +260,7 @@ int b200_latent_decode(const void* qa, long long ldqa, const void* q, long long 
     return -100;
   using bf = __nv_bfloat16;
   const int W = rank + rot, pitch = ((W / 8) | 1) * 16;
-  const int fixed = 4 * 16 * kLdSPitch * 4 + 16 * pitch, stage = kLdTok * pitch;
+  const int fixed = kLdFixed + 16 * pitch, stage = kLdTok * pitch;
   const int stages = fixed + 3 * stage <= 113 * 1024 ? 3 : 2;
   const int smem = fixed + stages * stage;
   LatentDecodeArgs a{(const bf*)qa, (const bf*)q, (const bf*)cache, ldqa, ldq, q_stride, q_off, block_table, seq_lens,
