@@ -371,27 +371,42 @@ struct DytTail {
   }
 };
 
+template <int BN>
 struct DytEpi {
   DytTail t;
   int M;
-  struct State { float al; };
+  // The residual of the next 32 columns is loaded ahead of the stores of the current ones: each thread walks along its
+  // own row, and without this every chunk would wait for a trip to memory.
+  struct State {
+    float al;
+    float4 h[8];
+  };
 
   __device__ __forceinline__ bool tile(int cta, int ncta, int it, int tiles_m, int tiles_n, int& m_blk,
                                        int& n_blk) const {
     return default_tile(cta, ncta, it, tiles_m, tiles_n, m_blk, n_blk);
   }
   __device__ __forceinline__ bool gate(int, int, volatile int*, int*) const { return true; }
-  __device__ __forceinline__ void begin(State& s, int, int, int) const { s.al = __bfloat162float(*t.alpha); }
+  __device__ __forceinline__ void fetch(State& s, int row, int col0) const {
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (row < M && col0 + 4 * i < t.N)  // N % 4 == 0
+        s.h[i] = ld4(t.res + static_cast<long long>(row) * t.N + col0 + 4 * i);
+  }
+  __device__ __forceinline__ void begin(State& s, int, int n_blk, int row) const {
+    s.al = __bfloat162float(*t.alpha);
+    fetch(s, row, n_blk * BN);
+  }
   __device__ __forceinline__ void end(State&, int, int, int) const {}
   __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
-    if (row >= M) return;
     float4 h[8];
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
-      h[i] = col0 + 4 * i < t.N ? ld4(t.res + static_cast<long long>(row) * t.N + col0 + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < 8; ++i) h[i] = s.h[i];
+    if ((col0 + 32) % BN) fetch(s, row, col0 + 32);
+    if (row >= M) return;
 #pragma unroll
     for (int i = 0; i < 8; ++i)
-      if (col0 + 4 * i < t.N)  // N % 4 == 0
+      if (col0 + 4 * i < t.N)
         t.apply4(s.al, row, col0 + 4 * i, make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]), h[i]);
   }
 };
@@ -608,6 +623,35 @@ int b200_gemm_bf16_splitk_rmsnorm(const void* A, const void* B, const void* bias
   return 0;
 }
 
+}  // extern "C"
+
+template <int BN>
+static int launch_dyt(const void* A, const void* B, const b200::DytTail& tail, int M, int N, int K, long long lda,
+                      long long ldb, cudaStream_t stream) {
+  using namespace b200;
+  using Cfg = GemmCfg<BN>;
+  CUtensorMap tmA, tmB;
+  int rc = make_tmap_2d(&tmA, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, K, lda * 2, kBM, 64);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tmB, B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, N, K, ldb * 2, BN, 64);
+  if (rc) return rc;
+  auto kern = gemm_tcgen05_kernel<BN, false, false, DytEpi<BN>>;
+  static bool attr_set = false;
+  if (!attr_set) {
+    B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
+    attr_set = true;
+  }
+  const long long tiles = static_cast<long long>((M + kBM - 1) / kBM) * ((N + BN - 1) / BN);
+  const int grid = static_cast<int>(tiles < sm_count() ? tiles : sm_count());
+  int* status = device_status_word();
+  if (!status) return -3;
+  kern<<<grid, kGemmThreads, Cfg::kSmemBytes, stream>>>(tmA, tmB, M, N, K, DytEpi<BN>{tail, M}, status);
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
+extern "C" {
+
 // A [M, K] . B [N, K]^T with the DytEpi tail: res [M, N] fp32 (in place), y [M, N] bf16, N % 4 == 0. splits > 1: split-K
 // into `workspace` (fp32 [splits * ceil(M/128)*128 * N]) with the tail in the reduction kernel.
 int b200_gemm_bf16_dyt(const void* A, const void* B, float* workspace, int M, int N, int K, long long lda,
@@ -630,26 +674,9 @@ int b200_gemm_bf16_dyt(const void* A, const void* B, float* workspace, int M, in
     B200_CHECK(cudaGetLastError());
     return 0;
   }
-  constexpr int BN = 128;
-  using Cfg = GemmCfg<BN>;
-  CUtensorMap tmA, tmB;
-  int rc = make_tmap_2d(&tmA, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, M, K, lda * 2, kBM, 64);
-  if (rc) return rc;
-  rc = make_tmap_2d(&tmB, B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, N, K, ldb * 2, BN, 64);
-  if (rc) return rc;
-  auto kern = gemm_tcgen05_kernel<BN, false, false, DytEpi>;
-  static bool attr_set = false;
-  if (!attr_set) {
-    B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
-    attr_set = true;
-  }
-  const long long tiles = static_cast<long long>((M + kBM - 1) / kBM) * ((N + BN - 1) / BN);
-  const int grid = static_cast<int>(tiles < sm_count() ? tiles : sm_count());
-  int* status = device_status_word();
-  if (!status) return -3;
-  kern<<<grid, kGemmThreads, Cfg::kSmemBytes, stream>>>(tmA, tmB, M, N, K, DytEpi{tail, M}, status);
-  B200_CHECK(cudaGetLastError());
-  return 0;
+  const long long tiles256 = static_cast<long long>((M + kBM - 1) / kBM) * ((N + 255) / 256);
+  return tiles256 >= 100 ? launch_dyt<256>(A, B, tail, M, N, K, lda, ldb, stream)
+                         : launch_dyt<128>(A, B, tail, M, N, K, lda, ldb, stream);
 }
 
 // Per-head products (HeadsEpi). A: [M][lda], head h reads columns [h * a_head, h * a_head + K). W is stacked:
