@@ -45,14 +45,27 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return t;
 }
 
+// 2^x and 1/x by the hardware approximations, denormals flushed (no range-scaling instructions around them)
+__device__ __forceinline__ float ex2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_fast(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float exp_fast(float x) { return ex2_fast(x * 1.4426950408889634f); }
+
 // tanh for results in the given dtype: fp32 gets the library function; for bf16 results 1 - 2 / (1 + e^2x), whose absolute
 // error (about 1e-7 of the range) is far below the result's rounding.
 __device__ __forceinline__ float tanh_as(float x, const float*) { return tanhf(x); }
 __device__ __forceinline__ float tanh_as(float x, const __nv_bfloat16*) {
-  return 1.f - __fdividef(2.f, 1.f + __expf(2.f * x));
+  return 1.f - 2.f * rcp_fast(1.f + exp_fast(2.f * x));
 }
 
 __device__ __forceinline__ float sigmoid_as(float x, const float*) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float sigmoid_as(float x, const __nv_bfloat16*) { return __fdividef(1.f, 1.f + __expf(-x)); }
+__device__ __forceinline__ float sigmoid_as(float x, const __nv_bfloat16*) { return rcp_fast(1.f + exp_fast(-x)); }
 
 }  // namespace b200

@@ -17,8 +17,8 @@ struct ScanArgs {
   int H, D, Dv, mode;
 };
 
-// x sigmoid(x) with the hardware exponential and quotient (a few ulp; 0 where exp(-x) overflows)
-__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+// x sigmoid(x) with the hardware exponential and reciprocal (a few ulp; -0 where exp(-x) overflows)
+__device__ __forceinline__ float silu_fast(float x) { return x * rcp_fast(1.f + exp_fast(-x)); }
 
 // q, f and k of one channel from the two projections u0, u1 (mode 0: with the channel's gate bias and lower bound;
 // mode 1: with the head's decay).
@@ -26,8 +26,8 @@ __device__ __forceinline__ void scan_activate(int mode, float u0, float u1, floa
                                               float& f, float& k) {
   q = silu_fast(u0);
   if (mode == 0) {
-    const float z = u1 + bias, e = __expf(-fabsf(z));
-    const float big = __fdividef(1.f, 1.f + e), small = e * big;  // sigmoid(|z|), sigmoid(-|z|)
+    const float z = u1 + bias, e = exp_fast(-fabsf(z));
+    const float big = rcp_fast(1.f + e), small = e * big;  // sigmoid(|z|), sigmoid(-|z|)
     // the smaller of f and 1 - f comes from the small sigmoid and the other by subtraction where needed: gates that
     // are nearly open keep their distance from 1 to full precision over long products
     if (z >= 0.f) {

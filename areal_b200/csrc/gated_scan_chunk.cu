@@ -173,7 +173,7 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
     if (d < DP) {
       const float other = sm.tot[half ^ 1][d], F = run * other;
       far = F < 0x1p-90f;
-      const float inv = far ? 0.f : __fdividef(1.f, F);
+      const float inv = far ? 0.f : rcp_fast(F);
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const int at = (half * 8 + i) * (DP + 8) + d;

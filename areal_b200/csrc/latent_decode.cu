@@ -138,10 +138,10 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
       // the running maximum is raised only when a score passes it by 2^8 (every tile holds at least one token)
       float corr = 1.f;
       if (mx > m[e] + 8.f) {
-        corr = m[e] == -INFINITY ? 0.f : exp2f(m[e] - mx);
+        corr = m[e] == -INFINITY ? 0.f : ex2_fast(m[e] - mx);
         m[e] = mx;
       }
-      const float w = exp2f(x - m[e]);
+      const float w = ex2_fast(x - m[e]);
       l[e] = l[e] * corr + w;
       const __nv_bfloat16 hi = __float2bfloat16(w);
       reinterpret_cast<__nv_bfloat16*>(sP + r * kLdPPitch)[lane] = hi;
@@ -220,7 +220,7 @@ __global__ void latent_merge_kernel(const float* __restrict__ o_part, const floa
   for (int s = 0; s < nsplit; ++s) m = fmaxf(m, ml[(u * nsplit + s) * 2]);
   for (int s = 0; s < nsplit; ++s) {
     const float ms = ml[(u * nsplit + s) * 2];
-    const float e = ms == -INFINITY ? 0.f : exp2f(ms - m);
+    const float e = ms == -INFINITY ? 0.f : ex2_fast(ms - m);
     l += ml[(u * nsplit + s) * 2 + 1] * e;
     if (threadIdx.x == 0) w[s] = e;
   }

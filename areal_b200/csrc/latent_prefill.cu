@@ -12,6 +12,7 @@
 //     (32 columns), and P V is two products with the A operand read from TMEM, so the weights keep fp32-like precision
 //     and take no shared memory.
 #include "common/host_utils.h"
+#include "common/io.cuh"
 #include "common/mma16.cuh"
 #include "common/ptx.cuh"
 
@@ -213,7 +214,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
           tc_fence_after();
         }
         const float mn = grow ? mx : m;
-        const float alpha = m == -INFINITY ? (mn == -INFINITY ? 1.f : 0.f) : exp2f(m - mn);
+        const float alpha = m == -INFINITY ? (mn == -INFINITY ? 1.f : 0.f) : ex2_fast(m - mn);
         l *= alpha;
         m = mn;
         if (j > 0) {
@@ -232,7 +233,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       uint32_t hi[32], lo[32];
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
-        const float a = exp2f(s[2 * i] - mref), b = exp2f(s[2 * i + 1] - mref);
+        const float a = ex2_fast(s[2 * i] - mref), b = ex2_fast(s[2 * i + 1] - mref);
         l += a + b;
         hi[i] = split2(a, b, lo[i]);
       }
@@ -300,16 +301,12 @@ static int launch_latent_prefill(const CUtensorMap& tmQ, const CUtensorMap& tmKV
 
 extern "C" {
 
-int b200_latent_prefill_ok(int D, int R, int Dv) {
-  return ((D == 64 || D == 128) && R >= 8 && R <= 64 && R % 8 == 0 && Dv >= 8 && Dv <= 128 && Dv % 8 == 0) ? 0 : -100;
-}
-
-// Contiguous q [T, H * (D + R)], kv [T, H * (D + Dv)], kr [T, R], o [T, H * Dv], 16-byte aligned; scale > 0.
+// Contiguous q [T, H * (D + R)], kv [T, H * (D + Dv)], kr [T, R], o [T, H * Dv], 16-byte aligned.
 int b200_latent_prefill(const void* q, const void* kv, const void* kr, void* o, const void* tiles, int n_tiles, int T,
                         int H, int D, int R, int Dv, float scale, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || n_tiles <= 0) return 0;
-  if (b200_latent_prefill_ok(D, R, Dv)) return -100;
+  if ((D != 64 && D != 128) || R < 8 || R > 64 || R % 8 || Dv < 8 || Dv > 128 || Dv % 8) return -100;
   CUtensorMap tmQ, tmKV, tmR;
   const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const uint64_t wq = static_cast<uint64_t>(H) * (D + R), wkv = static_cast<uint64_t>(H) * (D + Dv);

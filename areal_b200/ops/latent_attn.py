@@ -157,21 +157,41 @@ def _query_rows(meta):
     return got
 
 
+def _pad_heads(t: torch.Tensor, heads: int, width: int, to: int):
+    """``[T, heads, to]`` of ``t [T, heads * width]``, zero-filled."""
+    return torch.nn.functional.pad(t.reshape(t.shape[0], heads, width), (0, to - width))
+
+
+def _latent_prefill_mma(q, kv, kr, meta, H, D, R, Dv, scale):
+    """The tensor-core kernel takes unrotated parts of 64 or 128 and rotated parts and values in steps of 8; other widths
+    are padded with zeros, which add nothing to a score."""
+    T = q.shape[0]
+    Dp, Rp, Vp = (64 if D <= 64 else 128), -(-R // 8) * 8, -(-Dv // 8) * 8
+    if (Dp, Rp) != (D, R):
+        qh = q.view(T, H, D + R)
+        q = torch.cat((_pad_heads(qh[..., :D], H, D, Dp), _pad_heads(qh[..., D:], H, R, Rp)), -1).view(T, -1)
+    if (Dp, Vp) != (D, Dv):
+        kv = torch.cat((_pad_heads(kv[:, :H * D], H, D, Dp).view(T, -1), _pad_heads(kv[:, H * D:], H, Dv, Vp).view(T, -1)), -1)
+    if Rp != R:
+        kr = _pad_heads(kr, 1, R, Rp).view(T, Rp)
+    q, kv, kr = (t if t.is_contiguous() and t.data_ptr() % 16 == 0 else t.contiguous() for t in (q, kv, kr))
+    c = ctypes.c_int
+    out = torch.empty((T, H * Vp), dtype=q.dtype, device=q.device)
+    rc = _lib.kernels().b200_latent_prefill(
+        _lib.ptr(q), _lib.ptr(kv), _lib.ptr(kr), _lib.ptr(out), _lib.ptr(meta.fwd_tiles), c(meta.n_fwd), c(T), c(H), c(Dp),
+        c(Rp), c(Vp), ctypes.c_float(scale), _lib.stream_ptr())
+    _lib.check(rc, "b200_latent_prefill")
+    _lib.count_launch()
+    return out if Vp == Dv else out.view(T, H, Vp)[..., :Dv].reshape(T, H * Dv)
+
+
 def latent_attention(q, kv, kr, meta, H: int, D: int, rot: int, Dv: int, scale: float):
     """Causal attention of a packed batch: ``q [T, H * (D + rot)]``, ``kv [T, H * D | H * Dv]``, shared rotated part ``kr
     [T, rot]``. Returns ``[T, H * Dv]``."""
     if not kernel_ok(q, kv, kr):
         return latent_attention_ref(q, kv, kr, meta.cu_cpu, H, D, rot, Dv, scale)
-    if (q.dtype == torch.bfloat16 and _lib.kernels().b200_latent_prefill_ok(ctypes.c_int(D), ctypes.c_int(rot), ctypes.c_int(Dv)) == 0
-            and all(t.is_contiguous() and t.data_ptr() % 16 == 0 for t in (q, kv, kr))):
-        c = ctypes.c_int
-        out = torch.empty((q.shape[0], H * Dv), dtype=q.dtype, device=q.device)
-        rc = _lib.kernels().b200_latent_prefill(
-            _lib.ptr(q), _lib.ptr(kv), _lib.ptr(kr), _lib.ptr(out), _lib.ptr(meta.fwd_tiles), c(meta.n_fwd), c(q.shape[0]),
-            c(H), c(D), c(rot), c(Dv), ctypes.c_float(scale), _lib.stream_ptr())
-        _lib.check(rc, "b200_latent_prefill")
-        _lib.count_launch()
-        return out
+    if q.dtype == torch.bfloat16 and D <= 128 and rot <= 64 and Dv <= 128:
+        return _latent_prefill_mma(q, kv, kr, meta, H, D, rot, Dv, scale)
     start, length = _query_rows(meta)
     w = D + rot
     return _attend(q, w, q[:, D:], w, kv, D, kr, 0, kv[:, H * D:], Dv, D, rot, Dv, start, length, None, 1, H, 1, scale)

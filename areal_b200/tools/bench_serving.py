@@ -92,7 +92,8 @@ def serve(cfg: ModelConfig, prompts=8, length=2048, batch=64, steps=20) -> dict:
         r.step([TraceEntry(k, v) for k, v in toks.items()], list(toks))
 
     _lib.reset_launch_count()
-    pre_ms = _timed(prefill, 5, 2)
+    before = set(_lib.fallback_counts())
+    pre_ms = _timed(prefill, 5, 3)
     # decode: the requests enter in groups that fit one prefill step, then all of them step together
     s = eng.sched
     ids = []
@@ -121,20 +122,25 @@ def serve(cfg: ModelConfig, prompts=8, length=2048, batch=64, steps=20) -> dict:
     out = dict(params_m=round(cfg.num_params() / 1e6), prefill_ms=round(pre_ms, 3),
                prefill_tok_s=round(prompts * length / pre_ms * 1e3), decode_ms=round(dec_ms, 3),
                decode_tok_s=round(batch / dec_ms * 1e3), graph=eng._graphs is not None,
-               launches=_lib.launch_count(), fallbacks=sorted(_lib.fallback_counts()))
+               launches=_lib.launch_count(), fallbacks=sorted(set(_lib.fallback_counts()) - before))
     eng.destroy()
     eng.flat = eng.hybrid_state = eng._graphs = None
     return out
 
 
-def main(sizes: list[str], kernels: bool) -> int:
+def main(sizes: list[str], kernels: bool, sampler=None) -> int:
+    """``sampler``: samples the GPU's clocks while the models run (``start`` / ``stop``)."""
     t0 = time.time()
+    if sampler is not None:
+        sampler.start()
     res: dict = {"benchmark": "serving", "layers": LAYERS, "dtype": "bf16", "data": "random tokens, random weights",
                  "prefill": "8 x 2048 tokens", "decode": "64 sequences at 2048 tokens", "models": {}}
     for name in sizes:
         for fam, make in (("fofosun", fofosun_config), ("bailing_hybrid", bailing_config)):
             res["models"][f"{fam}-{name}"] = serve(make(**SIZES[name]))
             torch.cuda.empty_cache()
+    if sampler is not None:
+        res["clocks"] = sampler.stop()
     if kernels:
         from .bench_serving_kernels import run
 

@@ -31,6 +31,7 @@ def _row(name, fn, nbytes=0.0, flops=0.0, iters=10, flush=True):
 @torch.no_grad()
 def run() -> list[dict]:
     out = []
+    torch.manual_seed(0)
     H, D, n, L = 16, 128, 8, 2048
     T = n * L
     meta = VarlenMeta([L * i for i in range(n + 1)], "cuda")

@@ -26,7 +26,7 @@ def parse_args(argv=None) -> argparse.Namespace:
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--out", required=True, help="folder for the logits")
     ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
-    ap.add_argument("--max-requests", type=int, default=64, help="most requests that are live at any time")
+    ap.add_argument("--max-requests", type=int, default=256, help="most requests that are live at any time")
     ap.add_argument("--device", default=None)
     return ap.parse_args(argv)
 

@@ -271,7 +271,8 @@ def main():
     if args.serving:
         from areal_b200.tools import bench_serving
 
-        return bench_serving.main([x for x in args.serving_sizes.split(",") if x], args.serving_kernels)
+        return bench_serving.main([x for x in args.serving_sizes.split(",") if x], args.serving_kernels,
+                                  ClockSampler())
     if args.impl == "libstack":
         # context numbers from the installed libraries (vLLM, HF + FSDP2 + flash-attn, NCCL) on the benchmark's
         # shapes: NOT the reference, never a reference ratio (see baseline/libstack.py)

@@ -122,7 +122,7 @@ def _scan_oracle(x, spec, lens):
     return torch.cat(outs), states
 
 
-SCAN_SHAPES = [(1, 5, 3), (3, 24, 40), (2, 32, 32), (4, 64, 32), (3, 64, 128), (2, 128, 128), (2, 128, 64), (1, 160, 96)]
+SCAN_SHAPES = [(1, 5, 3), (3, 24, 40), (2, 32, 32), (5, 64, 32), (3, 64, 128), (2, 128, 128), (2, 128, 64), (1, 160, 96)]
 
 
 @pytest.mark.parametrize("dt", DTYPES)
@@ -203,7 +203,7 @@ def test_scan_of_a_long_sequence_keeps_what_the_first_token_wrote():
 
 
 @pytest.mark.parametrize("dt", DTYPES)
-@pytest.mark.parametrize("H,D,Dv", [(1, 5, 3), (4, 64, 32), (3, 128, 128)])
+@pytest.mark.parametrize("H,D,Dv", [(1, 5, 3), (5, 64, 32), (3, 128, 128)])
 def test_scan_step_with_the_head_norm(dt, H, D, Dv):
     from areal_b200.ops.gated_scan import scan_step
 
@@ -236,7 +236,7 @@ def _latent_oracle(q, kv, kr, lens, H, D, R, Dv, scale):
 
 
 LATENT_SHAPES = [(1, 5, 2, 3), (3, 24, 8, 40), (2, 64, 32, 64), (4, 64, 64, 32), (3, 128, 64, 128), (2, 128, 32, 64),
-                 (2, 32, 32, 32), (1, 128, 64, 256)]
+                 (2, 32, 16, 48), (2, 64, 8, 24), (1, 128, 64, 256)]
 
 
 @pytest.mark.parametrize("dt", DTYPES)
@@ -261,7 +261,7 @@ def test_latent_attention_of_packed_prompts(dt, H, D, R, Dv):
     _close(got[last], want[last], _tol(dt, 6e-3, 1e-5))
 
 
-DECODE_SHAPES = [(1, 5, 2, 13), (3, 24, 8, 40), (16, 64, 32, 128), (5, 64, 64, 512), (18, 32, 32, 96), (40, 128, 64, 512),
+DECODE_SHAPES = [(1, 5, 2, 13), (3, 24, 8, 40), (16, 64, 32, 128), (5, 64, 64, 512), (18, 32, 16, 112), (40, 128, 64, 512),
                  (2, 16, 16, 16), (8, 64, 32, 192)]
 
 
