@@ -136,7 +136,7 @@ def create_app(engine) -> FastAPI:
 def build_engine(args: argparse.Namespace):
     from .rollout_engine import NativeRolloutEngine
 
-    native = NativeRolloutConfig(model_path=args.model_path or "", model_preset=args.model_preset,
+    native = NativeRolloutConfig(model_path=args.model_path or "", model_preset=args.model_preset, dtype=args.dtype,
                                  context_length=args.context_length, max_num_seqs=args.max_num_seqs,
                                  max_num_batched_tokens=args.max_num_batched_tokens, seed=args.seed,
                                  cuda_graph=not args.disable_cuda_graph, num_kv_blocks=args.num_kv_blocks)
@@ -157,6 +157,8 @@ def parse_args(argv=None) -> argparse.Namespace:
     ap.add_argument("--max-num-seqs", type=int, default=512)
     ap.add_argument("--max-num-batched-tokens", type=int, default=16384)
     ap.add_argument("--num-kv-blocks", type=int, default=None)
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
+                    help="float32: true 32-bit serving (families whose kernels have a 32-bit form, e.g. fofosun)")
     ap.add_argument("--seed", type=int, default=1)
     ap.add_argument("--device", default=None)
     ap.add_argument("--disable-cuda-graph", action="store_true")
