@@ -27,6 +27,7 @@ import ctypes
 import hashlib
 import os
 import dataclasses
+import gc
 import threading
 import time
 from concurrent.futures import Future
@@ -194,6 +195,17 @@ class _DecodeGraphs:
         return (*sample(logits, self.temp[:b], None, None, self.u[:b]), hidden)
 
     def capture_all(self, stream):
+        # a graph of an engine that is garbage must not be destroyed in the middle of a capture: that invalidates it
+        gc.collect()
+        enabled = gc.isenabled()
+        gc.disable()
+        try:
+            self._capture_all(stream)
+        finally:
+            if enabled:
+                gc.enable()
+
+    def _capture_all(self, stream):
         with torch.cuda.stream(stream), torch.no_grad():
             for b in reversed(self.sizes):  # largest first: the shared pool is sized once
                 self._forward(b)  # warm-up outside capture (kernel attributes, workspace)
@@ -296,6 +308,7 @@ class NativeRolloutEngine(InferenceEngine):
         self.vision_tower_images = 0  # images that went through the tower (cache misses)
         self._lock = threading.Lock()
         self._executor = None
+        self._graphs = None
         self._gen_tokens = 0
         self._steps = 0
         self._step_error: BaseException | None = None
@@ -453,6 +466,7 @@ class NativeRolloutEngine(InferenceEngine):
             self._executor.destroy()
         if self.sched is not None:
             self.sched.close()
+        self._graphs = None  # releases the captured graphs now rather than at some later garbage collection
         self.kv_caches = None
         self.model = None
 
