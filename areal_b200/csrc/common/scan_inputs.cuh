@@ -17,28 +17,41 @@ struct ScanArgs {
   int H, D, Dv, mode;
 };
 
-// x sigmoid(x) with the hardware exponential and reciprocal (a few ulp; -0 where exp(-x) overflows)
+// x sigmoid(x): bf16 models take the hardware exponential and reciprocal (a few ulp; -0 where exp(-x) overflows), 32-bit
+// models the library's.
 __device__ __forceinline__ float silu_fast(float x) { return x * rcp_fast(1.f + exp_fast(-x)); }
+__device__ __forceinline__ float silu_as(float x, const __nv_bfloat16*) { return silu_fast(x); }
+__device__ __forceinline__ float silu_as(float x, const float*) { return x / (1.f + expf(-x)); }
+// sigmoid(|z|) and sigmoid(-|z|)
+__device__ __forceinline__ float2 sigmoid_pair(float z, const __nv_bfloat16*) {
+  const float e = exp_fast(-fabsf(z)), big = rcp_fast(1.f + e);
+  return make_float2(big, e * big);
+}
+__device__ __forceinline__ float2 sigmoid_pair(float z, const float*) {
+  const float e = expf(-fabsf(z));
+  return make_float2(1.f / (1.f + e), e / (1.f + e));
+}
 
 // q, f and k of one channel from the two projections u0, u1 (mode 0: with the channel's gate bias and lower bound;
 // mode 1: with the head's decay).
-__device__ __forceinline__ void scan_activate(int mode, float u0, float u1, float bias, float low, float decay, float& q,
-                                              float& f, float& k) {
-  q = silu_fast(u0);
+template <class T>
+__device__ __forceinline__ void scan_activate(const T* tag, int mode, float u0, float u1, float bias, float low,
+                                              float decay, float& q, float& f, float& k) {
+  q = silu_as(u0, tag);
   if (mode == 0) {
-    const float z = u1 + bias, e = exp_fast(-fabsf(z));
-    const float big = rcp_fast(1.f + e), small = e * big;  // sigmoid(|z|), sigmoid(-|z|)
+    const float z = u1 + bias;
+    const float2 s = sigmoid_pair(z, tag);
     // the smaller of f and 1 - f comes from the small sigmoid and the other by subtraction where needed: gates that
     // are nearly open keep their distance from 1 to full precision over long products
     if (z >= 0.f) {
-      k = (1.f - low) * small;
+      k = (1.f - low) * s.y;
       f = 1.f - k;
     } else {
-      k = (1.f - low) * big;
-      f = fmaf(1.f - low, small, low);
+      k = (1.f - low) * s.x;
+      f = fmaf(1.f - low, s.y, low);
     }
   } else {
-    k = silu_fast(u1);
+    k = silu_as(u1, tag);
     f = decay;
   }
 }
@@ -47,7 +60,7 @@ __device__ __forceinline__ void scan_channel(const ScanArgs& a, const T* row, in
                                              float& k) {
   const int hd = h * a.D + d;
   const bool gated = a.mode == 0;
-  scan_activate(a.mode, ld1(row + hd), ld1(row + a.H * a.D + hd), gated ? ld1(static_cast<const T*>(a.bias) + hd) : 0.f,
+  scan_activate(row, a.mode, ld1(row + hd), ld1(row + a.H * a.D + hd), gated ? ld1(static_cast<const T*>(a.bias) + hd) : 0.f,
                 gated ? ld1(static_cast<const T*>(a.lower) + hd) : 0.f, gated ? 0.f : a.decay[h], q, f, k);
 }
 // The value of a bf16 model is a bf16 number in both modes (the activated projection is rounded), so it enters tensor
@@ -57,7 +70,7 @@ __device__ __forceinline__ float round_as(float v, const __nv_bfloat16*) { retur
 template <class T>
 __device__ __forceinline__ float scan_value(const ScanArgs& a, const T* row, int h, int j) {
   const float v = ld1(row + 2 * a.H * a.D + h * a.Dv + j);
-  return a.mode == 0 ? v : round_as(silu_fast(v), row);
+  return a.mode == 0 ? v : round_as(silu_as(v, row), row);
 }
 
 }  // namespace b200

@@ -145,7 +145,7 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
       const int tok = half * 8 + i;
       q[i] = 0.f; k[i] = 0.f; f[i] = 1.f;
       if (dch && t0 + tok < seg.y)
-        scan_activate(mode, __bfloat162float(sm.raw[st][0][tok * 128 + d]), __bfloat162float(sm.raw[st][1][tok * 128 + d]),
+        scan_activate(x, mode, __bfloat162float(sm.raw[st][0][tok * 128 + d]), __bfloat162float(sm.raw[st][1][tok * 128 + d]),
                       bias, low, decay, q[i], f[i], k[i]);
       run *= f[i];
       q[i] *= run;  // q_i P_i, still without the gates of the first half
@@ -230,7 +230,7 @@ __global__ void __launch_bounds__(kScThreads, 2) scan_chunk_kernel(ScanChunkArgs
                 float qq, ff, kk;
                 const bool gated = mode == 0;
                 const int hd = h * D + c;
-                scan_activate(mode, __bfloat162float(sm.raw[st][0][i * 128 + c]), __bfloat162float(sm.raw[st][1][i * 128 + c]),
+                scan_activate(x, mode, __bfloat162float(sm.raw[st][0][i * 128 + c]), __bfloat162float(sm.raw[st][1][i * 128 + c]),
                               gated ? ld1(static_cast<const __nv_bfloat16*>(a.s.bias) + hd) : 0.f,
                               gated ? ld1(static_cast<const __nv_bfloat16*>(a.s.lower) + hd) : 0.f, decay_h, qq, ff, kk);
                 w[e] = i == j ? kk : w[e] * ff;
