@@ -68,4 +68,19 @@ __device__ __forceinline__ float tanh_as(float x, const __nv_bfloat16*) {
 __device__ __forceinline__ float sigmoid_as(float x, const float*) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float sigmoid_as(float x, const __nv_bfloat16*) { return rcp_fast(1.f + exp_fast(-x)); }
 
+// Gated activation g' * sigmoid(alpha * g') * (u' + beta) with g' = min(g, limit) and u' clamped to [-limit, limit]
+// (limit: infinity for none). SwiGLU is alpha 1, beta 0. The pointer names the result's dtype.
+struct GluParams {
+  float limit, alpha, beta;
+};
+template <class T>
+__device__ __forceinline__ float glu_act(float g, float u, GluParams p, const T*) {
+  g = fminf(g, p.limit);
+  u = fminf(fmaxf(u, -p.limit), p.limit);
+  return g * sigmoid_as(p.alpha * g, static_cast<const T*>(nullptr)) * (u + p.beta);
+}
+__device__ __forceinline__ float glu_act(float g, float u, GluParams p, const __nv_bfloat162*) {
+  return glu_act(g, u, p, static_cast<const __nv_bfloat16*>(nullptr));
+}
+
 }  // namespace b200

@@ -96,6 +96,28 @@ struct StoreEpi {
   }
 };
 
+// relu(x)^2 behind the product, on the fp32 accumulators (N % 8 == 0)
+struct Relu2Epi {
+  StoreEpi st;
+  using State = StoreEpi::State;
+  __device__ __forceinline__ bool tile(int cta, int ncta, int it, int tiles_m, int tiles_n, int& m_blk,
+                                       int& n_blk) const {
+    return default_tile(cta, ncta, it, tiles_m, tiles_n, m_blk, n_blk);
+  }
+  __device__ __forceinline__ bool gate(int, int, volatile int*, int*) const { return true; }
+  __device__ __forceinline__ void begin(State&, int, int, int) const {}
+  __device__ __forceinline__ void end(State&, int, int, int) const {}
+  __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
+    float u[32];
+#pragma unroll
+    for (int i = 0; i < 32; ++i) {
+      const float x = fmaxf(v[i], 0.f);
+      u[i] = x * x;
+    }
+    st.chunk(s, row, col0, u);
+  }
+};
+
 template <int BN, bool A_MN, bool B_MN>
 static int launch(const void* A, const void* B, void* C, const void* bias, int M, int N, int K,
                   long long lda, long long ldb, long long ldc, int out_fp32, int accumulate,
@@ -141,6 +163,7 @@ struct GroupedEpi {
   const int* tile_expert;
   const int* num_vm;
   int b_rows_per_expert;  // rows of the stacked B that belong to one expert
+  const int* src_of;      // when given, rows of padding (negative entries) are not written
   using State = StoreEpi::State;
 
   __device__ __forceinline__ bool tile(int cta, int ncta, int it, int, int tiles_n, int& m_blk, int& n_blk) const {
@@ -155,7 +178,46 @@ struct GroupedEpi {
   __device__ __forceinline__ void begin(State&, int, int, int) const {}
   __device__ __forceinline__ void end(State&, int, int, int) const {}
   __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
+    if (src_of && src_of[row] < 0) return;
     st.chunk(s, row, col0, v);
+  }
+};
+
+// The experts' first product with its gated activation on the accumulators. Gate and up rows of the weight alternate
+// (row 2i: gate i, row 2i + 1: up i), so neighbouring columns meet in one thread and half as many are written.
+struct GroupedGluEpi {
+  __nv_bfloat16* out;     // [rows, inter]
+  GluParams glu;
+  int inter;              // N / 2, a multiple of 8
+  const int *tile_expert, *num_vm, *src_of;
+  struct State { bool live; };
+
+  __device__ __forceinline__ bool tile(int cta, int ncta, int it, int, int tiles_n, int& m_blk, int& n_blk) const {
+    const long long t = static_cast<long long>(it) * ncta + cta;
+    if (t >= static_cast<long long>(*num_vm) * tiles_n) return false;
+    m_blk = static_cast<int>(t / tiles_n);
+    n_blk = static_cast<int>(t % tiles_n);
+    return true;
+  }
+  __device__ __forceinline__ int b_offset(int m_blk) const { return tile_expert[m_blk] * 2 * inter; }
+  __device__ __forceinline__ bool gate(int, int, volatile int*, int*) const { return true; }
+  __device__ __forceinline__ void begin(State& s, int, int, int row) const { s.live = src_of[row] >= 0; }
+  __device__ __forceinline__ void end(State&, int, int, int) const {}
+  __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
+    if (!s.live) return;
+    __nv_bfloat16* p = out + static_cast<long long>(row) * inter + col0 / 2;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      if (col0 / 2 + 8 * i >= inter) break;
+      uint4 o;
+      __nv_bfloat162* ob = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int c = 16 * i + 4 * j;
+        ob[j] = __floats2bfloat162_rn(glu_act(v[c], v[c + 1], glu, ob), glu_act(v[c + 2], v[c + 3], glu, ob));
+      }
+      reinterpret_cast<uint4*>(p)[i] = o;
+    }
   }
 };
 
@@ -188,7 +250,7 @@ struct GroupedWgradEpi {
 
 template <bool B_MN>
 static int launch_grouped(const void* A, const void* B, void* C, const int* tile_expert, const int* num_vm,
-                          int max_rows, int E, int N, int K, cudaStream_t stream) {
+                          int max_rows, int E, int N, int K, const int* src_of, cudaStream_t stream) {
   constexpr int BN = 128;
   using Cfg = GemmCfg<BN>;
   CUtensorMap tmA, tmB;
@@ -199,7 +261,7 @@ static int launch_grouped(const void* A, const void* B, void* C, const int* tile
   else       // stacked [E*N, K], K contiguous
     rc = make_tmap_2d(&tmB, B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (long long)E * N, K, (long long)K * 2, BN, 64);
   if (rc) return rc;
-  GroupedEpi epi{StoreEpi{C, nullptr, N, max_rows, N, 0, 0}, tile_expert, num_vm, B_MN ? K : N};
+  GroupedEpi epi{StoreEpi{C, nullptr, N, max_rows, N, 0, 0}, tile_expert, num_vm, B_MN ? K : N, src_of};
   auto kern = gemm_tcgen05_kernel<BN, false, B_MN, GroupedEpi>;
   static bool attr_set = false;
   if (!attr_set) {
@@ -251,6 +313,7 @@ struct SplitKEpi {
   }
 };
 
+template <bool RELU2>
 __global__ void splitk_reduce_kernel(const float* __restrict__ ws, const __nv_bfloat16* __restrict__ bias,
                                      __nv_bfloat16* __restrict__ out, long long ldc, int M, int N, int S,
                                      long long slice_stride) {
@@ -267,6 +330,10 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ ws, const __nv_bf
     if (bias) {
       acc.x += __bfloat162float(bias[c]); acc.y += __bfloat162float(bias[c + 1]);
       acc.z += __bfloat162float(bias[c + 2]); acc.w += __bfloat162float(bias[c + 3]);
+    }
+    if (RELU2) {
+      acc.x = fmaxf(acc.x, 0.f); acc.y = fmaxf(acc.y, 0.f); acc.z = fmaxf(acc.z, 0.f); acc.w = fmaxf(acc.w, 0.f);
+      acc.x *= acc.x; acc.y *= acc.y; acc.z *= acc.z; acc.w *= acc.w;
     }
     __nv_bfloat162 lo = __floats2bfloat162_rn(acc.x, acc.y), hi = __floats2bfloat162_rn(acc.z, acc.w);
     uint2 pk;
@@ -500,8 +567,49 @@ int b200_gemm_grouped(const void* A, const void* B, void* C, const int* tile_exp
   using namespace b200;
   if (max_rows <= 0 || N <= 0 || K <= 0) return 0;
   if ((N & 7) || (K & 7) || (b_mn && (K % 64))) return -100;
-  return b_mn ? launch_grouped<true>(A, B, C, tile_expert, num_vm, max_rows, E, N, K, stream)
-              : launch_grouped<false>(A, B, C, tile_expert, num_vm, max_rows, E, N, K, stream);
+  return b_mn ? launch_grouped<true>(A, B, C, tile_expert, num_vm, max_rows, E, N, K, nullptr, stream)
+              : launch_grouped<false>(A, B, C, tile_expert, num_vm, max_rows, E, N, K, nullptr, stream);
+}
+
+// The forward product for rows whose padding holds anything: padding rows (src_of < 0) are not written.
+int b200_gemm_grouped_rows(const void* A, const void* B, void* C, const int* tile_expert, const int* num_vm,
+                           const int* src_of, int max_rows, int E, int N, int K, cudaStream_t stream) {
+  using namespace b200;
+  if (max_rows <= 0 || N <= 0 || K <= 0) return 0;
+  if ((N & 7) || (K & 7)) return -100;
+  return launch_grouped<false>(A, B, C, tile_expert, num_vm, max_rows, E, N, K, src_of, stream);
+}
+
+// The same with the gated activation behind it: W stacked [E, 2 * inter, K] with alternating gate and up rows, C [rows,
+// inter]. inter % 8 == 0, K % 8 == 0.
+int b200_gemm_grouped_glu(const void* A, const void* B, void* C, const int* tile_expert, const int* num_vm,
+                          const int* src_of, int max_rows, int E, int inter, int K, float limit, float alpha,
+                          float beta, cudaStream_t stream) {
+  using namespace b200;
+  if (max_rows <= 0 || inter <= 0 || K <= 0) return 0;
+  if ((inter & 7) || (K & 7)) return -100;
+  constexpr int BN = 128;
+  using Cfg = GemmCfg<BN>;
+  const int N = 2 * inter;
+  CUtensorMap tmA, tmB;
+  int rc = make_tmap_2d(&tmA, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, max_rows, K, (long long)K * 2, kBM, 64);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tmB, B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (long long)E * N, K, (long long)K * 2, BN, 64);
+  if (rc) return rc;
+  GroupedGluEpi epi{(__nv_bfloat16*)C, GluParams{limit, alpha, beta}, inter, tile_expert, num_vm, src_of};
+  auto kern = gemm_tcgen05_kernel<BN, false, false, GroupedGluEpi>;
+  static bool attr_set = false;
+  if (!attr_set) {
+    B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
+    attr_set = true;
+  }
+  const long long tiles = static_cast<long long>((max_rows + kBM - 1) / kBM) * ((N + BN - 1) / BN);
+  const int grid = static_cast<int>(tiles < sm_count() ? tiles : sm_count());
+  int* status = device_status_word();
+  if (!status) return -3;
+  kern<<<grid, kGemmThreads, Cfg::kSmemBytes, stream>>>(tmA, tmB, max_rows, N, K, epi, status);
+  B200_CHECK(cudaGetLastError());
+  return 0;
 }
 
 // Grouped wgrad: dW[e] (+)= dY_e^T X_e with dY [max_rows, N], X [max_rows, K] in the padded layout
@@ -585,10 +693,18 @@ int b200_gemm_bf16_splitk(const void* A, const void* B, void* C, const void* bia
   long long rg = (total + 255) / 256;
   const long long maxg = static_cast<long long>(sm_count()) * 8;
   if (rg > maxg) rg = maxg;
-  splitk_reduce_kernel<<<(unsigned)rg, 256, 0, stream>>>(workspace, (const __nv_bfloat16*)bias, (__nv_bfloat16*)C, ldc,
+  splitk_reduce_kernel<false><<<(unsigned)rg, 256, 0, stream>>>(workspace, (const __nv_bfloat16*)bias, (__nv_bfloat16*)C, ldc,
                                                         M, N, S, stride);
   B200_CHECK(cudaGetLastError());
   return 0;
+}
+
+// The split-K product without its reduction, for callers that reduce the slices themselves: slice s of row r starts at
+// workspace + s * stride + r * N.
+int b200_gemm_bf16_splitk_partials(const void* A, const void* B, float* workspace, int M, int N, int K, long long lda,
+                                   long long ldb, int splits, int* S_out, long long* stride_out, cudaStream_t stream) {
+  if ((lda & 7) || (ldb & 7) || (N & 3) || splits < 1) return -100;
+  return launch_splitk_partials(A, B, workspace, M, N, K, lda, ldb, splits, S_out, stride_out, stream);
 }
 
 // Split-K projection followed, in the reduction kernel, by the residual add and RMSNorm:
@@ -625,9 +741,9 @@ int b200_gemm_bf16_splitk_rmsnorm(const void* A, const void* B, const void* bias
 
 }  // extern "C"
 
-template <int BN>
-static int launch_dyt(const void* A, const void* B, const b200::DytTail& tail, int M, int N, int K, long long lda,
-                      long long ldb, cudaStream_t stream) {
+template <int BN, class Epi>
+static int launch_epi(const void* A, const void* B, const Epi& epi, int M, int N, int K, long long lda, long long ldb,
+                      cudaStream_t stream) {
   using namespace b200;
   using Cfg = GemmCfg<BN>;
   CUtensorMap tmA, tmB;
@@ -635,7 +751,7 @@ static int launch_dyt(const void* A, const void* B, const b200::DytTail& tail, i
   if (rc) return rc;
   rc = make_tmap_2d(&tmB, B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, N, K, ldb * 2, BN, 64);
   if (rc) return rc;
-  auto kern = gemm_tcgen05_kernel<BN, false, false, DytEpi<BN>>;
+  auto kern = gemm_tcgen05_kernel<BN, false, false, Epi>;
   static bool attr_set = false;
   if (!attr_set) {
     B200_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmemBytes));
@@ -645,7 +761,7 @@ static int launch_dyt(const void* A, const void* B, const b200::DytTail& tail, i
   const int grid = static_cast<int>(tiles < sm_count() ? tiles : sm_count());
   int* status = device_status_word();
   if (!status) return -3;
-  kern<<<grid, kGemmThreads, Cfg::kSmemBytes, stream>>>(tmA, tmB, M, N, K, DytEpi<BN>{tail, M}, status);
+  kern<<<grid, kGemmThreads, Cfg::kSmemBytes, stream>>>(tmA, tmB, M, N, K, epi, status);
   B200_CHECK(cudaGetLastError());
   return 0;
 }
@@ -675,8 +791,32 @@ int b200_gemm_bf16_dyt(const void* A, const void* B, float* workspace, int M, in
     return 0;
   }
   const long long tiles256 = static_cast<long long>((M + kBM - 1) / kBM) * ((N + 255) / 256);
-  return tiles256 >= 100 ? launch_dyt<256>(A, B, tail, M, N, K, lda, ldb, stream)
-                         : launch_dyt<128>(A, B, tail, M, N, K, lda, ldb, stream);
+  return tiles256 >= 100 ? launch_epi<256>(A, B, DytEpi<256>{tail, M}, M, N, K, lda, ldb, stream)
+                         : launch_epi<128>(A, B, DytEpi<128>{tail, M}, M, N, K, lda, ldb, stream);
+}
+
+// C [M, N] (bf16, pitch N) = relu(A . B^T)^2. splits > 1: split-K with the activation in the reduction. N % 8 == 0.
+int b200_gemm_bf16_relu2(const void* A, const void* B, void* C, float* workspace, int M, int N, int K, long long lda,
+                         long long ldb, int splits, cudaStream_t stream) {
+  using namespace b200;
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((lda & 7) || (ldb & 7) || (N & 7)) return -100;
+  if (splits > 1) {
+    int S = 0;
+    long long stride = 0;
+    const int rc = launch_splitk_partials(A, B, workspace, M, N, K, lda, ldb, splits, &S, &stride, stream);
+    if (rc) return rc;
+    long long rg = (static_cast<long long>(M) * (N >> 2) + 255) / 256;
+    const long long maxg = static_cast<long long>(sm_count()) * 8;
+    if (rg > maxg) rg = maxg;
+    splitk_reduce_kernel<true><<<(unsigned)rg, 256, 0, stream>>>(workspace, nullptr, (__nv_bfloat16*)C, N, M, N, S, stride);
+    B200_CHECK(cudaGetLastError());
+    return 0;
+  }
+  const Relu2Epi epi{StoreEpi{C, nullptr, N, M, N, 0, 0}};
+  const long long tiles256 = static_cast<long long>((M + kBM - 1) / kBM) * ((N + 255) / 256);
+  return tiles256 >= 100 ? launch_epi<256>(A, B, epi, M, N, K, lda, ldb, stream)
+                         : launch_epi<128>(A, B, epi, M, N, K, lda, ldb, stream);
 }
 
 // Per-head products (HeadsEpi). A: [M][lda], head h reads columns [h * a_head, h * a_head + K). W is stacked:

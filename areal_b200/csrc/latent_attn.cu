@@ -4,12 +4,14 @@
 //   latent_prep   splits the down projection's row [q_rank | rank | rot]: RMS norm of the query latent, RMS norm of
 //                 the key / value latent, rotation of the shared key part, write of (latent | rotated part) into the
 //                 cache page of the token
+//   latent_qkv_prep  the same for a projection without query latent, [heads * (dim + rot) | rank | rot]: the queries'
+//                 rotated parts turn in place
 //   rope_pairs    rotates neighbouring pairs (2i, 2i+1) inside a slice of every head, in place
 //   attend        softmax attention of any widths, fp32 throughout: one warp per (query, head). Keys come in two
 //                 parts (per head, shared) and from rows of a packed batch (prefill) or from pages (decode, where the
 //                 per-head part is the latent itself, shared by the heads too, and the queries carry the key
 //                 up-projection). The tensor-core kernels cover the widths of real models; this one covers the rest
-//                 and fp32.
+//                 and fp32. A window bounds how far back a query sees; a gate scales every head's result by a sigmoid.
 #include "common/host_utils.h"
 #include "common/io.cuh"
 
@@ -106,6 +108,73 @@ __global__ void rope_pairs_kernel(T* __restrict__ x, long long ldx, int H, int h
   }
 }
 
+// One block per token; warp 0 takes the latent and the shared key part, the others (or, in a block of one warp, warp 0 as
+// well) the heads' rotated parts.
+template <class T, int V, bool PAIR>
+__global__ void latent_qkv_prep_kernel(T* __restrict__ x, long long ldx, int H, int D, const T* __restrict__ wc,
+                                       const float* __restrict__ cosT, const float* __restrict__ sinT,
+                                       const int* __restrict__ pos, int max_pos,
+                                       const long long* __restrict__ slot_mapping, T* __restrict__ c,
+                                       T* __restrict__ kr, T* __restrict__ cache, long long cache_rows, int rank,
+                                       int rot, float eps) {
+  const long long t = blockIdx.x;
+  const int half = rot >> 1, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int p = min(max(pos[t], 0), max_pos - 1);
+  const float* cr = cosT + static_cast<long long>(p) * half;
+  const float* sr = sinT + static_cast<long long>(p) * half;
+  T* row = x + t * ldx;
+  if (warp == 0) {
+    long long slot = slot_mapping ? slot_mapping[t] : -1;
+    if (slot >= cache_rows) slot = -1;
+    T* dst = slot >= 0 ? cache + slot * (rank + rot) : nullptr;
+    const T* lat = row + static_cast<long long>(H) * (D + rot);
+    float s = 0.f;
+    for (int i = lane * V; i < rank; i += 32 * V) {
+      if (V == 4) {
+        const float4 v = ld4(lat + i);
+        s = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+      } else {
+        s = fmaf(ld1(lat + i), ld1(lat + i), s);
+      }
+    }
+    const float k = 1.f / sqrtf(warp_sum(s) / rank + eps);
+    for (int i = lane * V; i < rank; i += 32 * V) {
+      if (V == 4) {
+        const float4 v = ld4(lat + i), w = ld4(wc + i);
+        const float4 y = make_float4(v.x * k * w.x, v.y * k * w.y, v.z * k * w.z, v.w * k * w.w);
+        if (c) st4(c + t * rank + i, y);
+        if (dst) st4(dst + i, y);
+      } else {
+        const float y = ld1(lat + i) * k * ld1(wc + i);
+        if (c) st1(c + t * rank + i, y);
+        if (dst) st1(dst + i, y);
+      }
+    }
+    lat += rank;
+    for (int i = lane; i < half; i += 32) {
+      const float u = ld1(lat + 2 * i), v = ld1(lat + 2 * i + 1);
+      const float a = u * cr[i] - v * sr[i], b = v * cr[i] + u * sr[i];
+      if (kr) { st1(kr + t * rot + 2 * i, a); st1(kr + t * rot + 2 * i + 1, b); }
+      if (dst) { st1(dst + rank + 2 * i, a); st1(dst + rank + 2 * i + 1, b); }
+    }
+    if (blockDim.x > 32) return;
+  }
+  const int first = blockDim.x > 32 ? threadIdx.x - 32 : threadIdx.x;
+  const int step = blockDim.x > 32 ? blockDim.x - 32 : blockDim.x;
+  for (int i = first; i < H * half; i += step) {
+    const int h = i / half, e = i - h * half;
+    T* q = row + static_cast<long long>(h) * (D + rot) + D + 2 * e;
+    const float2 uv = PAIR ? ld_pair(q) : make_float2(ld1(q), ld1(q + 1));
+    const float a = uv.x * cr[e] - uv.y * sr[e], b = uv.y * cr[e] + uv.x * sr[e];
+    if (PAIR) {
+      st_pair(q, a, b);
+    } else {
+      st1(q, a);
+      st1(q + 1, b);
+    }
+  }
+}
+
 struct AttendArgs {
   const void *qa, *qb;             // query parts: [rows][ld] + h * head stride
   long long ldqa, ldqb;
@@ -124,6 +193,9 @@ struct AttendArgs {
   long long ldo;
   int H, nsplit;
   float scale;
+  int window;                      // a query sees its last `window` keys; 0: all of them
+  const void* gate;                // null, or [n][ldg]: head h's result is multiplied by sigmoid(gate[h])
+  long long ldg;
 };
 
 // grid (n query rows, ceil(H / warps), nsplit)
@@ -138,8 +210,9 @@ __global__ void attend_kernel(AttendArgs a) {
   if (h >= a.H) return;                // whole warp; no block-wide barrier follows
   const long long r = blockIdx.x;
   const int L = a.kv_len[r];
-  const int per = (L + a.nsplit - 1) / a.nsplit;
-  const int k0 = blockIdx.z * per, k1 = min(L, k0 + per);
+  const int lo = a.window > 0 ? max(0, L - a.window) : 0;
+  const int per = (L - lo + a.nsplit - 1) / a.nsplit;
+  const int k0 = lo + blockIdx.z * per, k1 = min(L, k0 + per);
   for (int i = lane; i < a.da; i += 32) q[i] = ld1(static_cast<const T*>(a.qa) + r * a.ldqa + h * a.hqa + i);
   for (int i = lane; i < a.db; i += 32) q[a.da + i] = ld1(static_cast<const T*>(a.qb) + r * a.ldqb + h * a.hqb + i);
   for (int i = lane; i < a.dv; i += 32) acc[i] = 0.f;
@@ -181,7 +254,8 @@ __global__ void attend_kernel(AttendArgs a) {
     }
   }
   if (a.nsplit == 1) {
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (a.gate) inv *= sigmoid_as(ld1(static_cast<const T*>(a.gate) + r * a.ldg + h), static_cast<const T*>(nullptr));
     for (int i = lane; i < a.dv; i += 32)
       st1(static_cast<T*>(a.out) + r * a.ldo + static_cast<long long>(h) * a.dv + i, acc[i] * inv);
   } else {
@@ -194,7 +268,8 @@ __global__ void attend_kernel(AttendArgs a) {
 // Merge of split partials. m in natural-log units when LOG2 is false, in log2 units else.
 template <class T, bool LOG2>
 __global__ void attend_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ ml, T* __restrict__ out,
-                                    long long ldo, int H, int nsplit, int dv) {
+                                    long long ldo, int H, int nsplit, int dv, const T* __restrict__ gate,
+                                    long long ldg) {
   const long long u = blockIdx.x;
   const long long r = u / H;
   const int h = static_cast<int>(u % H);
@@ -205,7 +280,8 @@ __global__ void attend_merge_kernel(const float* __restrict__ o_part, const floa
     const float ms = ml[(u * nsplit + s) * 2];
     if (ms != -INFINITY) l += ml[(u * nsplit + s) * 2 + 1] * (LOG2 ? exp2f(ms - m) : expf(ms - m));
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if (gate) inv *= sigmoid_as(ld1(gate + r * ldg + h), gate);
   for (int i = threadIdx.x; i < dv; i += blockDim.x) {
     float t = 0.f;
     for (int s = 0; s < nsplit; ++s) {
@@ -241,6 +317,33 @@ int b200_latent_prep(const void* x, long long ldx, const void* wq, const void* w
   return 0;
 }
 
+// x [T][ldx]: [H * (D + rot) | rank | rot | ...]; the heads' last rot columns are rotated in place. c, kr, slot_mapping +
+// cache may be null.
+int b200_latent_qkv_prep(void* x, long long ldx, int H, int D, const void* wc, const float* cosT, const float* sinT,
+                         const int* pos, int max_pos, const long long* slot_mapping, void* c, void* kr, void* cache,
+                         long long cache_rows, int T, int rank, int rot, float eps, int fp32, cudaStream_t stream) {
+  using namespace b200;
+  if (T <= 0) return 0;
+  if ((rot & 1) || H < 1 || D < 0) return -100;
+  const long long q = static_cast<long long>(H) * (D + rot);
+  const bool v4 = q % 4 == 0 && rank % 4 == 0 && rot % 4 == 0 && ldx % 4 == 0;
+  const bool pair = !((ldx | D) & 1);
+  int block = 64;
+  while (block < 256 && block < 32 + H * (rot / 2)) block <<= 1;
+#define B200_LQ(T_, V_, P_)                                                                                         \
+  latent_qkv_prep_kernel<T_, V_, P_><<<T, block, 0, stream>>>((T_*)x, ldx, H, D, (const T_*)wc, cosT, sinT, pos,    \
+                                                              max_pos, slot_mapping, (T_*)c, (T_*)kr, (T_*)cache,   \
+                                                              cache_rows, rank, rot, eps)
+#define B200_LQV(T_)                                                                                                \
+  if (v4) { if (pair) B200_LQ(T_, 4, true); else B200_LQ(T_, 4, false); }                                           \
+  else { if (pair) B200_LQ(T_, 1, true); else B200_LQ(T_, 1, false); }
+  if (fp32) { B200_LQV(float) } else { B200_LQV(__nv_bfloat16) }
+#undef B200_LQV
+#undef B200_LQ
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
 // Rotates columns [offset, offset + dims) of every head of x [rows][ldx] in place; tables [max_pos, dims / 2].
 int b200_rope_pairs(void* x, long long ldx, int H, int head_stride, int offset, int dims, const float* cosT,
                     const float* sinT, const int* pos, int max_pos, long long rows, int fp32, cudaStream_t stream) {
@@ -265,11 +368,12 @@ int b200_attend(const void* qa, long long ldqa, int hqa, const void* qb, long lo
                 long long ldka, int hka, const void* kb, long long ldkb, int hkb, const void* v, long long ldv, int hv,
                 int da, int db, int dv, const int* seq_start, const int* kv_len, const int* block_table, int max_blocks,
                 int block_size, float* o_part, float* ml_part, void* out, long long ldo, int n, int H, int nsplit,
-                float scale, int fp32, cudaStream_t stream) {
+                float scale, int window, const void* gate, long long ldg, int fp32, cudaStream_t stream) {
   using namespace b200;
   if (n <= 0) return 0;
   AttendArgs a{qa, qb, ldqa, ldqb, hqa, hqb, ka, kb, v, ldka, ldkb, ldv, hka, hkb, hv, da, db, dv, seq_start, kv_len,
-               block_table, max_blocks, block_size, o_part, ml_part, out, ldo, H, nsplit, scale};
+               block_table, max_blocks, block_size, o_part, ml_part, out, ldo, H, nsplit, scale, window,
+               gate, ldg};
   int nw = H < 4 ? H : 4;
   const size_t per_warp = static_cast<size_t>(da + db + dv) * sizeof(float);
   while (nw > 1 && per_warp * nw > 48 * 1024) nw >>= 1;
@@ -280,10 +384,11 @@ int b200_attend(const void* qa, long long ldqa, int hqa, const void* qb, long lo
   else attend_kernel<__nv_bfloat16><<<grid, nw * 32, smem, stream>>>(a);
   B200_CHECK(cudaGetLastError());
   if (nsplit > 1) {
-    if (fp32) attend_merge_kernel<float, false><<<n * H, 128, 0, stream>>>(o_part, ml_part, (float*)out, ldo, H, nsplit, dv);
+    if (fp32) attend_merge_kernel<float, false><<<n * H, 128, 0, stream>>>(o_part, ml_part, (float*)out, ldo, H, nsplit, dv,
+                                                                                (const float*)gate, ldg);
     else
       attend_merge_kernel<__nv_bfloat16, false><<<n * H, 128, 0, stream>>>(o_part, ml_part, (__nv_bfloat16*)out, ldo, H,
-                                                                          nsplit, dv);
+                                                                          nsplit, dv, (const __nv_bfloat16*)gate, ldg);
     B200_CHECK(cudaGetLastError());
   }
   return 0;

@@ -7,7 +7,8 @@
 // scores of 8 tokens over half of the width; the [16, 32] scores meet in shared memory, every warp takes the softmax of two
 // heads (max, sum and weights in fp32, a lane per token) and, with all heads' weights, multiplies its share of the value
 // columns. The weights enter the product as two bf16 terms
-// (hi + lo), so they keep fp32-like precision.
+// (hi + lo), so they keep fp32-like precision. With a window the walk starts at the tile of the first visible token; a
+// gate scales a head's result by sigmoid(gate[sequence, head]) when it is written.
 #include "common/host_utils.h"
 #include "common/io.cuh"
 #include "common/mma16.cuh"
@@ -30,6 +31,9 @@ struct LatentDecodeArgs {
   float *o_part, *ml_part;
   int H, rank, rot, block_size, max_blocks, nsplit, pitch;  // pitch: bytes of a row in shared memory
   float scale_log2;
+  int window;           // 0: every cached token is visible
+  const __nv_bfloat16* gate;  // null or [B][ldg]
+  long long ldg;
 };
 
 __device__ __forceinline__ uint32_t sa32(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
@@ -48,8 +52,9 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
   const int b = blockIdx.x, h0 = blockIdx.y * 16, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int L = a.seq_lens[b];
-  const int tiles = (L + kLdTok - 1) / kLdTok, per = (tiles + a.nsplit - 1) / a.nsplit;
-  const int j0 = split * per, n = max(0, min(tiles, j0 + per) - j0);
+  const int lo = a.window > 0 ? max(0, L - a.window) : 0;  // first visible token
+  const int tiles = (L + kLdTok - 1) / kLdTok, t0 = lo / kLdTok, per = (tiles - t0 + a.nsplit - 1) / a.nsplit;
+  const int j0 = t0 + split * per, n = max(0, min(tiles, j0 + per) - j0);
   const int* bt = a.block_table + static_cast<long long>(b) * a.max_blocks;
   // queries: 16 rows of W, zero for heads past the last
   for (int i = threadIdx.x; i < 16 * (W / 8); i += blockDim.x) {
@@ -130,7 +135,8 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int r = 2 * warp + e;
-      const bool in = (j0 + j) * kLdTok + lane < L;
+      const int tok = (j0 + j) * kLdTok + lane;
+      const bool in = tok < L && tok >= lo;
       const float x = in ? (sS[r * kLdSPitch + lane] + sS[kHalf + r * kLdSPitch + lane]) * a.scale_log2 : -INFINITY;
       float mx = x;
 #pragma unroll
@@ -192,7 +198,9 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
     const int h = h0 + g + half * 8;
     if (h >= a.H) continue;
     const long long u = (static_cast<long long>(b) * a.H + h);
-    const float sum = sML[(g + half * 8) * 2 + 1], inv = sum > 0.f ? 1.f / sum : 0.f;
+    const float sum = sML[(g + half * 8) * 2 + 1];
+    float inv = sum > 0.f ? 1.f / sum : 0.f;
+    if (direct && a.gate) inv *= sigmoid_as(__bfloat162float(a.gate[b * a.ldg + h]), a.gate);
 #pragma unroll
     for (int i = 0; i < 2 * NP; ++i) {
       const int pr = warp + (i >> 1) * kLdWarps;
@@ -213,7 +221,8 @@ __global__ void __launch_bounds__(kLdWarps * 32, 2) latent_decode_kernel(LatentD
 
 // One block per (sequence, head); threads over the columns, two at a time.
 __global__ void latent_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ ml,
-                                    __nv_bfloat16* __restrict__ out, int nsplit, int rank) {
+                                    __nv_bfloat16* __restrict__ out, int nsplit, int rank,
+                                    const __nv_bfloat16* __restrict__ gate, long long ldg, int H) {
   __shared__ float w[64];
   const long long u = blockIdx.x;
   float m = -INFINITY, l = 0.f;
@@ -225,7 +234,8 @@ __global__ void latent_merge_kernel(const float* __restrict__ o_part, const floa
     if (threadIdx.x == 0) w[s] = e;
   }
   __syncthreads();
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if (gate) inv *= sigmoid_as(__bfloat162float(gate[u / H * ldg + u % H]), gate);
   for (int c = threadIdx.x * 2; c < rank; c += blockDim.x * 2) {
     float x = 0.f, y = 0.f;
     for (int s = 0; s < nsplit; ++s) {
@@ -253,7 +263,7 @@ int b200_latent_decode_ok(int rank, int rot) {
 int b200_latent_decode(const void* qa, long long ldqa, const void* q, long long ldq, int q_stride, int q_off,
                        const void* cache, const int* block_table, int max_blocks, int block_size, const int* seq_lens,
                        void* out, float* o_part, float* ml_part, int B, int H, int rank, int rot, int nsplit,
-                       float scale, cudaStream_t stream) {
+                       float scale, int window, const void* gate, long long ldg, cudaStream_t stream) {
   using namespace b200;
   if (B <= 0) return 0;
   if (b200_latent_decode_ok(rank, rot) || (ldqa & 7) || (ldq & 7) || (q_stride & 7) || (q_off & 7) || nsplit < 1 || nsplit > 64)
@@ -265,7 +275,7 @@ int b200_latent_decode(const void* qa, long long ldqa, const void* q, long long 
   const int smem = fixed + stages * stage;
   LatentDecodeArgs a{(const bf*)qa, (const bf*)q, (const bf*)cache, ldqa, ldq, q_stride, q_off, block_table, seq_lens,
                      (bf*)out, o_part, ml_part, H, rank, rot, block_size, max_blocks, nsplit, pitch,
-                     scale * 1.4426950408889634f};
+                     scale * 1.4426950408889634f, window, (const bf*)gate, ldg};
   dim3 grid(B, (H + 15) / 16, nsplit);
   const int np = (rank / 16 + kLdWarps - 1) / kLdWarps;
 #define B200_LDS(NP_, ST_)                                                                                          \
@@ -283,7 +293,8 @@ int b200_latent_decode(const void* qa, long long ldqa, const void* q, long long 
 #undef B200_LDS
   B200_CHECK(cudaGetLastError());
   if (nsplit > 1) {
-    latent_merge_kernel<<<B * H, rank >= 256 ? 256 : 128, 0, stream>>>(o_part, ml_part, (bf*)out, nsplit, rank);
+    latent_merge_kernel<<<B * H, rank >= 256 ? 256 : 128, 0, stream>>>(o_part, ml_part, (bf*)out, nsplit, rank,
+                                                                                (const bf*)gate, ldg, H);
     B200_CHECK(cudaGetLastError());
   }
   return 0;

@@ -11,6 +11,8 @@
 //   * the softmax weights stay in TMEM. They overwrite their own score buffer as two bf16 terms, hi (32 columns) and lo
 //     (32 columns), and P V is two products with the A operand read from TMEM, so the weights keep fp32-like precision
 //     and take no shared memory.
+//   * a window (query i sees keys i - window + 1 .. i) starts a tile's walk at the first block that any of its queries
+//     sees; a gate scales a head's result by sigmoid(gate[token, head]) on the way out.
 #include "common/host_utils.h"
 #include "common/io.cuh"
 #include "common/mma16.cuh"
@@ -50,7 +52,8 @@ template <int ND, int NV>
 __global__ void __launch_bounds__(kLpThreads, 2)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmKV,
                       const __grid_constant__ CUtensorMap tmR, const LatentTile* __restrict__ tiles,
-                      __nv_bfloat16* __restrict__ o, int H, int R, int Dv, float scale_log2, int* status) {
+                      __nv_bfloat16* __restrict__ o, int H, int R, int Dv, float scale_log2, int window,
+                      const __nv_bfloat16* __restrict__ gate, long long ldg, int* status) {
   using C = LpCfg<ND, NV>;
   constexpr int D = ND * 64, VS = C::kVStages;
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -66,7 +69,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const LatentTile tile = tiles[blockIdx.x];
   const int h = blockIdx.y;
-  const int nblk = (tile.kv_len + kLpK - 1) / kLpK;
+  const int blk0 = window > 0 ? max(0, tile.q_off - window + 1) / kLpK : 0;  // first block that a query of the tile sees
+  const int nblk = (tile.kv_len + kLpK - 1) / kLpK - blk0;
 
   if (threadIdx.x == 0) {
     abort_word = 0;
@@ -109,7 +113,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       for (int c = 0; c <= ND; ++c) tma_load_2d(sQ + c * C::kQBlk, &tmQ, q_full, h * (D + R) + c * 64, tile.q_start);
       bool ok = true;
       for (int j = 0; j < nblk; ++j) {
-        const int st = j & 1, row = tile.kv_start + j * kLpK;
+        const int st = j & 1, row = tile.kv_start + (blk0 + j) * kLpK;
         if (!mbar_wait(&k_empty[st], ((j >> 1) & 1) ^ 1, abort_flag)) { ok = false; break; }
         mbar_arrive_expect_tx(&k_full[st], C::kK);
         uint8_t* k = sK + st * C::kK;
@@ -179,7 +183,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     // ----------------------------------------------------------- softmax --
     const int r = warp * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
-    const int q_pos = tile.q_off + r;
+    const int q_pos = tile.q_off + r, q_lo = window > 0 ? q_pos - window + 1 : 0;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < nblk; ++j) {
@@ -195,11 +199,13 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 #pragma unroll
         for (int i = 0; i < 32; ++i) s[c * 32 + i] = __uint_as_float(raw[i]) * scale_log2;
       }
-      const int kv0 = j * kLpK;
-      if (kv0 + kLpK - 1 > tile.q_off || kv0 + kLpK > tile.kv_len) {  // the diagonal, or the end of the tile's keys
+      const int kv0 = (blk0 + j) * kLpK;
+      // the diagonal, the end of the tile's keys, or the window's edge for the tile's last query
+      if (kv0 + kLpK - 1 > tile.q_off || kv0 + kLpK > tile.kv_len ||
+          (window > 0 && kv0 < tile.q_off + kLpQ - window)) {
 #pragma unroll
         for (int i = 0; i < kLpK; ++i)
-          if (kv0 + i > q_pos || kv0 + i >= tile.kv_len) s[i] = -INFINITY;
+          if (kv0 + i > q_pos || kv0 + i >= tile.kv_len || kv0 + i < q_lo) s[i] = -INFINITY;
       }
       float mx = s[0];
 #pragma unroll
@@ -249,7 +255,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       tc_fence_after();
     }
     if (ok) {
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (gate && r < tile.q_len)
+        inv *= sigmoid_as(__bfloat162float(gate[static_cast<long long>(tile.q_start + r) * ldg + h]), gate);
       __nv_bfloat16* orow = o + (static_cast<long long>(tile.q_start + r) * H + h) * Dv;
 #pragma unroll 1
       for (int c = 0; c < NV * 2; ++c) {
@@ -285,14 +293,15 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 
 template <int ND, int NV>
 static int launch_latent_prefill(const CUtensorMap& tmQ, const CUtensorMap& tmKV, const CUtensorMap& tmR, const void* tiles,
-                                 int n_tiles, void* o, int H, int R, int Dv, float scale, cudaStream_t stream) {
+                                 int n_tiles, void* o, int H, int R, int Dv, float scale, int window,
+                                 const void* gate, long long ldg, cudaStream_t stream) {
   constexpr int smem = LpCfg<ND, NV>::kSmem;
   B200_CHECK(cudaFuncSetAttribute(latent_prefill_kernel<ND, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
   int* status = device_status_word();
   if (!status) return -3;
   latent_prefill_kernel<ND, NV><<<dim3(n_tiles, H), kLpThreads, smem, stream>>>(
       tmQ, tmKV, tmR, reinterpret_cast<const LatentTile*>(tiles), (__nv_bfloat16*)o, H, R, Dv,
-      scale * 1.4426950408889634f, status);
+      scale * 1.4426950408889634f, window, (const __nv_bfloat16*)gate, ldg, status);
   B200_CHECK(cudaGetLastError());
   return 0;
 }
@@ -301,26 +310,28 @@ static int launch_latent_prefill(const CUtensorMap& tmQ, const CUtensorMap& tmKV
 
 extern "C" {
 
-// Contiguous q [T, H * (D + R)], kv [T, H * (D + Dv)], kr [T, R], o [T, H * Dv], 16-byte aligned.
-int b200_latent_prefill(const void* q, const void* kv, const void* kr, void* o, const void* tiles, int n_tiles, int T,
-                        int H, int D, int R, int Dv, float scale, cudaStream_t stream) {
+// q [T][ldq] (H * (D + R) columns, pitch a multiple of 8); contiguous kv [T, H * (D + Dv)], kr [T, R], o [T, H * Dv]; all
+// 16-byte aligned. window: 0 for none. gate: null or [T][ldg], one number per head.
+int b200_latent_prefill(const void* q, long long ldq, const void* kv, const void* kr, void* o, const void* tiles,
+                        int n_tiles, int T, int H, int D, int R, int Dv, float scale, int window, const void* gate,
+                        long long ldg, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || n_tiles <= 0) return 0;
-  if ((D != 64 && D != 128) || R < 8 || R > 64 || R % 8 || Dv < 8 || Dv > 128 || Dv % 8) return -100;
+  if ((D != 64 && D != 128) || R < 8 || R > 64 || R % 8 || (ldq & 7) || Dv < 8 || Dv > 128 || Dv % 8) return -100;
   CUtensorMap tmQ, tmKV, tmR;
   const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const uint64_t wq = static_cast<uint64_t>(H) * (D + R), wkv = static_cast<uint64_t>(H) * (D + Dv);
-  int rc = make_tmap_2d(&tmQ, q, bf, 2, T, wq, wq * 2, kLpQ, 64);
+  int rc = make_tmap_2d(&tmQ, q, bf, 2, T, wq, static_cast<uint64_t>(ldq) * 2, kLpQ, 64);
   if (rc) return rc;
   rc = make_tmap_2d(&tmKV, kv, bf, 2, T, wkv, wkv * 2, kLpK, 64);
   if (rc) return rc;
   rc = make_tmap_2d(&tmR, kr, bf, 2, T, R, static_cast<uint64_t>(R) * 2, kLpK, 64);
   if (rc) return rc;
   if (D == 64)
-    return Dv <= 64 ? launch_latent_prefill<1, 1>(tmQ, tmKV, tmR, tiles, n_tiles, o, H, R, Dv, scale, stream)
-                    : launch_latent_prefill<1, 2>(tmQ, tmKV, tmR, tiles, n_tiles, o, H, R, Dv, scale, stream);
-  return Dv <= 64 ? launch_latent_prefill<2, 1>(tmQ, tmKV, tmR, tiles, n_tiles, o, H, R, Dv, scale, stream)
-                  : launch_latent_prefill<2, 2>(tmQ, tmKV, tmR, tiles, n_tiles, o, H, R, Dv, scale, stream);
+    return Dv <= 64 ? launch_latent_prefill<1, 1>(tmQ, tmKV, tmR, tiles, n_tiles, o, H, R, Dv, scale, window, gate, ldg, stream)
+                    : launch_latent_prefill<1, 2>(tmQ, tmKV, tmR, tiles, n_tiles, o, H, R, Dv, scale, window, gate, ldg, stream);
+  return Dv <= 64 ? launch_latent_prefill<2, 1>(tmQ, tmKV, tmR, tiles, n_tiles, o, H, R, Dv, scale, window, gate, ldg, stream)
+                  : launch_latent_prefill<2, 2>(tmQ, tmKV, tmR, tiles, n_tiles, o, H, R, Dv, scale, window, gate, ldg, stream);
 }
 
 }  // extern "C"

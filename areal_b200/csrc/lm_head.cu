@@ -18,8 +18,25 @@
 // 3-4 all-reduces (areal/utils/functional/vocab_parallel.py:84-372).
 #include "common/gemm_core.cuh"
 #include "common/host_utils.h"
+#include "common/io.cuh"
 
 namespace b200 {
+
+// Soft cap of the logits, cap * tanh(z / cap), ahead of the temperature; cap 0: none. `slope`: the derivative, from the
+// capped logit.
+struct SoftCap {
+  float cap, inv;
+  __device__ __forceinline__ void apply(const float (&v)[32], float (&z)[32]) const {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) z[i] = v[i];
+    if (cap > 0.f) {  // one branch for all columns: models without a cap pay no tanh
+#pragma unroll
+      for (int i = 0; i < 32; ++i) z[i] = cap * tanh_as(z[i] * inv, static_cast<const __nv_bfloat16*>(nullptr));
+    }
+  }
+  __device__ __forceinline__ float slope(float capped) const { return 1.f - (capped * inv) * (capped * inv); }
+};
+static SoftCap soft_cap(float cap) { return SoftCap{cap, cap > 0.f ? 1.f / cap : 0.f}; }
 
 struct LmStatsEpi {
   float* partials;          // [nsplit, T, 4] : m, l, sx, target
@@ -34,6 +51,7 @@ struct LmStatsEpi {
   int nb_per;               // n-blocks per split
   int nsplit;
   float inv_temp;
+  SoftCap cap;
   struct State {
     float m, l, sx, t;
   };
@@ -60,10 +78,11 @@ struct LmStatsEpi {
     if (row >= T || col0 >= N) return;
     const int label = labels[row] - vocab_start;
     float x[32];
+    cap.apply(v, x);
     float cm = -INFINITY;
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
-      x[i] = (col0 + i < N) ? v[i] * inv_temp : -INFINITY;
+      x[i] = (col0 + i < N) ? x[i] * inv_temp : -INFINITY;
       cm = fmaxf(cm, x[i]);
     }
     if (label >= col0 && label < col0 + 32) {
@@ -135,6 +154,7 @@ struct LmDlogitsEpi {
   long long ldz;
   int T, N, vocab_start;
   float inv_temp;
+  SoftCap cap;
   struct State {
     float gl, ge, lz, e;
     int label;
@@ -157,12 +177,13 @@ struct LmDlogitsEpi {
   __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
     if (row >= T || col0 >= N) return;
     float d[32];
+    cap.apply(v, d);
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
-      const float y = v[i] * inv_temp;
+      const float z = d[i], y = z * inv_temp;
       const float p = __expf(y - s.lz);
       const float onehot = (col0 + i == s.label) ? 1.f : 0.f;
-      d[i] = (s.gl * (onehot - p) + s.ge * p * (s.e - y)) * inv_temp;
+      d[i] = (s.gl * (onehot - p) + s.ge * p * (s.e - y)) * inv_temp * cap.slope(z);  // (no cap: slope 1)
     }
     __nv_bfloat16* out = dz + static_cast<long long>(row) * ldz + col0;
     if (col0 + 32 <= N && (ldz & 7) == 0) {
@@ -226,6 +247,7 @@ struct LmSampleEpi {
   const unsigned long long* rng;  // [0] seed, [1] step counter
   int T, N;
   int nb_per, nsplit;
+  SoftCap cap;
   struct State {
     float m, l, best, bx, inv_t;
     int bi;
@@ -262,10 +284,11 @@ struct LmSampleEpi {
   __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
     if (row >= T || col0 >= N) return;
     float x[32];
+    cap.apply(v, x);
     float cm = -INFINITY;
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
-      x[i] = (col0 + i < N) ? v[i] * s.inv_t : -INFINITY;
+      x[i] = (col0 + i < N) ? x[i] * s.inv_t : -INFINITY;
       cm = fmaxf(cm, x[i]);
     }
     const float m_new = fmaxf(s.m, cm);
@@ -396,14 +419,15 @@ int b200_lm_head_nsplit(int T, int V) {
 // partials: fp32 [nsplit, T, 4] with nsplit = b200_lm_head_nsplit(T, V).
 int b200_lm_head_stats(const void* X, const void* W, const int* labels, float* partials, int T,
                        int V, int H, long long ldx, long long ldw, int vocab_start,
-                       float inv_temp, cudaStream_t stream) {
+                       float inv_temp, float softcap, cudaStream_t stream) {
   using namespace b200;
   if (T == 0 || V == 0) return 0;
   const int tiles_m = (T + 127) / 128;
   const int tiles_n = (V + 255) / 256;
   const int nsplit = b200_lm_head_nsplit(T, V);
   const int nb_per = (tiles_n + nsplit - 1) / nsplit;
-  LmStatsEpi epi{partials, {}, 0, 0, labels, T, V, vocab_start, nb_per, nsplit, inv_temp};
+  LmStatsEpi epi{partials, {}, 0, 0, labels, T, V, vocab_start, nb_per, nsplit, inv_temp,
+                 soft_cap(softcap)};
   return launch_lm(X, W, T, V, H, ldx, ldw, epi, static_cast<long long>(tiles_m) * nsplit,
                    stream);
 }
@@ -414,7 +438,7 @@ int b200_lm_head_stats(const void* X, const void* W, const int* labels, float* p
 // among the ranks must separate this launch from b200_lm_head_combine over the local buffer.
 int b200_lm_head_stats_peers(const void* X, const void* W, const int* labels, void* const* peer_partials,
                              int n_peers, int rank, int T, int V, int H, long long ldx, long long ldw,
-                             int vocab_start, float inv_temp, cudaStream_t stream) {
+                             int vocab_start, float inv_temp, float softcap, cudaStream_t stream) {
   using namespace b200;
   if (n_peers < 1 || n_peers > 8) return -100;
   if (T == 0 || V == 0) return 0;
@@ -422,7 +446,8 @@ int b200_lm_head_stats_peers(const void* X, const void* W, const int* labels, vo
   const int tiles_n = (V + 255) / 256;
   const int nsplit = b200_lm_head_nsplit(T, V);
   const int nb_per = (tiles_n + nsplit - 1) / nsplit;
-  LmStatsEpi epi{nullptr, {}, n_peers, rank * nsplit, labels, T, V, vocab_start, nb_per, nsplit, inv_temp};
+  LmStatsEpi epi{nullptr, {}, n_peers, rank * nsplit, labels, T, V, vocab_start, nb_per, nsplit, inv_temp,
+                 soft_cap(softcap)};
   for (int p = 0; p < n_peers; ++p) epi.peers[p] = reinterpret_cast<float*>(peer_partials[p]);
   return launch_lm(X, W, T, V, H, ldx, ldw, epi, static_cast<long long>(tiles_m) * nsplit, stream);
 }
@@ -459,13 +484,14 @@ int b200_lm_head_sample_nsplit(int B, int V) {
 // rng: two 64-bit words on the device (seed, step counter), the counter is advanced by one.
 int b200_lm_head_sample(const void* X, const void* W, const float* temperature, void* partials, int* part_idx,
                         unsigned long long* rng, int* tokens, float* logprobs, int B, int V, int H,
-                        long long ldx, long long ldw, cudaStream_t stream) {
+                        long long ldx, long long ldw, float softcap, cudaStream_t stream) {
   using namespace b200;
   if (B == 0 || V == 0) return 0;
   const int tiles_m = (B + 127) / 128;
   const int nb_per = b200_lm_head_sample_nb_per(B, V);
   const int nsplit = b200_lm_head_sample_nsplit(B, V);
-  LmSampleEpi epi{reinterpret_cast<LmSampleRec*>(partials), part_idx, temperature, rng, B, V, nb_per, nsplit};
+  LmSampleEpi epi{reinterpret_cast<LmSampleRec*>(partials), part_idx, temperature, rng, B, V, nb_per, nsplit,
+                  soft_cap(softcap)};
   int rc = launch_lm(X, W, B, V, H, ldx, ldw, epi, static_cast<long long>(tiles_m) * nsplit, stream);
   if (rc) return rc;
   lm_sample_combine_kernel<<<(B + 3) / 4, 128, 0, stream>>>(reinterpret_cast<const LmSampleRec*>(partials),
@@ -488,11 +514,11 @@ int b200_lm_head_combine(const float* partials, int nparts, int T, float* logp, 
 int b200_lm_head_dlogits(const void* X, const void* W, const int* labels, const float* g_logp,
                          const float* g_ent, const float* logz, const float* ey, void* dz, int T,
                          int V, int H, long long ldx, long long ldw, long long ldz,
-                         int vocab_start, float inv_temp, cudaStream_t stream) {
+                         int vocab_start, float inv_temp, float softcap, cudaStream_t stream) {
   using namespace b200;
   if (T == 0 || V == 0) return 0;
   LmDlogitsEpi epi{reinterpret_cast<__nv_bfloat16*>(dz), labels, g_logp, g_ent, logz, ey, ldz, T, V,
-                   vocab_start, inv_temp};
+                   vocab_start, inv_temp, soft_cap(softcap)};
   const long long tiles = static_cast<long long>((T + 127) / 128) * ((V + 255) / 256);
   return launch_lm(X, W, T, V, H, ldx, ldw, epi, tiles, stream);
 }

@@ -15,64 +15,115 @@
 #include <stdint.h>
 
 #include "common/host_utils.h"
+#include "common/io.cuh"
 
 namespace b200 {
 
 constexpr int kMaxE = 1024;
 constexpr int kChunk = 256;  // flat entries per warp in the sort
 
-// One warp per token. logits [T, E] fp32 → idx [T, k] int32, w [T, k] fp32.
-// score = softmax over all experts; the k largest are kept (ties: lowest index) and
-// optionally renormalised to sum to one.
-template <int PER>  // experts per lane = ceil(E / 32)
-__global__ void moe_route_kernel(const float* __restrict__ logits, int* __restrict__ idx, float* __restrict__ w,
-                                 int T, int E, int k, int renorm) {
-  const long long t = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
+// A warp routes one token. z: this lane's logits (experts lane + 32 i). Scores are the softmax over all experts; the k
+// experts with the largest score (plus correction, when there is one) are chosen, ties going to the lowest index, and
+// weighted by their score without the correction, optionally renormalised to sum to one.
+template <int PER, class C>
+__device__ __forceinline__ void route_token(const float (&z)[PER], const C* __restrict__ correction, int E, int k,
+                                            int renorm, int* __restrict__ idx, float* __restrict__ w) {
   const int lane = threadIdx.x & 31;
-  if (t >= T) return;
-  float v[PER];
+  float s[PER], pick[PER];
   float mx = -INFINITY;
 #pragma unroll
-  for (int i = 0; i < PER; ++i) {
-    const int e = lane + 32 * i;
-    v[i] = e < E ? logits[t * E + e] : -INFINITY;
-    mx = fmaxf(mx, v[i]);
-  }
+  for (int i = 0; i < PER; ++i) mx = fmaxf(mx, lane + 32 * i < E ? z[i] : -INFINITY);
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
   float sum = 0.f;
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
-    v[i] = (lane + 32 * i < E) ? expf(v[i] - mx) : -1.f;  // -1 marks "not available"
-    if (v[i] > 0.f) sum += v[i];
+    s[i] = lane + 32 * i < E ? expf(z[i] - mx) : 0.f;
+    sum += s[i];
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
   const float inv = 1.f / sum;
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int e = lane + 32 * i;
+    s[i] *= inv;
+    pick[i] = e < E ? s[i] + (correction ? ld1(correction + e) : 0.f) : -INFINITY;  // -inf: not available
+  }
   float picked_sum = 0.f;
   float my_w = 0.f;
   int my_e = 0;
   for (int j = 0; j < k; ++j) {
-    float best = -1.f;
+    float best = -INFINITY, bs = 0.f;
     int be = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < PER; ++i)
-      if (v[i] > best) { best = v[i]; be = lane + 32 * i; }
+      if (pick[i] > best) { best = pick[i]; bs = s[i]; be = lane + 32 * i; }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, bs, o);
       const int oe = __shfl_xor_sync(0xffffffffu, be, o);
-      if (ob > best || (ob == best && oe < be)) { best = ob; be = oe; }
+      if (ob > best || (ob == best && oe < be)) { best = ob; bs = os; be = oe; }
     }
 #pragma unroll
     for (int i = 0; i < PER; ++i)
-      if (lane + 32 * i == be) v[i] = -1.f;
-    picked_sum += best * inv;
-    if (lane == j) { my_w = best * inv; my_e = be; }
+      if (lane + 32 * i == be) pick[i] = -INFINITY;
+    picked_sum += bs;
+    if (lane == j) { my_w = bs; my_e = be < E ? be : 0; }  // (be >= E only if every score is NaN)
   }
   if (lane < k) {
-    idx[t * k + lane] = my_e;
-    w[t * k + lane] = renorm ? my_w / picked_sum : my_w;
+    idx[lane] = my_e;
+    w[lane] = renorm ? my_w / picked_sum : my_w;
+  }
+}
+
+// One warp per token: logits [T, E] fp32 → idx [T, k] int32, w [T, k] fp32. PER: experts per lane = ceil(E / 32)
+template <int PER, class C>
+__global__ void moe_route_kernel(const float* __restrict__ logits, const C* __restrict__ correction,
+                                 int* __restrict__ idx, float* __restrict__ w, int T, int E, int k, int renorm) {
+  const long long t = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
+  const int lane = threadIdx.x & 31;
+  if (t >= T) return;
+  float z[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i) z[i] = lane + 32 * i < E ? logits[t * E + lane + 32 * i] : 0.f;
+  route_token<PER>(z, correction, E, k, renorm, idx + t * k, w + t * k);
+}
+
+// Router projection and choice of a few tokens (a decode step): one block per token, the token's vector in shared memory,
+// a warp per expert in turn. Products and sums in fp32.
+template <int PER, class D>
+__global__ void moe_router_kernel(const D* __restrict__ x, long long ldx, const D* __restrict__ wr,
+                                  const D* __restrict__ correction, int* __restrict__ idx, float* __restrict__ w, int H,
+                                  int E, int k, int renorm) {
+  extern __shared__ float rsm[];  // [H] vector, [E] logits
+  float* z = rsm + H;
+  const long long t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  for (int c = threadIdx.x; c < H; c += blockDim.x) rsm[c] = ld1(x + t * ldx + c);
+  __syncthreads();
+  const bool v4 = H % 4 == 0;
+  for (int e = warp; e < E; e += nw) {
+    const D* row = wr + static_cast<long long>(e) * H;
+    float s = 0.f;
+    if (v4) {
+#pragma unroll 4
+      for (int c = lane * 4; c < H; c += 128) {
+        const float4 a = ld4(row + c), b = *reinterpret_cast<const float4*>(rsm + c);
+        s = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, s))));
+      }
+    } else {
+      for (int c = lane; c < H; c += 32) s = fmaf(ld1(row + c), rsm[c], s);
+    }
+    s = warp_sum(s);
+    if (lane == 0) z[e] = s;
+  }
+  __syncthreads();
+  if (warp == 0) {
+    float v[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) v[i] = lane + 32 * i < E ? z[lane + 32 * i] : 0.f;
+    route_token<PER>(v, correction, E, k, renorm, idx + t * k, w + t * k);
   }
 }
 
@@ -153,6 +204,154 @@ __global__ void moe_place_kernel(const int* __restrict__ idx, int n, int E, cons
     __syncwarp();
     if (valid && lane == (__ffs(peers) - 1)) run[e] += __popc(peers);
     __syncwarp();
+  }
+}
+
+// The whole sort of a few copies (n <= 1024, a decode step) in one block: thread i owns copy i. Same result as the three
+// passes above. Shared memory: [warps][E] counts, then [E + 1] first tiles.
+__global__ void moe_sort_small_kernel(const int* __restrict__ idx, int n, int E, int* __restrict__ counts,
+                                      int* __restrict__ prow0, int* __restrict__ tile_expert, int* __restrict__ num_vm,
+                                      int* __restrict__ dest, int* __restrict__ src_of) {
+  extern __shared__ int ssm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  int* first = ssm + nw * E;
+  __shared__ int s_warp[32];
+  for (int i = threadIdx.x; i < nw * E; i += blockDim.x) ssm[i] = 0;
+  __syncthreads();
+  const int i = threadIdx.x;
+  const bool valid = i < n;
+  const int e = valid ? idx[i] : -1 - lane;  // invalid lanes match nobody
+  const unsigned peers = __match_any_sync(0xffffffffu, e);
+  const int rank = __popc(peers & ((1u << lane) - 1u));
+  if (valid && lane == __ffs(peers) - 1) ssm[warp * E + e] = __popc(peers);
+  __syncthreads();
+  // thread x owns experts x, x + blockDim.x, ...: counts of the earlier warps, then tiles
+  for (int x = threadIdx.x; x < E; x += blockDim.x) {
+    int run = 0;
+    for (int v = 0; v < nw; ++v) {
+      const int c = ssm[v * E + x];
+      ssm[v * E + x] = run;
+      run += c;
+    }
+    counts[x] = run;
+    first[x] = (run + 127) >> 7;
+  }
+  __syncthreads();
+  // exclusive scan of the tile counts, a block's width at a time
+  int base = 0;
+  for (int x0 = 0; x0 < E; x0 += blockDim.x) {
+    const int x = x0 + threadIdx.x;
+    const int mine = x < E ? first[x] : 0;
+    int inc = mine;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, inc, o);
+      if (lane >= o) inc += v;
+    }
+    __syncthreads();  // the previous round's readers of s_warp are done
+    if (lane == 31) s_warp[warp] = inc;
+    __syncthreads();
+    int before = base, total = base;
+    for (int v = 0; v < nw; ++v) {
+      if (v < warp) before += s_warp[v];
+      total += s_warp[v];
+    }
+    if (x < E) {
+      const int t0 = before + inc - mine;
+      first[x] = t0;
+      prow0[x] = t0 << 7;
+      for (int vm = t0; vm < t0 + mine; ++vm) tile_expert[vm] = x;
+    }
+    base = total;
+  }
+  if (threadIdx.x == 0) {
+    prow0[E] = base << 7;
+    *num_vm = base;
+  }
+  for (int r = threadIdx.x; r < base << 7; r += blockDim.x) src_of[r] = -1;
+  __syncthreads();
+  if (valid) {
+    const int pos = (first[e] << 7) + ssm[warp * E + e] + rank;
+    dest[i] = pos;
+    src_of[pos] = i;
+  }
+}
+
+// out[dest[t * k + j]] = x[t]: a token's vector is read once and written to the rows of its k choices. Rows of padding keep
+// what they hold. One warp per (token, part of its vector).
+__global__ void moe_scatter_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const int* __restrict__ dest,
+                                   int T, int k, int H, int parts, __nv_bfloat16* __restrict__ out) {
+  const int vec = H >> 3, lane = threadIdx.x & 31;
+  const long long warps = (static_cast<long long>(gridDim.x) * blockDim.x) >> 5;
+  for (long long u = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
+       u < static_cast<long long>(T) * parts; u += warps) {
+    const long long t = u / parts;
+    const uint4* in = reinterpret_cast<const uint4*>(x + t * ldx);
+    for (int c = static_cast<int>(u % parts) * 32 + lane; c < vec; c += 32 * parts) {
+      const uint4 v = in[c];
+      for (int j = 0; j < k; ++j)
+        reinterpret_cast<uint4*>(out + static_cast<long long>(__ldg(dest + t * k + j)) * H)[c] = v;
+    }
+  }
+}
+
+// Grouped product of any sizes in fp32 arithmetic (32-bit models, sizes that the tensor-core kernel does not take), over
+// the same padded expert-sorted rows: C[r] = A[row] . W[e(r)]^T for the 64 x 64 tile of a half tile of rows and 64
+// weight rows. gather_k > 0: row r of A is x[src_of[r] / gather_k], else A's own row r. GLU: weight rows alternate
+// between gate and up and the gated activation follows; C is half as wide.
+template <class T, bool GLU>
+__global__ void __launch_bounds__(256) moe_gemm_simt_kernel(const T* __restrict__ a, long long lda, int gather_k,
+                                                            const T* __restrict__ w, T* __restrict__ c, long long ldc,
+                                                            const int* __restrict__ tile_expert,
+                                                            const int* __restrict__ num_vm,
+                                                            const int* __restrict__ src_of, int N, int K, GluParams glu) {
+  __shared__ float sa[16][68], sb[16][68];
+  __shared__ long long arow[64];
+  const int vm = blockIdx.x >> 1, r0 = vm * 128 + (blockIdx.x & 1) * 64, n0 = blockIdx.y * 64;
+  if (vm >= *num_vm || src_of[r0] < 0) return;  // a segment's rows come first in its tile
+  const int e = tile_expert[vm];
+  if (threadIdx.x < 64) {
+    const int s = src_of[r0 + threadIdx.x];
+    arow[threadIdx.x] = s < 0 ? -1 : (gather_k > 0 ? s / gather_k : r0 + static_cast<int>(threadIdx.x));
+  }
+  __syncthreads();
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const T* wb = w + static_cast<long long>(e) * N * K;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+    for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+      const int kk = i & 15, r = i >> 4;
+      const bool in = k0 + kk < K;
+      sa[kk][r] = in && arow[r] >= 0 ? ld1(a + arow[r] * lda + k0 + kk) : 0.f;
+      sb[kk][r] = in && n0 + r < N ? ld1(wb + static_cast<long long>(n0 + r) * K + k0 + kk) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < 16; ++kk) {
+      const float4 av = *reinterpret_cast<const float4*>(&sa[kk][ty * 4]);
+      const float4 bv = *reinterpret_cast<const float4*>(&sb[kk][tx * 4]);
+      const float aa[4] = {av.x, av.y, av.z, av.w}, bb[4] = {bv.x, bv.y, bv.z, bv.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(aa[i], bb[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    if (arow[ty * 4 + i] < 0) continue;
+    T* row = c + static_cast<long long>(r0 + ty * 4 + i) * ldc;
+    const int col = n0 + tx * 4;
+    if (GLU) {
+#pragma unroll
+      for (int j = 0; j < 4; j += 2)
+        if (col + j < N) st1(row + (col + j) / 2, glu_act(acc[i][j], acc[i][j + 1], glu, row));
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (col + j < N) st1(row + col + j, acc[i][j]);
+    }
   }
 }
 
@@ -425,15 +624,92 @@ __global__ void rowdot_scale_kernel(__nv_bfloat16* __restrict__ a, const __nv_bf
 
 extern "C" {
 
-int b200_moe_route(const float* logits, int* idx, float* w, int T, int E, int k, int renorm, cudaStream_t stream) {
+// correction: null or [E], bf16 or fp32 (correction_fp32)
+int b200_moe_route(const float* logits, const void* correction, int correction_fp32, int* idx, float* w, int T, int E,
+                   int k, int renorm, cudaStream_t stream) {
   using namespace b200;
   if (T == 0) return 0;
   if (E > 256 || k > 32 || k > E) return -100;
   const unsigned grid = (static_cast<long long>(T) * 32 + 255) / 256;
   const int per = (E + 31) / 32;
-#define RT(P) moe_route_kernel<P><<<grid, 256, 0, stream>>>(logits, idx, w, T, E, k, renorm)
-  if (per <= 1) RT(1); else if (per <= 2) RT(2); else if (per <= 4) RT(4); else RT(8);
+#define RT(P, C) moe_route_kernel<P, C><<<grid, 256, 0, stream>>>(logits, (const C*)correction, idx, w, T, E, k, renorm)
+#define RTP(C) if (per <= 1) RT(1, C); else if (per <= 2) RT(2, C); else if (per <= 4) RT(4, C); else RT(8, C);
+  if (correction_fp32) { RTP(float) } else { RTP(__nv_bfloat16) }
+#undef RTP
 #undef RT
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// x [T][ldx], wr [E, H], correction null or [E]: all bf16 or all fp32. For few tokens (every block reads all of wr).
+int b200_moe_router(const void* x, long long ldx, const void* wr, const void* correction, int* idx, float* w, int T, int H,
+                    int E, int k, int renorm, int fp32, cudaStream_t stream) {
+  using namespace b200;
+  if (T == 0) return 0;
+  const size_t smem = static_cast<size_t>(H + E) * sizeof(float);
+  if (E > 256 || k > 32 || k > E || smem > 200 * 1024) return -100;
+  const int per = (E + 31) / 32, block = E > 64 ? 512 : 256;
+#define RT(P, D)                                                                                                    \
+  {                                                                                                                 \
+    if (smem > 48 * 1024)                                                                                           \
+      B200_CHECK(cudaFuncSetAttribute(moe_router_kernel<P, D>, cudaFuncAttributeMaxDynamicSharedMemorySize,         \
+                                      static_cast<int>(smem)));                                                     \
+    moe_router_kernel<P, D><<<T, block, smem, stream>>>((const D*)x, ldx, (const D*)wr, (const D*)correction, idx, w, H, \
+                                                        E, k, renorm);                                              \
+  }
+#define RTP(D) if (per <= 1) RT(1, D) else if (per <= 2) RT(2, D) else if (per <= 4) RT(4, D) else RT(8, D)
+  if (fp32) { RTP(float) } else { RTP(__nv_bfloat16) }
+#undef RTP
+#undef RT
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// The sort for n <= 1024 copies; outputs as b200_moe_sort (src_of is set for the tiles in use only).
+int b200_moe_sort_small(const int* idx, int n, int E, int* counts, int* prow0, int* tile_expert, int* num_vm, int* dest,
+                        int* src_of, int max_vm, cudaStream_t stream) {
+  using namespace b200;
+  if (n < 1 || n > 1024 || E > 256) return -100;
+  if (max_vm < (n + 127) / 128 + E) return -101;
+  const int block = (n + 31) / 32 * 32;
+  const size_t sh = (static_cast<size_t>(block / 32) * E + E + 1) * sizeof(int);
+  moe_sort_small_kernel<<<1, block, sh, stream>>>(idx, n, E, counts, prow0, tile_expert, num_vm, dest, src_of);
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// bf16 rows of tokens to the padded rows of their choices (padding keeps what it holds). H % 8 == 0.
+int b200_moe_scatter(const void* x, long long ldx, const int* dest, int T, int k, int H, void* out, cudaStream_t stream) {
+  using namespace b200;
+  if (H % 8 || ldx % 8) return -100;
+  if (T == 0) return 0;
+  int parts = 1;
+  while (parts < 8 && static_cast<long long>(T) * parts < 16LL * sm_count() && 32 * parts < H / 8) parts <<= 1;
+  long long grid = (static_cast<long long>(T) * parts * 32 + 255) / 256;
+  const long long maxg = static_cast<long long>(sm_count()) * 16;
+  if (grid > maxg) grid = maxg;
+  moe_scatter_kernel<<<(unsigned)grid, 256, 0, stream>>>((const __nv_bfloat16*)x, ldx, dest, T, k, H, parts,
+                                                        (__nv_bfloat16*)out);
+  B200_CHECK(cudaGetLastError());
+  return 0;
+}
+
+// See moe_gemm_simt_kernel. w [E, N, K]; N even with glu. gather_k 0: a holds padded rows.
+int b200_moe_gemm_simt(const void* a, long long lda, int gather_k, const void* w, void* c, long long ldc,
+                       const int* tile_expert, const int* num_vm, const int* src_of, int max_vm, int N, int K, int glu,
+                       float limit, float alpha, float beta, int fp32, cudaStream_t stream) {
+  using namespace b200;
+  if (max_vm <= 0 || N <= 0 || K <= 0) return 0;
+  if (glu && (N & 1)) return -100;
+  const dim3 grid(max_vm * 2, (N + 63) / 64);
+  const GluParams g{limit, alpha, beta};
+  using bf = __nv_bfloat16;
+#define MS(T_, G_)                                                                                                  \
+  moe_gemm_simt_kernel<T_, G_><<<grid, 256, 0, stream>>>((const T_*)a, lda, gather_k, (const T_*)w, (T_*)c, ldc,    \
+                                                         tile_expert, num_vm, src_of, N, K, g)
+  if (fp32) { if (glu) MS(float, true); else MS(float, false); }
+  else { if (glu) MS(bf, true); else MS(bf, false); }
+#undef MS
   B200_CHECK(cudaGetLastError());
   return 0;
 }

@@ -190,7 +190,8 @@ class _DecodeGraphs:
                                 self.slots[:b], max_seq_len=e.ncfg.context_length, **extra)
         if self.fused_sampling:
             # the token is drawn in the LM-head GEMM's epilogue: no [B, V] logits, no separate sampler pass
-            return (*lm_head_sample(hidden, e.model.output_weight(), self.temp[:b], self.rng_state), hidden)
+            return (*lm_head_sample(hidden, e.model.output_weight(), self.temp[:b], self.rng_state,
+                                     softcap=e.model.cfg.logit_softcap), hidden)
         logits = e.model.logits(hidden, out_dtype=torch.float32)
         return (*sample(logits, self.temp[:b], None, None, self.u[:b]), hidden)
 

@@ -491,7 +491,7 @@ class B200TrainEngine(TrainEngine):
                 return self.model.values(hidden), None
             labels = torch.roll(ids, shifts=-1, dims=0)
             logp, ent = lm_head_logprobs(hidden, self.model.output_weight(), labels,
-                                         self.config.temperature)
+                                         self.config.temperature, softcap=self.model.cfg.logit_softcap)
             return logp, ent
         return self._forward_mb_parallel(mb, meta, stage_input, chunk)
 

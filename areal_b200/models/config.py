@@ -87,6 +87,11 @@ class ModelConfig:
     # decoders given as an explicit list of layers (`models/layered.py`): every entry names the mixer's type and sizes
     # and the feed-forward's (None: the layer has none); the sizes above then only summarise the list
     layer_specs: list[dict] = field(default_factory=list)
+    # what such a decoder wraps its sublayers in: "dynamic_tanh" (norm in front, learned scale on the result) or
+    # "layer_norm" (one norm in front and one on the result)
+    layer_norms: str = "dynamic_tanh"
+    # logits <- cap * tanh(logits / cap); 0 = none
+    logit_softcap: float = 0.0
     moe_group_score_top: int = 2  # a group's score: the sum of its this many best experts
     decoder_sparse_step: int = 1
     mlp_only_layers: list[int] = field(default_factory=list)
@@ -132,10 +137,16 @@ class ModelConfig:
         """Paged-cache tensors of layer ``i`` as ``(heads, width)`` per token; empty for layers without a cache."""
         if self.is_layered:
             m = self.layer_specs[i]["mixer"]
-            return [(1, m["kv_rank"] + m["rot_dim"])] if self.layer_type(i) == "latent_attention" else []
+            own = self.layer_type(i) == "latent_attention" and m.get("kv_from") is None
+            return [(1, m["kv_rank"] + m["rot_dim"])] if own else []
         if self.layer_type(i) != "full_attention":
             return []
         return [(self.num_key_value_heads, self.head_dim)] * 2
+
+    def cache_layer(self, i: int) -> int:
+        """The layer whose cache layer ``i`` attends to: its own, or an earlier layer's that it shares."""
+        src = self.layer_specs[i]["mixer"].get("kv_from") if self.is_layered else None
+        return i if src is None else src
 
     def recurrent_shape(self, i: int) -> tuple[int, int, int] | None:
         """State of layer ``i`` per sequence ``(heads, key width, value width)``, None for layers without one. Covers
@@ -196,26 +207,37 @@ class ModelConfig:
     def kv_size(self) -> int:
         return self.num_key_value_heads * self.head_dim
 
-    def _layered_params(self, i: int) -> int:
+    def _layered_params(self, i: int, active: bool = False) -> int:
+        """Parameters of layer ``i`` of a layered decoder; ``active``: only those that one token passes through."""
         h, spec = self.hidden_size, self.layer_specs[i]
         m, t = spec["mixer"], spec["type"]
         H, D, Dv = m["heads"], m["dim"], m["vdim"]
+        # what surrounds a sublayer: Dynamic Tanh (weight, bias, alpha) and a scale, or two layer norms
+        wrap = 4 * h if self.layer_norms == "layer_norm" else 3 * h + 1
         if t == "latent_attention":
-            n = (h * (m["q_rank"] + m["kv_rank"] + m["rot_dim"]) + m["q_rank"] * (1 + H * (D + m["rot_dim"]))
-                 + m["kv_rank"] * (1 + H * (D + Dv)))
+            rq, rank, R = m.get("q_rank", 0), m["kv_rank"], m["rot_dim"]
+            n = h * rq + rq * (1 + H * (D + R)) if rq else h * H * (D + R)
+            if m.get("kv_from") is None:
+                n += h * (rank + R) + rank
+            n += rank * H * (D + Dv) + (h * H if m.get("gate") else 0)
         elif t == "hgrn2":
             n = h * H * (2 * D + Dv) + 2 * H * D + Dv
         else:
             n = h * H * (2 * D + 2 * Dv) + H * Dv
-        n += h * H * Dv + 3 * h + 1
-        if spec["mlp"] is not None:
-            n += 2 * h * spec["mlp"]["ff"] + 4 + 3 * h + 1
-        return n
+        n += h * H * Dv + wrap
+        mlp = spec["mlp"]
+        if mlp is None:
+            return n
+        if mlp["kind"] == "moe":
+            r = mlp["router"]
+            return n + wrap + (h + 1) * r["experts"] + 3 * h * mlp["expert"]["ff"] * (r["top"] if active else r["experts"])
+        return n + wrap + 2 * h * mlp["ff"] + (4 if mlp.get("act", "polynorm") == "polynorm" else 0)
 
     def num_params(self) -> int:
         h, L = self.hidden_size, self.num_hidden_layers
         if self.is_layered:
-            return 2 * self.vocab_size * h + 2 * h + 1 + sum(self._layered_params(i) for i in range(L))
+            final = 2 * h + (self.layer_norms == "dynamic_tanh")
+            return 2 * self.vocab_size * h + final + sum(self._layered_params(i) for i in range(L))
         attn = self.attn_params()
         if self.attention_bias:
             attn += self.q_size + 2 * self.kv_size
@@ -261,9 +283,10 @@ class ModelConfig:
             total = 2 * h * self.vocab_size
             for i, spec in enumerate(self.layer_specs):
                 m = spec["mixer"]
-                total += 2 * self._layered_params(i)
+                total += 2 * self._layered_params(i, active=True)
                 if spec["type"] == "latent_attention":
-                    total += 2 * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"]) * (seq_len / 2)
+                    keys = min(seq_len / 2, m.get("window") or seq_len)
+                    total += 2 * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"]) * keys
                 else:
                     total += 4 * m["heads"] * m["dim"] * m["vdim"]
             return total * (3 if backward else 1)
@@ -285,6 +308,8 @@ class ModelConfig:
         top = cfg
         if cfg.get("architecture") == "Fofosun":
             return cls._from_fofosun(cfg, overrides)
+        if cfg.get("architecture") == "Gatolix":
+            return cls._from_gatolix(cfg, overrides)
         if "text_config" in cfg:  # composite (vision-language) checkpoints nest the decoder's config
             cfg = cfg["text_config"]
         mt = cfg.get("model_type", "qwen3")
@@ -430,25 +455,78 @@ class ModelConfig:
                 raise NotImplementedError(f"layer {i}: mixer {t!r}; supported are {sorted(keys)}")
             spec = {k: m[k] for k in keys[t]}
             if t == "latent_attention":
-                spec["rot"] = {"base": float(m["rot"]["base"]), "dims": int(m["rot"]["dims"])}
-                if spec["rot"]["dims"] != spec["rot_dim"] or spec["rot_dim"] % 2:
-                    raise NotImplementedError(f"layer {i}: the rotated part must be rotated whole, in pairs")
+                spec["rot"] = _rotation({k: m["rot"][k] for k in ("base", "dims")}, m["rot_dim"], i)
             if t == "lightning" and len(spec["decay"]) != spec["heads"]:
                 raise ValueError(f"layer {i}: {len(spec['decay'])} decays for {spec['heads']} heads")
             if mlp is not None and mlp.get("kind", "dense") != "dense":
                 raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']!r}; supported is 'dense'")
             specs.append({"type": t, "mixer": spec, "mlp": None if mlp is None else {"kind": "dense", "ff": mlp["ff"]}})
+        return cls._layered("fofosun", cfg, specs, overrides)
+
+    @classmethod
+    def _layered(cls, model_type: str, cfg: dict, specs: list[dict], overrides: dict, **fields) -> "ModelConfig":
         heads = max((s["mixer"]["heads"] for s in specs), default=1)
-        out = cls(model_type="fofosun", vocab_size=cfg["vocab"], hidden_size=cfg["width"], layer_specs=specs,
+        moe = [s["mlp"] for s in specs if s["mlp"] and s["mlp"]["kind"] == "moe"]
+        out = cls(model_type=model_type, vocab_size=cfg["vocab"], hidden_size=cfg["width"], layer_specs=specs,
                   num_hidden_layers=len(specs), rms_norm_eps=cfg["norm"]["eps"],
-                  intermediate_size=max((s["mlp"]["ff"] for s in specs if s["mlp"]), default=0),
+                  intermediate_size=max((s["mlp"]["ff"] for s in specs if s["mlp"] and "ff" in s["mlp"]), default=0),
                   num_attention_heads=heads, num_key_value_heads=heads,
-                  head_dim=max((s["mixer"]["dim"] for s in specs), default=1), tie_word_embeddings=False, qk_norm=False)
+                  head_dim=max((s["mixer"]["dim"] for s in specs), default=1), tie_word_embeddings=False, qk_norm=False,
+                  num_experts=max((m["router"]["experts"] for m in moe), default=0),
+                  num_experts_per_tok=max((m["router"]["top"] for m in moe), default=0),
+                  moe_intermediate_size=max((m["expert"]["ff"] for m in moe), default=0), **fields)
         for k, v in overrides.items():
             setattr(out, k, v)
         return out
 
+    @classmethod
+    def _from_gatolix(cls, cfg: dict, overrides: dict) -> "ModelConfig":
+        """``config.json`` of a Gatolix checkpoint: ``layers`` as in a Fofosun one, with windowed, gated latent attention
+        (a layer may read an earlier layer's latents: ``kv_from``) and dense or mixture-of-experts feed-forwards."""
+        specs = []
+        for i, layer in enumerate(cfg["layers"]):
+            t, m, mlp = layer["type"], layer["mixer"], layer.get("mlp")
+            if t != "latent_attention":
+                raise NotImplementedError(f"layer {i}: mixer {t!r}; supported is 'latent_attention'")
+            rot, src = _rotation(m["rot"], m["rot_dim"], i), m.get("kv_from")
+            if src is not None:
+                own = specs[src]["mixer"] if 0 <= src < i else {"kv_from": -1}
+                if own.get("kv_from") is not None:
+                    raise ValueError(f"layer {i}: layer {src} keeps no latents that it could read")
+                if (own["kv_rank"], own["rot_dim"], own["rot"]) != (m["kv_rank"], m["rot_dim"], rot):
+                    raise ValueError(f"layer {i}: its latents' sizes or rotation differ from those of layer {src}")
+            spec = {k: m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale")}
+            spec.update(rot=rot, window=(m.get("mask") or {}).get("size"), kv_from=src, gate=True)
+            if mlp is None:
+                ff = None
+            elif mlp["kind"] == "dense":
+                ff = {"kind": "dense", "ff": mlp["ff"], "act": "relu2"}
+            elif mlp["kind"] == "moe":
+                ff = {"kind": "moe", "router": {k: mlp["router"][k] for k in ("experts", "top")},
+                      "expert": {k: mlp["expert"][k] for k in ("ff", "limit")}}
+            else:
+                raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']!r}; supported are 'dense' and 'moe'")
+            specs.append({"type": t, "mixer": spec, "mlp": ff})
+        return cls._layered("gatolix", cfg, specs, overrides, layer_norms="layer_norm",
+                            logit_softcap=float(cfg.get("logit_softcap") or 0.0))
+
+    def _to_gatolix(self) -> dict:
+        layers = []
+        for s in self.layer_specs:
+            m = {k: s["mixer"][k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "scale", "rot")}
+            if s["mixer"]["window"] is not None:
+                m["mask"] = {"size": s["mixer"]["window"]}
+            if s["mixer"]["kv_from"] is not None:
+                m["kv_from"] = s["mixer"]["kv_from"]
+            mlp = None if s["mlp"] is None else {k: v for k, v in s["mlp"].items() if k != "act"}
+            layers.append({"type": s["type"], "mixer": m, "mlp": mlp})
+        out = {"architecture": "Gatolix", "layers": layers, "norm": {"eps": self.rms_norm_eps},
+               "vocab": self.vocab_size, "width": self.hidden_size}
+        return dict(out, logit_softcap=self.logit_softcap) if self.logit_softcap else out
+
     def to_hf_config(self) -> dict:
+        if self.model_type == "gatolix":
+            return self._to_gatolix()
         if self.model_type == "fofosun":
             return {"architecture": "Fofosun", "layers": self.layer_specs, "norm": {"eps": self.rms_norm_eps},
                     "vocab": self.vocab_size, "width": self.hidden_size}
@@ -578,6 +656,21 @@ _VL_TYPES = ("qwen2_5_vl", "qwen2_vl", "qwen3_vl", "qwen3_vl_moe")
 _TEXT_TYPES = {"qwen2", "qwen3", "qwen3_moe", "qwen3_5", "llama", "mistral", "qwen2_moe", "mixtral", "deepseek_v2", "deepseek_v3", "bailing_hybrid"}
 
 # Named shapes used by the benchmark configurations (random-init, synthetic data).
+
+
+def _rotation(rot: dict, width: int, layer: int) -> dict:
+    """A latent-attention layer's rotation: base, number of rotated dimensions and, when given, YaRN scaling."""
+    out = {"base": float(rot["base"]), "dims": int(rot["dims"])}
+    if out["dims"] != width or width % 2:
+        raise NotImplementedError(f"layer {layer}: the rotated part must be rotated whole, in pairs")
+    if rot.get("scaling"):
+        out["scaling"] = {k: rot["scaling"][k] for k in ("factor", "original", "fast", "slow")}
+    return out
+
+
+_TINY_LATENT = {"heads": 4, "dim": 32, "rot_dim": 16, "vdim": 24, "kv_rank": 80, "scale": 0.15, "mask": {"size": 50},
+                "rot": {"base": 1e4, "dims": 16, "scaling": {"factor": 4.0, "original": 512, "fast": 16.0, "slow": 1.0}}}
+
 PRESETS: dict[str, ModelConfig] = {
     "tiny-qwen2": ModelConfig(model_type="qwen2", vocab_size=1024, hidden_size=256,
                               intermediate_size=688, num_hidden_layers=2, num_attention_heads=4,
@@ -694,6 +787,13 @@ PRESETS: dict[str, ModelConfig] = {
              "mlp": None},
             {"type": "lightning", "mixer": {"heads": 2, "dim": 48, "vdim": 64, "decay": [0.7, 0.99]},
              "mlp": {"kind": "dense", "ff": 320}}]}, {}),
+    # Gatolix at test size: windows, shared latents, a dense and a mixture feed-forward and a layer without one
+    "tiny-gatolix": ModelConfig._from_gatolix({
+        "vocab": 1024, "width": 192, "norm": {"eps": 1e-6}, "logit_softcap": 20.0, "layers": [
+            {"type": "latent_attention", "mixer": dict(_TINY_LATENT), "mlp": {"kind": "dense", "ff": 320}},
+            {"type": "latent_attention", "mixer": dict(_TINY_LATENT, heads=6, kv_from=0, mask={"size": 24}), "mlp": None},
+            {"type": "latent_attention", "mixer": dict(_TINY_LATENT), "mlp": {
+                "kind": "moe", "router": {"experts": 6, "top": 2}, "expert": {"ff": 96, "limit": 3.0}}}]}, {}),
     # DeepSeek-V2-Lite: latent attention without the query bottleneck, softmax routing, two shared experts
     "deepseek-v2-lite": ModelConfig(model_type="deepseek_v2", vocab_size=102400, hidden_size=2048,
                                     intermediate_size=10944, num_hidden_layers=27, num_attention_heads=16,

@@ -1,36 +1,41 @@
 """Decoders described as a list of layers (``ModelConfig.layer_specs``), each with its own mixer, its own sizes and an
-optional feed-forward, on an fp32 residual stream. The Fofosun family is built this way:
+optional feed-forward, on an fp32 residual stream:
 
     x = embed[token]
-    x = x + ls1 * mixer(norm1(x));   x = x + ls2 * ff(norm2(x))     per layer; a layer may have no feed-forward
+    x = x + wrap1(mixer(norm1(x)));   x = x + wrap2(ff(norm2(x)))     per layer; a layer may have no feed-forward
     logits = head norm(x)
 
-Norms are Dynamic Tanh, ``tanh(alpha x) * w + b`` (Zhu, Chen, He, LeCun, Liu, "Transformers without Normalization"),
-the feed-forward is ``W_down polynorm(W_up x)``. Every sublayer hands the activations in front of its output
-projection to :func:`ops.dyt.linear_residual_dyt`, which projects, scales, adds to the residual and applies the NEXT
-sublayer's norm in one kernel, so the model is a flat list of sublayers between the embedding and the head.
+Norms (``ModelConfig.layer_norms``): Dynamic Tanh, ``tanh(alpha x) * w + b`` (Zhu, Chen, He, LeCun, Liu, "Transformers
+without Normalization") with a learned per-column scale as ``wrap``, or layer norm with a second layer norm as ``wrap``.
+Every sublayer hands the activations in front of its output projection to the next norm's ``join``, which projects,
+wraps, adds to the residual and normalises in as few kernels as the shapes allow (``ops/dyt.py``, ``ops/layer_norm.py``),
+so the model is a flat list of sublayers between the embedding and the head.
 
 Mixers (``MIXERS``): HGRN2 (``models/hgrn2.py``), lightning attention with configured decays
-(``models/lightning.py``), latent attention over a compressed cache (``models/mla.py``). A mixer has
-``hidden(y, ctx, cache, rec)``, an output projection ``o`` and ``tensors(prefix)``; what it keeps per sequence is
+(``models/lightning.py``), latent attention over a compressed cache (``models/mla.py``). Feed-forwards (``make_mlp``):
+dense with PolyNorm or squared ReLU, mixture of gated experts. A sublayer has ``hidden(y, ctx, cache, rec)``, an output
+projection ``o`` (None: ``hidden`` is the sublayer's result) and ``tensors(prefix)``; what a mixer keeps per sequence is
 declared by ``ModelConfig.cache_shapes`` / ``recurrent_shape``, allocated by the rollout engine and passed in.
 
-The class shares loading, the head and the engine interface (``prefill`` / ``decode``) with ``QwenModel``. It is served
-by the rollout engine and runs forward and backward for training on one process per replica (data parallelism).
+The Fofosun and Gatolix families are built this way. The class shares loading, the head and the engine interface
+(``prefill`` / ``decode``) with ``QwenModel``. It is served by the rollout engine and runs forward and backward for
+training on one process per replica (data parallelism).
 """
 
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import Any, Iterator
 
 import torch
 import torch.nn as nn
 
-from ..ops import dyt
+from ..ops import dyt, layer_norm as ln
 from ..ops.attention import VarlenMeta
-from ..ops.gemm import linear
+from ..ops.gemm import linear, linear_relu2
 from ..ops.latent_attn import rotary_tables
+from ..ops.lm_head import soft_cap_
+from ..ops.moe import ExpertRows, GatedAct, gated_experts, route_tokens
 from .config import ModelConfig
 from .hgrn2 import HGRN2
 from .lightning import ConstantDecayLightning
@@ -40,8 +45,19 @@ from .qwen import QwenModel
 MIXERS = {"hgrn2": HGRN2, "lightning": ConstantDecayLightning, "latent_attention": LatentAttention}
 
 
-class DynamicTanh(nn.Module):
+class ColumnScale(nn.Module):
+    """Learned scale on a sublayer's result."""
+
     def __init__(self, n: int, dtype, device):
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(n, dtype=dtype, device=device))
+
+    def tensors(self, name: str):
+        yield name, self.weight
+
+
+class DynamicTanh(nn.Module):
+    def __init__(self, n: int, eps: float, dtype, device):
         super().__init__()
         self.weight = nn.Parameter(torch.ones(n, dtype=dtype, device=device))
         self.bias = nn.Parameter(torch.zeros(n, dtype=dtype, device=device))
@@ -51,10 +67,107 @@ class DynamicTanh(nn.Module):
     def args(self):
         return self.alpha, self.weight, self.bias
 
+    def embed(self, ids, table):
+        """``(norm(res), res)`` of ``res = table[ids]``."""
+        return dyt.embed_dyt(ids, table, self.args)
+
+    def join(self, a, o, wrap: ColumnScale, res):
+        """``(norm(res), res)`` of ``res + wrap * (a @ o.T)``: this norm stands in front of the next sublayer."""
+        if o is None:
+            return dyt.residual_dyt(a, wrap.weight, res, self.args)
+        return dyt.linear_residual_dyt(a, o, wrap.weight, res, self.args)
+
     def tensors(self, name: str):
         yield name, self.weight
         yield name + ".b", self.bias
         yield name + ".alpha", self.alpha
+
+
+class LayerNorm(nn.Module):
+    def __init__(self, n: int, eps: float, dtype, device):
+        super().__init__()
+        self.eps = eps
+        self.weight = nn.Parameter(torch.ones(n, dtype=dtype, device=device))
+        self.bias = nn.Parameter(torch.zeros(n, dtype=dtype, device=device))
+
+    @property
+    def args(self):
+        return self.weight, self.bias
+
+    def embed(self, ids, table):
+        return ln.embed_ln(ids, table, self.args, self.eps)
+
+    def join(self, a, o, wrap: "LayerNorm", res):
+        """``(norm(res), res)`` of ``res + wrap(a @ o.T)``; without ``o``, ``a`` is the sublayer's result, also as the
+        experts' uncombined rows."""
+        if isinstance(a, ExpertRows):
+            return ln.experts_residual_ln(a, wrap.args, res, self.args, self.eps)
+        if o is None:
+            return ln.residual_ln(a, wrap.args, res, self.args, self.eps)
+        return ln.linear_residual_ln(a, o, wrap.args, res, self.args, self.eps)
+
+    def tensors(self, name: str):
+        yield name, self.weight
+        yield name + ".b", self.bias
+
+
+# norm, what is wrapped around a sublayer's result, and the latter's checkpoint names
+NORMS = {"dynamic_tanh": (DynamicTanh, lambda n, eps, dtype, device: ColumnScale(n, dtype, device), ("ls1", "ls2")),
+         "layer_norm": (LayerNorm, LayerNorm, ("norm1b", "norm2b"))}
+
+
+class Relu2MLP(nn.Module):
+    """``relu(W_up y)^2``, to be projected by ``o`` (the down projection)."""
+
+    def __init__(self, hidden: int, spec: dict, eps: float, dtype, device):
+        super().__init__()
+        self.up = nn.Parameter(torch.empty(spec["ff"], hidden, dtype=dtype, device=device))
+        self.o = nn.Parameter(torch.empty(hidden, spec["ff"], dtype=dtype, device=device))
+
+    def hidden(self, y, ctx=None, cache=None, rec=None):
+        return linear_relu2(y, self.up)
+
+    def tensors(self, p: str):
+        yield p + "up", self.up
+        yield p + "down", self.o
+
+
+class ExpertsMLP(nn.Module):
+    """Mixture of gated experts: ``sum_e s_e W_down,e act(W_gate,e y, W_up,e y)`` over a token's chosen experts. Scores ``s``
+    are the softmax of the router's logits (32-bit) over all experts; the ``top`` largest of ``s + correction`` are chosen
+    and weighted by ``s``, not renormalised. The activation is ``ops/moe.py::GatedAct`` with the family's constants. Gate
+    and up rows alternate in ``gate_up`` so that the activation runs in the product's epilogue."""
+
+    o = None
+
+    def __init__(self, hidden: int, spec: dict, act: GatedAct, dtype, device):
+        super().__init__()
+        E, ff = spec["router"]["experts"], spec["expert"]["ff"]
+        mk = lambda *shape: nn.Parameter(torch.empty(*shape, dtype=dtype, device=device))
+        self.top, self.act = spec["router"]["top"], act
+        self.router = mk(E, hidden)
+        self.correction = nn.Parameter(torch.zeros(E, dtype=dtype, device=device))
+        self.gate_up = mk(E, 2 * ff, hidden)
+        self.down = mk(E, hidden, ff)
+
+    def hidden(self, y, ctx=None, cache=None, rec=None):
+        idx, w = route_tokens(y, self.router, self.top, False, self.correction)
+        return gated_experts(y, idx, w, self.gate_up, self.down, self.act)
+
+    def tensors(self, p: str):
+        for e in range(self.router.shape[0]):
+            yield f"{p}e{e}.gate", self.gate_up[e, 0::2]
+            yield f"{p}e{e}.up", self.gate_up[e, 1::2]
+            yield f"{p}e{e}.down", self.down[e]
+        yield p + "router", self.router
+        yield p + "correction", self.correction
+
+
+def make_mlp(hidden: int, spec: dict, eps: float, dtype, device):
+    if spec["kind"] == "moe":
+        # x * sigmoid(1.702 x) approximates GELU (Hendrycks and Gimpel, "Gaussian Error Linear Units")
+        return ExpertsMLP(hidden, spec, GatedAct(alpha=1.702, beta=1.0, limit=float(spec["expert"]["limit"])), dtype, device)
+    return {"polynorm": PolyNormMLP, "relu2": Relu2MLP}[spec.get("act", "polynorm")](hidden, spec, eps, dtype, device)
 
 
 class PolyNormMLP(nn.Module):
@@ -80,25 +193,26 @@ class PolyNormMLP(nn.Module):
 class LayeredBlock(nn.Module):
     def __init__(self, cfg: ModelConfig, i: int, dtype, device):
         super().__init__()
-        h, spec = cfg.hidden_size, cfg.layer_specs[i]
-        scale = lambda: nn.Parameter(torch.ones(h, dtype=dtype, device=device))
-        self.norm1 = DynamicTanh(h, dtype, device)
-        self.attn = MIXERS[spec["type"]](h, spec["mixer"], cfg.rms_norm_eps, dtype, device)
-        self.ls1 = scale()
-        self.norm2 = self.mlp = self.ls2 = None
+        h, spec, eps = cfg.hidden_size, cfg.layer_specs[i], cfg.rms_norm_eps
+        norm, wrap, self.wrap_names = NORMS[cfg.layer_norms]
+        self.norm1 = norm(h, eps, dtype, device)
+        self.attn = MIXERS[spec["type"]](h, spec["mixer"], eps, dtype, device)
+        self.attn.index = i
+        self.wrap1 = wrap(h, eps, dtype, device)
+        self.norm2 = self.mlp = self.wrap2 = None
         if spec["mlp"] is not None:
-            self.norm2 = DynamicTanh(h, dtype, device)
-            self.mlp = PolyNormMLP(h, spec["mlp"], cfg.rms_norm_eps, dtype, device)
-            self.ls2 = scale()
+            self.norm2 = norm(h, eps, dtype, device)
+            self.mlp = make_mlp(h, spec["mlp"], eps, dtype, device)
+            self.wrap2 = wrap(h, eps, dtype, device)
 
     def tensors(self, p: str):
         yield from self.norm1.tensors(p + "norm1")
         yield from self.attn.tensors(p + "mix.")
-        yield p + "ls1", self.ls1
+        yield from self.wrap1.tensors(p + self.wrap_names[0])
         if self.mlp is not None:
             yield from self.norm2.tensors(p + "norm2")
             yield from self.mlp.tensors(p + "mlp.")
-            yield p + "ls2", self.ls2
+            yield from self.wrap2.tensors(p + self.wrap_names[1])
 
 
 @dataclass
@@ -115,10 +229,13 @@ class StepContext:
     seq_lens: torch.Tensor | None = None
     max_seq_len: int | None = None
     state_slots: torch.Tensor | None = None
+    # latents and rotated key parts of the batch, by layer, of the layers in ``shared`` (those that others read)
+    shared: frozenset = frozenset()
+    latents: dict = field(default_factory=dict)
 
-    def rotary(self, dims: int, base: float):
+    def rotary(self, rot: dict):
         n = self.max_seq_len if self.decode else self.meta.max_seqlen
-        return self.model.rotary(dims, base, n or 1, self.pos.device)
+        return self.model.rotary(rot, n or 1, self.pos.device)
 
 
 class LayeredModel(QwenModel):
@@ -137,12 +254,13 @@ class LayeredModel(QwenModel):
         mk = lambda *shape: nn.Parameter(torch.empty(*shape, dtype=dtype, device=device))
         self.embed = mk(cfg.vocab_size, cfg.hidden_size)
         self.layers = nn.ModuleList(LayeredBlock(cfg, i, dtype, device) for i in self.layer_ids)
-        self.norm = DynamicTanh(cfg.hidden_size, dtype, device)
+        self.norm = NORMS[cfg.layer_norms][0](cfg.hidden_size, cfg.rms_norm_eps, dtype, device)
         self.lm_head = mk(cfg.vocab_size, cfg.hidden_size)
         self.score = None
         self.checkpoint_every = 0
-        self._tables: dict[tuple[int, float], tuple[torch.Tensor, torch.Tensor]] = {}
+        self._tables: dict[tuple, tuple[torch.Tensor, torch.Tensor]] = {}
         self._positions = 1
+        self._shared = frozenset(j for i in self.layer_ids if (j := cfg.cache_layer(i)) != i)
 
     @torch.no_grad()
     def init_weights(self, seed: int = 0, std: float = 0.02):
@@ -162,25 +280,32 @@ class LayeredModel(QwenModel):
         keeps their addresses)."""
         self._positions = max(self._positions, int(n))
 
-    def rotary(self, dims: int, base: float, n: int, device):
-        t = self._tables.get((dims, base))
+    def rotary(self, rot: dict, n: int, device):
+        dims, base, scaling = rot["dims"], rot["base"], rot.get("scaling")
+        key = (dims, base, tuple(sorted(scaling.items())) if scaling else None)
+        t = self._tables.get(key)
         if t is None or t[0].shape[0] < n or t[0].device != device:
-            t = self._tables[(dims, base)] = rotary_tables(max(n, self._positions), dims, base, device)
+            t = self._tables[key] = rotary_tables(max(n, self._positions), dims, base, device, scaling)
         return t
+
+    def logits(self, hidden, out_dtype=torch.float32):
+        return soft_cap_(super().logits(hidden, out_dtype), self.cfg.logit_softcap)
 
     # -------------------------------------------------------------------- forward
     def _run(self, input_ids, ctx: StepContext, kv_caches=None, state=None):
         """Embedding, every sublayer, final norm: ``[T, hidden]`` in the model's dtype."""
-        subs = []  # (sublayer, its scale, its norm, its cache, its state)
+        ctx.shared = self._shared
+        subs = []  # (sublayer, its wrap, its norm, its cache, its state)
         for i, layer in enumerate(self.layers):
-            cache = kv_caches[i][0] if kv_caches is not None and kv_caches[i] is not None else None
-            subs.append((layer.attn, layer.ls1, layer.norm1, cache, state.rec[i] if state is not None else None))
+            src = kv_caches[self.cfg.cache_layer(i)] if kv_caches is not None else None
+            cache = src[0] if src is not None else None
+            subs.append((layer.attn, layer.wrap1, layer.norm1, cache, state.rec[i] if state is not None else None))
             if layer.mlp is not None:
-                subs.append((layer.mlp, layer.ls2, layer.norm2, None, None))
+                subs.append((layer.mlp, layer.wrap2, layer.norm2, None, None))
         norms = [s[2] for s in subs] + [self.norm]
-        y, res = dyt.embed_dyt(input_ids, self.embed, norms[0].args)
-        for k, (sub, scale, _, cache, rec) in enumerate(subs):
-            y, res = dyt.linear_residual_dyt(sub.hidden(y, ctx, cache, rec), sub.o, scale, res, norms[k + 1].args)
+        y, res = norms[0].embed(input_ids, self.embed)
+        for k, (sub, wrap, _, cache, rec) in enumerate(subs):
+            y, res = norms[k + 1].join(sub.hidden(y, ctx, cache, rec), sub.o, wrap, res)
         return y
 
     def forward(self, input_ids, position_ids, meta: VarlenMeta, attn_fn=None, **unsupported):

@@ -176,48 +176,77 @@ class LatentAttention(nn.Module):
     """Latent attention served from a compressed cache: a token leaves its normed latent and one rotated key part
     shared by all heads (``rank + rot`` numbers) instead of every head's keys and values.
 
-        c_q = rmsnorm(W_dq x);  q = W_uq c_q          per head [unrotated | rotated]
-        c, r = split(W_dkv x);  c = rmsnorm(c)        latent, shared rotated key part
+        q = W_uq rmsnorm(W_dq x), or W_q x without ``q_rank``     per head [unrotated | rotated]
+        c, r = split(W_dkv x);  c = rmsnorm(c)                    latent, shared rotated key part
         k_h = [W_uk,h c | rope(r)],  v_h = W_uv,h c;  softmax(q k^T * scale) v, causal
+        times sigmoid(W_g x)_h per head with ``gate``
 
-    Rotation turns neighbouring pairs and keeps the layout. A mixer of the layered decoder (``models/layered.py``):
-    ``hidden`` returns the concatenated heads in front of the output projection. Prefills expand keys and values
-    (``ops/latent_attn.py::latent_attention``); decode steps stay in the latent space (``latent_decode``)."""
+    ``window``: a token sees itself and the ``window - 1`` before it. ``kv_from``: the layer has no W_dkv and reads the
+    latents and rotated key parts of that earlier layer (in a prefill its rows of the batch, in a decode step its cache)
+    through its own W_uk and W_uv. Rotation turns neighbouring pairs and keeps the layout, optionally with YaRN scaling. A
+    mixer of the layered decoder (``models/layered.py``): ``hidden`` returns the concatenated heads in front of the output
+    projection. Prefills expand keys and values (``ops/latent_attn.py::latent_attention``); decode steps stay in the
+    latent space (``latent_decode``)."""
 
     def __init__(self, hidden: int, spec: dict, eps: float, dtype, device):
         super().__init__()
         self.H, self.D, self.R, self.Dv = spec["heads"], spec["dim"], spec["rot_dim"], spec["vdim"]
-        self.q_rank, self.rank, self.scale, self.eps = spec["q_rank"], spec["kv_rank"], float(spec["scale"]), eps
-        self.rot_base = float(spec["rot"]["base"])
+        self.q_rank, self.rank, self.scale, self.eps = spec.get("q_rank", 0), spec["kv_rank"], float(spec["scale"]), eps
+        self.rot, self.window, self.kv_from = spec["rot"], spec.get("window"), spec.get("kv_from")
+        self.index = 0  # its place in the decoder, by which other layers refer to its latents
+        self.nq = self.q_rank or self.H * (self.D + self.R)
+        self.nkv = self.rank + self.R if self.kv_from is None else 0
+        self.ng = self.H if spec.get("gate") else 0
         mk = lambda *shape: nn.Parameter(torch.empty(*shape, dtype=dtype, device=device))
         ones = lambda n: nn.Parameter(torch.ones(n, dtype=dtype, device=device))
-        self.down = mk(self.q_rank + self.rank + self.R, hidden)        # dq | dkv (latent, rotated part)
-        self.q_norm, self.c_norm = ones(self.q_rank), ones(self.rank)
-        self.uq = mk(self.H * (self.D + self.R), self.q_rank)
+        self.inp = mk(self.nq + self.nkv + self.ng, hidden)             # dq or q | dkv (latent, rotated part) | g
+        self.q_norm = ones(self.q_rank) if self.q_rank else None
+        self.c_norm = ones(self.rank) if self.nkv else None
+        self.uq = mk(self.H * (self.D + self.R), self.q_rank) if self.q_rank else None
         self.ukv = mk(self.H * (self.D + self.Dv), self.rank)           # uk | uv
         self.o = mk(hidden, self.H * self.Dv)
+        if self.q_rank and not self.nkv:
+            raise NotImplementedError("a layer that reads another layer's latents has no query latent")
 
     def hidden(self, y, ctx, cache=None, rec=None):
         from ..ops import latent_attn as la
 
         H, D, R = self.H, self.D, self.R
-        cos, sin = ctx.rotary(R, self.rot_base)
-        cq, c, kr = la.latent_prep(linear(y, self.down), self.q_norm, self.c_norm, self.rank, R, self.eps, cos, sin,
-                                   ctx.pos, cache, ctx.slot_mapping, want_rows=not ctx.decode)
-        q = la.rope_pairs_(linear(cq, self.uq), H, D, R, cos, sin, ctx.pos)
+        cos, sin = ctx.rotary(self.rot)
+        x = linear(y, self.inp)
+        gate = x[:, self.nq + self.nkv:] if self.ng else None
+        if self.q_rank:
+            cq, c, kr = la.latent_prep(x[:, :self.nq + self.nkv], self.q_norm, self.c_norm, self.rank, R, self.eps, cos, sin,
+                                       ctx.pos, cache, ctx.slot_mapping, want_rows=not ctx.decode)
+            q = la.rope_pairs_(linear(cq, self.uq), H, D, R, cos, sin, ctx.pos)
+        elif self.nkv:
+            q, c, kr = la.latent_qkv_prep(x, H, D, self.c_norm, self.rank, R, self.eps, cos, sin, ctx.pos, cache,
+                                          ctx.slot_mapping, want_rows=not ctx.decode)
+        else:
+            q = la.rope_pairs_(x[:, :self.nq], H, D, R, cos, sin, ctx.pos)
+            c, kr = ctx.latents.get(self.kv_from, (None, None))
+        if self.index in ctx.shared:
+            ctx.latents[self.index] = (c, kr)
         if not ctx.decode:
-            return la.latent_attention(q, linear(c, self.ukv), kr, ctx.meta, H, D, R, self.Dv, self.scale)
+            return la.latent_attention(q, linear(c, self.ukv), kr, ctx.meta, H, D, R, self.Dv, self.scale, self.window, gate)
         qa = la.heads_matmul(q, H, D, self.ukv[:H * D], transposed=True)
         ol = la.latent_decode(qa, q, cache, ctx.block_table, ctx.seq_lens, H, D, R, self.rank, self.scale,
-                              ctx.max_seq_len)
+                              ctx.max_seq_len, self.window, gate)
         return la.heads_matmul(ol, H, self.rank, self.ukv[H * D:], transposed=False)
 
     def tensors(self, p: str):
-        yield p + "dq", self.down[:self.q_rank]
-        yield p + "dkv", self.down[self.q_rank:]
-        yield p + "dq.norm", self.q_norm
-        yield p + "dkv.norm", self.c_norm
-        yield p + "uq", self.uq
+        kv = slice(self.nq, self.nq + self.nkv)
+        if self.q_rank:
+            yield p + "dq", self.inp[:self.nq]
+            yield p + "dq.norm", self.q_norm
+            yield p + "uq", self.uq
+        else:
+            yield p + "q", self.inp[:self.nq]
+        if self.nkv:
+            yield p + "dkv", self.inp[kv]
+            yield p + "dkv.norm", self.c_norm
         yield p + "uk", self.ukv[:self.H * self.D]
         yield p + "uv", self.ukv[self.H * self.D:]
+        if self.ng:
+            yield p + "g", self.inp[self.nq + self.nkv:]
         yield p + "o", self.o

@@ -133,6 +133,33 @@ def _splitk_plan(M: int, N: int, K: int) -> int:
     return splits if splits >= 2 else 0
 
 
+def linear_relu2(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``relu(x @ w.T)^2``. On the bf16 kernels the activation runs on the product's fp32 accumulators (for decode-sized
+    products in the split-K reduction)."""
+    grad = torch.is_grad_enabled() and (x.requires_grad or w.requires_grad)
+    if not (_lib.use_cuda_kernels(x, w) and x.dtype in (torch.bfloat16, torch.float32)) or grad:
+        return torch.relu(linear(x, w)).square()
+    M, K = x.shape
+    N = w.shape[0]
+    if not (x.dtype == torch.bfloat16 and N % 8 == 0 and K % 8 == 0 and x.stride(1) == 1 and w.is_contiguous()
+            and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
+        z = linear(x, w)
+        rc = _lib.kernels().b200_relu2(_lib.ptr(z), ctypes.c_longlong(z.numel()), ctypes.c_int(int(z.dtype == torch.float32)),
+                                       _lib.stream_ptr())
+        _lib.check(rc, "b200_relu2")
+        _lib.count_launch()
+        return z
+    splits = _splitk_plan(M, N, K)
+    ws = torch.empty((splits * -(-M // 128) * 128, N), dtype=torch.float32, device=x.device) if splits else None
+    y = torch.empty((M, N), dtype=x.dtype, device=x.device)
+    rc = _lib.kernels().b200_gemm_bf16_relu2(
+        _lib.ptr(x), _lib.ptr(w), _lib.ptr(y), _lib.ptr(ws), ctypes.c_int(M), ctypes.c_int(N), ctypes.c_int(K),
+        ctypes.c_longlong(x.stride(0)), ctypes.c_longlong(w.stride(0)), ctypes.c_int(splits), _lib.stream_ptr())
+    _lib.check(rc, "b200_gemm_bf16_relu2")
+    _lib.count_launch(2 if splits else 1)
+    return y
+
+
 @torch.no_grad()
 def linear_rmsnorm(x: torch.Tensor, w: torch.Tensor, norm_w: torch.Tensor, eps: float,
                    residual: torch.Tensor | None = None):

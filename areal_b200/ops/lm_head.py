@@ -25,10 +25,29 @@ from .gemm import gemm
 _BWD_ROW_CHUNK = 4096
 
 
-def lm_head_logprobs_ref(x, w, labels, temperature=1.0, tp_group=None, vocab_start=0):
+def soft_cap(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap * tanh(logits / cap)``; 0: no cap."""
+    return cap * torch.tanh(logits / cap) if cap else logits
+
+
+def soft_cap_(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    """:func:`soft_cap` in place where the kernel takes it (fp32, no gradient)."""
+    if not cap or logits.numel() == 0:
+        return logits
+    if not (_lib.use_cuda_kernels(logits) and logits.dtype == torch.float32 and logits.is_contiguous()) or (
+            torch.is_grad_enabled() and logits.requires_grad):
+        return soft_cap(logits, cap)
+    rc = _lib.kernels().b200_softcap(_lib.ptr(logits), ctypes.c_longlong(logits.numel()), ctypes.c_float(cap),
+                                     _lib.stream_ptr())
+    _lib.check(rc, "b200_softcap")
+    _lib.count_launch()
+    return logits
+
+
+def lm_head_logprobs_ref(x, w, labels, temperature=1.0, tp_group=None, vocab_start=0, softcap=0.0):
     """fp32 reference (also the CPU path). With ``tp_group`` the local shard's
     statistics are all-reduced like the reference implementation does."""
-    logits = (x.float() @ w.float().t()) / temperature
+    logits = soft_cap(x.float() @ w.float().t(), softcap) / temperature
     if tp_group is None or dist.get_world_size(tp_group) == 1:
         lse = torch.logsumexp(logits, -1)
         tgt = logits.gather(-1, labels.long()[:, None]).squeeze(-1)
@@ -64,7 +83,8 @@ class _AllReduceSum(torch.autograd.Function):
 
 class _LMHead(torch.autograd.Function):
     @staticmethod
-    def forward(ctx, x, w, labels, temperature, tp_group, vocab_start, tp_fused=None):
+    def forward(ctx, x, w, labels, temperature, tp_group, vocab_start, tp_fused=None, softcap=0.0):
+        ctx.softcap = float(softcap)
         T, H = x.shape
         V = w.shape[0]
         x = x if x.is_contiguous() else x.contiguous()
@@ -86,7 +106,7 @@ class _LMHead(torch.autograd.Function):
                                               ctypes.c_int(tp_fused.rank), ctypes.c_int(T), ctypes.c_int(V),
                                               ctypes.c_int(H), ctypes.c_longlong(x.stride(0)),
                                               ctypes.c_longlong(w.stride(0)), ctypes.c_int(vocab_start),
-                                              ctypes.c_float(inv_t), _lib.stream_ptr())
+                                              ctypes.c_float(inv_t), ctypes.c_float(ctx.softcap), _lib.stream_ptr())
             _lib.check(rc, "b200_lm_head_stats_peers")
             tp_fused.barrier.sync()
             half = bufs.nbytes // 2
@@ -98,7 +118,7 @@ class _LMHead(torch.autograd.Function):
                                     ctypes.c_int(T), ctypes.c_int(V), ctypes.c_int(H),
                                     ctypes.c_longlong(x.stride(0)), ctypes.c_longlong(w.stride(0)),
                                     ctypes.c_int(vocab_start), ctypes.c_float(inv_t),
-                                    _lib.stream_ptr())
+                                    ctypes.c_float(ctx.softcap), _lib.stream_ptr())
         _lib.check(rc, "b200_lm_head_stats")
         if tp > 1:
             # ranks may pick different split counts only if their shard sizes differ; pad to max
@@ -164,7 +184,7 @@ class _LMHead(torch.autograd.Function):
                 ctypes.c_int(n), ctypes.c_int(V), ctypes.c_int(H),
                 ctypes.c_longlong(x.stride(0)), ctypes.c_longlong(w.stride(0)),
                 ctypes.c_longlong(Vp), ctypes.c_int(ctx.vocab_start), ctypes.c_float(ctx.inv_t),
-                _lib.stream_ptr())
+                ctypes.c_float(ctx.softcap), _lib.stream_ptr())
             _lib.check(rc, "b200_lm_head_dlogits")
             _lib.count_launch()
             dzv = dz[:n, :V]
@@ -178,7 +198,7 @@ class _LMHead(torch.autograd.Function):
         dw = None
         if need_dw and main is None:
             dw = dw_acc.to(w.dtype)
-        return dx, dw, None, None, None, None, None
+        return dx, dw, None, None, None, None, None, None
 
 
 def _peer_partials(fctx, nbytes: int):
@@ -203,17 +223,18 @@ def _peer_partials(fctx, nbytes: int):
     return st[0], st[1], calls
 
 
-def lm_head_logprobs(x, w, labels, temperature: float = 1.0, tp_group=None, vocab_start: int = 0, tp_fused=None):
+def lm_head_logprobs(x, w, labels, temperature: float = 1.0, tp_group=None, vocab_start: int = 0, tp_fused=None,
+                     softcap: float = 0.0):
     """Per-token log-probability of ``labels`` and entropy of the next-token
     distribution ``softmax(x @ w.T / temperature)``. ``w`` may be this rank's
     vocabulary shard starting at global id ``vocab_start``; the gradient with respect to ``x``
     is then this shard's partial contribution, to be summed over ``tp_group`` by the caller
     (``parallel.tensor_parallel.gather_seq`` does so in its backward). With ``tp_fused`` (the tp group's
     ``FusedCommContext``) the statistics are exchanged by peer stores from the GEMM epilogue instead
-    of an NCCL all-gather."""
+    of an NCCL all-gather. ``softcap``: the logits are ``cap * tanh(x @ w.T / cap)`` (0: uncapped)."""
     if _lib.use_cuda_kernels(x, w) and x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0:
-        return _LMHead.apply(x, w, labels, temperature, tp_group, vocab_start, tp_fused)
-    return lm_head_logprobs_ref(x, w, labels, temperature, tp_group, vocab_start)
+        return _LMHead.apply(x, w, labels, temperature, tp_group, vocab_start, tp_fused, softcap)
+    return lm_head_logprobs_ref(x, w, labels, temperature, tp_group, vocab_start, softcap)
 
 
 # --------------------------------------------------------------------------- fused sampling head
@@ -226,10 +247,10 @@ def new_sampling_rng(seed: int, device) -> torch.Tensor:
     return torch.tensor([int(seed) & 0x7FFFFFFFFFFFFFFF, 0], dtype=torch.int64, device=device)
 
 
-def lm_head_sample_ref(x, w, temperature, rng_state):
+def lm_head_sample_ref(x, w, temperature, rng_state, softcap=0.0):
     """PyTorch statement of the fused head: Gumbel-max over ``x @ w.T / temperature`` (argmax where the
     temperature is not positive) and the token's log-probability under the unfiltered distribution."""
-    logits = x.float() @ w.float().t()
+    logits = soft_cap(x.float() @ w.float().t(), softcap)
     t = temperature.float()
     noisy = t > 0
     scaled = logits / torch.where(noisy, t, torch.ones_like(t))[:, None]
@@ -242,14 +263,15 @@ def lm_head_sample_ref(x, w, temperature, rng_state):
     return tokens.to(torch.int32), logp
 
 
-def lm_head_sample(x: torch.Tensor, w: torch.Tensor, temperature: torch.Tensor, rng_state: torch.Tensor):
+def lm_head_sample(x: torch.Tensor, w: torch.Tensor, temperature: torch.Tensor, rng_state: torch.Tensor,
+                   softcap: float = 0.0):
     """Draws ``tokens[b] ~ softmax(x[b] @ w.T / temperature[b])`` inside the LM-head GEMM's epilogue (the
     ``[B, V]`` logits are never written) and returns ``(tokens int32 [B], logprobs f32 [B])``; rows with
     ``temperature <= 0`` take the argmax. Top-k / top-p filtering needs the whole row and goes through
     ``rollout_ops.sample`` on materialised logits instead. The inference servers the reference drives
     sample on materialised logits (areal/engine/sglang_remote.py:43-127 ``sampling_params``)."""
     if not (_lib.use_cuda_kernels(x, w) and x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0):
-        return lm_head_sample_ref(x, w, temperature, rng_state)
+        return lm_head_sample_ref(x, w, temperature, rng_state, softcap)
     B, H = x.shape
     V = w.shape[0]
     lib = _lib.kernels()
@@ -264,7 +286,7 @@ def lm_head_sample(x: torch.Tensor, w: torch.Tensor, temperature: torch.Tensor, 
     rc = lib.b200_lm_head_sample(_lib.ptr(x), _lib.ptr(w), _lib.ptr(temperature), _lib.ptr(partials),
                                  _lib.ptr(part_idx), _lib.ptr(rng_state), _lib.ptr(tokens), _lib.ptr(logps),
                                  ctypes.c_int(B), ctypes.c_int(V), ctypes.c_int(H), ctypes.c_longlong(x.stride(0)),
-                                 ctypes.c_longlong(w.stride(0)), _lib.stream_ptr())
+                                 ctypes.c_longlong(w.stride(0)), ctypes.c_float(softcap), _lib.stream_ptr())
     _lib.check(rc, "b200_lm_head_sample")
     _lib.count_launch(2)
     return tokens, logps

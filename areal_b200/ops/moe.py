@@ -25,15 +25,20 @@ from dataclasses import dataclass
 import torch
 
 from . import _lib, fused
-from .gemm import linear
+from .dyt import fp32_flag, kernel_ok
+from .gemm import gemm, linear
 
 
 # --------------------------------------------------------------------------- references
 
 
-def route_ref(logits: torch.Tensor, k: int, renorm: bool):
+def route_ref(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None):
     probs = logits.float().softmax(-1)
-    w, idx = probs.topk(k, dim=-1)
+    if correction is None:
+        w, idx = probs.topk(k, dim=-1)
+    else:
+        idx = (probs + correction.float()).topk(k, dim=-1).indices
+        w = probs.gather(-1, idx)
     if renorm:
         w = w / w.sum(-1, keepdim=True)
     return idx.to(torch.int32), w
@@ -72,19 +77,45 @@ def moe_experts_ref(x, idx, w, gate_up, down):
 # --------------------------------------------------------------------------- CUDA pieces
 
 
-def route(logits: torch.Tensor, k: int, renorm: bool):
-    """``logits [T, E]`` fp32 → ``(idx [T,k] int32, w [T,k] fp32)``."""
+def route(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None):
+    """``logits [T, E]`` fp32 → ``(idx [T,k] int32, w [T,k] fp32)``. ``correction [E]`` is added to the scores when the
+    experts are chosen; their weights are the scores without it."""
     T, E = logits.shape
-    if not (_lib.use_cuda_kernels(logits) and logits.dtype == torch.float32 and E <= 256 and k <= 32):
-        return route_ref(logits, k, renorm)
+    if not (_lib.use_cuda_kernels(logits) and logits.dtype == torch.float32 and E <= 256 and k <= 32
+            and (correction is None or correction.dtype in (torch.float32, torch.bfloat16))):
+        return route_ref(logits, k, renorm, correction)
     logits = logits if logits.is_contiguous() else logits.contiguous()
     idx = torch.empty((T, k), dtype=torch.int32, device=logits.device)
     w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
-    rc = _lib.kernels().b200_moe_route(_lib.ptr(logits), _lib.ptr(idx), _lib.ptr(w), ctypes.c_int(T), ctypes.c_int(E),
+    rc = _lib.kernels().b200_moe_route(_lib.ptr(logits), _lib.ptr(correction),
+                                       ctypes.c_int(int(correction is not None and correction.dtype == torch.float32)),
+                                       _lib.ptr(idx), _lib.ptr(w), ctypes.c_int(T), ctypes.c_int(E),
                                        ctypes.c_int(k), ctypes.c_int(int(renorm)), _lib.stream_ptr())
     _lib.check(rc, "b200_moe_route")
     _lib.count_launch()
     return idx, w
+
+
+def route_tokens(x: torch.Tensor, router: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None):
+    """Router projection (fp32 products and sums) and choice: ``x [T, H]``, ``router [E, H]``. A decode step's few tokens
+    take one kernel."""
+    T, H = x.shape
+    E = router.shape[0]
+    if kernel_ok(x, router) and T <= 256 and E <= 256 and k <= 32 and (H + E) * 4 <= 200 * 1024:
+        x = x if x.stride(1) == 1 and x.data_ptr() % 16 == 0 and x.stride(0) % 4 == 0 else x.contiguous()
+        idx = torch.empty((T, k), dtype=torch.int32, device=x.device)
+        w = torch.empty((T, k), dtype=torch.float32, device=x.device)
+        rc = _lib.kernels().b200_moe_router(
+            _lib.ptr(x), ctypes.c_longlong(x.stride(0)), _lib.ptr(router), _lib.ptr(correction), _lib.ptr(idx), _lib.ptr(w),
+            ctypes.c_int(T), ctypes.c_int(H), ctypes.c_int(E), ctypes.c_int(k), ctypes.c_int(int(renorm)), fp32_flag(x),
+            _lib.stream_ptr())
+        _lib.check(rc, "b200_moe_router")
+        _lib.count_launch()
+        return idx, w
+    if kernel_ok(x, router):
+        logits = gemm(x, router, out_dtype=torch.float32) if x.dtype == torch.bfloat16 else torch.nn.functional.linear(x, router)
+        return route(logits, k, renorm, correction)
+    return route_ref(torch.nn.functional.linear(x.float(), router.float()), k, renorm, correction)
 
 
 @dataclass
@@ -112,6 +143,14 @@ def sort_by_expert(idx: torch.Tensor, num_experts: int) -> ExpertSort:
     ints = lambda m: torch.empty(m, dtype=torch.int32, device=dev)
     s = ExpertSort(n, k, num_experts, max_vm * 128, ints(n), ints(max_vm * 128), ints(num_experts),
                    ints(num_experts + 1), ints(max_vm), ints(1))
+    if 0 < n <= 1024 and num_experts <= 256 and not _lib.checked():
+        rc = _lib.kernels().b200_moe_sort_small(_lib.ptr(idx), ctypes.c_int(n), ctypes.c_int(num_experts), _lib.ptr(s.counts),
+                                                _lib.ptr(s.prow0), _lib.ptr(s.tile_expert), _lib.ptr(s.num_vm),
+                                                _lib.ptr(s.dest), _lib.ptr(s.src_of), ctypes.c_int(max_vm),
+                                                _lib.stream_ptr())
+        _lib.check(rc, "b200_moe_sort_small")
+        _lib.count_launch()
+        return s
     chunk_hist = ints(max((n + 255) // 256, 1) * num_experts)
     if _lib.checked():
         _lib.check_index("moe_sort.expert_ids", idx, num_experts)
@@ -256,3 +295,81 @@ def moe_experts_forward(x, idx, w, gate_up, down):
     if not ok:
         return moe_experts_ref(x, idx, w, gate_up, down)
     return _MoEExperts.apply(x.contiguous(), idx, w, gate_up, down)
+
+
+# --------------------------------------------------------------------------- gated experts, forward only
+
+
+@dataclass(frozen=True)
+class GatedAct:
+    """``g' * sigmoid(alpha * g') * (u' + beta)`` with ``g' = min(g, limit)`` and ``u'`` clamped to ``[-limit, limit]``.
+    SwiGLU is ``GatedAct()``."""
+
+    alpha: float = 1.0
+    beta: float = 0.0
+    limit: float = float("inf")
+
+    def __call__(self, g, u):
+        gf, uf = g.float().clamp(max=self.limit), u.float().clamp(-self.limit, self.limit)
+        return (gf * torch.sigmoid(self.alpha * gf) * (uf + self.beta)).to(g.dtype)
+
+
+@dataclass
+class ExpertRows:
+    """Results of the chosen experts, not yet combined: row ``dest[t * k + j]`` of ``rows`` belongs to choice ``j`` of
+    token ``t`` and counts ``w[t, j]``."""
+
+    rows: torch.Tensor
+    dest: torch.Tensor
+    w: torch.Tensor
+
+
+def gated_experts_ref(x, idx, w, gate_up, down, act: GatedAct):
+    """``sum_j w[t,j] * down_e(act(gate_e x, up_e x))`` with the rows of ``gate_up [E, 2I, H]`` alternating between gate
+    and up; fp32 ``[T, H]``. Differentiable."""
+    out = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
+    for e in range(gate_up.shape[0]):
+        t, j = (idx == e).nonzero(as_tuple=True)
+        if t.numel() == 0:
+            continue
+        z = linear(x[t], gate_up[e])
+        y = linear(act(z[:, 0::2], z[:, 1::2]), down[e])
+        out = out.index_add(0, t, y.float() * w[t, j][:, None].float())
+    return out
+
+
+def gated_experts(x, idx, w, gate_up, down, act: GatedAct):
+    """The chosen experts of every token: ``x [T, H]``, ``idx / w [T, k]``, ``gate_up [E, 2I, H]`` (gate and up rows
+    alternate), ``down [E, H, I]``. On the kernels the result is an :class:`ExpertRows`, which the following norm combines
+    (``ops/layer_norm.py::experts_residual_ln``); elsewhere the combined ``[T, H]``. bf16 sizes in steps of 8 run on the
+    grouped tensor-core products with the activation in the first one's epilogue; 32-bit models and other sizes on a
+    grouped fp32 kernel. Everything stays on the device."""
+    if not kernel_ok(x, gate_up, down, w):
+        return gated_experts_ref(x, idx, w, gate_up, down, act)
+    T, H = x.shape
+    E, I2, _ = gate_up.shape
+    I, k = I2 // 2, idx.shape[1]
+    s = sort_by_expert(idx, E)
+    c, ll, f, p = ctypes.c_int, ctypes.c_longlong, ctypes.c_float, _lib.ptr
+    x = x if x.stride(1) == 1 and x.data_ptr() % 16 == 0 and x.stride(0) % 8 == 0 else x.contiguous()
+    new = lambda n: torch.empty((s.max_rows, n), dtype=x.dtype, device=x.device)
+    a, y = new(I), new(H)
+    glu = (f(act.limit), f(act.alpha), f(act.beta))
+    lib = _lib.kernels()
+    if x.dtype == torch.bfloat16 and H % 8 == 0 and I % 8 == 0 and T > 0:
+        xs = new(H)
+        _lib.check(lib.b200_moe_scatter(p(x), ll(x.stride(0)), p(s.dest), c(T), c(k), c(H), p(xs), _lib.stream_ptr()),
+                   "b200_moe_scatter")
+        _lib.check(lib.b200_gemm_grouped_glu(p(xs), p(gate_up), p(a), p(s.tile_expert), p(s.num_vm), p(s.src_of),
+                                             c(s.max_rows), c(E), c(I), c(H), *glu, _lib.stream_ptr()), "b200_gemm_grouped_glu")
+        _lib.check(lib.b200_gemm_grouped_rows(p(a), p(down), p(y), p(s.tile_expert), p(s.num_vm), p(s.src_of),
+                                              c(s.max_rows), c(E), c(H), c(I), _lib.stream_ptr()), "b200_gemm_grouped_rows")
+        _lib.count_launch(3)
+    else:
+        fp32, max_vm = fp32_flag(x), c(s.max_rows // 128)
+        for src, ld, gather, w_, out, n, kk, on in ((x, x.stride(0), k, gate_up, a, I2, H, 1), (a, I, 0, down, y, H, I, 0)):
+            _lib.check(lib.b200_moe_gemm_simt(p(src), ll(ld), c(gather), p(w_), p(out), ll(out.shape[1]), p(s.tile_expert),
+                                              p(s.num_vm), p(s.src_of), max_vm, c(n), c(kk), c(on), *glu, fp32,
+                                              _lib.stream_ptr()), "b200_moe_gemm_simt")
+        _lib.count_launch(2)
+    return ExpertRows(y, s.dest, w.float().contiguous())
