@@ -211,7 +211,7 @@ __global__ void moe_place_kernel(const int* __restrict__ idx, int n, int E, cons
 // passes above. Shared memory: [warps][E] counts, then [E + 1] first tiles.
 __global__ void moe_sort_small_kernel(const int* __restrict__ idx, int n, int E, int* __restrict__ counts,
                                       int* __restrict__ prow0, int* __restrict__ tile_expert, int* __restrict__ num_vm,
-                                      int* __restrict__ dest, int* __restrict__ src_of) {
+                                      int* __restrict__ dest, int* __restrict__ src_of, int max_rows) {
   extern __shared__ int ssm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   int* first = ssm + nw * E;
@@ -268,7 +268,7 @@ __global__ void moe_sort_small_kernel(const int* __restrict__ idx, int n, int E,
     prow0[E] = base << 7;
     *num_vm = base;
   }
-  for (int r = threadIdx.x; r < base << 7; r += blockDim.x) src_of[r] = -1;
+  for (int r = threadIdx.x; r < max_rows; r += blockDim.x) src_of[r] = -1;
   __syncthreads();
   if (valid) {
     const int pos = (first[e] << 7) + ssm[warp * E + e] + rank;
@@ -665,7 +665,7 @@ int b200_moe_router(const void* x, long long ldx, const void* wr, const void* co
   return 0;
 }
 
-// The sort for n <= 1024 copies; outputs as b200_moe_sort (src_of is set for the tiles in use only).
+// The sort for n <= 1024 copies; outputs as b200_moe_sort.
 int b200_moe_sort_small(const int* idx, int n, int E, int* counts, int* prow0, int* tile_expert, int* num_vm, int* dest,
                         int* src_of, int max_vm, cudaStream_t stream) {
   using namespace b200;
@@ -673,7 +673,8 @@ int b200_moe_sort_small(const int* idx, int n, int E, int* counts, int* prow0, i
   if (max_vm < (n + 127) / 128 + E) return -101;
   const int block = (n + 31) / 32 * 32;
   const size_t sh = (static_cast<size_t>(block / 32) * E + E + 1) * sizeof(int);
-  moe_sort_small_kernel<<<1, block, sh, stream>>>(idx, n, E, counts, prow0, tile_expert, num_vm, dest, src_of);
+  moe_sort_small_kernel<<<1, block, sh, stream>>>(idx, n, E, counts, prow0, tile_expert, num_vm, dest, src_of,
+                                               max_vm * 128);
   B200_CHECK(cudaGetLastError());
   return 0;
 }
