@@ -37,7 +37,7 @@ import torch.nn.functional as F
 
 from ..ops import fused
 from ..ops.attention import VarlenMeta, varlen_attention
-from ..ops.gemm import linear
+from ..ops.gemm import linear, linear_pitched
 from .config import ModelConfig
 
 
@@ -213,7 +213,7 @@ class LatentAttention(nn.Module):
 
         H, D, R = self.H, self.D, self.R
         cos, sin = ctx.rotary(self.rot)
-        x = linear(y, self.inp)
+        x = linear_pitched(y, self.inp)
         gate = x[:, self.nq + self.nkv:] if self.ng else None
         if self.q_rank:
             cq, c, kr = la.latent_prep(x[:, :self.nq + self.nkv], self.q_norm, self.c_norm, self.rank, R, self.eps, cos, sin,

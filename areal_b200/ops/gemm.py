@@ -133,6 +133,16 @@ def _splitk_plan(M: int, N: int, K: int) -> int:
     return splits if splits >= 2 else 0
 
 
+def linear_pitched(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``x @ w.T`` whose rows start 16-byte aligned whatever the number of columns: slices of them feed kernels that want
+    aligned pitches."""
+    N = w.shape[0]
+    grad = torch.is_grad_enabled() and (x.requires_grad or w.requires_grad)
+    if N % 8 == 0 or grad or not (_lib.use_cuda_kernels(x, w) and x.dtype == torch.bfloat16):
+        return linear(x, w)
+    return gemm(x, w, out=torch.empty((x.shape[0], -(-N // 8) * 8), dtype=x.dtype, device=x.device)[:, :N])
+
+
 def linear_relu2(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     """``relu(x @ w.T)^2``. On the bf16 kernels the activation runs on the product's fp32 accumulators (for decode-sized
     products in the split-K reduction)."""

@@ -149,8 +149,8 @@ def heads_matmul(a: torch.Tensor, heads: int, width: int, w: torch.Tensor, trans
     B, stride = a.shape[0], a.shape[1] // heads
     n = w.shape[1] if transposed else w.shape[0] // heads
     if (a.dtype == torch.bfloat16 and kernel_ok(a, w) and stride % 8 == 0 and n % 8 == 0 and width % 8 == 0
-            and (not transposed or width % 64 == 0) and a.stride(1) == 1 and a.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0
-            and w.data_ptr() % 16 == 0):
+            and (not transposed or width % 64 == 0) and w.data_ptr() % 16 == 0):
+        a = _aligned(a, heads * stride)
         out = torch.empty((B, heads * n), dtype=a.dtype, device=a.device)
         rc = _lib.kernels().b200_gemm_heads(
             _lib.ptr(a), ctypes.c_longlong(a.stride(0)), ctypes.c_int(stride), _lib.ptr(w), ctypes.c_longlong(w.stride(0)),
@@ -162,6 +162,13 @@ def heads_matmul(a: torch.Tensor, heads: int, width: int, w: torch.Tensor, trans
     ah = a.view(B, heads, stride)[..., :width].transpose(0, 1)
     wh = w.view(heads, width, n) if transposed else w.view(heads, n, width).transpose(1, 2)
     return torch.bmm(ah, wh).transpose(0, 1).reshape(B, heads * n)
+
+
+def _aligned(t: torch.Tensor, width: int) -> torch.Tensor:
+    """``t [rows, width]`` as the tensor-core kernels take it: unit inner stride, 16-byte aligned rows."""
+    if t.shape[0] == 1 and t.stride(1) == 1:
+        t = t.as_strided(t.shape, (width, 1))  # the pitch of a single row means nothing
+    return t if t.stride(1) == 1 and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 else t.contiguous()
 
 
 def _ptrs(*ts):
@@ -242,7 +249,7 @@ def _latent_prefill_mma(q, kv, kr, meta, H, D, R, Dv, scale, window, gate):
     if Rp != R:
         kr = _pad_heads(kr, 1, R, Rp).view(T, Rp)
     kv, kr = (t if t.is_contiguous() and t.data_ptr() % 16 == 0 else t.contiguous() for t in (kv, kr))
-    q = q if q.stride(1) == 1 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 else q.contiguous()
+    q = _aligned(q, H * (Dp + Rp))
     c = ctypes.c_int
     out = torch.empty((T, H * Vp), dtype=q.dtype, device=q.device)
     rc = _lib.kernels().b200_latent_prefill(
@@ -321,9 +328,8 @@ def latent_decode(qa, q, cache, block_table, seq_lens, H: int, D: int, rot: int,
     rows = cache.view(-1, rank + rot)
     span = min(max_seq_len, window) if window else max_seq_len  # most keys that a query sees
     if (q.dtype == torch.bfloat16 and _lib.kernels().b200_latent_decode_ok(ctypes.c_int(rank), ctypes.c_int(rot)) == 0
-            and D % 8 == 0 and cache.is_contiguous() and cache.data_ptr() % 16 == 0
-            and all(t.stride(1) == 1 and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (qa, q))):
-        return _latent_decode_mma(qa, q, cache, block_table, seq_lens, H, D, rot, rank, scale, span, window, gate)
+            and D % 8 == 0 and cache.is_contiguous() and cache.data_ptr() % 16 == 0):
+        return _latent_decode_mma(_aligned(qa, H * rank), _aligned(q, H * (D + rot)), cache, block_table, seq_lens, H, D, rot, rank, scale, span, window, gate)
     nsplit = 1
     while B * -(-H // 4) * nsplit < 1184 and nsplit < 64 and span // (nsplit * 2) >= 64:
         nsplit *= 2

@@ -100,3 +100,15 @@ def random_weights(cfg, seed=0, sharp=1.0):
     nrm("final.norm")
     lin("head", cfg["vocab"], d, 3.0)
     return {n: t.to(torch.bfloat16).float() for n, t in out.items()}
+
+
+def settle_routing(cfg, w, seed=0):
+    """Corrections that decide every token's choice by themselves (scores are below 1): with reduced precision a close call
+    may fall either way, and a comparison must not rest on it. Weights still follow the token's scores."""
+    g = torch.Generator().manual_seed(seed)
+    for i, L in enumerate(cfg["layers"]):
+        if L["mlp"] is not None and L["mlp"]["kind"] == "moe":
+            c = torch.zeros(L["mlp"]["router"]["experts"])
+            c[torch.randperm(len(c), generator=g)[:L["mlp"]["router"]["top"]]] = 2.0
+            w[f"l{i}.mlp.correction"] = c
+    return w
