@@ -1,10 +1,12 @@
-"""Serving throughput of a layered (Fofosun) model beside the closest other family, the Bailing hybrid, at equal sizes,
-and the new kernels one by one beside their counterparts.
+"""Serving throughput of a layered model beside the closest other family at equal sizes, and its kernels one by one beside
+their counterparts.
 
-    python bench.py --serving [--serving-sizes s,m,l] [--serving-kernels]
+    python bench.py --serving [--serving-family fofosun|gatolix] [--serving-sizes s,m,l] [--serving-kernels]
 
-Models: 8 layers of the given width with random weights, 6 recurrent and 2 latent-attention layers, a feed-forward of the
-same width on each. Both run through the rollout engine's scheduler and step functions (captured decode graphs where the
+Fofosun beside the Bailing hybrid: 8 layers of the given width with random weights, 6 recurrent and 2 latent-attention
+layers, a feed-forward of the same width on each. Gatolix beside DeepSeek-V2: 8 layers of latent attention with a plain
+query projection, a dense feed-forward on the first, mixtures of 64 experts (6 per token) on the others; Gatolix with
+windows of 512 tokens and half of its layers reading another layer's latents. Both run through the rollout engine's scheduler and step functions (captured decode graphs where the
 family has them). Prefill: 8 prompts of 2048 tokens in one step. Decode: 64 sequences at a context of 2048 tokens.
 Times are CUDA events on the launching stream; weights, caches and states exceed the L2. Kernel timings flush the L2
 between iterations; fractions are of the measured peaks.
@@ -27,6 +29,8 @@ SIZES = {  # width, heads, query latent, latent, feed-forward
     "m": dict(width=2048, heads=16, q_rank=768, kv_rank=512, ff=6144),
     "l": dict(width=4096, heads=32, q_rank=1536, kv_rank=512, ff=12288),
 }
+EXPERT_FF = {"s": 704, "m": 1408, "l": 2048}
+EXPERTS, TOP, WINDOW = 64, 6, 512
 VOCAB, LAYERS = 32000, 8
 
 
@@ -49,6 +53,34 @@ def bailing_config(width, heads, q_rank, kv_rank, ff) -> ModelConfig:
                        kv_lora_rank=kv_rank, qk_nope_head_dim=128, qk_rope_head_dim=64, v_head_dim=128,
                        rope_interleave=True, lightning_group_size=4, lightning_head_dim=128, lightning_norm_groups=1,
                        partial_rotary_factor=0.5, max_position_embeddings=8192)
+
+
+def gatolix_config(width, heads, q_rank, kv_rank, ff, expert_ff) -> ModelConfig:
+    layers = []
+    for i in range(LAYERS):
+        m = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": kv_rank, "scale": 192 ** -0.5,
+             "mask": {"size": WINDOW}, "rot": {"base": 1e4, "dims": 64, "scaling": {
+                 "factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        if i >= LAYERS // 2:
+            m["kv_from"] = LAYERS // 2 - 1
+        mlp = {"kind": "dense", "ff": ff} if i == 0 else {
+            "kind": "moe", "router": {"experts": EXPERTS, "top": TOP}, "expert": {"ff": expert_ff, "limit": 7.0}}
+        layers.append({"type": "latent_attention", "mixer": m, "mlp": mlp})
+    return ModelConfig.from_hf_config({"architecture": "Gatolix", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6},
+                                       "logit_softcap": 30.0, "layers": layers})
+
+
+def deepseek_config(width, heads, q_rank, kv_rank, ff, expert_ff) -> ModelConfig:
+    return ModelConfig(model_type="deepseek_v2", vocab_size=VOCAB, hidden_size=width, intermediate_size=ff,
+                       num_hidden_layers=LAYERS, num_attention_heads=heads, num_key_value_heads=heads, head_dim=192,
+                       rope_theta=1e4, tie_word_embeddings=False, qk_norm=False, num_experts=EXPERTS,
+                       num_experts_per_tok=TOP, moe_intermediate_size=expert_ff, norm_topk_prob=False,
+                       moe_group_score_top=1, mlp_only_layers=[0], kv_lora_rank=kv_rank, qk_nope_head_dim=128,
+                       qk_rope_head_dim=64, v_head_dim=128, rope_interleave=True, max_position_embeddings=8192)
+
+
+FAMILIES = {"fofosun": (("fofosun", fofosun_config), ("bailing_hybrid", bailing_config)),
+            "gatolix": (("gatolix", gatolix_config), ("deepseek_v2", deepseek_config))}
 
 
 def _engine(cfg: ModelConfig, seqs: int, context: int, tokens: int):
@@ -128,7 +160,7 @@ def serve(cfg: ModelConfig, prompts=8, length=2048, batch=64, steps=20) -> dict:
     return out
 
 
-def main(sizes: list[str], kernels: bool, sampler=None) -> int:
+def main(sizes: list[str], kernels: bool, sampler=None, family: str = "fofosun") -> int:
     """``sampler``: samples the GPU's clocks while the models run (``start`` / ``stop``)."""
     t0 = time.time()
     if sampler is not None:
@@ -136,15 +168,16 @@ def main(sizes: list[str], kernels: bool, sampler=None) -> int:
     res: dict = {"benchmark": "serving", "layers": LAYERS, "dtype": "bf16", "data": "random tokens, random weights",
                  "prefill": "8 x 2048 tokens", "decode": "64 sequences at 2048 tokens", "models": {}}
     for name in sizes:
-        for fam, make in (("fofosun", fofosun_config), ("bailing_hybrid", bailing_config)):
-            res["models"][f"{fam}-{name}"] = serve(make(**SIZES[name]))
+        more = dict(expert_ff=EXPERT_FF[name]) if family == "gatolix" else {}
+        for fam, make in FAMILIES[family]:
+            res["models"][f"{fam}-{name}"] = serve(make(**SIZES[name], **more))
             torch.cuda.empty_cache()
     if sampler is not None:
         res["clocks"] = sampler.stop()
     if kernels:
-        from .bench_serving_kernels import run
+        from .bench_serving_kernels import run, run_gatolix
 
-        res["kernels"] = run()
+        res["kernels"] = run_gatolix() if family == "gatolix" else run()
     res["seconds"] = round(time.time() - t0)
     print(json.dumps(res), flush=True)
     return 0

@@ -3,14 +3,17 @@ algorithmic FLOPs over the measured bf16 peak and algorithmic bytes over the mea
 
 from __future__ import annotations
 
+import ctypes
+
 import numpy as np
 import torch
 
-from ..ops import dyt, fused, latent_attn as la
+from ..ops import _lib, dyt, fused, latent_attn as la, layer_norm as ln, moe
 from ..ops.attention import VarlenMeta, varlen_attention
 from ..ops.gated_scan import ScanSpec, scan_prefill, scan_step
-from ..ops.gemm import linear_rmsnorm
+from ..ops.gemm import linear, linear_relu2, linear_rmsnorm
 from ..ops.linear_attn import linear_attn_prefill, linear_attn_step
+from ..ops.lm_head import lm_head_sample, new_sampling_rng
 from ..ops.microbench import peaks, timeit
 from ..ops.rollout_ops import paged_decode
 
@@ -117,4 +120,120 @@ def run() -> list[dict]:
     ids = torch.from_numpy(np.random.default_rng(0).integers(0, 32000, T)).to("cuda")
     table = _rand(32000, W)
     out.append(_row("embed_dyt 16384 x 2048", lambda: dyt.embed_dyt(ids, table, norm), T * W * 8))
+    return out
+
+
+@torch.no_grad()
+def run_gatolix() -> list[dict]:
+    """Kernels of the Gatolix family beside those of the families with like ones."""
+    out = []
+    torch.manual_seed(0)
+    H, D, R, rank, n, L, B, W, win = 16, 128, 64, 512, 8, 2048, 64, 2048, 512
+    T = n * L
+    add = lambda *a, **k: out.append(_row(*a, **k))
+    # --- latent attention: FLOPs of the visible pairs, bytes of the visible rows
+    meta = VarlenMeta([L * i for i in range(n + 1)], "cuda")
+    x, kv, kr = _rand(T, H * (D + R) + rank + R + H), _rand(T, H * 2 * D), _rand(T, R)
+    q, gate = x[:, :H * (D + R)], x[:, -H:]
+    qc = q.contiguous()
+    per = 2 * (D + R + D) * n * H
+    pairs = L * L / 2
+    seen = sum(min(i + 1, win) for i in range(L))
+    add("latent_prefill 8x2048, window 512, gate", lambda: la.latent_attention(q, kv, kr, meta, H, D, R, D, 0.07, win, gate), 0, per * seen)
+    add("latent_prefill 8x2048, gate", lambda: la.latent_attention(q, kv, kr, meta, H, D, R, D, 0.07, None, gate), 0, per * pairs)
+    add("[fofosun] latent_prefill 8x2048", lambda: la.latent_attention(qc, kv, kr, meta, H, D, R, D, 0.07), 0, per * pairs)
+    ctx, bs = 2048, 16
+    nb = B * ctx // bs
+    bt = torch.randperm(nb, device="cuda").view(B, -1).int()
+    lens = torch.full((B,), ctx, device="cuda", dtype=torch.int32)
+    cache = _rand(nb, 1, bs, rank + R)
+    qa = _rand(B, H * rank, s=0.1)
+    row = (rank + R) * 2
+    add("latent_decode 64 x 2048, window 512, gate", lambda: la.latent_decode(qa, q[:B], cache, bt, lens, H, D, R, rank, 0.07, ctx, win, gate[:B]), B * win * row)
+    add("latent_decode 64 x 2048, window 2048, gate", lambda: la.latent_decode(qa, q[:B], cache, bt, lens, H, D, R, rank, 0.07, ctx, ctx, gate[:B]), B * ctx * row)
+    add("[fofosun] latent_decode 64 x 512", lambda: la.latent_decode(qa, qc[:B], cache, bt, lens // 4, H, D, R, rank, 0.07, win), B * win * row)
+    add("[fofosun] latent_decode 64 x 2048", lambda: la.latent_decode(qa, qc[:B], cache, bt, lens, H, D, R, rank, 0.07, ctx), B * ctx * row)
+    cos, sin = la.rotary_tables(L, R, 1e4, "cuda")
+    pos = torch.arange(L, device="cuda", dtype=torch.int32).repeat(n)
+    wq, wc = _rand(768), _rand(rank)
+    moved = (H * R + rank + R) * 4
+    add("latent_qkv_prep 16384 tokens", lambda: la.latent_qkv_prep(x, H, D, wc, rank, R, 1e-6, cos, sin, pos), T * moved)
+    add("latent_qkv_prep batch 64", lambda: la.latent_qkv_prep(x[:B], H, D, wc, rank, R, 1e-6, cos, sin, pos[:B]), B * moved)
+    xd = _rand(T, 768 + rank + R)
+    add("[fofosun] latent_prep 16384 tokens", lambda: la.latent_prep(xd, wq, wc, rank, R, 1e-6, cos, sin, pos), T * (768 + rank + R) * 4)
+    add("rope_pairs 16384 tokens x 16 heads x 64, in wider rows", lambda: la.rope_pairs_(q, H, D, R, cos, sin, pos), T * H * R * 4)
+    add("[fofosun] rope_pairs 16384 tokens x 16 heads x 64", lambda: la.rope_pairs_(qc, H, D, R, cos, sin, pos), T * H * R * 4)
+    # --- norms around the residual
+    v = lambda: (_rand(W), _rand(W))
+    post, norm, res, resb, wn = v(), v(), _rand(T, W, dt=F32), _rand(T, W), _rand(W)
+    dn = (torch.tensor(0.5, device="cuda", dtype=BF), _rand(W), _rand(W))
+    aw, ww = _rand(T, W), _rand(W, W, s=W ** -0.5)
+    add("residual_ln 16384 x 2048 (two norms)", lambda: ln.residual_ln(aw, post, res, norm, 1e-6), T * W * 12)
+    add("[fofosun] residual_dyt 16384 x 2048", lambda: dyt.residual_dyt(aw, wn, res, dn), T * W * 12)
+    add("[deepseek] rmsnorm + residual 16384 x 2048", lambda: fused.rmsnorm(aw, wn, 1e-6, residual=resb), T * W * 8)
+    add("residual_ln 64 x 2048", lambda: ln.residual_ln(aw[:B], post, res[:B], norm, 1e-6), B * W * 12, iters=20)
+    add("[deepseek] rmsnorm + residual 64 x 2048", lambda: fused.rmsnorm(aw[:B], wn, 1e-6, residual=resb[:B]), B * W * 8, iters=20)
+    add("linear_residual_ln 16384 x 2048 x 2048", lambda: ln.linear_residual_ln(aw, ww, post, res, norm, 1e-6), T * W * 12, 2.0 * T * W * W)
+    add("[fofosun] linear_residual_dyt 16384 x 2048 x 2048", lambda: dyt.linear_residual_dyt(aw, ww, wn, res, dn), T * W * 12, 2.0 * T * W * W)
+    add("[deepseek] linear + rmsnorm 16384 x 2048 x 2048", lambda: linear_rmsnorm(aw, ww, wn, 1e-6, resb), T * W * 10, 2.0 * T * W * W)
+    add("linear_residual_ln 64 x 2048 x 2048", lambda: ln.linear_residual_ln(aw[:B], ww, post, res[:B], norm, 1e-6), W * W * 2, iters=20)
+    add("[deepseek] linear_rmsnorm 64 x 2048 x 2048", lambda: linear_rmsnorm(aw[:B], ww, wn, 1e-6, resb[:B]), W * W * 2, iters=20)
+    ids = torch.from_numpy(np.random.default_rng(0).integers(0, 32000, T)).to("cuda")
+    table = _rand(32000, W)
+    add("embed_ln 16384 x 2048", lambda: ln.embed_ln(ids, table, norm, 1e-6), T * W * 8)
+    add("[fofosun] embed_dyt 16384 x 2048", lambda: dyt.embed_dyt(ids, table, dn), T * W * 8)
+    # --- dense feed-forward
+    F = 6144
+    wu = _rand(F, W, s=W ** -0.5)
+    add("linear_relu2 16384 x 2048 -> 6144", lambda: linear_relu2(aw, wu), T * (W + F) * 2, 2.0 * T * W * F)
+    add("[any] linear 16384 x 2048 -> 6144", lambda: linear(aw, wu), T * (W + F) * 2, 2.0 * T * W * F)
+    add("linear_relu2 64 x 2048 -> 6144", lambda: linear_relu2(aw[:B], wu), W * F * 2, iters=20)
+    add("[any] linear 64 x 2048 -> 6144", lambda: linear(aw[:B], wu), W * F * 2, iters=20)
+    # --- mixture of experts
+    E, k, ff = 64, 6, 1408
+    rw, corr = _rand(E, W, s=W ** -0.5), _rand(E, s=0.1)
+    gu, down = _rand(E, 2 * ff, W, s=W ** -0.5), _rand(E, W, ff, s=ff ** -0.5)
+    act = moe.GatedAct(1.702, 1.0, 7.0)
+    for t in (T, B):
+        xt = aw[:t]
+        it = 20 if t == B else 10
+        route_bytes = t * W * 2 + E * W * 2
+        add(f"route_tokens {t} x 2048, 64 experts", lambda: moe.route_tokens(xt, rw, k, False, corr), route_bytes, iters=it)
+        add(f"[deepseek] fp32 router projection + route {t}", lambda: moe.route(torch.nn.functional.linear(xt.float(), rw.float()), k, False), route_bytes, iters=it)
+        idx, w = moe.route_tokens(xt, rw, k, False, corr)
+        add(f"sort {t} x 6", lambda: moe.sort_by_expert(idx, E), t * k * 16, iters=it)
+        s = moe.sort_by_expert(idx, E)
+        live = int((s.counts > 0).sum())
+        weights = lambda m: live * m * W * 2
+        rows = t * k
+        xs = moe.gather_rows(xt, s)
+        p, c, st = _lib.ptr, ctypes.c_int, _lib.stream_ptr
+        lib = _lib.kernels()
+        h, y = torch.empty(s.max_rows, ff, device="cuda", dtype=BF), torch.empty(s.max_rows, W, device="cuda", dtype=BF)
+        glu = tuple(ctypes.c_float(f) for f in (act.limit, act.alpha, act.beta))
+        tail = (p(s.tile_expert), p(s.num_vm), p(s.src_of), c(s.max_rows), c(E))
+        add(f"moe_scatter {t} x 6", lambda: lib.b200_moe_scatter(p(xt), ctypes.c_longlong(W), p(s.dest), c(t), c(k), c(W), p(xs), st()),
+            (t + rows) * W * 2, iters=it)
+        add(f"[deepseek] gather {t} x 6", lambda: moe.gather_rows(xt, s), (t + rows) * W * 2, iters=it)
+        add(f"grouped gate | up + activation {t} x 6", lambda: lib.b200_gemm_grouped_glu(p(xs), p(gu), p(h), *tail, c(ff), c(W), *glu, st()),
+            weights(2 * ff) + rows * (W + ff) * 2, 4.0 * rows * W * ff, iters=it)
+        add(f"[deepseek] grouped gate | up, then SwiGLU {t} x 6", lambda: moe._swiglu_raw(moe.grouped_gemm(xs, gu, s)),
+            weights(2 * ff) + rows * (W + ff) * 2, 4.0 * rows * W * ff, iters=it)
+        add(f"grouped down {t} x 6", lambda: lib.b200_gemm_grouped_rows(p(h), p(down), p(y), *tail, c(W), c(ff), st()),
+            weights(ff) + rows * (W + ff) * 2, 2.0 * rows * W * ff, iters=it)
+        add(f"[deepseek] grouped down {t} x 6", lambda: moe.grouped_gemm(h, down, s),
+            weights(ff) + rows * (W + ff) * 2, 2.0 * rows * W * ff, iters=it)
+        e = moe.ExpertRows(y, s.dest, w)
+        add(f"experts_residual_ln {t} x 6 (combine, two norms)", lambda: ln.experts_residual_ln(e, post, res[:t], norm, 1e-6),
+            t * W * (2 * k + 10), iters=it)
+        add(f"[deepseek] combine {t} x 6, then rmsnorm + residual", lambda: fused.rmsnorm(moe.combine_rows(y, s, w), wn, 1e-6, residual=resb[:t]),
+            t * W * (2 * k + 8), iters=it)
+        add(f"route, experts, combine, norms {t}", lambda: ln.experts_residual_ln(moe.gated_experts(xt, *moe.route_tokens(xt, rw, k, False, corr), gu, down, act), post, res[:t], norm, 1e-6),
+            weights(3 * ff), 6.0 * rows * W * ff, iters=it)
+        add(f"[deepseek] route, experts, combine, norm {t}", lambda: fused.rmsnorm(moe.moe_experts_forward(xt, *moe.route(torch.nn.functional.linear(xt.float(), rw.float()), k, False), gu, down), wn, 1e-6, residual=resb[:t]),
+            weights(3 * ff), 6.0 * rows * W * ff, iters=it)
+    # --- head
+    wl, temp, rng = _rand(32000, W, s=W ** -0.5), torch.ones(B, device="cuda"), new_sampling_rng(0, "cuda")
+    add("lm_head_sample batch 64, soft cap", lambda: lm_head_sample(aw[:B], wl, temp, rng, softcap=30.0), 32000 * W * 2, iters=20)
+    add("[any] lm_head_sample batch 64", lambda: lm_head_sample(aw[:B], wl, temp, rng), 32000 * W * 2, iters=20)
     return out
