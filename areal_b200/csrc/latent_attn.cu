@@ -161,6 +161,16 @@ __global__ void latent_qkv_prep_kernel(T* __restrict__ x, long long ldx, int H, 
   }
   const int first = blockDim.x > 32 ? threadIdx.x - 32 : threadIdx.x;
   const int step = blockDim.x > 32 ? blockDim.x - 32 : blockDim.x;
+  if (V == 4 && PAIR && !(half & 1) && !(D & 3)) {  // two pairs at a time
+    for (int i = first; i < H * (half >> 1); i += step) {
+      const int h = i / (half >> 1), e = (i - h * (half >> 1)) * 2;
+      T* q = row + static_cast<long long>(h) * (D + rot) + D + 2 * e;
+      const float4 v = ld4(q);
+      const float2 cs = *reinterpret_cast<const float2*>(cr + e), sn = *reinterpret_cast<const float2*>(sr + e);
+      st4(q, make_float4(v.x * cs.x - v.y * sn.x, v.y * cs.x + v.x * sn.x, v.z * cs.y - v.w * sn.y, v.w * cs.y + v.z * sn.y));
+    }
+    return;
+  }
   for (int i = first; i < H * half; i += step) {
     const int h = i / half, e = i - h * half;
     T* q = row + static_cast<long long>(h) * (D + rot) + D + 2 * e;

@@ -90,8 +90,25 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const C* __re
   route_token<PER>(z, correction, E, k, renorm, idx + t * k, w + t * k);
 }
 
+__device__ __forceinline__ float dot8(const float* w, const float* x, float s) {
+  const float4 a = ld4(w), b = ld4(w + 4), c = ld4(x), d = ld4(x + 4);
+  s = fmaf(a.x, c.x, fmaf(a.y, c.y, fmaf(a.z, c.z, fmaf(a.w, c.w, s))));
+  return fmaf(b.x, d.x, fmaf(b.y, d.y, fmaf(b.z, d.z, fmaf(b.w, d.w, s))));
+}
+__device__ __forceinline__ float dot8(const __nv_bfloat16* w, const float* x, float s) {
+  const uint4 raw = *reinterpret_cast<const uint4*>(w);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 f = __bfloat1622float2(h[j]), g = *reinterpret_cast<const float2*>(x + 2 * j);
+    s = fmaf(f.x, g.x, fmaf(f.y, g.y, s));
+  }
+  return s;
+}
+
 // Router projection and choice of a few tokens (a decode step): one block per token, the token's vector in shared memory,
-// a warp per expert in turn. Products and sums in fp32.
+// a warp per pair of experts in turn (the weights come from L2: two rows with several loads each in flight hide its
+// latency). Products and sums in fp32.
 template <int PER, class D>
 __global__ void moe_router_kernel(const D* __restrict__ x, long long ldx, const D* __restrict__ wr,
                                   const D* __restrict__ correction, int* __restrict__ idx, float* __restrict__ w, int H,
@@ -102,21 +119,30 @@ __global__ void moe_router_kernel(const D* __restrict__ x, long long ldx, const 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   for (int c = threadIdx.x; c < H; c += blockDim.x) rsm[c] = ld1(x + t * ldx + c);
   __syncthreads();
-  const bool v4 = H % 4 == 0;
-  for (int e = warp; e < E; e += nw) {
+  const bool v8 = H % 8 == 0;
+  for (int e = warp * 2; e < E; e += nw * 2) {
+    const int e1 = min(e + 1, E - 1);
     const D* row = wr + static_cast<long long>(e) * H;
-    float s = 0.f;
-    if (v4) {
+    const D* row1 = wr + static_cast<long long>(e1) * H;
+    float s = 0.f, s1 = 0.f;
+    if (v8) {
 #pragma unroll 4
-      for (int c = lane * 4; c < H; c += 128) {
-        const float4 a = ld4(row + c), b = *reinterpret_cast<const float4*>(rsm + c);
-        s = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, s))));
+      for (int c = lane * 8; c < H; c += 256) {
+        s = dot8(row + c, rsm + c, s);
+        s1 = dot8(row1 + c, rsm + c, s1);
       }
     } else {
-      for (int c = lane; c < H; c += 32) s = fmaf(ld1(row + c), rsm[c], s);
+      for (int c = lane; c < H; c += 32) {
+        s = fmaf(ld1(row + c), rsm[c], s);
+        s1 = fmaf(ld1(row1 + c), rsm[c], s1);
+      }
     }
     s = warp_sum(s);
-    if (lane == 0) z[e] = s;
+    s1 = warp_sum(s1);
+    if (lane == 0) {
+      z[e] = s;
+      z[e1] = e1 == e ? s : s1;
+    }
   }
   __syncthreads();
   if (warp == 0) {
@@ -648,7 +674,7 @@ int b200_moe_router(const void* x, long long ldx, const void* wr, const void* co
   if (T == 0) return 0;
   const size_t smem = static_cast<size_t>(H + E) * sizeof(float);
   if (E > 256 || k > 32 || k > E || smem > 200 * 1024) return -100;
-  const int per = (E + 31) / 32, block = E > 64 ? 512 : 256;
+  const int per = (E + 31) / 32, block = E > 32 ? 1024 : (E > 16 ? 512 : 256);
 #define RT(P, D)                                                                                                    \
   {                                                                                                                 \
     if (smem > 48 * 1024)                                                                                           \
