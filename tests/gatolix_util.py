@@ -31,8 +31,8 @@ def config(layers, width=48, vocab=97, eps=1e-5, cap=9.0):
 
 Y = (4.0, 64, 8.0, 1.0)  # YaRN whose ramp lies inside the pairs of the small rotations below
 
-# name -> configuration. "odd": no size is a multiple of 8; "ones": sizes and counts of one; "tile": sizes that the
-# tensor-core kernels take.
+# name -> configuration. "odd": no size is a multiple of 8; "ones": sizes and counts of one; "padded": sizes
+# that are padded for the tensor-core kernels; "tile": sizes that these take as they are.
 CONFIGS = {
     "mixed": config([latent(3, 16, 8, 24, 32, 0.2, 12, 500.0, Y, mlp=moe(5, 2, 24, 1.5)),
                      latent(2, 24, 16, 16, 40, 0.17, 33, 300.0, (8.0, 100, 4.0, 0.5), mlp=dense(56)),
@@ -46,6 +46,8 @@ CONFIGS = {
                     latent(1, 2, 2, 1, 1, 0.9, 2, 10.0, (1.0, 2048, 32.0, 1.0), kv_from=0, mlp=dense(1))], width=16, vocab=31),
     "plain": config([latent(2, 16, 4, 16, 24, 0.2, mlp=dense(32)), latent(2, 16, 4, 8, 24, 0.2, kv_from=0)], width=40,
                     vocab=70, cap=None),
+    "padded": config([latent(4, 96, 48, 80, 96, 0.11, 45, 2e3, (3.0, 300, 12.0, 2.0), mlp=moe(10, 5, 40, 1.8)),
+                      latent(12, 40, 48, 104, 96, 0.15, 17, 2e3, (3.0, 300, 12.0, 2.0), kv_from=0, mlp=dense(200))], width=136, vocab=120),
     "tile": config([latent(3, 64, 32, 64, 128, 0.12, 100, 1e4, (4.0, 256, 16.0, 1.0), mlp=moe(12, 4, 72, 2.0)),
                     latent(18, 64, 64, 32, 192, 0.1, 31, 5e3, (16.0, 128, 8.0, 1.0), mlp=dense(1056)),
                     latent(2, 128, 64, 128, 192, 0.07, 64, 5e3, (16.0, 128, 8.0, 1.0), kv_from=1, mlp=moe(20, 2, 136, 1.5)),
