@@ -18,6 +18,15 @@ from tests import gatolix_oracle as oracle
 from tests.fofosun_util import TraceReplay, make_engine, rel_error, run_batch, tokens, write_checkpoint
 from tests.gatolix_util import CONFIGS, Y, config, dense, latent, moe, random_weights
 
+@pytest.fixture(autouse=True)
+def _few_threads():
+    """Everything here is tiny: waking a host's cores for each step only costs time."""
+    n = torch.get_num_threads()
+    torch.set_num_threads(1)
+    yield
+    torch.set_num_threads(n)
+
+
 ROOT = Path(__file__).resolve().parent.parent
 TOL = 3e-5
 
