@@ -34,6 +34,8 @@ class TraceReplay:
 
     def __init__(self, engine):
         self.e = engine
+        # every request runs its own prompt: a request that forks from an equal prompt has no hidden states for it
+        engine.sched.set_prompt_sharing(False)
         self.rid: dict[str, int] = {}      # live requests
         self.planned: list[int] = []       # request ids of the last plan, in its order; their next tokens are due
 

@@ -502,3 +502,22 @@ def test_trace_runner_command(tmp_path):
     for i, t in {0: wa[[0, 17]], 1: wb[[8]], 2: wa[[19]], 3: wb[[3]]}.items():
         got = torch.from_numpy(np.fromfile(tmp_path / "out" / f"{i}.f32", dtype="<f4")).view(-1, cfg["vocab"])
         assert rel_error(got, t) < TOL
+
+
+def test_replay_of_equal_prompts_in_one_batch(tmp_path):
+    """Requests that start alike still run each by itself, and go on differently."""
+    cfg = CONFIGS["mixed"]
+    w = random_weights(cfg, 29)
+    write_checkpoint(tmp_path, cfg, w)
+    a = tokens(40, cfg["vocab"], 1)
+    reqs = {"a": a, "b": list(a), "c": a[:33] + tokens(5, cfg["vocab"], 2), "d": tokens(9, cfg["vocab"], 3)}
+    eng = make_engine(tmp_path)
+    try:
+        r = TraceReplay(eng)
+        for cuts in ({"a": 30, "b": 30, "c": 30, "d": 5}, {"a": 32, "b": 35, "c": 32, "d": 9}):
+            got = run_batch(r, reqs, cuts)
+            for k, v in reqs.items():
+                assert rel_error(got[k], oracle.forward(cfg, w, v)) < TOL
+        assert eng.sched.stats()["prompt_forks"] == 0
+    finally:
+        eng.destroy()

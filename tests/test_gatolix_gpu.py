@@ -393,11 +393,13 @@ def test_greedy_generation_with_decode_graphs(tmp_path, dtype):
     if dtype == "bfloat16":
         settle_routing(cfg, w)
     write_checkpoint(tmp_path, cfg, w)
-    prompts = [tokens(n, cfg["vocab"], 20 + n) for n in (1, 19, 2, 33, 47, 11, 16)]
-    new = [9, 24, 30, 6, 15, 20, 17]
+    prompts = [tokens(n, cfg["vocab"], 20 + n) for n in (1, 19, 2, 33, 47, 11, 16)] + [tokens(37, cfg["vocab"], 18)] * 3
+    new = [9, 24, 30, 6, 15, 20, 17, 12, 25, 40]
     eng = make_engine(tmp_path, "cuda", dtype, start_loop=True, seqs=4, blocks=64, context=128)
     try:
-        for p, n, r in zip(prompts, new, _generate(eng, prompts, new)):
+        outs = _generate(eng, prompts, new)
+        assert eng.sched.stats()["prompt_forks"] > 0                             # the last three share their prompt's pages
+        for p, n, r in zip(prompts, new, outs):
             assert len(r.output_tokens) == n
             lg = oracle.forward(cfg, w, p + r.output_tokens)[len(p) - 1:-1]
             got = lg.gather(1, torch.tensor(r.output_tokens)[:, None]).squeeze(1)
