@@ -183,14 +183,35 @@ struct GroupedEpi {
   }
 };
 
+// 32 neighbouring accumulators (alternating gate and up, times `scale`) to 16 activations of a row
+__device__ __forceinline__ void store_glu(__nv_bfloat16* out, int inter, int row, int col0, const float (&v)[32], float scale,
+                                          GluParams glu) {
+  __nv_bfloat16* p = out + static_cast<long long>(row) * inter + col0 / 2;
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    if (col0 / 2 + 8 * i >= inter) break;
+    uint4 o;
+    __nv_bfloat162* ob = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = 16 * i + 4 * j;
+      ob[j] = __floats2bfloat162_rn(glu_act(v[c] * scale, v[c + 1] * scale, glu, ob),
+                                    glu_act(v[c + 2] * scale, v[c + 3] * scale, glu, ob));
+    }
+    reinterpret_cast<uint4*>(p)[i] = o;
+  }
+}
+
 // The experts' first product with its gated activation on the accumulators. Gate and up rows of the weight alternate
-// (row 2i: gate i, row 2i + 1: up i), so neighbouring columns meet in one thread and half as many are written.
+// (row 2i: gate i, row 2i + 1: up i), so neighbouring columns meet in one thread and half as many are written. scale (null:
+// none): a row's products count scale[src_of[row]] times ahead of the activation.
 struct GroupedGluEpi {
   __nv_bfloat16* out;     // [rows, inter]
   GluParams glu;
   int inter;              // N / 2, a multiple of 8
   const int *tile_expert, *num_vm, *src_of;
-  struct State { bool live; };
+  const float* scale;
+  struct State { bool live; float s; };
 
   __device__ __forceinline__ bool tile(int cta, int ncta, int it, int, int tiles_n, int& m_blk, int& n_blk) const {
     const long long t = static_cast<long long>(it) * ncta + cta;
@@ -201,23 +222,32 @@ struct GroupedGluEpi {
   }
   __device__ __forceinline__ int b_offset(int m_blk) const { return tile_expert[m_blk] * 2 * inter; }
   __device__ __forceinline__ bool gate(int, int, volatile int*, int*) const { return true; }
-  __device__ __forceinline__ void begin(State& s, int, int, int row) const { s.live = src_of[row] >= 0; }
+  __device__ __forceinline__ void begin(State& s, int, int, int row) const {
+    const int src = src_of[row];
+    s.live = src >= 0;
+    s.s = scale && s.live ? scale[src] : 1.f;
+  }
   __device__ __forceinline__ void end(State&, int, int, int) const {}
   __device__ __forceinline__ void chunk(State& s, int row, int col0, const float (&v)[32]) const {
-    if (!s.live) return;
-    __nv_bfloat16* p = out + static_cast<long long>(row) * inter + col0 / 2;
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      if (col0 / 2 + 8 * i >= inter) break;
-      uint4 o;
-      __nv_bfloat162* ob = reinterpret_cast<__nv_bfloat162*>(&o);
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int c = 16 * i + 4 * j;
-        ob[j] = __floats2bfloat162_rn(glu_act(v[c], v[c + 1], glu, ob), glu_act(v[c + 2], v[c + 3], glu, ob));
-      }
-      reinterpret_cast<uint4*>(p)[i] = o;
-    }
+    if (s.live) store_glu(out, inter, row, col0, v, s.s, glu);
+  }
+};
+
+// The same activation behind a plain product
+struct GluEpi {
+  __nv_bfloat16* out;     // [M, inter]
+  GluParams glu;
+  int M, inter;
+  struct State {};
+  __device__ __forceinline__ bool tile(int cta, int ncta, int it, int tiles_m, int tiles_n, int& m_blk,
+                                       int& n_blk) const {
+    return default_tile(cta, ncta, it, tiles_m, tiles_n, m_blk, n_blk);
+  }
+  __device__ __forceinline__ bool gate(int, int, volatile int*, int*) const { return true; }
+  __device__ __forceinline__ void begin(State&, int, int, int) const {}
+  __device__ __forceinline__ void end(State&, int, int, int) const {}
+  __device__ __forceinline__ void chunk(State&, int row, int col0, const float (&v)[32]) const {
+    if (row < M) store_glu(out, inter, row, col0, v, 1.f, glu);
   }
 };
 
@@ -340,6 +370,22 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ ws, const __nv_bf
     pk.x = *reinterpret_cast<uint32_t*>(&lo);
     pk.y = *reinterpret_cast<uint32_t*>(&hi);
     *reinterpret_cast<uint2*>(out + static_cast<long long>(row) * ldc + c) = pk;
+  }
+}
+
+__global__ void splitk_reduce_glu_kernel(const float* __restrict__ ws, __nv_bfloat16* __restrict__ out, int M, int N, int S,
+                                         long long slice_stride, GluParams glu) {
+  const int nq = N >> 2;
+  const long long total = static_cast<long long>(M) * nq;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < S; ++s) {
+      const float4 v = *reinterpret_cast<const float4*>(ws + s * slice_stride + i * 4);
+      acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
+    }
+    __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(out) + i;
+    *o = __floats2bfloat162_rn(glu_act(acc.x, acc.y, glu, o), glu_act(acc.z, acc.w, glu, o));
   }
 }
 
@@ -583,8 +629,8 @@ int b200_gemm_grouped_rows(const void* A, const void* B, void* C, const int* til
 // The same with the gated activation behind it: W stacked [E, 2 * inter, K] with alternating gate and up rows, C [rows,
 // inter]. inter % 8 == 0, K % 8 == 0.
 int b200_gemm_grouped_glu(const void* A, const void* B, void* C, const int* tile_expert, const int* num_vm,
-                          const int* src_of, int max_rows, int E, int inter, int K, float limit, float alpha,
-                          float beta, cudaStream_t stream) {
+                          const int* src_of, const float* scale, int max_rows, int E, int inter, int K, float limit,
+                          float alpha, float beta, cudaStream_t stream) {
   using namespace b200;
   if (max_rows <= 0 || inter <= 0 || K <= 0) return 0;
   if ((inter & 7) || (K & 7)) return -100;
@@ -596,7 +642,7 @@ int b200_gemm_grouped_glu(const void* A, const void* B, void* C, const int* tile
   if (rc) return rc;
   rc = make_tmap_2d(&tmB, B, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (long long)E * N, K, (long long)K * 2, BN, 64);
   if (rc) return rc;
-  GroupedGluEpi epi{(__nv_bfloat16*)C, GluParams{limit, alpha, beta}, inter, tile_expert, num_vm, src_of};
+  GroupedGluEpi epi{(__nv_bfloat16*)C, GluParams{limit, alpha, beta}, inter, tile_expert, num_vm, src_of, scale};
   auto kern = gemm_tcgen05_kernel<BN, false, false, GroupedGluEpi>;
   static bool attr_set = false;
   if (!attr_set) {
@@ -814,6 +860,33 @@ int b200_gemm_bf16_relu2(const void* A, const void* B, void* C, float* workspace
     return 0;
   }
   const Relu2Epi epi{StoreEpi{C, nullptr, N, M, N, 0, 0}};
+  const long long tiles256 = static_cast<long long>((M + kBM - 1) / kBM) * ((N + 255) / 256);
+  return tiles256 >= 100 ? launch_epi<256>(A, B, epi, M, N, K, lda, ldb, stream)
+                         : launch_epi<128>(A, B, epi, M, N, K, lda, ldb, stream);
+}
+
+// C [M, inter] (bf16, pitch inter) = the gated activation of A . B^T, B [2 * inter, K] with alternating gate and up rows.
+// splits > 1: split-K with the activation in the reduction. inter % 8 == 0.
+int b200_gemm_bf16_glu(const void* A, const void* B, void* C, float* workspace, int M, int inter, int K, long long lda,
+                       long long ldb, int splits, float limit, float alpha, float beta, cudaStream_t stream) {
+  using namespace b200;
+  if (M <= 0 || inter <= 0 || K <= 0) return 0;
+  if ((lda & 7) || (ldb & 7) || (inter & 7)) return -100;
+  const GluParams glu{limit, alpha, beta};
+  const int N = 2 * inter;
+  if (splits > 1) {
+    int S = 0;
+    long long stride = 0;
+    const int rc = launch_splitk_partials(A, B, workspace, M, N, K, lda, ldb, splits, &S, &stride, stream);
+    if (rc) return rc;
+    long long rg = (static_cast<long long>(M) * (N >> 2) + 255) / 256;
+    const long long maxg = static_cast<long long>(sm_count()) * 8;
+    if (rg > maxg) rg = maxg;
+    splitk_reduce_glu_kernel<<<(unsigned)rg, 256, 0, stream>>>(workspace, (__nv_bfloat16*)C, M, N, S, stride, glu);
+    B200_CHECK(cudaGetLastError());
+    return 0;
+  }
+  const GluEpi epi{(__nv_bfloat16*)C, glu, M, inter};
   const long long tiles256 = static_cast<long long>((M + kBM - 1) / kBM) * ((N + 255) / 256);
   return tiles256 >= 100 ? launch_epi<256>(A, B, epi, M, N, K, lda, ldb, stream)
                          : launch_epi<128>(A, B, epi, M, N, K, lda, ldb, stream);

@@ -58,6 +58,7 @@ struct Request {
 
 struct Scheduler {
   int num_blocks, block_size, max_num_seqs, max_batched_tokens, max_blocks_per_seq;
+  int max_len = INT32_MAX;  // most tokens that a sequence may reach (models with a table of positions)
   std::vector<int32_t> free_blocks;
   std::vector<int32_t> refcnt;  // pages may be shared by requests with the same prompt (read-only full pages)
   std::unordered_map<uint64_t, int64_t> prompt_leader;  // prompt hash -> request whose prompt pages can be shared
@@ -134,6 +135,9 @@ void* b200_sched_create(int num_blocks, int block_size, int max_num_seqs, int ma
   return s;
 }
 
+// Sequences end (reason: length) when they would grow past this many tokens; longer prompts are refused.
+void b200_sched_set_max_len(void* h, int max_len) { static_cast<Scheduler*>(h)->max_len = max_len; }
+
 void b200_sched_destroy(void* h) { delete static_cast<Scheduler*>(h); }
 
 // Returns the request id (> 0) or -1 when the prompt can never fit. share_len: number of leading tokens that
@@ -144,7 +148,7 @@ int64_t b200_sched_add_shared(void* h, const int32_t* prompt, int n_prompt, int 
   auto* s = static_cast<Scheduler*>(h);
   std::lock_guard<std::mutex> lk(s->mu);
   const int64_t total = static_cast<int64_t>(n_prompt) + max_new_tokens;
-  if (n_prompt <= 0 || n_prompt > s->max_batched_tokens ||
+  if (n_prompt <= 0 || n_prompt > s->max_batched_tokens || n_prompt > s->max_len ||
       (n_prompt + s->block_size - 1) / s->block_size > s->max_blocks_per_seq)
     return -1;
   (void)total;
@@ -256,9 +260,14 @@ int b200_sched_plan(void* h, PlanHeader* hdr, int64_t* seq_ids, int32_t* cu_seql
           }
         }
       }
+      if (L > s->max_len) {  // preempted with its last token: nothing is left to generate
+        s->waiting.pop_front();
+        s->finish(r, kLength);
+        continue;
+      }
       if (L > budget) break;
       // keep one page of head-room per running sequence so decode can proceed
-      if (!s->ensure_blocks(r, L + 1)) {
+      if (!s->ensure_blocks(r, std::min(L + 1, s->max_len))) {
         s->release(r);
         break;
       }
@@ -295,11 +304,11 @@ int b200_sched_plan(void* h, PlanHeader* hdr, int64_t* seq_ids, int32_t* cu_seql
   for (size_t i = 0; i < s->running.size();) {
     Request& r = s->reqs[s->running[i]];
     const int32_t L = static_cast<int32_t>(r.tokens.size());
-    if (s->ensure_blocks(r, L)) {
+    if (L <= s->max_len && s->ensure_blocks(r, L)) {
       ++i;
       continue;
     }
-    if (static_cast<int32_t>((L + s->block_size - 1) / s->block_size) > s->max_blocks_per_seq) {
+    if (L > s->max_len || static_cast<int32_t>((L + s->block_size - 1) / s->block_size) > s->max_blocks_per_seq) {
       // context limit reached
       const int64_t id = r.id;
       s->finish(r, kLength);

@@ -12,6 +12,8 @@
 //                 per-head part is the latent itself, shared by the heads too, and the queries carry the key
 //                 up-projection). The tensor-core kernels cover the widths of real models; this one covers the rest
 //                 and fp32. A window bounds how far back a query sees; a gate scales every head's result by a sigmoid.
+//                 Grouped-query attention runs here too: keys and values per group of heads, first tokens that a window
+//                 keeps, a soft cap on the scores, a sink in the softmax.
 #include "common/host_utils.h"
 #include "common/io.cuh"
 
@@ -206,7 +208,23 @@ struct AttendArgs {
   int window;                      // a query sees its last `window` keys; 0: all of them
   const void* gate;                // null, or [n][ldg]: head h's result is multiplied by sigmoid(gate[h])
   long long ldg;
+  int group;                       // query heads per key / value head (head strides of keys and values count those)
+  int page_rows;                   // paged: key rows per page, a multiple of block_size (the heads' rows follow each other)
+  int keep;                        // with a window: the first `keep` keys are always visible
+  float softcap;                   // score <- softcap * tanh(score / softcap); 0: none
+  const void* sink;                // null, or [H]: exp(sink[h]) joins head h's denominator
 };
+
+// The factor on a head's accumulators from their reference m and sum l, with the sink's term.
+__device__ __forceinline__ float attend_factor(float m, float l, const float* sink) {
+  float f = 1.f;
+  if (sink) {
+    const float mn = fmaxf(m, *sink);
+    f = m == -INFINITY ? 0.f : expf(m - mn);
+    l = l * f + expf(*sink - mn);
+  }
+  return l > 0.f ? f / l : 0.f;
+}
 
 // grid (n query rows, ceil(H / warps), nsplit)
 template <class T>
@@ -221,8 +239,9 @@ __global__ void attend_kernel(AttendArgs a) {
   const long long r = blockIdx.x;
   const int L = a.kv_len[r];
   const int lo = a.window > 0 ? max(0, L - a.window) : 0;
-  const int per = (L - lo + a.nsplit - 1) / a.nsplit;
-  const int k0 = lo + blockIdx.z * per, k1 = min(L, k0 + per);
+  const int nk = min(a.keep, lo), n_seen = L - lo + nk;  // kept keys, then those inside the window
+  const int per = (n_seen + a.nsplit - 1) / a.nsplit, hg = h / a.group;
+  const int k0 = blockIdx.z * per, k1 = min(n_seen, k0 + per);
   for (int i = lane; i < a.da; i += 32) q[i] = ld1(static_cast<const T*>(a.qa) + r * a.ldqa + h * a.hqa + i);
   for (int i = lane; i < a.db; i += 32) q[a.da + i] = ld1(static_cast<const T*>(a.qb) + r * a.ldqb + h * a.hqb + i);
   for (int i = lane; i < a.dv; i += 32) acc[i] = 0.f;
@@ -231,24 +250,25 @@ __global__ void attend_kernel(AttendArgs a) {
   const int* bt = a.block_table ? a.block_table + r * a.max_blocks : nullptr;
   float m = -INFINITY, l = 0.f;
   for (int kb = k0; kb < k1; kb += 32) {
-    const int j = kb + lane;
+    const int i_seen = kb + lane, j = i_seen < nk ? i_seen : i_seen + lo - nk;
     long long row = 0;
     float s = -INFINITY;
-    if (j < k1) {
-      row = bt ? static_cast<long long>(bt[j / a.block_size]) * a.block_size + j % a.block_size : first + j;
-      const T* ka = static_cast<const T*>(a.ka) + row * a.ldka + h * a.hka;
-      const T* kp = static_cast<const T*>(a.kb) + row * a.ldkb + h * a.hkb;
+    if (i_seen < k1) {
+      row = bt ? static_cast<long long>(bt[j / a.block_size]) * a.page_rows + j % a.block_size : first + j;
+      const T* ka = static_cast<const T*>(a.ka) + row * a.ldka + static_cast<long long>(hg) * a.hka;
+      const T* kp = static_cast<const T*>(a.kb) + row * a.ldkb + static_cast<long long>(hg) * a.hkb;
       float d = 0.f;
       for (int i = 0; i < a.da; ++i) d = fmaf(q[i], ld1(ka + i), d);
       for (int i = 0; i < a.db; ++i) d = fmaf(q[a.da + i], ld1(kp + i), d);
       s = d * a.scale;
+      if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
     }
     float mx = s;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
     const float mn = fmaxf(m, mx);
     const float sc = m == -INFINITY ? 0.f : expf(m - mn);
-    const float p = j < k1 ? expf(s - mn) : 0.f;
+    const float p = i_seen < k1 ? expf(s - mn) : 0.f;
     l = l * sc + warp_sum(p);
     m = mn;
     const int n = min(32, k1 - kb);
@@ -258,13 +278,14 @@ __global__ void attend_kernel(AttendArgs a) {
       for (int e = 0; e < n; ++e) {
         const long long rr = __shfl_sync(0xffffffffu, row, e);
         const float pe = __shfl_sync(0xffffffffu, p, e);
-        if (i < a.dv) t = fmaf(pe, ld1(static_cast<const T*>(a.v) + rr * a.ldv + h * a.hv + i), t);
+        if (i < a.dv) t = fmaf(pe, ld1(static_cast<const T*>(a.v) + rr * a.ldv + static_cast<long long>(hg) * a.hv + i), t);
       }
       if (i < a.dv) acc[i] = fmaf(acc[i], sc, t);
     }
   }
   if (a.nsplit == 1) {
-    float inv = l > 0.f ? 1.f / l : 0.f;
+    const float sink = a.sink ? ld1(static_cast<const T*>(a.sink) + h) : 0.f;
+    float inv = attend_factor(m, l, a.sink ? &sink : nullptr);
     if (a.gate) inv *= sigmoid_as(ld1(static_cast<const T*>(a.gate) + r * a.ldg + h), static_cast<const T*>(nullptr));
     for (int i = lane; i < a.dv; i += 32)
       st1(static_cast<T*>(a.out) + r * a.ldo + static_cast<long long>(h) * a.dv + i, acc[i] * inv);
@@ -275,11 +296,11 @@ __global__ void attend_kernel(AttendArgs a) {
   }
 }
 
-// Merge of split partials. m in natural-log units when LOG2 is false, in log2 units else.
-template <class T, bool LOG2>
+// Merge of split partials.
+template <class T>
 __global__ void attend_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ ml, T* __restrict__ out,
                                     long long ldo, int H, int nsplit, int dv, const T* __restrict__ gate,
-                                    long long ldg) {
+                                    long long ldg, const T* __restrict__ sink) {
   const long long u = blockIdx.x;
   const long long r = u / H;
   const int h = static_cast<int>(u % H);
@@ -288,18 +309,44 @@ __global__ void attend_merge_kernel(const float* __restrict__ o_part, const floa
   float l = 0.f;
   for (int s = 0; s < nsplit; ++s) {
     const float ms = ml[(u * nsplit + s) * 2];
-    if (ms != -INFINITY) l += ml[(u * nsplit + s) * 2 + 1] * (LOG2 ? exp2f(ms - m) : expf(ms - m));
+    if (ms != -INFINITY) l += ml[(u * nsplit + s) * 2 + 1] * expf(ms - m);
   }
-  float inv = l > 0.f ? 1.f / l : 0.f;
+  const float sv = sink ? ld1(sink + h) : 0.f;
+  float inv = attend_factor(m, l, sink ? &sv : nullptr);
   if (gate) inv *= sigmoid_as(ld1(gate + r * ldg + h), gate);
   for (int i = threadIdx.x; i < dv; i += blockDim.x) {
     float t = 0.f;
     for (int s = 0; s < nsplit; ++s) {
       const float ms = ml[(u * nsplit + s) * 2];
-      if (ms != -INFINITY) t = fmaf(o_part[(u * nsplit + s) * dv + i], LOG2 ? exp2f(ms - m) : expf(ms - m), t);
+      if (ms != -INFINITY) t = fmaf(o_part[(u * nsplit + s) * dv + i], expf(ms - m), t);
     }
     st1(out + r * ldo + static_cast<long long>(h) * dv + i, t * inv);
   }
+}
+
+// Launches the attention and, for several splits, their merge.
+static int launch_attend(const AttendArgs& a, int n, int fp32, cudaStream_t stream) {
+  const int H = a.H, nsplit = a.nsplit;
+  int nw = H < 4 ? H : 4;
+  const size_t per_warp = static_cast<size_t>(a.da + a.db + a.dv) * sizeof(float);
+  while (nw > 1 && per_warp * nw > 48 * 1024) nw >>= 1;
+  const size_t smem = per_warp * nw;
+  if (smem > 48 * 1024) return -100;
+  dim3 grid(n, (H + nw - 1) / nw, nsplit);
+  if (fp32) attend_kernel<float><<<grid, nw * 32, smem, stream>>>(a);
+  else attend_kernel<__nv_bfloat16><<<grid, nw * 32, smem, stream>>>(a);
+  B200_CHECK(cudaGetLastError());
+  if (nsplit > 1) {
+    if (fp32)
+      attend_merge_kernel<float><<<n * H, 128, 0, stream>>>(a.o_part, a.ml_part, (float*)a.out, a.ldo, H, nsplit, a.dv,
+                                                            (const float*)a.gate, a.ldg, (const float*)a.sink);
+    else
+      attend_merge_kernel<__nv_bfloat16><<<n * H, 128, 0, stream>>>(
+          a.o_part, a.ml_part, (__nv_bfloat16*)a.out, a.ldo, H, nsplit, a.dv, (const __nv_bfloat16*)a.gate, a.ldg,
+          (const __nv_bfloat16*)a.sink);
+    B200_CHECK(cudaGetLastError());
+  }
+  return 0;
 }
 
 }  // namespace b200
@@ -383,25 +430,26 @@ int b200_attend(const void* qa, long long ldqa, int hqa, const void* qb, long lo
   if (n <= 0) return 0;
   AttendArgs a{qa, qb, ldqa, ldqb, hqa, hqb, ka, kb, v, ldka, ldkb, ldv, hka, hkb, hv, da, db, dv, seq_start, kv_len,
                block_table, max_blocks, block_size, o_part, ml_part, out, ldo, H, nsplit, scale, window,
-               gate, ldg};
-  int nw = H < 4 ? H : 4;
-  const size_t per_warp = static_cast<size_t>(da + db + dv) * sizeof(float);
-  while (nw > 1 && per_warp * nw > 48 * 1024) nw >>= 1;
-  const size_t smem = per_warp * nw;
-  if (smem > 48 * 1024) return -100;
-  dim3 grid(n, (H + nw - 1) / nw, nsplit);
-  if (fp32) attend_kernel<float><<<grid, nw * 32, smem, stream>>>(a);
-  else attend_kernel<__nv_bfloat16><<<grid, nw * 32, smem, stream>>>(a);
-  B200_CHECK(cudaGetLastError());
-  if (nsplit > 1) {
-    if (fp32) attend_merge_kernel<float, false><<<n * H, 128, 0, stream>>>(o_part, ml_part, (float*)out, ldo, H, nsplit, dv,
-                                                                                (const float*)gate, ldg);
-    else
-      attend_merge_kernel<__nv_bfloat16, false><<<n * H, 128, 0, stream>>>(o_part, ml_part, (__nv_bfloat16*)out, ldo, H,
-                                                                          nsplit, dv, (const __nv_bfloat16*)gate, ldg);
-    B200_CHECK(cudaGetLastError());
-  }
-  return 0;
+               gate, ldg, 1, block_size, 0, 0.f, nullptr};
+  return launch_attend(a, n, fp32, stream);
+}
+
+// Grouped-query form: q [n][ldq] + h * hq; keys and values per kv head g at g * hk / g * hv of a row. Packed (seq_start): rows
+// of the batch. Paged (block_table): page p's rows start at p * page_rows, and hk, hv lead from one head's rows of a page
+// to the next one's. window, keep, softcap: 0 for none; sink [H], gate [n][ldg]: null for none.
+int b200_attend_grouped(const void* q, long long ldq, int hq, const void* k, long long ldk, int hk, const void* v,
+                        long long ldv, int hv, int d, int dv, const int* seq_start, const int* kv_len,
+                        const int* block_table, int max_blocks, int block_size, int page_rows, float* o_part,
+                        float* ml_part, void* out, long long ldo, int n, int H, int G, int nsplit, float scale, int window,
+                        int keep, float softcap, const void* sink, const void* gate, long long ldg, int fp32,
+                        cudaStream_t stream) {
+  using namespace b200;
+  if (n <= 0) return 0;
+  if (G < 1 || H % G || block_size < 1) return -100;
+  AttendArgs a{q, nullptr, ldq, 0, hq, 0, k, nullptr, v, ldk, 0, ldv, hk, 0, hv, d, 0, dv, seq_start, kv_len, block_table,
+               max_blocks, block_size, o_part, ml_part, out, ldo, H, nsplit, scale, window, gate, ldg, H / G, page_rows,
+               keep, softcap, sink};
+  return launch_attend(a, n, fp32, stream);
 }
 
 }  // extern "C"

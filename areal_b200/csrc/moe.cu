@@ -22,28 +22,34 @@ namespace b200 {
 constexpr int kMaxE = 1024;
 constexpr int kChunk = 256;  // flat entries per warp in the sort
 
-// A warp routes one token. z: this lane's logits (experts lane + 32 i). Scores are the softmax over all experts; the k
-// experts with the largest score (plus correction, when there is one) are chosen, ties going to the lowest index, and
+// A warp routes one token. z: this lane's logits (experts lane + 32 i). Scores are the softmax over all experts, or with
+// `sigmoid` each expert's 1 / (1 + e^-z); the k experts with the largest score (plus correction, when there is one) are chosen, ties going to the lowest index, and
 // weighted by their score without the correction, optionally renormalised to sum to one.
 template <int PER, class C>
 __device__ __forceinline__ void route_token(const float (&z)[PER], const C* __restrict__ correction, int E, int k,
-                                            int renorm, int* __restrict__ idx, float* __restrict__ w) {
+                                            int renorm, int sigmoid, int* __restrict__ idx, float* __restrict__ w) {
   const int lane = threadIdx.x & 31;
   float s[PER], pick[PER];
-  float mx = -INFINITY;
+  float inv = 1.f;
+  if (sigmoid) {
 #pragma unroll
-  for (int i = 0; i < PER; ++i) mx = fmaxf(mx, lane + 32 * i < E ? z[i] : -INFINITY);
+    for (int i = 0; i < PER; ++i) s[i] = 1.f / (1.f + expf(-z[i]));
+  } else {
+    float mx = -INFINITY;
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-  float sum = 0.f;
+    for (int i = 0; i < PER; ++i) mx = fmaxf(mx, lane + 32 * i < E ? z[i] : -INFINITY);
 #pragma unroll
-  for (int i = 0; i < PER; ++i) {
-    s[i] = lane + 32 * i < E ? expf(z[i] - mx) : 0.f;
-    sum += s[i];
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      s[i] = lane + 32 * i < E ? expf(z[i] - mx) : 0.f;
+      sum += s[i];
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    inv = 1.f / sum;
   }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-  const float inv = 1.f / sum;
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i;
@@ -80,14 +86,15 @@ __device__ __forceinline__ void route_token(const float (&z)[PER], const C* __re
 // One warp per token: logits [T, E] fp32 → idx [T, k] int32, w [T, k] fp32. PER: experts per lane = ceil(E / 32)
 template <int PER, class C>
 __global__ void moe_route_kernel(const float* __restrict__ logits, const C* __restrict__ correction,
-                                 int* __restrict__ idx, float* __restrict__ w, int T, int E, int k, int renorm) {
+                                 int* __restrict__ idx, float* __restrict__ w, int T, int E, int k, int renorm,
+                                 int sigmoid) {
   const long long t = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (t >= T) return;
   float z[PER];
 #pragma unroll
   for (int i = 0; i < PER; ++i) z[i] = lane + 32 * i < E ? logits[t * E + lane + 32 * i] : 0.f;
-  route_token<PER>(z, correction, E, k, renorm, idx + t * k, w + t * k);
+  route_token<PER>(z, correction, E, k, renorm, sigmoid, idx + t * k, w + t * k);
 }
 
 __device__ __forceinline__ float dot8(const float* w, const float* x, float s) {
@@ -112,7 +119,7 @@ __device__ __forceinline__ float dot8(const __nv_bfloat16* w, const float* x, fl
 template <int PER, class D>
 __global__ void moe_router_kernel(const D* __restrict__ x, long long ldx, const D* __restrict__ wr,
                                   const D* __restrict__ correction, int* __restrict__ idx, float* __restrict__ w, int H,
-                                  int E, int k, int renorm) {
+                                  int E, int k, int renorm, int sigmoid) {
   extern __shared__ float rsm[];  // [H] vector, [E] logits
   float* z = rsm + H;
   const long long t = blockIdx.x;
@@ -149,7 +156,7 @@ __global__ void moe_router_kernel(const D* __restrict__ x, long long ldx, const 
     float v[PER];
 #pragma unroll
     for (int i = 0; i < PER; ++i) v[i] = lane + 32 * i < E ? z[lane + 32 * i] : 0.f;
-    route_token<PER>(v, correction, E, k, renorm, idx + t * k, w + t * k);
+    route_token<PER>(v, correction, E, k, renorm, sigmoid, idx + t * k, w + t * k);
   }
 }
 
@@ -324,13 +331,15 @@ __global__ void moe_scatter_kernel(const __nv_bfloat16* __restrict__ x, long lon
 // Grouped product of any sizes in fp32 arithmetic (32-bit models, sizes that the tensor-core kernel does not take), over
 // the same padded expert-sorted rows: C[r] = A[row] . W[e(r)]^T for the 64 x 64 tile of a half tile of rows and 64
 // weight rows. gather_k > 0: row r of A is x[src_of[r] / gather_k], else A's own row r. GLU: weight rows alternate
-// between gate and up and the gated activation follows; C is half as wide.
+// between gate and up and the gated activation follows; C is half as wide. scale (null: none): row r's products count
+// scale[src_of[r]] times ahead of the activation.
 template <class T, bool GLU>
 __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(const T* __restrict__ a, long long lda, int gather_k,
                                                             const T* __restrict__ w, T* __restrict__ c, long long ldc,
                                                             const int* __restrict__ tile_expert,
                                                             const int* __restrict__ num_vm,
-                                                            const int* __restrict__ src_of, int N, int K, GluParams glu) {
+                                                            const int* __restrict__ src_of,
+                                                            const float* __restrict__ scale, int N, int K, GluParams glu) {
   __shared__ float sa[16][68], sb[16][68];
   __shared__ long long arow[64];
   const int vm = blockIdx.x >> 1, r0 = vm * 128 + (blockIdx.x & 1) * 64, n0 = blockIdx.y * 64;
@@ -367,6 +376,11 @@ __global__ void __launch_bounds__(256) moe_gemm_simt_kernel(const T* __restrict_
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     if (arow[ty * 4 + i] < 0) continue;
+    if (scale) {
+      const float f = scale[src_of[r0 + ty * 4 + i]];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] *= f;
+    }
     T* row = c + static_cast<long long>(r0 + ty * 4 + i) * ldc;
     const int col = n0 + tx * 4;
     if (GLU) {
@@ -652,13 +666,13 @@ extern "C" {
 
 // correction: null or [E], bf16 or fp32 (correction_fp32)
 int b200_moe_route(const float* logits, const void* correction, int correction_fp32, int* idx, float* w, int T, int E,
-                   int k, int renorm, cudaStream_t stream) {
+                   int k, int renorm, int sigmoid, cudaStream_t stream) {
   using namespace b200;
   if (T == 0) return 0;
   if (E > 256 || k > 32 || k > E) return -100;
   const unsigned grid = (static_cast<long long>(T) * 32 + 255) / 256;
   const int per = (E + 31) / 32;
-#define RT(P, C) moe_route_kernel<P, C><<<grid, 256, 0, stream>>>(logits, (const C*)correction, idx, w, T, E, k, renorm)
+#define RT(P, C) moe_route_kernel<P, C><<<grid, 256, 0, stream>>>(logits, (const C*)correction, idx, w, T, E, k, renorm, sigmoid)
 #define RTP(C) if (per <= 1) RT(1, C); else if (per <= 2) RT(2, C); else if (per <= 4) RT(4, C); else RT(8, C);
   if (correction_fp32) { RTP(float) } else { RTP(__nv_bfloat16) }
 #undef RTP
@@ -669,7 +683,7 @@ int b200_moe_route(const float* logits, const void* correction, int correction_f
 
 // x [T][ldx], wr [E, H], correction null or [E]: all bf16 or all fp32. For few tokens (every block reads all of wr).
 int b200_moe_router(const void* x, long long ldx, const void* wr, const void* correction, int* idx, float* w, int T, int H,
-                    int E, int k, int renorm, int fp32, cudaStream_t stream) {
+                    int E, int k, int renorm, int sigmoid, int fp32, cudaStream_t stream) {
   using namespace b200;
   if (T == 0) return 0;
   const size_t smem = static_cast<size_t>(H + E) * sizeof(float);
@@ -681,7 +695,7 @@ int b200_moe_router(const void* x, long long ldx, const void* wr, const void* co
       B200_CHECK(cudaFuncSetAttribute(moe_router_kernel<P, D>, cudaFuncAttributeMaxDynamicSharedMemorySize,         \
                                       static_cast<int>(smem)));                                                     \
     moe_router_kernel<P, D><<<T, block, smem, stream>>>((const D*)x, ldx, (const D*)wr, (const D*)correction, idx, w, H, \
-                                                        E, k, renorm);                                              \
+                                                        E, k, renorm, sigmoid);                                     \
   }
 #define RTP(D) if (per <= 1) RT(1, D) else if (per <= 2) RT(2, D) else if (per <= 4) RT(4, D) else RT(8, D)
   if (fp32) { RTP(float) } else { RTP(__nv_bfloat16) }
@@ -723,7 +737,8 @@ int b200_moe_scatter(const void* x, long long ldx, const int* dest, int T, int k
 
 // See moe_gemm_simt_kernel. w [E, N, K]; N even with glu. gather_k 0: a holds padded rows.
 int b200_moe_gemm_simt(const void* a, long long lda, int gather_k, const void* w, void* c, long long ldc,
-                       const int* tile_expert, const int* num_vm, const int* src_of, int max_vm, int N, int K, int glu,
+                       const int* tile_expert, const int* num_vm, const int* src_of, const float* scale, int max_vm,
+                       int N, int K, int glu,
                        float limit, float alpha, float beta, int fp32, cudaStream_t stream) {
   using namespace b200;
   if (max_vm <= 0 || N <= 0 || K <= 0) return 0;
@@ -733,7 +748,7 @@ int b200_moe_gemm_simt(const void* a, long long lda, int gather_k, const void* w
   using bf = __nv_bfloat16;
 #define MS(T_, G_)                                                                                                  \
   moe_gemm_simt_kernel<T_, G_><<<grid, 256, 0, stream>>>((const T_*)a, lda, gather_k, (const T_*)w, (T_*)c, ldc,    \
-                                                         tile_expert, num_vm, src_of, N, K, g)
+                                                         tile_expert, num_vm, src_of, scale, N, K, g)
   if (fp32) { if (glu) MS(float, true); else MS(float, false); }
   else { if (glu) MS(bf, true); else MS(bf, false); }
 #undef MS

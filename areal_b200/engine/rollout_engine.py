@@ -138,6 +138,9 @@ class PagedScheduler:
     def set_prompt_sharing(self, on: bool):
         self.lib.b200_sched_set_prompt_sharing(self.h, ctypes.c_int(int(on)))
 
+    def set_max_len(self, n: int):
+        self.lib.b200_sched_set_max_len(self.h, ctypes.c_int(n))
+
     def close(self):
         if self.h:
             self.lib.b200_sched_destroy(self.h)
@@ -365,6 +368,8 @@ class NativeRolloutEngine(InferenceEngine):
         self.kv_caches = self._alloc_kv(nblocks, dtype)
         self.sched = PagedScheduler(nblocks, bs, ncfg.max_num_seqs, ncfg.max_num_batched_tokens,
                                     max_blocks_per_seq)
+        if mc.position_limit is not None:
+            self.sched.set_max_len(mc.position_limit)
         # Hybrid models: per-sequence state of the linear-attention layers, addressed by a slot that a
         # request keeps from its first prefill until it finishes. Prompts are not shared (a shared page
         # says nothing about the recurrent state).

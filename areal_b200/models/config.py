@@ -88,8 +88,13 @@ class ModelConfig:
     # and the feed-forward's (None: the layer has none); the sizes above then only summarise the list
     layer_specs: list[dict] = field(default_factory=list)
     # what such a decoder wraps its sublayers in: "dynamic_tanh" (norm in front, learned scale on the result) or
-    # "layer_norm" (one norm in front and one on the result)
+    # "layer_norm" (one norm in front and one on the result) or "post_rms" (RMS norm on the result only)
     layer_norms: str = "dynamic_tanh"
+    # input: embed[token] * embedding_scale, plus a learned vector per position (table of `max_position_embeddings` rows,
+    # which then bounds the length of a sequence)
+    embedding_scale: float = 1.0
+    learned_positions: bool = False
+    logit_scale: float = 1.0  # logits = head(x) * logit_scale
     # logits <- cap * tanh(logits / cap); 0 = none
     logit_softcap: float = 0.0
     moe_group_score_top: int = 2  # a group's score: the sum of its this many best experts
@@ -137,6 +142,8 @@ class ModelConfig:
         """Paged-cache tensors of layer ``i`` as ``(heads, width)`` per token; empty for layers without a cache."""
         if self.is_layered:
             m = self.layer_specs[i]["mixer"]
+            if self.layer_type(i) == "grouped_attention":  # widths in steps of 16: what a tensor-core tile takes
+                return [(m["kv_heads"], -(-n // 16) * 16) for n in (m["dim"], m["vdim"])]
             own = self.layer_type(i) == "latent_attention" and m.get("kv_from") is None
             return [(1, m["kv_rank"] + m["rot_dim"])] if own else []
         if self.layer_type(i) != "full_attention":
@@ -147,6 +154,16 @@ class ModelConfig:
         """The layer whose cache layer ``i`` attends to: its own, or an earlier layer's that it shares."""
         src = self.layer_specs[i]["mixer"].get("kv_from") if self.is_layered else None
         return i if src is None else src
+
+    def weights_layer(self, i: int) -> int:
+        """The layer whose parameters layer ``i`` runs with: its own, or an earlier layer's (with a cache of its own)."""
+        j = self.layer_specs[i].get("weights_of") if self.is_layered else None
+        return i if j is None else self.weights_layer(j)
+
+    @property
+    def position_limit(self) -> int | None:
+        """Longest sequence that the model's tables hold (None: positions are computed)."""
+        return self.max_position_embeddings if self.learned_positions else None
 
     def recurrent_shape(self, i: int) -> tuple[int, int, int] | None:
         """State of layer ``i`` per sequence ``(heads, key width, value width)``, None for layers without one. Covers
@@ -212,14 +229,17 @@ class ModelConfig:
         h, spec = self.hidden_size, self.layer_specs[i]
         m, t = spec["mixer"], spec["type"]
         H, D, Dv = m["heads"], m["dim"], m["vdim"]
-        # what surrounds a sublayer: Dynamic Tanh (weight, bias, alpha) and a scale, or two layer norms
-        wrap = 4 * h if self.layer_norms == "layer_norm" else 3 * h + 1
+        # what surrounds a sublayer: Dynamic Tanh (weight, bias, alpha) and a scale, two layer norms, or an RMS norm
+        wrap = {"layer_norm": 4 * h, "post_rms": h}.get(self.layer_norms, 3 * h + 1)
         if t == "latent_attention":
             rq, rank, R = m.get("q_rank", 0), m["kv_rank"], m["rot_dim"]
             n = h * rq + rq * (1 + H * (D + R)) if rq else h * H * (D + R)
             if m.get("kv_from") is None:
                 n += h * (rank + R) + rank
             n += rank * H * (D + Dv) + (h * H if m.get("gate") else 0)
+        elif t == "grouped_attention":
+            rows = H * D + m["kv_heads"] * (D + Dv)
+            n = h * rows + (rows if m["bias"] else 0) + (H if m["sink"] else 0) + (h * H if m["gate"] else 0)
         elif t == "hgrn2":
             n = h * H * (2 * D + Dv) + 2 * H * D + Dv
         else:
@@ -230,14 +250,18 @@ class ModelConfig:
             return n
         if mlp["kind"] == "moe":
             r = mlp["router"]
-            return n + wrap + (h + 1) * r["experts"] + 3 * h * mlp["expert"]["ff"] * (r["top"] if active else r["experts"])
+            n += 3 * h * mlp["shared"]["ff"] if mlp.get("shared") else 0
+            n += (h + bool(r.get("correction", True))) * r["experts"]
+            return n + wrap + 3 * h * mlp["expert"]["ff"] * (r["top"] if active else r["experts"])
         return n + wrap + 2 * h * mlp["ff"] + (4 if mlp.get("act", "polynorm") == "polynorm" else 0)
 
     def num_params(self) -> int:
         h, L = self.hidden_size, self.num_hidden_layers
         if self.is_layered:
-            final = 2 * h + (self.layer_norms == "dynamic_tanh")
-            return 2 * self.vocab_size * h + final + sum(self._layered_params(i) for i in range(L))
+            final = {"layer_norm": 2 * h, "post_rms": h}.get(self.layer_norms, 2 * h + 1)
+            final += self.max_position_embeddings * h if self.learned_positions else 0
+            return 2 * self.vocab_size * h + final + sum(self._layered_params(i) for i in range(L)
+                                                         if self.weights_layer(i) == i)
         attn = self.attn_params()
         if self.attention_bias:
             attn += self.q_size + 2 * self.kv_size
@@ -287,6 +311,9 @@ class ModelConfig:
                 if spec["type"] == "latent_attention":
                     keys = min(seq_len / 2, m.get("window") or seq_len)
                     total += 2 * m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"]) * keys
+                elif spec["type"] == "grouped_attention":
+                    keys = min(seq_len / 2, m["window"] + m["keep_first"]) if m["window"] else seq_len / 2
+                    total += 2 * m["heads"] * (m["dim"] + m["vdim"]) * keys
                 else:
                     total += 4 * m["heads"] * m["dim"] * m["vdim"]
             return total * (3 if backward else 1)
@@ -310,6 +337,8 @@ class ModelConfig:
             return cls._from_fofosun(cfg, overrides)
         if cfg.get("architecture") == "Gatolix":
             return cls._from_gatolix(cfg, overrides)
+        if cfg.get("architecture") == "Felosun":
+            return cls._from_felosun(cfg, overrides)
         if "text_config" in cfg:  # composite (vision-language) checkpoints nest the decoder's config
             cfg = cfg["text_config"]
         mt = cfg.get("model_type", "qwen3")
@@ -470,7 +499,8 @@ class ModelConfig:
         out = cls(model_type=model_type, vocab_size=cfg["vocab"], hidden_size=cfg["width"], layer_specs=specs,
                   num_hidden_layers=len(specs), rms_norm_eps=cfg["norm"]["eps"],
                   intermediate_size=max((s["mlp"]["ff"] for s in specs if s["mlp"] and "ff" in s["mlp"]), default=0),
-                  num_attention_heads=heads, num_key_value_heads=heads,
+                  num_attention_heads=heads,
+                  num_key_value_heads=max((s["mixer"].get("kv_heads", s["mixer"]["heads"]) for s in specs), default=1),
                   head_dim=max((s["mixer"]["dim"] for s in specs), default=1), tie_word_embeddings=False, qk_norm=False,
                   num_experts=max((m["router"]["experts"] for m in moe), default=0),
                   num_experts_per_tok=max((m["router"]["top"] for m in moe), default=0),
@@ -524,7 +554,74 @@ class ModelConfig:
                "vocab": self.vocab_size, "width": self.hidden_size}
         return dict(out, logit_softcap=self.logit_softcap) if self.logit_softcap else out
 
+    @classmethod
+    def _from_felosun(cls, cfg: dict, overrides: dict) -> "ModelConfig":
+        """``config.json`` of a Felosun checkpoint: two kinds of grouped-query attention (``attention`` with biases,
+        neighbouring rotary pairs, a window that keeps the first tokens, and a sink; ``attention_2`` with split rotary
+        pairs, soft-capped scores and a gate per head), mixtures of clamped gated experts with a shared expert, and layers
+        that run with an earlier layer's weights (``weights_of``)."""
+        specs = []
+        for i, layer in enumerate(cfg["layers"]):
+            t, m, mlp, src = layer["type"], layer["mixer"], layer.get("mlp"), layer.get("weights_of")
+            if t not in ("attention", "attention_2"):
+                raise NotImplementedError(f"layer {i}: mixer {t!r}; supported are 'attention' and 'attention_2'")
+            second = t == "attention_2"
+            if m["heads"] % m["kv_heads"]:
+                raise ValueError(f"layer {i}: {m['heads']} query heads do not divide into {m['kv_heads']} groups")
+            spec = {k: m[k] for k in ("heads", "kv_heads", "dim", "vdim", "scale")}
+            rot, mask = m["rot"], m.get("mask") or {}
+            spec["rot"] = {"base": float(rot["base"]), "dims": int(rot["dims"])}
+            if rot["dims"] % 2 or not 0 <= rot["dims"] <= m["dim"]:
+                raise ValueError(f"layer {i}: {rot['dims']} rotated dimensions in heads of {m['dim']}")
+            if rot.get("scaling"):
+                spec["rot"]["scaling"] = {"factor": float(rot["scaling"]["factor"])}
+            if mask.get("size") is not None and mask["size"] < 1:
+                raise ValueError(f"layer {i}: a window of {mask['size']} tokens")
+            spec.update(window=mask.get("size"), keep_first=int(mask.get("keep_first") or 0),
+                        softcap=float(m.get("softcap") or 0.0), bias=not second, sink=not second, gate=second,
+                        rot_halves=second, unit_qk=True)
+            ff = None
+            if mlp is not None:
+                if mlp["kind"] != "moe":
+                    raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']!r}; supported is 'moe'")
+                ff = {"kind": "moe", "router": dict({k: mlp["router"][k] for k in ("experts", "top")}, score="sigmoid",
+                                                    correction=False),
+                      "expert": {k: mlp["expert"][k] for k in ("ff", "limit")}, "weight": "input"}
+                if mlp.get("shared"):
+                    ff["shared"] = {k: mlp["shared"][k] for k in ("ff", "limit")}
+            out = {"type": "grouped_attention", "mixer": spec, "mlp": ff}
+            if src is not None:
+                if not 0 <= src < i or {k: specs[src][k] for k in out} != out:
+                    raise ValueError(f"layer {i}: it cannot run with the weights of layer {src}")
+                out["weights_of"] = src
+            specs.append(out)
+        emb = cfg.get("embedding") or {}
+        return cls._layered("felosun", cfg, specs, overrides, layer_norms="post_rms", learned_positions=True,
+                            max_position_embeddings=int(cfg["max_positions"]), embedding_scale=float(emb.get("scale", 1.0)),
+                            logit_scale=float(cfg.get("logit_scale", 1.0)))
+
+    def _to_felosun(self) -> dict:
+        layers = []
+        for s in self.layer_specs:
+            a, mlp = s["mixer"], s["mlp"]
+            m = {k: a[k] for k in ("heads", "kv_heads", "dim", "vdim", "scale", "rot")}
+            if a["window"] is not None:
+                m["mask"] = {"size": a["window"], "keep_first": a["keep_first"]}
+            if a["softcap"]:
+                m["softcap"] = a["softcap"]
+            if mlp is not None:
+                mlp = dict({"kind": "moe", "router": {k: mlp["router"][k] for k in ("experts", "top")},
+                            "expert": mlp["expert"]}, **({"shared": mlp["shared"]} if mlp.get("shared") else {}))
+            layers.append({"type": "attention_2" if a["gate"] else "attention", "mixer": m, "mlp": mlp})
+            if s.get("weights_of") is not None:
+                layers[-1]["weights_of"] = s["weights_of"]
+        return {"architecture": "Felosun", "embedding": {"scale": self.embedding_scale}, "layers": layers,
+                "logit_scale": self.logit_scale, "max_positions": self.max_position_embeddings,
+                "norm": {"eps": self.rms_norm_eps}, "vocab": self.vocab_size, "width": self.hidden_size}
+
     def to_hf_config(self) -> dict:
+        if self.model_type == "felosun":
+            return self._to_felosun()
         if self.model_type == "gatolix":
             return self._to_gatolix()
         if self.model_type == "fofosun":
@@ -671,6 +768,11 @@ def _rotation(rot: dict, width: int, layer: int) -> dict:
 _TINY_LATENT = {"heads": 4, "dim": 32, "rot_dim": 16, "vdim": 24, "kv_rank": 80, "scale": 0.15, "mask": {"size": 50},
                 "rot": {"base": 1e4, "dims": 16, "scaling": {"factor": 4.0, "original": 512, "fast": 16.0, "slow": 1.0}}}
 
+_TINY_WINDOWED = {"heads": 6, "kv_heads": 2, "dim": 32, "vdim": 40, "scale": 0.25, "mask": {"size": 24, "keep_first": 5},
+                  "rot": {"base": 1e4, "dims": 16}}
+_TINY_MIXTURE = {"kind": "moe", "router": {"experts": 6, "top": 2}, "expert": {"ff": 96, "limit": 3.0},
+                 "shared": {"ff": 64, "limit": 2.0}}
+
 PRESETS: dict[str, ModelConfig] = {
     "tiny-qwen2": ModelConfig(model_type="qwen2", vocab_size=1024, hidden_size=256,
                               intermediate_size=688, num_hidden_layers=2, num_attention_heads=4,
@@ -794,6 +896,14 @@ PRESETS: dict[str, ModelConfig] = {
             {"type": "latent_attention", "mixer": dict(_TINY_LATENT, heads=6, kv_from=0, mask={"size": 24}), "mlp": None},
             {"type": "latent_attention", "mixer": dict(_TINY_LATENT), "mlp": {
                 "kind": "moe", "router": {"experts": 6, "top": 2}, "expert": {"ff": 96, "limit": 3.0}}}]}, {}),
+    # Felosun at test size: both kinds of attention, grouped heads, a repeated layer and one without a feed-forward
+    "tiny-felosun": ModelConfig._from_felosun({
+        "vocab": 1024, "width": 192, "norm": {"eps": 1e-6}, "embedding": {"scale": 5.0}, "logit_scale": 0.5,
+        "max_positions": 512, "layers": [
+            {"type": "attention", "mixer": _TINY_WINDOWED, "mlp": _TINY_MIXTURE},
+            {"type": "attention_2", "mixer": {"heads": 4, "kv_heads": 4, "dim": 48, "vdim": 32, "scale": 0.2, "softcap": 20.0,
+                                              "rot": {"base": 5e3, "dims": 24, "scaling": {"factor": 2.0}}}, "mlp": None},
+            {"type": "attention", "mixer": _TINY_WINDOWED, "mlp": _TINY_MIXTURE, "weights_of": 0}]}, {}),
     # DeepSeek-V2-Lite: latent attention without the query bottleneck, softmax routing, two shared experts
     "deepseek-v2-lite": ModelConfig(model_type="deepseek_v2", vocab_size=102400, hidden_size=2048,
                                     intermediate_size=10944, num_hidden_layers=27, num_attention_heads=16,

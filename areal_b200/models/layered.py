@@ -1,23 +1,26 @@
 """Decoders described as a list of layers (``ModelConfig.layer_specs``), each with its own mixer, its own sizes and an
 optional feed-forward, on an fp32 residual stream:
 
-    x = embed[token]
+    x = embed[token] * scale (+ positions[p])
     x = x + wrap1(mixer(norm1(x)));   x = x + wrap2(ff(norm2(x)))     per layer; a layer may have no feed-forward
-    logits = head norm(x)
+    logits = head norm(x) * scale
 
 Norms (``ModelConfig.layer_norms``): Dynamic Tanh, ``tanh(alpha x) * w + b`` (Zhu, Chen, He, LeCun, Liu, "Transformers
-without Normalization") with a learned per-column scale as ``wrap``, or layer norm with a second layer norm as ``wrap``.
+without Normalization") with a learned per-column scale as ``wrap``; layer norm with a second layer norm as ``wrap``; no
+norm in front and an RMS norm as ``wrap`` (the sublayers then read the stream itself).
 Every sublayer hands the activations in front of its output projection to the next norm's ``join``, which projects,
 wraps, adds to the residual and normalises in as few kernels as the shapes allow (``ops/dyt.py``, ``ops/layer_norm.py``),
 so the model is a flat list of sublayers between the embedding and the head.
 
 Mixers (``MIXERS``): HGRN2 (``models/hgrn2.py``), lightning attention with configured decays
-(``models/lightning.py``), latent attention over a compressed cache (``models/mla.py``). Feed-forwards (``make_mlp``):
-dense with PolyNorm or squared ReLU, mixture of gated experts. A sublayer has ``hidden(y, ctx, cache, rec)``, an output
+(``models/lightning.py``), latent attention over a compressed cache (``models/mla.py``), grouped-query attention
+(``models/gqa.py``). Feed-forwards (``make_mlp``): dense with PolyNorm or squared ReLU, mixture of gated experts, with or
+without a shared expert. A layer may run with an earlier layer's weights (``ModelConfig.weights_layer``) and a cache of
+its own. A sublayer has ``hidden(y, ctx, cache, rec)``, an output
 projection ``o`` (None: ``hidden`` is the sublayer's result) and ``tensors(prefix)``; what a mixer keeps per sequence is
 declared by ``ModelConfig.cache_shapes`` / ``recurrent_shape``, allocated by the rollout engine and passed in.
 
-The Fofosun and Gatolix families are built this way. The class shares loading, the head and the engine interface
+The Fofosun, Gatolix and Felosun families are built this way. The class shares loading, the head and the engine interface
 (``prefill`` / ``decode``) with ``QwenModel``. It is served by the rollout engine and runs forward and backward for
 training on one process per replica (data parallelism).
 """
@@ -30,19 +33,21 @@ from typing import Any, Iterator
 import torch
 import torch.nn as nn
 
-from ..ops import dyt, layer_norm as ln
+from ..ops import dyt, layer_norm as ln, residual_rms as rms
 from ..ops.attention import VarlenMeta
-from ..ops.gemm import linear, linear_relu2
+from ..ops.gemm import linear, linear_relu2, linear_slices
 from ..ops.latent_attn import rotary_tables
 from ..ops.lm_head import soft_cap_
-from ..ops.moe import ExpertRows, GatedAct, gated_experts, route_tokens
+from ..ops.moe import ExpertRows, GatedAct, gated_experts, gated_linear, route_tokens
 from .config import ModelConfig
+from .gqa import GroupedAttention
 from .hgrn2 import HGRN2
 from .lightning import ConstantDecayLightning
 from .mla import LatentAttention
 from .qwen import QwenModel
 
-MIXERS = {"hgrn2": HGRN2, "lightning": ConstantDecayLightning, "latent_attention": LatentAttention}
+MIXERS = {"hgrn2": HGRN2, "lightning": ConstantDecayLightning, "latent_attention": LatentAttention,
+          "grouped_attention": GroupedAttention}
 
 
 class ColumnScale(nn.Module):
@@ -111,9 +116,44 @@ class LayerNorm(nn.Module):
         yield name + ".b", self.bias
 
 
-# norm, what is wrapped around a sublayer's result, and the latter's checkpoint names
-NORMS = {"dynamic_tanh": (DynamicTanh, lambda n, eps, dtype, device: ColumnScale(n, dtype, device), ("ls1", "ls2")),
-         "layer_norm": (LayerNorm, LayerNorm, ("norm1b", "norm2b"))}
+class Stream(nn.Module):
+    """No norm: the next sublayer reads the residual stream, rounded to the model's dtype. Results are RMS normed."""
+
+    def __init__(self, n: int, eps: float, dtype, device):
+        super().__init__()
+        self.eps, self.scale, self.weight = eps, 1.0, None
+
+    def embed(self, ids, table, scale: float = 1.0, pos=None, pos_table=None):
+        return rms.embed_residual(ids, table, scale, pos, pos_table, self.weight, self.eps, self.scale)
+
+    def join(self, a, o, wrap: "RMSNorm", res):
+        """``(norm(res), res)`` of ``res + wrap(a @ o.T)``; without ``o``, ``a`` is the sublayer's result, also as the
+        experts' uncombined rows."""
+        tail = (wrap.weight, res, self.weight, self.eps, self.scale)
+        if isinstance(a, ExpertRows):
+            return rms.experts_residual_rms(a, *tail)
+        return rms.residual_rms(a, *tail) if o is None else rms.linear_residual_rms(a, o, *tail)
+
+    def tensors(self, name: str):
+        return iter(())
+
+
+class RMSNorm(Stream):
+    """RMS norm of the stream (behind the last layer, where ``scale`` multiplies its result) or of a sublayer's result."""
+
+    def __init__(self, n: int, eps: float, dtype, device, scale: float = 1.0):
+        super().__init__(n, eps, dtype, device)
+        self.scale = scale
+        self.weight = nn.Parameter(torch.ones(n, dtype=dtype, device=device))
+
+    def tensors(self, name: str):
+        yield name, self.weight
+
+
+# norm, what is wrapped around a sublayer's result, the latter's checkpoint names, and the norm in front of the head
+NORMS = {"dynamic_tanh": (DynamicTanh, lambda n, eps, dtype, device: ColumnScale(n, dtype, device), ("ls1", "ls2"), DynamicTanh),
+         "layer_norm": (LayerNorm, LayerNorm, ("norm1b", "norm2b"), LayerNorm),
+         "post_rms": (Stream, RMSNorm, ("norm1", "norm2"), RMSNorm)}
 
 
 class Relu2MLP(nn.Module):
@@ -133,26 +173,39 @@ class Relu2MLP(nn.Module):
 
 
 class ExpertsMLP(nn.Module):
-    """Mixture of gated experts: ``sum_e s_e W_down,e act(W_gate,e y, W_up,e y)`` over a token's chosen experts. Scores ``s``
-    are the softmax of the router's logits (32-bit) over all experts; the ``top`` largest of ``s + correction`` are chosen
-    and weighted by ``s``, not renormalised. The activation is ``ops/moe.py::GatedAct`` with the family's constants. Gate
-    and up rows alternate in ``gate_up`` so that the activation runs in the product's epilogue."""
+    """Mixture of gated experts. Scores ``s`` are the softmax of the router's logits (32-bit) over all experts, or each
+    expert's sigmoid (``router["score"]``); the ``top`` largest of ``s``, plus a learned correction unless
+    ``router["correction"]`` is false, are chosen and weighted by ``s``, not renormalised. The weight multiplies an expert's
+    result, or what goes into it (``spec["weight"]`` "input"). Every token also passes through the ``shared`` expert, when
+    there is one. An expert is ``W_down act(W_gate y, W_up y)`` with the activation of ``ops/moe.py::GatedAct``. Gate and
+    up rows alternate in ``gate_up`` so that the activation runs in the product's epilogue."""
 
     o = None
 
-    def __init__(self, hidden: int, spec: dict, act: GatedAct, dtype, device):
+    def __init__(self, hidden: int, spec: dict, act, dtype, device):
+        """``act``: the activation for an expert's ``limit``."""
         super().__init__()
-        E, ff = spec["router"]["experts"], spec["expert"]["ff"]
+        router = spec["router"]
+        E, ff = router["experts"], spec["expert"]["ff"]
         mk = lambda *shape: nn.Parameter(torch.empty(*shape, dtype=dtype, device=device))
-        self.top, self.act = spec["router"]["top"], act
+        self.top, self.score = router["top"], router.get("score", "softmax")
+        self.act, self.scale_input = act(spec["expert"]["limit"]), spec.get("weight") == "input"
         self.router = mk(E, hidden)
-        self.correction = nn.Parameter(torch.zeros(E, dtype=dtype, device=device))
+        self.correction = nn.Parameter(torch.zeros(E, dtype=dtype, device=device)) if router.get("correction", True) else None
         self.gate_up = mk(E, 2 * ff, hidden)
         self.down = mk(E, hidden, ff)
+        self.shared = GatedMLP(hidden, spec["shared"]["ff"], act(spec["shared"]["limit"]), dtype, device) \
+            if spec.get("shared") else None
 
     def hidden(self, y, ctx=None, cache=None, rec=None):
-        idx, w = route_tokens(y, self.router, self.top, False, self.correction)
-        return gated_experts(y, idx, w, self.gate_up, self.down, self.act)
+        idx, w = route_tokens(y, self.router, self.top, False, self.correction, self.score)
+        e = gated_experts(y, idx, w, self.gate_up, self.down, self.act, self.scale_input)
+        if self.shared is None:
+            return e
+        if not isinstance(e, ExpertRows):
+            return e + linear(self.shared.hidden(y), self.shared.o).float()
+        e.add = linear_slices(self.shared.hidden(y), self.shared.o)
+        return e
 
     def tensors(self, p: str):
         for e in range(self.router.shape[0]):
@@ -160,13 +213,34 @@ class ExpertsMLP(nn.Module):
             yield f"{p}e{e}.up", self.gate_up[e, 1::2]
             yield f"{p}e{e}.down", self.down[e]
         yield p + "router", self.router
-        yield p + "correction", self.correction
+        if self.correction is not None:
+            yield p + "correction", self.correction
+        if self.shared is not None:
+            yield from self.shared.tensors(p + "shared.")
+
+
+class GatedMLP(nn.Module):
+    """``act(W_gate y, W_up y)``, to be projected by ``o`` (the down projection); gate and up rows alternate in ``gate_up``."""
+
+    def __init__(self, hidden: int, ff: int, act: GatedAct, dtype, device):
+        super().__init__()
+        self.act = act
+        self.gate_up = nn.Parameter(torch.empty(2 * ff, hidden, dtype=dtype, device=device))
+        self.o = nn.Parameter(torch.empty(hidden, ff, dtype=dtype, device=device))
+
+    def hidden(self, y, ctx=None, cache=None, rec=None):
+        return gated_linear(y, self.gate_up, self.act)
+
+    def tensors(self, p: str):
+        yield p + "gate", self.gate_up[0::2]
+        yield p + "up", self.gate_up[1::2]
+        yield p + "down", self.o
 
 
 def make_mlp(hidden: int, spec: dict, eps: float, dtype, device):
     if spec["kind"] == "moe":
         # x * sigmoid(1.702 x) approximates GELU (Hendrycks and Gimpel, "Gaussian Error Linear Units")
-        return ExpertsMLP(hidden, spec, GatedAct(alpha=1.702, beta=1.0, limit=float(spec["expert"]["limit"])), dtype, device)
+        return ExpertsMLP(hidden, spec, lambda limit: GatedAct(alpha=1.702, beta=1.0, limit=float(limit)), dtype, device)
     return {"polynorm": PolyNormMLP, "relu2": Relu2MLP}[spec.get("act", "polynorm")](hidden, spec, eps, dtype, device)
 
 
@@ -194,7 +268,7 @@ class LayeredBlock(nn.Module):
     def __init__(self, cfg: ModelConfig, i: int, dtype, device):
         super().__init__()
         h, spec, eps = cfg.hidden_size, cfg.layer_specs[i], cfg.rms_norm_eps
-        norm, wrap, self.wrap_names = NORMS[cfg.layer_norms]
+        norm, wrap, self.wrap_names, _ = NORMS[cfg.layer_norms]
         self.norm1 = norm(h, eps, dtype, device)
         self.attn = MIXERS[spec["type"]](h, spec["mixer"], eps, dtype, device)
         self.attn.index = i
@@ -253,8 +327,14 @@ class LayeredModel(QwenModel):
         self.layer_start, self.layer_end = 0, cfg.num_hidden_layers
         mk = lambda *shape: nn.Parameter(torch.empty(*shape, dtype=dtype, device=device))
         self.embed = mk(cfg.vocab_size, cfg.hidden_size)
-        self.layers = nn.ModuleList(LayeredBlock(cfg, i, dtype, device) for i in self.layer_ids)
-        self.norm = NORMS[cfg.layer_norms][0](cfg.hidden_size, cfg.rms_norm_eps, dtype, device)
+        self.pos = mk(cfg.max_position_embeddings, cfg.hidden_size) if cfg.learned_positions else None
+        self.layers = nn.ModuleList()
+        for i in self.layer_ids:  # a layer that runs with another's weights is the same module once more
+            j = cfg.weights_layer(i)
+            self.layers.append(LayeredBlock(cfg, i, dtype, device) if j == i else self.layers[j])
+        # the head is linear: the logits' scale is the last norm's
+        scaled = dict(scale=cfg.logit_scale) if cfg.logit_scale != 1.0 else {}
+        self.norm = NORMS[cfg.layer_norms][3](cfg.hidden_size, cfg.rms_norm_eps, dtype, device, **scaled)
         self.lm_head = mk(cfg.vocab_size, cfg.hidden_size)
         self.score = None
         self.checkpoint_every = 0
@@ -297,13 +377,17 @@ class LayeredModel(QwenModel):
         ctx.shared = self._shared
         subs = []  # (sublayer, its wrap, its norm, its cache, its state)
         for i, layer in enumerate(self.layers):
-            src = kv_caches[self.cfg.cache_layer(i)] if kv_caches is not None else None
-            cache = src[0] if src is not None else None
+            cache = kv_caches[self.cfg.cache_layer(i)] if kv_caches is not None else None
+            if cache is not None and len(cache) == 1:
+                cache = cache[0]
             subs.append((layer.attn, layer.wrap1, layer.norm1, cache, state.rec[i] if state is not None else None))
             if layer.mlp is not None:
                 subs.append((layer.mlp, layer.wrap2, layer.norm2, None, None))
         norms = [s[2] for s in subs] + [self.norm]
-        y, res = norms[0].embed(input_ids, self.embed)
+        extra = {}
+        if self.pos is not None or self.cfg.embedding_scale != 1.0:
+            extra = dict(scale=self.cfg.embedding_scale, pos=ctx.pos, pos_table=self.pos)
+        y, res = norms[0].embed(input_ids, self.embed, **extra)
         for k, (sub, wrap, _, cache, rec) in enumerate(subs):
             y, res = norms[k + 1].join(sub.hidden(y, ctx, cache, rec), sub.o, wrap, res)
         return y
@@ -331,8 +415,11 @@ class LayeredModel(QwenModel):
     # ----------------------------------------------------------------- checkpoint
     def to_hf_local(self, export: bool = False) -> Iterator[tuple[str, torch.Tensor]]:
         yield "embed", self.embed
+        if self.pos is not None:
+            yield "pos", self.pos
         for i, layer in enumerate(self.layers):
-            yield from layer.tensors(f"l{i}.")
+            if self.cfg.weights_layer(i) == i:
+                yield from layer.tensors(f"l{i}.")
         yield from self.norm.tensors("final.norm")
         yield "head", self.lm_head
 

@@ -16,6 +16,7 @@ Counterpart of the cuBLAS-backed ``nn.Linear`` calls of the reference
 from __future__ import annotations
 
 import ctypes
+from dataclasses import dataclass
 
 import torch
 
@@ -133,14 +134,46 @@ def _splitk_plan(M: int, N: int, K: int) -> int:
     return splits if splits >= 2 else 0
 
 
-def linear_pitched(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    """``x @ w.T`` whose rows start 16-byte aligned whatever the number of columns: slices of them feed kernels that want
-    aligned pitches."""
+def linear_pitched(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None) -> torch.Tensor:
+    """``x @ w.T (+ bias)`` whose rows start 16-byte aligned whatever the number of columns: slices of them feed kernels
+    that want aligned pitches."""
     N = w.shape[0]
     grad = torch.is_grad_enabled() and (x.requires_grad or w.requires_grad)
     if N % 8 == 0 or grad or not (_lib.use_cuda_kernels(x, w) and x.dtype == torch.bfloat16):
+        return linear(x, w, bias)
+    return gemm(x, w, bias=bias, out=torch.empty((x.shape[0], -(-N // 8) * 8), dtype=x.dtype, device=x.device)[:, :N])
+
+
+@dataclass
+class Slices:
+    """A product whose reduction is still split: row ``r`` is the sum over ``s < n`` of the fp32 rows at ``s * stride + r *
+    columns`` of ``ws``. The kernel that reads it does the sum."""
+
+    ws: torch.Tensor
+    stride: int
+    n: int
+
+
+def _tma_rows(*ts: torch.Tensor) -> bool:
+    return all(t.stride(1) == 1 and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in ts)
+
+
+def linear_slices(x: torch.Tensor, w: torch.Tensor) -> "torch.Tensor | Slices":
+    """``x @ w.T``, as :class:`Slices` where the product is decode-sized and split over its reduction."""
+    M, K = x.shape
+    N = w.shape[0]
+    splits = _splitk_plan(M, N, K) if x.dtype == torch.bfloat16 and _lib.use_cuda_kernels(x, w) else 0
+    if not (splits and K % 8 == 0 and _tma_rows(x, w)):
         return linear(x, w)
-    return gemm(x, w, out=torch.empty((x.shape[0], -(-N // 8) * 8), dtype=x.dtype, device=x.device)[:, :N])
+    ws = torch.empty((splits * -(-M // 128) * 128, N), dtype=torch.float32, device=x.device)
+    S, stride = ctypes.c_int(0), ctypes.c_longlong(0)
+    rc = _lib.kernels().b200_gemm_bf16_splitk_partials(
+        _lib.ptr(x), _lib.ptr(w), _lib.ptr(ws), ctypes.c_int(M), ctypes.c_int(N), ctypes.c_int(K),
+        ctypes.c_longlong(x.stride(0)), ctypes.c_longlong(w.stride(0)), ctypes.c_int(splits), ctypes.byref(S),
+        ctypes.byref(stride), _lib.stream_ptr())
+    _lib.check(rc, "b200_gemm_bf16_splitk_partials")
+    _lib.count_launch()
+    return Slices(ws, stride.value, S.value)
 
 
 def linear_relu2(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:

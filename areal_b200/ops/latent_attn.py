@@ -25,12 +25,15 @@ from .dyt import fp32_flag, kernel_ok
 def rotary_tables(n: int, dims: int, base: float, device, scaling: dict | None = None):
     """``cos, sin [n, dims / 2]`` (fp32) of ``p * f_i``, ``f_i = base^(-2i / dims)``, the angles taken in double precision.
 
-    ``scaling`` (``factor, original, fast, slow``) is YaRN's: pairs that turn fewer than ``slow`` times within ``original``
-    positions are slowed down by ``factor``, those that turn more than ``fast`` times keep their frequency, with a linear
-    ramp over the pair index in between; ``cos`` and ``sin`` are multiplied by ``0.1 ln(factor) + 1``."""
+    ``scaling`` with a ``factor`` alone divides every ``f_i`` by it. With ``factor, original, fast, slow`` it is YaRN's:
+    pairs that turn fewer than ``slow`` times within ``original`` positions are slowed down by ``factor``, those that turn
+    more than ``fast`` times keep their frequency, with a linear ramp over the pair index in between; ``cos`` and ``sin``
+    are multiplied by ``0.1 ln(factor) + 1``."""
     f = base ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
     mag = 1.0
-    if scaling:
+    if scaling and "original" not in scaling:
+        f = f / scaling["factor"]
+    elif scaling:
         at = lambda turns: dims * math.log(scaling["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
         lo, hi = max(math.floor(at(scaling["fast"])), 0), min(math.ceil(at(scaling["slow"])), dims - 1)
         ramp = ((torch.arange(dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0, 1)

@@ -83,13 +83,12 @@ def linear_residual_ln(a: torch.Tensor, w: torch.Tensor, post, res: torch.Tensor
 
 
 def experts_residual_ln(e, post, res: torch.Tensor, norm, eps: float):
-    """The weighted sum of a token's chosen experts (``e``: :class:`ops.moe.ExpertRows`), its norm, the residual add and
+    """The weighted sum of a token's chosen experts and addend (``e``: :class:`ops.moe.ExpertRows`), its norm, the residual add and
     the next sublayer's norm in one kernel."""
     T, W = res.shape
     y = torch.empty((T, W), dtype=norm[0].dtype, device=res.device)
-    rc = _lib.kernels().b200_experts_residual_ln(*_p(e.rows, e.dest, e.w), ctypes.c_int(e.w.shape[1]), *_p(*post, res, *norm, y),
-                                                 ctypes.c_longlong(T), ctypes.c_int(W), ctypes.c_float(eps), fp32_flag(y),
-                                                 _lib.stream_ptr())
+    rc = _lib.kernels().b200_experts_residual_ln(*e.args(), *_p(*post, res, *norm, y), ctypes.c_longlong(T),
+                                                 ctypes.c_int(W), ctypes.c_float(eps), fp32_flag(y), _lib.stream_ptr())
     _lib.check(rc, "b200_experts_residual_ln")
     _lib.count_launch()
     return y, res

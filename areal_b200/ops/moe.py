@@ -26,14 +26,17 @@ import torch
 
 from . import _lib, fused
 from .dyt import fp32_flag, kernel_ok
-from .gemm import gemm, linear
+from .gemm import Slices, _splitk_plan, _tma_rows, gemm, linear
 
 
 # --------------------------------------------------------------------------- references
 
 
-def route_ref(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None):
-    probs = logits.float().softmax(-1)
+_SCORES = {"softmax": 0, "sigmoid": 1}
+
+
+def route_ref(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None, score: str = "softmax"):
+    probs = logits.float().softmax(-1) if score == "softmax" else torch.sigmoid(logits.float())
     if correction is None:
         w, idx = probs.topk(k, dim=-1)
     else:
@@ -77,26 +80,29 @@ def moe_experts_ref(x, idx, w, gate_up, down):
 # --------------------------------------------------------------------------- CUDA pieces
 
 
-def route(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None):
-    """``logits [T, E]`` fp32 → ``(idx [T,k] int32, w [T,k] fp32)``. ``correction [E]`` is added to the scores when the
-    experts are chosen; their weights are the scores without it."""
+def route(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None, score: str = "softmax"):
+    """``logits [T, E]`` fp32 → ``(idx [T,k] int32, w [T,k] fp32)``. Scores are the softmax over all experts or each
+    expert's sigmoid. ``correction [E]`` is added to the scores when the experts are chosen; their weights are the scores
+    without it."""
     T, E = logits.shape
     if not (_lib.use_cuda_kernels(logits) and logits.dtype == torch.float32 and E <= 256 and k <= 32
             and (correction is None or correction.dtype in (torch.float32, torch.bfloat16))):
-        return route_ref(logits, k, renorm, correction)
+        return route_ref(logits, k, renorm, correction, score)
     logits = logits if logits.is_contiguous() else logits.contiguous()
     idx = torch.empty((T, k), dtype=torch.int32, device=logits.device)
     w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
     rc = _lib.kernels().b200_moe_route(_lib.ptr(logits), _lib.ptr(correction),
                                        ctypes.c_int(int(correction is not None and correction.dtype == torch.float32)),
                                        _lib.ptr(idx), _lib.ptr(w), ctypes.c_int(T), ctypes.c_int(E),
-                                       ctypes.c_int(k), ctypes.c_int(int(renorm)), _lib.stream_ptr())
+                                       ctypes.c_int(k), ctypes.c_int(int(renorm)), ctypes.c_int(_SCORES[score]),
+                                       _lib.stream_ptr())
     _lib.check(rc, "b200_moe_route")
     _lib.count_launch()
     return idx, w
 
 
-def route_tokens(x: torch.Tensor, router: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None):
+def route_tokens(x: torch.Tensor, router: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None,
+                 score: str = "softmax"):
     """Router projection (fp32 products and sums) and choice: ``x [T, H]``, ``router [E, H]``. A decode step's few tokens
     take one kernel."""
     T, H = x.shape
@@ -107,15 +113,15 @@ def route_tokens(x: torch.Tensor, router: torch.Tensor, k: int, renorm: bool, co
         w = torch.empty((T, k), dtype=torch.float32, device=x.device)
         rc = _lib.kernels().b200_moe_router(
             _lib.ptr(x), ctypes.c_longlong(x.stride(0)), _lib.ptr(router), _lib.ptr(correction), _lib.ptr(idx), _lib.ptr(w),
-            ctypes.c_int(T), ctypes.c_int(H), ctypes.c_int(E), ctypes.c_int(k), ctypes.c_int(int(renorm)), fp32_flag(x),
-            _lib.stream_ptr())
+            ctypes.c_int(T), ctypes.c_int(H), ctypes.c_int(E), ctypes.c_int(k), ctypes.c_int(int(renorm)),
+            ctypes.c_int(_SCORES[score]), fp32_flag(x), _lib.stream_ptr())
         _lib.check(rc, "b200_moe_router")
         _lib.count_launch()
         return idx, w
     if kernel_ok(x, router):
         logits = gemm(x, router, out_dtype=torch.float32) if x.dtype == torch.bfloat16 else torch.nn.functional.linear(x, router)
-        return route(logits, k, renorm, correction)
-    return route_ref(torch.nn.functional.linear(x.float(), router.float()), k, renorm, correction)
+        return route(logits, k, renorm, correction, score)
+    return route_ref(torch.nn.functional.linear(x.float(), router.float()), k, renorm, correction, score)
 
 
 @dataclass
@@ -317,35 +323,52 @@ class GatedAct:
 @dataclass
 class ExpertRows:
     """Results of the chosen experts, not yet combined: row ``dest[t * k + j]`` of ``rows`` belongs to choice ``j`` of
-    token ``t`` and counts ``w[t, j]``."""
+    token ``t`` and counts ``w[t, j]`` (None: 1). ``add``: what every token adds to the sum of its ``k`` choices."""
 
     rows: torch.Tensor
     dest: torch.Tensor
-    w: torch.Tensor
+    k: int
+    w: torch.Tensor | None
+    add: "torch.Tensor | Slices | None" = None
+
+    def args(self):
+        """``rows, dest, w, k`` and the addend's ``rows, pitch, slices, slice stride, number of slices`` for the kernels
+        that combine."""
+        ll, c, p = ctypes.c_longlong, ctypes.c_int, _lib.ptr
+        sl = self.add if isinstance(self.add, Slices) else None
+        add = self.add if sl is None else None
+        if add is not None and not (add.stride(1) == 1 and add.stride(0) % 4 == 0 and add.data_ptr() % 16 == 0):
+            add = self.add = add.contiguous()
+        return (p(self.rows), p(self.dest), p(self.w), c(self.k), p(add), ll(add.stride(0) if add is not None else 0),
+                p(sl.ws if sl else None), ll(sl.stride if sl else 0), c(sl.n if sl else 0))
 
 
-def gated_experts_ref(x, idx, w, gate_up, down, act: GatedAct):
+def gated_experts_ref(x, idx, w, gate_up, down, act: GatedAct, scale_input: bool = False):
     """``sum_j w[t,j] * down_e(act(gate_e x, up_e x))`` with the rows of ``gate_up [E, 2I, H]`` alternating between gate
-    and up; fp32 ``[T, H]``. Differentiable."""
+    and up; fp32 ``[T, H]``. ``scale_input``: ``sum_j down_e(act(gate_e (w x), up_e (w x)))``. Differentiable."""
     out = torch.zeros(x.shape, dtype=torch.float32, device=x.device)
     for e in range(gate_up.shape[0]):
         t, j = (idx == e).nonzero(as_tuple=True)
         if t.numel() == 0:
             continue
-        z = linear(x[t], gate_up[e])
+        z, s = linear(x[t], gate_up[e]), w[t, j][:, None].float()
+        if scale_input:
+            z, s = (z.float() * s).to(z.dtype), 1.0
         y = linear(act(z[:, 0::2], z[:, 1::2]), down[e])
-        out = out.index_add(0, t, y.float() * w[t, j][:, None].float())
+        out = out.index_add(0, t, y.float() * s)
     return out
 
 
-def gated_experts(x, idx, w, gate_up, down, act: GatedAct):
+def gated_experts(x, idx, w, gate_up, down, act: GatedAct, scale_input: bool = False):
     """The chosen experts of every token: ``x [T, H]``, ``idx / w [T, k]``, ``gate_up [E, 2I, H]`` (gate and up rows
     alternate), ``down [E, H, I]``. On the kernels the result is an :class:`ExpertRows`, which the following norm combines
-    (``ops/layer_norm.py::experts_residual_ln``); elsewhere the combined ``[T, H]``. bf16 sizes in steps of 8 run on the
-    grouped tensor-core products with the activation in the first one's epilogue; 32-bit models and other sizes on a
-    grouped fp32 kernel. Everything stays on the device."""
+    (``ops/layer_norm.py::experts_residual_ln``, ``ops/residual_rms.py::experts_residual_rms``); elsewhere the combined
+    ``[T, H]``. bf16 sizes in steps of 8 run on the grouped tensor-core products with the activation in the first one's
+    epilogue; 32-bit models and other sizes on a grouped fp32 kernel. Everything stays on the device. ``scale_input``: an
+    expert's weight multiplies what goes into it instead of its result; as the first product is linear, its fp32
+    accumulators are scaled."""
     if not kernel_ok(x, gate_up, down, w):
-        return gated_experts_ref(x, idx, w, gate_up, down, act)
+        return gated_experts_ref(x, idx, w, gate_up, down, act, scale_input)
     T, H = x.shape
     E, I2, _ = gate_up.shape
     I, k = I2 // 2, idx.shape[1]
@@ -353,7 +376,8 @@ def gated_experts(x, idx, w, gate_up, down, act: GatedAct):
     c, ll, f, p = ctypes.c_int, ctypes.c_longlong, ctypes.c_float, _lib.ptr
     x = x if x.stride(1) == 1 and x.data_ptr() % 16 == 0 and x.stride(0) % 8 == 0 else x.contiguous()
     new = lambda n: torch.empty((s.max_rows, n), dtype=x.dtype, device=x.device)
-    a, y = new(I), new(H)
+    a, y, w = new(I), new(H), w.float().contiguous()
+    ws = p(w if scale_input else None)
     glu = (f(act.limit), f(act.alpha), f(act.beta))
     lib = _lib.kernels()
     if x.dtype == torch.bfloat16 and H % 8 == 0 and I % 8 == 0 and T > 0:
@@ -361,7 +385,8 @@ def gated_experts(x, idx, w, gate_up, down, act: GatedAct):
         _lib.check(lib.b200_moe_scatter(p(x), ll(x.stride(0)), p(s.dest), c(T), c(k), c(H), p(xs), _lib.stream_ptr()),
                    "b200_moe_scatter")
         _lib.check(lib.b200_gemm_grouped_glu(p(xs), p(gate_up), p(a), p(s.tile_expert), p(s.num_vm), p(s.src_of),
-                                             c(s.max_rows), c(E), c(I), c(H), *glu, _lib.stream_ptr()), "b200_gemm_grouped_glu")
+                                             ws, c(s.max_rows), c(E), c(I), c(H), *glu, _lib.stream_ptr()),
+                   "b200_gemm_grouped_glu")
         _lib.check(lib.b200_gemm_grouped_rows(p(a), p(down), p(y), p(s.tile_expert), p(s.num_vm), p(s.src_of),
                                               c(s.max_rows), c(E), c(H), c(I), _lib.stream_ptr()), "b200_gemm_grouped_rows")
         _lib.count_launch(3)
@@ -369,7 +394,32 @@ def gated_experts(x, idx, w, gate_up, down, act: GatedAct):
         fp32, max_vm = fp32_flag(x), c(s.max_rows // 128)
         for src, ld, gather, w_, out, n, kk, on in ((x, x.stride(0), k, gate_up, a, I2, H, 1), (a, I, 0, down, y, H, I, 0)):
             _lib.check(lib.b200_moe_gemm_simt(p(src), ll(ld), c(gather), p(w_), p(out), ll(out.shape[1]), p(s.tile_expert),
-                                              p(s.num_vm), p(s.src_of), max_vm, c(n), c(kk), c(on), *glu, fp32,
-                                              _lib.stream_ptr()), "b200_moe_gemm_simt")
+                                              p(s.num_vm), p(s.src_of), ws if on else p(None), max_vm, c(n), c(kk),
+                                              c(on), *glu, fp32, _lib.stream_ptr()), "b200_moe_gemm_simt")
         _lib.count_launch(2)
-    return ExpertRows(y, s.dest, w.float().contiguous())
+    return ExpertRows(y, s.dest, k, None if scale_input else w)
+
+
+def gated_linear(x: torch.Tensor, gate_up: torch.Tensor, act: GatedAct) -> torch.Tensor:
+    """``act(W_gate x, W_up x)`` with alternating gate and up rows ``gate_up [2I, H]``: ``[T, I]``. On the bf16 kernels the
+    activation runs on the product's fp32 accumulators (for decode-sized products in the split-K reduction)."""
+    if not kernel_ok(x, gate_up):
+        z = linear(x, gate_up)
+        return act(z[:, 0::2], z[:, 1::2])
+    T, H = x.shape
+    I = gate_up.shape[0] // 2
+    c, ll, f, p = ctypes.c_int, ctypes.c_longlong, ctypes.c_float, _lib.ptr
+    glu = (f(act.limit), f(act.alpha), f(act.beta))
+    out = torch.empty((T, I), dtype=x.dtype, device=x.device)
+    lib = _lib.kernels()
+    if x.dtype == torch.bfloat16 and I % 8 == 0 and H % 8 == 0 and _tma_rows(x, gate_up):
+        splits = _splitk_plan(T, 2 * I, H)
+        ws = torch.empty((splits * -(-T // 128) * 128, 2 * I), dtype=torch.float32, device=x.device) if splits else None
+        _lib.check(lib.b200_gemm_bf16_glu(p(x), p(gate_up), p(out), p(ws), c(T), c(I), c(H), ll(x.stride(0)),
+                                          ll(gate_up.stride(0)), c(splits), *glu, _lib.stream_ptr()), "b200_gemm_bf16_glu")
+        _lib.count_launch(2 if splits else 1)
+        return out
+    z = linear(x, gate_up).contiguous()
+    _lib.check(lib.b200_glu_pairs(p(z), p(out), ll(out.numel()), *glu, fp32_flag(x), _lib.stream_ptr()), "b200_glu_pairs")
+    _lib.count_launch()
+    return out

@@ -212,10 +212,11 @@ def run_gatolix() -> list[dict]:
         h, y = torch.empty(s.max_rows, ff, device="cuda", dtype=BF), torch.empty(s.max_rows, W, device="cuda", dtype=BF)
         glu = tuple(ctypes.c_float(f) for f in (act.limit, act.alpha, act.beta))
         tail = (p(s.tile_expert), p(s.num_vm), p(s.src_of), c(s.max_rows), c(E))
+        glu_tail = (*tail[:3], p(None), *tail[3:])
         add(f"moe_scatter {t} x 6", lambda: lib.b200_moe_scatter(p(xt), ctypes.c_longlong(W), p(s.dest), c(t), c(k), c(W), p(xs), st()),
             (t + rows) * W * 2, iters=it)
         add(f"[deepseek] gather {t} x 6", lambda: moe.gather_rows(xt, s), (t + rows) * W * 2, iters=it)
-        add(f"grouped gate | up + activation {t} x 6", lambda: lib.b200_gemm_grouped_glu(p(xs), p(gu), p(h), *tail, c(ff), c(W), *glu, st()),
+        add(f"grouped gate | up + activation {t} x 6", lambda: lib.b200_gemm_grouped_glu(p(xs), p(gu), p(h), *glu_tail, c(ff), c(W), *glu, st()),
             weights(2 * ff) + rows * (W + ff) * 2, 4.0 * rows * W * ff, iters=it)
         add(f"[deepseek] grouped gate | up, then SwiGLU {t} x 6", lambda: moe._swiglu_raw(moe.grouped_gemm(xs, gu, s)),
             weights(2 * ff) + rows * (W + ff) * 2, 4.0 * rows * W * ff, iters=it)
@@ -223,7 +224,7 @@ def run_gatolix() -> list[dict]:
             weights(ff) + rows * (W + ff) * 2, 2.0 * rows * W * ff, iters=it)
         add(f"[deepseek] grouped down {t} x 6", lambda: moe.grouped_gemm(h, down, s),
             weights(ff) + rows * (W + ff) * 2, 2.0 * rows * W * ff, iters=it)
-        e = moe.ExpertRows(y, s.dest, w)
+        e = moe.ExpertRows(y, s.dest, k, w)
         add(f"experts_residual_ln {t} x 6 (combine, two norms)", lambda: ln.experts_residual_ln(e, post, res[:t], norm, 1e-6),
             t * W * (2 * k + 10), iters=it)
         add(f"[deepseek] combine {t} x 6, then rmsnorm + residual", lambda: fused.rmsnorm(moe.combine_rows(y, s, w), wn, 1e-6, residual=resb[:t]),
