@@ -88,7 +88,7 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   uint8_t* sK = sQ + C::kQ;
   uint8_t* sV = sK + 2 * C::kK;
   uint64_t *q_full = &bars[0], *k_full = &bars[1], *k_empty = &bars[3], *v_full = &bars[5], *v_empty = &bars[7],
-           *s_full = &bars[9], *p_ready = &bars[11], *pv_done = &bars[12];
+           *s_full = &bars[9], *p_ready = &bars[11], *pv_done = &bars[13];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const GqaTile tile = a.tiles[blockIdx.x];
   const int h = blockIdx.y, hk = h / a.group;
@@ -113,9 +113,10 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       mbar_init(&v_full[i], 1);
       mbar_init(&v_empty[i], 1);
       mbar_init(&s_full[i], 1);
+      // one per score buffer: a role may be a whole block ahead of what another has looked at
+      mbar_init(&p_ready[i], 128);
+      mbar_init(&pv_done[i], 1);
     }
-    mbar_init(p_ready, 128);
-    mbar_init(pv_done, 1);
     fence_mbar_init();
     prefetch_tmap(&tmQ);
     prefetch_tmap(&tmK);
@@ -186,7 +187,7 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         // the other score buffer held the weights of block j - 1, whose product was issued before this one: products
         // of one CTA run in issue order
         if (j + 1 < nblk && !issue_s(j + 1)) { ok = false; break; }
-        if (!mbar_wait(p_ready, j & 1, abort_flag)) { ok = false; break; }
+        if (!mbar_wait(&p_ready[j & 1], (j >> 1) & 1, abort_flag)) { ok = false; break; }
         if (!mbar_wait(&v_full[vs], (j / VS) & 1, abort_flag)) { ok = false; break; }
         tc_fence_after();
         const uint32_t v_addr = smem_u32(sV + vs * C::kV), p_addr = tmem_base + (j & 1) * kGpK;
@@ -196,7 +197,7 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           gqa_umma_ts(tmem_O, p_addr + k * 8, b, idesc_o, (j > 0 || k > 0) ? 1u : 0u);
         }
         umma_commit(&v_empty[vs]);
-        umma_commit(pv_done);
+        umma_commit(&pv_done[j & 1]);
       }
       if (!ok) {
         *abort_flag = 1;
@@ -255,7 +256,7 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         const bool grow = mx > m + 8.f;
         if (__any_sync(0xffffffffu, grow)) {
           if (j > 0) {
-            if (!mbar_wait(pv_done, (j - 1) & 1, abort_flag)) { ok = false; break; }
+            if (!mbar_wait(&pv_done[(j - 1) & 1], ((j - 1) >> 1) & 1, abort_flag)) { ok = false; break; }
             tc_fence_after();
           }
           const float mn = grow ? mx : m;
@@ -287,11 +288,10 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       tmem_st_32x32(s_addr + 32, lo);
       tmem_st_wait();
       tc_fence_before();
-      mbar_arrive(p_ready);
+      mbar_arrive(&p_ready[j & 1]);
     }
     if (ok && nblk > 0) {
-      ok = nblk < 2 || mbar_wait(pv_done, nblk & 1, abort_flag);  // phases are waited for in order
-      ok = ok && mbar_wait(pv_done, (nblk - 1) & 1, abort_flag);
+      ok = mbar_wait(&pv_done[(nblk - 1) & 1], ((nblk - 1) >> 1) & 1, abort_flag);  // products run in issue order
       tc_fence_after();
     }
     if (ok) {
