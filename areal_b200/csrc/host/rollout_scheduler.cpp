@@ -328,6 +328,7 @@ int b200_sched_plan(void* h, PlanHeader* hdr, int64_t* seq_ids, int32_t* cu_seql
     if (s->running.empty()) return kIdle;
     i = 0;  // re-check from the start with the freed pages
   }
+  if (s->running.empty()) return kIdle;  // every sequence was at its limit
   // Sequences that share prefix pages sit next to each other in the batch (equal first page): the attention
   // kernel's blocks of one group then run at about the same time and read the shared pages from L2.
   std::vector<int64_t> order(s->running.begin(), s->running.end());

@@ -20,6 +20,16 @@ def _few_cpu_threads():
     torch.set_num_threads(n)
 
 
+@pytest.fixture(autouse=True)
+def _no_wait_ran_out():
+    """A kernel whose bounded wait runs out leaves its results unwritten and a code in the status word."""
+    from areal_b200.ops import _lib
+
+    _lib.read_status()
+    yield
+    assert _lib.read_status() == 0
+
+
 DTYPES = [torch.bfloat16, torch.float32]
 
 
@@ -278,6 +288,28 @@ def test_attention_of_packed_prompts(dt, H, G, D, Dv, opt, unit):
             if 0 <= row < m and float(want[row].abs().max()) > 1e-2:  # (a dominant sink leaves little)
                 _close(got[s0 + row], want[row], _tol(dt, 8e-3, 2e-5))
         s0 = e
+
+
+@pytest.mark.parametrize("unit,cap", [(False, 30.0), (True, 30.0), (False, 0.0)])
+def test_repeated_launches_agree(unit, cap):
+    """Many launches over a batch of many short tiles, into memory that holds no numbers: every launch writes every row,
+    and always the same bits (its warps meet in a different order each time)."""
+    from areal_b200.ops.attention import VarlenMeta
+    from areal_b200.ops.gqa import prefill
+
+    H, G, D, Dv, lens = 20, 1, 80, 64, [1, 64, 65, 129, 300]
+    T = sum(lens)
+    a = _spec(H, G, D, Dv, softcap=cap, unit_eps=1e-6 if unit else None)
+    q, k, v = _rand(T, H, D, seed=1), _rand(T, G, D, seed=2), _rand(T, G, Dv, seed=3)
+    if unit:
+        q, k = (t / t.pow(2).mean(-1, keepdim=True).sqrt() for t in (q, k))
+    q, k, v = (t.to(torch.bfloat16) for t in (q, k, v))
+    meta = VarlenMeta([0] + np.cumsum(lens).tolist(), "cuda")
+    first = prefill(q, k, v, meta, a)
+    for _ in range(400):
+        junk = torch.full_like(first, float("nan"))
+        del junk
+        assert torch.equal(prefill(q, k, v, meta, a), first)
 
 
 @pytest.mark.parametrize("dt", DTYPES)
