@@ -1,12 +1,15 @@
 """Serving throughput of a layered model beside the closest other family at equal sizes, and its kernels one by one beside
 their counterparts.
 
-    python bench.py --serving [--serving-family fofosun|gatolix] [--serving-sizes s,m,l] [--serving-kernels]
+    python bench.py --serving [--serving-family fofosun|gatolix|felosun] [--serving-sizes s,m,l] [--serving-kernels]
 
 Fofosun beside the Bailing hybrid: 8 layers of the given width with random weights, 6 recurrent and 2 latent-attention
 layers, a feed-forward of the same width on each. Gatolix beside DeepSeek-V2: 8 layers of latent attention with a plain
 query projection, a dense feed-forward on the first, mixtures of 64 experts (6 per token) on the others; Gatolix with
-windows of 512 tokens and half of its layers reading another layer's latents. Both run through the rollout engine's scheduler and step functions (captured decode graphs where the
+windows of 512 tokens and half of its layers reading another layer's latents. Felosun beside Qwen3-MoE with a shared
+expert: 8 layers of grouped-query attention (heads of 128, four query heads per key / value head), mixtures of 64 experts (6
+per token) and a shared expert twice as wide on each; in Felosun every other layer sees a window of 512 tokens and the first
+64. Both run through the rollout engine's scheduler and step functions (captured decode graphs where the
 family has them). Prefill: 8 prompts of 2048 tokens in one step. Decode: 64 sequences at a context of 2048 tokens.
 Times are CUDA events on the launching stream; weights, caches and states exceed the L2. Kernel timings flush the L2
 between iterations; fractions are of the measured peaks.
@@ -79,8 +82,29 @@ def deepseek_config(width, heads, q_rank, kv_rank, ff, expert_ff) -> ModelConfig
                        qk_rope_head_dim=64, v_head_dim=128, rope_interleave=True, max_position_embeddings=8192)
 
 
+def felosun_config(width, heads, q_rank, kv_rank, ff, expert_ff) -> ModelConfig:
+    size = {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    a = {"type": "attention", "mixer": dict(size, mask={"size": WINDOW, "keep_first": 64}, rot={"base": 1e4, "dims": 64})}
+    b = {"type": "attention_2", "mixer": dict(size, softcap=50.0, rot={"base": 1e4, "dims": 128, "scaling": {"factor": 4.0}})}
+    mlp = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP}, "expert": {"ff": expert_ff, "limit": 7.0},
+           "shared": {"ff": 2 * expert_ff, "limit": 7.0}}
+    return ModelConfig.from_hf_config({"architecture": "Felosun", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6},
+                                       "embedding": {"scale": 1.0}, "logit_scale": 1.0, "max_positions": 8192,
+                                       "layers": [dict(x, mlp=mlp) for x in [a, b] * (LAYERS // 2)]})
+
+
+def qwen_moe_config(width, heads, q_rank, kv_rank, ff, expert_ff) -> ModelConfig:
+    return ModelConfig(model_type="qwen3_moe", vocab_size=VOCAB, hidden_size=width, intermediate_size=ff,
+                       num_hidden_layers=LAYERS, num_attention_heads=heads, num_key_value_heads=heads // 4, head_dim=128,
+                       rope_theta=1e4, tie_word_embeddings=False, qk_norm=True, num_experts=EXPERTS,
+                       num_experts_per_tok=TOP, moe_intermediate_size=expert_ff, norm_topk_prob=False,
+                       shared_expert_intermediate_size=2 * expert_ff, shared_expert_gated=False,
+                       max_position_embeddings=8192)
+
+
 FAMILIES = {"fofosun": (("fofosun", fofosun_config), ("bailing_hybrid", bailing_config)),
-            "gatolix": (("gatolix", gatolix_config), ("deepseek_v2", deepseek_config))}
+            "gatolix": (("gatolix", gatolix_config), ("deepseek_v2", deepseek_config)),
+            "felosun": (("felosun", felosun_config), ("qwen3_moe", qwen_moe_config))}
 
 
 def _engine(cfg: ModelConfig, seqs: int, context: int, tokens: int):
@@ -168,16 +192,16 @@ def main(sizes: list[str], kernels: bool, sampler=None, family: str = "fofosun")
     res: dict = {"benchmark": "serving", "layers": LAYERS, "dtype": "bf16", "data": "random tokens, random weights",
                  "prefill": "8 x 2048 tokens", "decode": "64 sequences at 2048 tokens", "models": {}}
     for name in sizes:
-        more = dict(expert_ff=EXPERT_FF[name]) if family == "gatolix" else {}
+        more = dict(expert_ff=EXPERT_FF[name]) if family != "fofosun" else {}
         for fam, make in FAMILIES[family]:
             res["models"][f"{fam}-{name}"] = serve(make(**SIZES[name], **more))
             torch.cuda.empty_cache()
     if sampler is not None:
         res["clocks"] = sampler.stop()
     if kernels:
-        from .bench_serving_kernels import run, run_gatolix
+        from . import bench_serving_kernels as k
 
-        res["kernels"] = run_gatolix() if family == "gatolix" else run()
+        res["kernels"] = {"fofosun": k.run, "gatolix": k.run_gatolix, "felosun": k.run_felosun}[family]()
     res["seconds"] = round(time.time() - t0)
     print(json.dumps(res), flush=True)
     return 0

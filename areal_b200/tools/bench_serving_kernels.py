@@ -8,10 +8,10 @@ import ctypes
 import numpy as np
 import torch
 
-from ..ops import _lib, dyt, fused, latent_attn as la, layer_norm as ln, moe
+from ..ops import _lib, dyt, fused, gqa, latent_attn as la, layer_norm as ln, moe, residual_rms as rr
 from ..ops.attention import VarlenMeta, varlen_attention
 from ..ops.gated_scan import ScanSpec, scan_prefill, scan_step
-from ..ops.gemm import linear, linear_relu2, linear_rmsnorm
+from ..ops.gemm import linear, linear_relu2, linear_rmsnorm, linear_slices
 from ..ops.linear_attn import linear_attn_prefill, linear_attn_step
 from ..ops.lm_head import lm_head_sample, new_sampling_rng
 from ..ops.microbench import peaks, timeit
@@ -237,4 +237,133 @@ def run_gatolix() -> list[dict]:
     wl, temp, rng = _rand(32000, W, s=W ** -0.5), torch.ones(B, device="cuda"), new_sampling_rng(0, "cuda")
     add("lm_head_sample batch 64, soft cap", lambda: lm_head_sample(aw[:B], wl, temp, rng, softcap=30.0), 32000 * W * 2, iters=20)
     add("[any] lm_head_sample batch 64", lambda: lm_head_sample(aw[:B], wl, temp, rng), 32000 * W * 2, iters=20)
+    return out
+
+
+@torch.no_grad()
+def run_felosun() -> list[dict]:
+    """Kernels of the Felosun family beside those of the families with like ones."""
+    out = []
+    torch.manual_seed(0)
+    H, G, D, n, L, B, W, win, keep = 16, 4, 128, 8, 2048, 64, 2048, 512, 64
+    T = n * L
+    add = lambda *a, **k: out.append(_row(*a, **k))
+    unit = lambda t: (t.float() / t.float().pow(2).mean(-1, keepdim=True).sqrt()).to(BF)
+    spec = lambda h=H, g=G, d=D, **kw: gqa.GroupedSpec(h, g, d, d, d ** -0.5, rot_dims=kw.pop("rot", 64), unit_eps=1e-6, **kw)
+    # --- prompts: FLOPs of the visible pairs
+    meta = VarlenMeta([L * i for i in range(n + 1)], "cuda")
+    pairs = n * L * L / 2
+    seen = n * sum(min(i + 1, win + min(keep, max(0, i + 1 - win))) for i in range(L))
+    q, k, v, sink, gate = unit(_rand(T, H, D)), unit(_rand(T, G, D)), _rand(T, G, D), _rand(H), _rand(T, H)
+    flops = lambda p, h=H, d=D: p * h * 4 * d
+    add("gqa.prefill 8x2048, 16 / 4 heads of 128, window 512 + 64, sink", lambda: gqa.prefill(q, k, v, meta, spec(window=win, keep_first=keep), sink), 0, flops(seen))
+    add("gqa.prefill 8x2048, cap, gate", lambda: gqa.prefill(q, k, v, meta, spec(softcap=50.0), None, gate), 0, flops(pairs))
+    add("gqa.prefill 8x2048, small cap, gate", lambda: gqa.prefill(q, k, v, meta, spec(softcap=15.0), None, gate), 0, flops(pairs))
+    add("gqa.prefill 8x2048", lambda: gqa.prefill(q, k, v, meta, spec()), 0, flops(pairs))
+    add("[qwen3] attn_fwd 8x2048, 16 / 4 heads of 128", lambda: varlen_attention(q, k, v, meta), 0, flops(pairs))
+    x4, g4 = _rand(T, H * 192 + 512 + 64 + H), _rand(T, H)
+    ql, kv4, kr = x4[:, :H * 192], _rand(T, H * 256), _rand(T, 64)
+    add("[gatolix] latent_prefill 8x2048, window 512, gate", lambda: la.latent_attention(ql, kv4, kr, meta, H, 128, 64, 128, 0.07, win, g4), 0,
+        n * H * 2 * 320 * sum(min(i + 1, win) for i in range(L)))
+    add("[gatolix] latent_prefill 8x2048, gate", lambda: la.latent_attention(ql, kv4, kr, meta, H, 128, 64, 128, 0.07, None, g4), 0, pairs * H * 2 * 320)
+    for d in (64, 96):
+        qd, kd, vd = unit(_rand(T, H, d)), unit(_rand(T, G, d)), _rand(T, G, d)
+        add(f"gqa.prefill 8x2048, 16 / 4 heads of {d}", lambda: gqa.prefill(qd, kd, vd, meta, spec(d=d)), 0, flops(pairs, d=d))
+    # --- decoding: the visible rows once
+    ctx, bs = 2048, 16
+    nb = B * ctx // bs
+    bt = torch.randperm(nb, device="cuda").view(B, -1).int()
+    lens = torch.full((B,), ctx, device="cuda", dtype=torch.int32)
+    for h, g in ((16, 4), (8, 8)):
+        kc, vc, qd = unit(_rand(nb, g, bs, D)), _rand(nb, g, bs, D), unit(_rand(B, h, D))
+        rows = lambda m: 2 * B * m * g * D * 2
+        s1, g1 = _rand(h), _rand(B, h)
+        add(f"gqa.decode 64 x 2048, {h} / {g} heads of 128, window 512 + 64, sink", lambda: gqa.decode(qd, kc, vc, bt, lens, spec(h, g, window=win, keep_first=keep), s1, None, ctx), rows(win + keep))
+        add(f"[qwen3] paged_decode 64 x 576, {h} / {g} heads", lambda: paged_decode(qd, kc, vc, bt, lens // 2048 * 576, max_seq_len=576), rows(576))
+        add(f"gqa.decode 64 x 2048, {h} / {g} heads of 128, cap, gate", lambda: gqa.decode(qd, kc, vc, bt, lens, spec(h, g, softcap=50.0), None, g1, ctx), rows(ctx))
+        add(f"[qwen3] paged_decode 64 x 2048, {h} / {g} heads", lambda: paged_decode(qd, kc, vc, bt, lens, max_seq_len=ctx), rows(ctx))
+    kc, vc, qd = unit(_rand(nb, G, bs, 64)), _rand(nb, G, bs, 64), unit(_rand(B, H, 64))
+    add("gqa.decode 64 x 2048, 16 / 4 heads of 64", lambda: gqa.decode(qd, kc, vc, bt, lens, spec(d=64), None, None, ctx), 2 * B * ctx * G * 64 * 2)
+    # --- rotation, norms, cache write
+    pos = torch.arange(L, device="cuda", dtype=torch.int32).repeat(n)
+    kc, vc = _rand(nb * n // 4, G, bs, D), _rand(nb * n // 4, G, bs, D)
+    slots = torch.arange(T, device="cuda")
+    xq, wn = _rand(T, (H + 2 * G) * D), _rand(D)
+    moved = (2 * H + 5 * G) * D * 2  # queries and keys in and out, values in, keys and values to the cache
+    for halves, rot in ((False, 64), (True, 128)):
+        cos, sin = la.rotary_tables(L, rot, 1e4, "cuda")
+        a = spec(rot=rot, rot_halves=halves)
+        add(f"gqa.qkv_prep 16384 tokens, {'split' if halves else 'neighbouring'} pairs of {rot}", lambda: gqa.qkv_prep(xq, a, cos, sin, pos, (kc, vc), slots), T * moved)
+        add(f"gqa.qkv_prep batch 64, {'split' if halves else 'neighbouring'} pairs of {rot}", lambda: gqa.qkv_prep(xq[:B], a, cos, sin, pos[:B], (kc, vc), slots[:B], False), B * (moved - 2 * G * D), iters=20)
+    cs, sn = fused.rope_tables(L, D, 1e4, "cuda")[:2]
+    from ..ops.rollout_ops import kv_cache_write
+
+    def qwen_prep():
+        qq, kk, vv = fused.qknorm_rope(xq, wn, wn, cs, sn, pos, H, G, D)
+        kv_cache_write(kk, vv, slots, kc, vc)
+
+    add("[qwen3] qknorm_rope, kv_cache_write 16384 tokens", qwen_prep, T * moved)
+    add("[qwen3] qknorm_rope_kvwrite batch 64", lambda: fused.qknorm_rope_kvwrite(xq[:B], wn, wn, cs, sn, pos[:B], H, G, D, 1e-6, slots[:B], kc, vc), B * (moved - 2 * G * D), iters=20)
+    # --- norms around the residual
+    post, norm, res, resb = _rand(W), _rand(W), _rand(T, W, dt=F32), _rand(T, W)
+    pair = lambda: (_rand(W), _rand(W))
+    lpost, lnorm = pair(), pair()
+    aw, ww = _rand(T, W), _rand(W, W, s=W ** -0.5)
+    for t in (T, B):
+        it = 20 if t == B else 10
+        add(f"residual_rms {t} x 2048", lambda: rr.residual_rms(aw[:t], post, res[:t], None, 1e-6), t * W * 12, iters=it)
+        add(f"[gatolix] residual_ln {t} x 2048", lambda: ln.residual_ln(aw[:t], lpost, res[:t], lnorm, 1e-6), t * W * 12, iters=it)
+        add(f"[qwen3] rmsnorm + residual {t} x 2048", lambda: fused.rmsnorm(aw[:t], norm, 1e-6, residual=resb[:t]), t * W * 8, iters=it)
+        nbytes, fl = (t * W * 12, 2.0 * t * W * W) if t == T else (W * W * 2, 0)
+        add(f"linear_residual_rms {t} x 2048 x 2048", lambda: rr.linear_residual_rms(aw[:t], ww, post, res[:t], None, 1e-6), nbytes, fl, iters=it)
+        add(f"[qwen3] linear_rmsnorm {t} x 2048 x 2048", lambda: linear_rmsnorm(aw[:t], ww, norm, 1e-6, resb[:t]), nbytes, fl, iters=it)
+    ids = torch.from_numpy(np.random.default_rng(0).integers(0, 32000, T)).to("cuda")
+    table, at = _rand(32000, W), _rand(8192, W)
+    add("embed_residual 16384 x 2048, positions", lambda: rr.embed_residual(ids, table, 3.0, pos, at, None, 1e-6), T * W * 8 + L * W * 2)
+    add("[gatolix] embed_ln 16384 x 2048", lambda: ln.embed_ln(ids, table, lnorm, 1e-6), T * W * 8)
+    # --- mixture of experts
+    E, top, ff = 64, 6, 1408
+    rw = _rand(E, W, s=W ** -0.5)
+    gu, down = _rand(E, 2 * ff, W, s=W ** -0.5), _rand(E, W, ff, s=ff ** -0.5)
+    sgu, sdown = _rand(4 * ff, W, s=W ** -0.5), _rand(W, 2 * ff, s=ff ** -0.5)
+    act = moe.GatedAct(1.702, 1.0, 7.0)
+    p, c, st, lib = _lib.ptr, ctypes.c_int, _lib.stream_ptr, _lib.kernels()
+    glu = tuple(ctypes.c_float(f) for f in (act.limit, act.alpha, act.beta))
+    for t in (T, B):
+        xt, it = aw[:t], 20 if t == B else 10
+        route_bytes = t * W * 2 + E * W * 2
+        add(f"route_tokens {t} x 2048, 64 experts, sigmoid", lambda: moe.route_tokens(xt, rw, top, False, None, "sigmoid"), route_bytes, iters=it)
+        add(f"[gatolix] route_tokens {t}, softmax", lambda: moe.route_tokens(xt, rw, top, False), route_bytes, iters=it)
+        idx, w = moe.route_tokens(xt, rw, top, False, None, "sigmoid")
+        s = moe.sort_by_expert(idx, E)
+        live, rows = int((s.counts > 0).sum()), t * top
+        xs = moe.gather_rows(xt, s)
+        h, y = torch.empty(s.max_rows, ff, device="cuda", dtype=BF), torch.empty(s.max_rows, W, device="cuda", dtype=BF)
+        for name, scale in (("", w), ("[gatolix] ", None)):
+            add(f"{name}grouped gate | up + activation {t} x 6{', scaled inputs' if scale is not None else ''}",
+                lambda: lib.b200_gemm_grouped_glu(p(xs), p(gu), p(h), p(s.tile_expert), p(s.num_vm), p(s.src_of), p(scale), c(s.max_rows), c(E), c(ff), c(W), *glu, st()),
+                live * 2 * ff * W * 2 + rows * (W + ff) * 2, 4.0 * rows * W * ff, iters=it)
+        sh_bytes, sh_flops = 4 * ff * W * 2 + t * (W + 2 * ff) * 2, 8.0 * t * W * ff
+        add(f"gated_linear {t} x 2048 -> 2816 (shared expert)", lambda: moe.gated_linear(xt, sgu, act), sh_bytes, sh_flops, iters=it)
+        add(f"[qwen3] linear, then SwiGLU {t} x 2048 -> 2816", lambda: fused.swiglu(linear(xt, sgu)), sh_bytes, sh_flops, iters=it)
+        hs = moe.gated_linear(xt, sgu, act)
+        e = moe.ExpertRows(y, s.dest, top, None, linear_slices(hs, sdown))
+        add(f"experts_residual_rms {t} x 6 + shared", lambda: rr.experts_residual_rms(e, post, res[:t], None, 1e-6), t * W * (2 * top + 2 + 10), iters=it)
+        ew = moe.ExpertRows(y, s.dest, top, w)
+        add(f"[gatolix] experts_residual_ln {t} x 6", lambda: ln.experts_residual_ln(ew, lpost, res[:t], lnorm, 1e-6), t * W * (2 * top + 10), iters=it)
+
+        def felosun():
+            i2, w2 = moe.route_tokens(xt, rw, top, False, None, "sigmoid")
+            r = moe.gated_experts(xt, i2, w2, gu, down, act, True)
+            r.add = linear_slices(moe.gated_linear(xt, sgu, act), sdown)
+            return rr.experts_residual_rms(r, post, res[:t], None, 1e-6)
+
+        def qwen():
+            i2, w2 = moe.route(torch.nn.functional.linear(xt.float(), rw.float()), top, False)
+            r = moe.moe_experts_forward(xt, i2, w2, gu, down) + linear(fused.swiglu(linear(xt, sgu)), sdown)
+            return fused.rmsnorm(r, norm, 1e-6, residual=resb[:t])
+
+        nbytes, fl = live * 3 * ff * W * 2 + 6 * ff * W * 2, 6.0 * (rows + 2 * t) * W * ff
+        add(f"mixture with shared expert and norm {t}", felosun, nbytes, fl, iters=it)
+        add(f"[qwen3] mixture with shared expert and norm {t}", qwen, nbytes, fl, iters=it)
     return out
