@@ -55,21 +55,21 @@ struct GqaPrefillArgs {
   int H, group, D, Dv;     // D in steps of 16
   int hq, hk, hv;          // head strides
   float scale, cap;        // cap: 0 for none
-  int cap_poly;            // |score / cap| is small enough for the polynomial
+  int cap_terms;           // > 0: |score / cap| is small enough for the first 4 or 6 terms of tanh's series, whose
+  float cap_c[6];          // coefficients, in powers of (q . k)^2, give the capped score over q . k in units of log 2
   int window, keep;        // 0: none
   const __nv_bfloat16* sink;
   const __nv_bfloat16* gate;
   long long ldg;
 };
 
-// tanh by its Taylor polynomial: relative error below 1e-6 for |x| <= 0.5
-__device__ __forceinline__ float tanh_small(float x) {
-  const float t = x * x;
-  float p = fmaf(t, -1382.f / 155925.f, 62.f / 2835.f);
-  p = fmaf(t, p, -17.f / 315.f);
-  p = fmaf(t, p, 2.f / 15.f);
-  p = fmaf(t, p, -1.f / 3.f);
-  return fmaf(x * t, p, x);
+template <int N>
+__device__ __forceinline__ float cap_series(float x, const float* c) {
+  const float u = x * x;
+  float p = c[N - 1];
+#pragma unroll
+  for (int i = N - 2; i >= 0; --i) p = fmaf(u, p, c[i]);
+  return x * p;
 }
 
 template <int ND, int NV, bool BOUNDED>
@@ -229,9 +229,12 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       if (a.cap <= 0.f) {
 #pragma unroll
         for (int i = 0; i < kGpK; ++i) s[i] *= scale_log2;
-      } else if (a.cap_poly) {
+      } else if (a.cap_terms == 4) {
 #pragma unroll
-        for (int i = 0; i < kGpK; ++i) s[i] = cap_log2 * tanh_small(s[i] * to_cap);
+        for (int i = 0; i < kGpK; ++i) s[i] = cap_series<4>(s[i], a.cap_c);
+      } else if (a.cap_terms == 6) {
+#pragma unroll
+        for (int i = 0; i < kGpK; ++i) s[i] = cap_series<6>(s[i], a.cap_c);
       } else {
 #pragma unroll
         for (int i = 0; i < kGpK; ++i) s[i] = cap_log2 * tanh_as(s[i] * to_cap, a.o);
@@ -394,9 +397,17 @@ int b200_gqa_prefill(const void* q, long long ldq, int hq, const void* k, long l
   const float log2e = 1.4426950408889634f;
   float bound = score_bound;
   if (softcap > 0.f && (bound <= 0.f || softcap < bound)) bound = softcap;
-  const GqaPrefillArgs a{reinterpret_cast<const GqaTile*>(tiles), (__nv_bfloat16*)o, H, H / G, D, Dv, hq, hk, hv, scale,
-                         softcap, softcap > 0.f && score_bound > 0.f && score_bound <= 0.5f * softcap, window, keep,
-                         (const __nv_bfloat16*)sink, (const __nv_bfloat16*)gate, ldg};
+  GqaPrefillArgs a{reinterpret_cast<const GqaTile*>(tiles), (__nv_bfloat16*)o, H, H / G, D, Dv, hq, hk, hv, scale, softcap,
+                   0, {}, window, keep, (const __nv_bfloat16*)sink, (const __nv_bfloat16*)gate, ldg};
+  if (softcap > 0.f && score_bound > 0.f && score_bound <= 0.5f * softcap) {
+    // cap * tanh(s / cap) = s (1 - r / 3 + 2 r^2 / 15 - 17 r^3 / 315 + ...), r = (s / cap)^2. What is left out is below 1e-6
+    // of the score: 4 terms up to s / cap = 0.25, 6 terms up to 0.5.
+    const double c[6] = {1.0, -1.0 / 3, 2.0 / 15, -17.0 / 315, 62.0 / 2835, -1382.0 / 155925};
+    const double r = static_cast<double>(scale) / softcap;
+    double f = static_cast<double>(scale) * 1.4426950408889634;
+    for (int i = 0; i < 6; ++i, f *= r * r) a.cap_c[i] = static_cast<float>(c[i] * f);
+    a.cap_terms = score_bound <= 0.25f * softcap ? 4 : 6;
+  }
   // 2^(-64 .. 64): neither the weights, their sums nor the two-term split leave the range of fp32 and bf16
   return bound > 0.f && bound * log2e <= 64.f ? pick_gqa_prefill<true>(tmQ, tmK, tmV, a, n_tiles, stream)
                                               : pick_gqa_prefill<false>(tmQ, tmK, tmV, a, n_tiles, stream);

@@ -4,7 +4,8 @@
 //
 //   k_cache [blocks, G, block_size, Dp], v_cache [blocks, G, block_size, Vp]      Dp, Vp: D, Dv in steps of 16, zero-filled
 //
-// One warp per (token, head); everything is computed in fp32 and rounded once.
+// One warp per (token, head), or for bf16 widths in steps of 8 one part of a warp, eight numbers to a lane; everything is
+// computed in fp32 and rounded once.
 #include "common/host_utils.h"
 #include "common/io.cuh"
 
@@ -47,6 +48,97 @@ template <class T, int V>
 __device__ __forceinline__ void stvec(T* p, const Vec<V>& a) {
   if constexpr (V == 4) st4(p, make_float4(a.e[0], a.e[1], a.e[2], a.e[3]));
   else st1(p, a.e[0]);
+}
+
+// a cos + b sin, rounded the same way wherever it is compiled
+__device__ __forceinline__ float turned(float a, float b, float c, float s) { return fmaf(a, c, __fmul_rn(b, s)); }
+
+__device__ __forceinline__ void ld8(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 raw = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 b = __bfloat1622float2(h[j]);
+    f[2 * j] = b.x;
+    f[2 * j + 1] = b.y;
+  }
+}
+__device__ __forceinline__ void ld8(const float* p, float (&f)[8]) {
+  const float4 a = ld4(p), b = ld4(p + 4);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
+// LPH: lanes per head (8 * LPH >= Dp, Vp); 32 / LPH heads per warp
+template <int LPH>
+__global__ void __launch_bounds__(256) gqa_prep8_kernel(GqaPrepArgs a) {
+  using T = __nv_bfloat16;
+  const int units = a.H + 2 * a.G, lane = threadIdx.x & 31;
+  const int u = (blockIdx.x * 8 + (threadIdx.x >> 5)) * (32 / LPH) + lane / LPH, c = (lane % LPH) * 8;
+  const bool live = u < a.T * units;  // (whole warps stay for the shuffles)
+  const int t = live ? u / units : 0, r = live ? u - t * units : 0;
+  const bool is_q = r < a.H, is_v = r >= a.H + a.G;
+  const int g = is_q ? r : (is_v ? r - a.H - a.G : r - a.H);
+  const int width = is_v ? a.Dv : a.D, padded = is_v ? a.Vp : a.Dp;
+  const T* src = static_cast<const T*>(a.x) + t * a.ldx + (is_v ? (a.H + a.G) * a.D + g * a.Dv : r * a.D);
+  const bool in = live && c < width;
+  float f[8] = {};
+  if (in) ld8(src + c, f);
+  if (in && !is_v && c < a.rot) {
+    const int half = a.rot >> 1;
+    const long long at = static_cast<long long>(min(max(a.pos[t], 0), a.max_pos - 1)) * half;
+    if (a.halves) {
+      const bool low = c < half;
+      const int e = low ? c : c - half;
+      float o[8], cs[8], sn[8];
+      ld8(src + (low ? c + half : e), o);
+      ld8(a.cosT + at + e, cs);
+      ld8(a.sinT + at + e, sn);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] = turned(f[j], low ? -o[j] : o[j], cs[j], sn[j]);
+    } else {
+      const float4 cs = ld4(a.cosT + at + (c >> 1)), sn = ld4(a.sinT + at + (c >> 1));
+      const float cc[4] = {cs.x, cs.y, cs.z, cs.w}, ss[4] = {sn.x, sn.y, sn.z, sn.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float x = f[2 * j], y = f[2 * j + 1];
+        f[2 * j] = turned(x, -y, cc[j], ss[j]);
+        f[2 * j + 1] = turned(y, x, cc[j], ss[j]);
+      }
+    }
+  }
+  if (a.eps >= 0.f) {
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s = fmaf(f[j], f[j], s);
+#pragma unroll
+    for (int d = LPH / 2; d > 0; d >>= 1) s += __shfl_xor_sync(0xffffffffu, s, d);
+    // the warp's loads are all done here: the results may overwrite the source
+    const float k = is_v ? 1.f : 1.f / sqrtf(s / a.D + a.eps);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[j] *= k;
+  } else {
+    __syncwarp();
+  }
+  if (!live || c >= padded) return;
+  uint4 out;
+  __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&out);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) h[j] = __floats2bfloat162_rn(f[2 * j], f[2 * j + 1]);
+  T* dst = nullptr;
+  if (is_q) dst = static_cast<T*>(a.q) + t * a.ldq + g * a.hq;
+  else if (is_v) dst = a.v ? static_cast<T*>(a.v) + t * a.ldv + g * a.hv : nullptr;
+  else dst = a.k ? static_cast<T*>(a.k) + t * a.ldk + g * a.hk : nullptr;
+  if (dst) *reinterpret_cast<uint4*>(dst + c) = out;
+  if (!is_q && a.slots) {
+    const long long slot = a.slots[t];
+    if (slot >= 0 && slot < a.cache_rows) {
+      const int blk = static_cast<int>(slot) / a.block_size, off = static_cast<int>(slot) - blk * a.block_size;
+      T* page = static_cast<T*>(is_v ? a.v_cache : a.k_cache) +
+                ((static_cast<long long>(blk) * a.G + g) * a.block_size + off) * padded;
+      *reinterpret_cast<uint4*>(page + c) = out;
+    }
+  }
 }
 
 // V: elements per access; N: accesses per lane (32 * V * N >= Dp, Vp)
@@ -97,17 +189,17 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(GqaPrepArgs a) {
         const Vec<V> o = ldvec<T, V>(src + (low ? c + half : e));
         const Vec<V> cs = ldvec<float, V>(cr + e), sn = ldvec<float, V>(sr + e);
 #pragma unroll
-        for (int j = 0; j < V; ++j) f[i].e[j] = f[i].e[j] * cs.e[j] + (low ? -o.e[j] : o.e[j]) * sn.e[j];
+        for (int j = 0; j < V; ++j) f[i].e[j] = turned(f[i].e[j], low ? -o.e[j] : o.e[j], cs.e[j], sn.e[j]);
       } else if constexpr (V == 4) {
         const float2 cs = *reinterpret_cast<const float2*>(cr + (c >> 1)), sn = *reinterpret_cast<const float2*>(sr + (c >> 1));
         const Vec<V> o = f[i];
-        f[i].e[0] = o.e[0] * cs.x - o.e[1] * sn.x;
-        f[i].e[1] = o.e[1] * cs.x + o.e[0] * sn.x;
-        f[i].e[2] = o.e[2] * cs.y - o.e[3] * sn.y;
-        f[i].e[3] = o.e[3] * cs.y + o.e[2] * sn.y;
+        f[i].e[0] = turned(o.e[0], -o.e[1], cs.x, sn.x);
+        f[i].e[1] = turned(o.e[1], o.e[0], cs.x, sn.x);
+        f[i].e[2] = turned(o.e[2], -o.e[3], cs.y, sn.y);
+        f[i].e[3] = turned(o.e[3], o.e[2], cs.y, sn.y);
       } else {
         const float o = ld1(src + (c ^ 1)), cs = cr[c >> 1], sn = sr[c >> 1];
-        f[i].e[0] = f[i].e[0] * cs + ((c & 1) ? o : -o) * sn;
+        f[i].e[0] = turned(f[i].e[0], (c & 1) ? o : -o, cs, sn);
       }
     }
 #pragma unroll
@@ -153,8 +245,20 @@ int b200_gqa_prep(const void* x, long long ldx, int H, int G, int D, int Dv, con
                 slots, k_cache, v_cache, block_size, cache_rows, T};
   const bool v4 = D % 4 == 0 && Dv % 4 == 0 && rot % 4 == 0 && (!halves || rot % 8 == 0) && ldx % 4 == 0 && ldq % 4 == 0 &&
                   ldk % 4 == 0 && ldv % 4 == 0 && hq % 4 == 0 && hk % 4 == 0 && hv % 4 == 0;
-  const unsigned grid = static_cast<unsigned>((units + 7) / 8);
   const int w = Dp > Vp ? Dp : Vp;
+  const bool v8 = !fp32 && w <= 256 && cache_rows < 0x7fffffff && D % 8 == 0 && Dv % 8 == 0 && rot % (halves ? 16 : 8) == 0 &&
+                  !((ldx | ldq | ldk | ldv | hq | hk | hv) & 7) && !(reinterpret_cast<uintptr_t>(x) & 15);
+  if (v8) {
+    const int lph = w <= 64 ? 8 : (w <= 128 ? 16 : 32);
+    const long long heads = 8LL * (32 / lph);
+    const unsigned grid8 = static_cast<unsigned>((units + heads - 1) / heads);
+    if (lph == 8) gqa_prep8_kernel<8><<<grid8, 256, 0, stream>>>(a);
+    else if (lph == 16) gqa_prep8_kernel<16><<<grid8, 256, 0, stream>>>(a);
+    else gqa_prep8_kernel<32><<<grid8, 256, 0, stream>>>(a);
+    B200_CHECK(cudaGetLastError());
+    return 0;
+  }
+  const unsigned grid = static_cast<unsigned>((units + 7) / 8);
   using bf = __nv_bfloat16;
 #define B200_GP(T_, V_, N_) gqa_prep_kernel<T_, V_, N_><<<grid, 256, 0, stream>>>(a)
 #define B200_GPN(T_)                                                                               \

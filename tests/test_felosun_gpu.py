@@ -174,7 +174,7 @@ def _spec(H, G, D, Dv, **kw):
 @pytest.mark.parametrize("dt", DTYPES)
 @pytest.mark.parametrize("H,G,D,Dv,rot,halves", [(3, 1, 7, 5, 6, False), (4, 2, 64, 64, 32, True), (2, 2, 96, 40, 96, False), (5, 5, 40, 24, 24, True),
                                                  (2, 1, 256, 136, 100, True), (1, 1, 1, 1, 0, False), (6, 3, 272, 400, 272, False),
-                                                 (4, 4, 20, 36, 12, True), (8, 2, 128, 128, 128, True)])
+                                                 (4, 4, 20, 36, 12, True), (8, 2, 128, 128, 128, True), (3, 1, 24, 40, 8, False), (2, 2, 96, 112, 32, True)])
 @pytest.mark.parametrize("unit,extra", [(True, 0), (False, 0), (True, 3)])
 def test_qkv_prep(dt, H, G, D, Dv, rot, halves, unit, extra):
     from areal_b200.ops.gqa import pad16, qkv_prep
@@ -223,7 +223,7 @@ def test_qkv_prep(dt, H, G, D, Dv, rot, halves, unit, extra):
 SHAPES = [(3, 1, 7, 5), (4, 2, 24, 40), (6, 2, 64, 64), (4, 4, 96, 96), (2, 1, 128, 128), (5, 5, 48, 112), (20, 1, 80, 64),
           (2, 1, 192, 256), (2, 2, 256, 72), (2, 1, 272, 32)]
 OPTIONS = [dict(), dict(window=40, keep_first=20, sink=True), dict(window=1, sink=True), dict(window=64, keep_first=64),
-           dict(window=63, keep_first=65, gate=True, softcap=5.0), dict(window=65, keep_first=1, sink=True),
+           dict(window=63, keep_first=65, gate=True, softcap=5.0), dict(window=65, keep_first=1, sink=True), dict(softcap=45.0),
            dict(softcap=30.0, gate=True), dict(window=128, keep_first=130, softcap=2.0, sink=True, gate=True), dict(window=500, keep_first=3)]
 
 
