@@ -67,7 +67,7 @@ def parse_args():
     p.add_argument("--no-fused-comm-check", action="store_true",
                    help="N >= 2: skip the untimed check of the fused compute+collective kernels")
     p.add_argument("--serving", action="store_true",
-                   help="instead of the training benchmark: prefill and decode throughput of a layered (Fofosun) model "
+                   help="instead of the training benchmark: prefill and decode throughput of a layered model "
                         "beside the closest other family at equal sizes (one GPU; see areal_b200/tools/bench_serving.py)")
     p.add_argument("--serving-family", default="fofosun", choices=["fofosun", "gatolix", "felosun"], help="with --serving: which family")
     p.add_argument("--serving-sizes", default="s,m,l", help="with --serving: which sizes")

@@ -48,7 +48,7 @@ _MIXED = [windowed(4, 2, 16, 24, 8, 0.5, 12, 3, 500.0, moe(5, 2, 24, 1.5, 40, 0.
 _ODD = [windowed(3, 1, 7, 5, 6, 0.8, 9, 2, 77.0, moe(3, 2, 11, 1.1, 13, 0.6)), capped(5, 5, 5, 9, 2, 0.7, 3.0, 1.5, 30.0)]
 _PADDED = [windowed(4, 2, 40, 56, 24, 0.2, 45, 17, 2e3, moe(10, 5, 40, 1.8, 72, 1.2)),
            capped(3, 1, 104, 72, 100, 0.12, 9.0, 3.0, 2e3, moe(4, 1, 24, 0.9, 24, 0.9))]
-_TILE = [windowed(6, 2, 64, 64, 32, 0.2, 100, 70, 1e4, moe(12, 4, 72, 2.0, 136, 1.5)),
+_TILE = [windowed(6, 3, 64, 64, 48, 0.2, 100, 70, 1e4, moe(12, 4, 72, 2.0, 136, 1.5)),
          capped(4, 4, 128, 128, 128, 0.1, 30.0, 4.0, 5e3, moe(20, 2, 136, 1.5, 1056, 3.0)),
          windowed(20, 1, 80, 112, 80, 0.15, 31, 64, 5e3, moe(3, 1, 64, 2.5))]
 _WIDE = [windowed(2, 1, 192, 256, 64, 0.09, 70, 5, 1e4, moe(4, 2, 40, 2.0, 48, 1.0)),

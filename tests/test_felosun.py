@@ -74,7 +74,7 @@ def test_scaled_embedding_with_positions():
 
 
 @pytest.mark.parametrize("dims,width,halves,base,factor", [(8, 8, False, 1e4, None), (8, 8, True, 1e4, 1.0), (6, 11, False, 50.0, 3.0),
-                                                           (6, 11, True, 50.0, 3.0), (2, 2, True, 1e6, 8.0), (64, 96, True, 2e4, 4.0), (0, 4, False, 1e4, None)])
+                                                           (6, 11, True, 50.0, 3.0), (2, 2, True, 1e6, 8.0), (64, 80, True, 3e4, 5.0), (0, 4, False, 1e4, None)])
 def test_rotation_of_leading_dimensions(dims, width, halves, base, factor):
     from areal_b200.ops.gqa import rotate_ref
     from areal_b200.ops.latent_attn import rotary_tables

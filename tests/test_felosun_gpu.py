@@ -220,9 +220,9 @@ def test_qkv_prep(dt, H, G, D, Dv, rot, halves, unit, extra):
             assert bool((flat[rest] == 7.0).all())
 
 
-SHAPES = [(3, 1, 7, 5), (4, 2, 24, 40), (6, 2, 64, 64), (4, 4, 96, 96), (2, 1, 128, 128), (5, 5, 48, 112), (20, 1, 80, 64),
+SHAPES = [(3, 1, 7, 5), (4, 2, 24, 40), (6, 3, 64, 64), (4, 4, 96, 80), (2, 1, 128, 128), (5, 5, 48, 112), (20, 1, 80, 64),
           (2, 1, 192, 256), (2, 2, 256, 72), (2, 1, 272, 32)]
-OPTIONS = [dict(), dict(window=40, keep_first=20, sink=True), dict(window=1, sink=True), dict(window=64, keep_first=64),
+OPTIONS = [dict(), dict(window=45, keep_first=19, sink=True), dict(window=1, sink=True), dict(window=64, keep_first=64),
            dict(window=63, keep_first=65, gate=True, softcap=5.0), dict(window=65, keep_first=1, sink=True), dict(softcap=45.0),
            dict(softcap=30.0, gate=True), dict(window=128, keep_first=130, softcap=2.0, sink=True, gate=True), dict(window=500, keep_first=3)]
 
