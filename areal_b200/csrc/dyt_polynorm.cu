@@ -3,7 +3,7 @@
 //   embed_dyt     res = table[id];                 y = tanh(alpha * res) * w + b
 //   residual_dyt  res += scale * delta;            y = tanh(alpha * res) * w + b
 //   polynorm      y = a N(z) + b N(z^2) + c N(z^3) + e,   N(u) = u / sqrt(mean(u^2) + eps)
-//   group_rms     y = N(o per group of columns) * w (* sigmoid(gate))
+//   group_rms     y = N(o per group of columns) * w (* sigmoid(gate), or gate * sigmoid(gate))
 //
 // Dynamic Tanh: Zhu, Chen, He, LeCun, Liu, "Transformers without Normalization". The residual stream and everything
 // computed here is fp32; inputs, weights and y have the model's dtype (bf16 or fp32). Dynamic Tanh needs no row
@@ -121,11 +121,13 @@ __global__ void polynorm_kernel(const T* __restrict__ z, long long ldz, const T*
 }
 
 // o [rows, groups * n] fp32. One warp per (row, group) when a group is narrow, one block per (row, group) else.
-// w: [n] shared by the groups (w_per_group 0) or [groups * n]. gate: null or [rows, groups * n] with pitch ld_gate.
+// w: [n] shared by the groups (w_per_group 0) or [groups * n]. gate: null or [rows, groups * n] with pitch ld_gate; silu: the
+// result is multiplied by gate * sigmoid(gate) instead of sigmoid(gate).
 template <class T, bool WARP, int V>
 __global__ void group_rms_kernel(const float* __restrict__ o, const T* __restrict__ w, int w_per_group,
-                                 const T* __restrict__ gate, long long ld_gate, T* __restrict__ y, long long rows,
-                                 int groups, int n, float eps) {
+                                 const T* __restrict__ gate, long long ld_gate, int silu, T* __restrict__ y,
+                                 long long rows, int groups, int n, float eps) {
+  auto act = [&](float u) { return sigmoid_as(u, y) * (silu ? u : 1.f); };
   __shared__ float red[33];
   const int nthr = WARP ? 32 : blockDim.x, tid = WARP ? (threadIdx.x & 31) : threadIdx.x;
   const long long unit = WARP ? static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5)
@@ -155,12 +157,12 @@ __global__ void group_rms_kernel(const float* __restrict__ o, const T* __restric
       v.x *= k * ww.x; v.y *= k * ww.y; v.z *= k * ww.z; v.w *= k * ww.w;
       if (gb) {
         const float4 u = ld4(gb + c);
-        v.x *= sigmoid_as(u.x, y); v.y *= sigmoid_as(u.y, y); v.z *= sigmoid_as(u.z, y); v.w *= sigmoid_as(u.w, y);
+        v.x *= act(u.x); v.y *= act(u.y); v.z *= act(u.z); v.w *= act(u.w);
       }
       st4(yb + c, v);
     } else {
       float v = ob[c] * k * ld1(wb + c);
-      if (gb) v *= sigmoid_as(ld1(gb + c), y);
+      if (gb) v *= act(ld1(gb + c));
       st1(yb + c, v);
     }
   }
@@ -242,7 +244,7 @@ int b200_polynorm(const void* z, long long ldz, const void* coef, void* y, long 
   return 0;
 }
 
-int b200_group_rms(const float* o, const void* w, int w_per_group, const void* gate, long long ld_gate, void* y,
+int b200_group_rms(const float* o, const void* w, int w_per_group, const void* gate, long long ld_gate, int silu, void* y,
                    long long rows, int groups, int n, float eps, int fp32, cudaStream_t stream) {
   using namespace b200;
   if (rows <= 0 || groups <= 0 || n <= 0) return 0;
@@ -255,7 +257,7 @@ int b200_group_rms(const float* o, const void* w, int w_per_group, const void* g
   const unsigned grid = static_cast<unsigned>(warp ? (units + 7) / 8 : units);
 #define B200_GR(T_, W_, V_)                                                                                         \
   group_rms_kernel<T_, W_, V_><<<grid, block, 0, stream>>>(o, (const T_*)w, w_per_group, (const T_*)gate, ld_gate,  \
-                                                           (T_*)y, rows, groups, n, eps)
+                                                           silu, (T_*)y, rows, groups, n, eps)
 #define B200_GRV(T_)                                                                                                \
   if (warp) { if (v4) B200_GR(T_, true, 4); else B200_GR(T_, true, 1); }                                            \
   else { if (v4) B200_GR(T_, false, 4); else B200_GR(T_, false, 1); }

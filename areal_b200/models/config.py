@@ -88,12 +88,17 @@ class ModelConfig:
     # and the feed-forward's (None: the layer has none); the sizes above then only summarise the list
     layer_specs: list[dict] = field(default_factory=list)
     # what such a decoder wraps its sublayers in: "dynamic_tanh" (norm in front, learned scale on the result) or
-    # "layer_norm" (one norm in front and one on the result) or "post_rms" (RMS norm on the result only)
+    # "layer_norm" (one norm in front and one on the result) or "post_rms" (RMS norm on the result only) or "parallel" (one
+    # layer norm per layer, which both sublayers read; the sum of their results times `residual_mult` is added)
     layer_norms: str = "dynamic_tanh"
+    residual_mult: float = 1.0
+    # the mixer reads h + conv(h), a causal convolution over this many tokens on every channel (0: it reads h)
+    input_conv: int = 0
     # input: embed[token] * embedding_scale, plus a learned vector per position (table of `max_position_embeddings` rows,
     # which then bounds the length of a sequence)
     embedding_scale: float = 1.0
     learned_positions: bool = False
+    sinusoid_positions: bool = False  # a computed vector of sines and cosines per position instead
     logit_scale: float = 1.0  # logits = head(x) * logit_scale
     # logits <- cap * tanh(logits / cap); 0 = none
     logit_softcap: float = 0.0
@@ -132,7 +137,7 @@ class ModelConfig:
     def has_recurrent_state(self) -> bool:
         """Some layers carry a per-sequence recurrent state through generation (linear-attention layers)."""
         return (self.is_hybrid or self.lightning_group_size > 1
-                or any(self.recurrent_shape(i) is not None for i in range(len(self.layer_specs))))
+                or any(self.state_shapes(i) for i in range(len(self.layer_specs))))
 
     @property
     def is_layered(self) -> bool:
@@ -142,7 +147,9 @@ class ModelConfig:
         """Paged-cache tensors of layer ``i`` as ``(heads, width)`` per token; empty for layers without a cache."""
         if self.is_layered:
             m = self.layer_specs[i]["mixer"]
-            if self.layer_type(i) == "grouped_attention":  # widths in steps of 16: what a tensor-core tile takes
+            if self.layer_type(i) == "mixer_pair":  # the left one attends
+                m = m["left"]
+            if "kv_heads" in m:  # grouped attention; widths in steps of 16: what a tensor-core tile takes
                 return [(m["kv_heads"], -(-n // 16) * 16) for n in (m["dim"], m["vdim"])]
             own = self.layer_type(i) == "latent_attention" and m.get("kv_from") is None
             return [(1, m["kv_rank"] + m["rot_dim"])] if own else []
@@ -169,11 +176,31 @@ class ModelConfig:
         """State of layer ``i`` per sequence ``(heads, key width, value width)``, None for layers without one. Covers
         the families whose state is one matrix per head (the Qwen3.5 hybrid also keeps convolution inputs)."""
         if self.is_layered:
-            m = self.layer_specs[i]["mixer"]
-            return (m["heads"], m["dim"], m["vdim"]) if self.layer_type(i) in ("hgrn2", "lightning") else None
+            m, t = self.layer_specs[i]["mixer"], self.layer_type(i)
+            if t == "mixer_pair":
+                m = m["right"]
+            return (m["heads"], m["dim"], m["vdim"]) if t in ("hgrn2", "lightning", "mlstm", "mixer_pair") else None
         if self.layer_is_lightning(i):
             return (self.num_attention_heads, self.lightning_head_dim, self.lightning_head_dim)
         return None
+
+    def state_shapes(self, i: int) -> dict[str, tuple[tuple[int, ...], bool]]:
+        """What layer ``i`` keeps per sequence: name -> (shape, kept in 32-bit); else in the model's dtype. ``S`` is the
+        matrix state of :meth:`recurrent_shape`; ``n`` and ``m`` are the normaliser and the running maximum of an mLSTM;
+        ``conv`` and ``qkv`` are rings of the last inputs of the layer's input convolution and of a mixer's short
+        convolution, one row per position modulo the number of taps."""
+        S = self.recurrent_shape(i)
+        out = {} if S is None else {"S": (S, True)}
+        if self.is_layered:
+            m, t = self.layer_specs[i]["mixer"], self.layer_type(i)
+            if t == "mlstm":
+                out.update(n=((m["heads"], m["dim"]), True), m=((m["heads"],), True))
+            if t == "mixer_pair":
+                r = m["right"]
+                out["qkv"] = ((r["conv"], 2 * r["kv_heads"] * r["dim"] + r["heads"] * r["vdim"]), False)
+            if self.input_conv:
+                out["conv"] = ((self.input_conv, self.hidden_size), False)
+        return out
 
     @property
     def graph_decode(self) -> bool:
@@ -224,8 +251,31 @@ class ModelConfig:
     def kv_size(self) -> int:
         return self.num_key_value_heads * self.head_dim
 
+    def _parallel_params(self, i: int, active: bool) -> int:
+        h, spec = self.hidden_size, self.layer_specs[i]
+        m, mlp = spec["mixer"], spec["mlp"]
+        n = 2 * h + h * self.input_conv
+        if spec["type"] == "mlstm":
+            H, D, Dv = m["heads"], m["dim"], m["vdim"]
+            n += h * H * (2 * D + 3 * Dv + 2) + 2 * H + H * Dv
+        else:
+            a, r = m["left"], m["right"]
+            n += h * (a["heads"] * (a["dim"] + a["vdim"]) + a["kv_heads"] * (a["dim"] + a["vdim"])) + a["heads"]
+            H, Dv = r["heads"], r["vdim"]
+            qkv = 2 * r["kv_heads"] * r["dim"] + H * Dv
+            n += qkv * (h + r["conv"]) + h * (2 * H + 2 * H * Dv) + 2 * H + Dv + 2 * h
+        if mlp is None:
+            return n
+        if mlp["kind"] == "dense":
+            return n + 3 * h * mlp["ff"]
+        r = mlp["router"]
+        n += h * (3 * mlp["shared"]["ff"] + 1) if mlp.get("shared") else 0
+        return n + (h + 1) * r["experts"] + 3 * h * mlp["expert"]["ff"] * (r["top"] if active else r["experts"])
+
     def _layered_params(self, i: int, active: bool = False) -> int:
         """Parameters of layer ``i`` of a layered decoder; ``active``: only those that one token passes through."""
+        if self.layer_norms == "parallel":
+            return self._parallel_params(i, active)
         h, spec = self.hidden_size, self.layer_specs[i]
         m, t = spec["mixer"], spec["type"]
         H, D, Dv = m["heads"], m["dim"], m["vdim"]
@@ -258,7 +308,7 @@ class ModelConfig:
     def num_params(self) -> int:
         h, L = self.hidden_size, self.num_hidden_layers
         if self.is_layered:
-            final = {"layer_norm": 2 * h, "post_rms": h}.get(self.layer_norms, 2 * h + 1)
+            final = {"layer_norm": 2 * h, "parallel": 2 * h, "post_rms": h}.get(self.layer_norms, 2 * h + 1)
             final += self.max_position_embeddings * h if self.learned_positions else 0
             return 2 * self.vocab_size * h + final + sum(self._layered_params(i) for i in range(L)
                                                          if self.weights_layer(i) == i)
@@ -314,6 +364,9 @@ class ModelConfig:
                 elif spec["type"] == "grouped_attention":
                     keys = min(seq_len / 2, m["window"] + m["keep_first"]) if m["window"] else seq_len / 2
                     total += 2 * m["heads"] * (m["dim"] + m["vdim"]) * keys
+                elif spec["type"] == "mixer_pair":
+                    a, r = m["left"], m["right"]
+                    total += a["heads"] * (a["dim"] + a["vdim"]) * seq_len + 6 * r["heads"] * r["dim"] * r["vdim"]
                 else:
                     total += 4 * m["heads"] * m["dim"] * m["vdim"]
             return total * (3 if backward else 1)
@@ -339,6 +392,8 @@ class ModelConfig:
             return cls._from_gatolix(cfg, overrides)
         if cfg.get("architecture") == "Felosun":
             return cls._from_felosun(cfg, overrides)
+        if cfg.get("architecture") == "Dikopel":
+            return cls._from_dikopel(cfg, overrides)
         if "text_config" in cfg:  # composite (vision-language) checkpoints nest the decoder's config
             cfg = cfg["text_config"]
         mt = cfg.get("model_type", "qwen3")
@@ -494,14 +549,15 @@ class ModelConfig:
 
     @classmethod
     def _layered(cls, model_type: str, cfg: dict, specs: list[dict], overrides: dict, **fields) -> "ModelConfig":
-        heads = max((s["mixer"]["heads"] for s in specs), default=1)
+        mixers = [m.get("left", m) for m in (s["mixer"] for s in specs)]
+        heads = max((m["heads"] for m in mixers), default=1)
         moe = [s["mlp"] for s in specs if s["mlp"] and s["mlp"]["kind"] == "moe"]
         out = cls(model_type=model_type, vocab_size=cfg["vocab"], hidden_size=cfg["width"], layer_specs=specs,
                   num_hidden_layers=len(specs), rms_norm_eps=cfg["norm"]["eps"],
                   intermediate_size=max((s["mlp"]["ff"] for s in specs if s["mlp"] and "ff" in s["mlp"]), default=0),
                   num_attention_heads=heads,
-                  num_key_value_heads=max((s["mixer"].get("kv_heads", s["mixer"]["heads"]) for s in specs), default=1),
-                  head_dim=max((s["mixer"]["dim"] for s in specs), default=1), tie_word_embeddings=False, qk_norm=False,
+                  num_key_value_heads=max((m.get("kv_heads", m["heads"]) for m in mixers), default=1),
+                  head_dim=max((m["dim"] for m in mixers), default=1), tie_word_embeddings=False, qk_norm=False,
                   num_experts=max((m["router"]["experts"] for m in moe), default=0),
                   num_experts_per_tok=max((m["router"]["top"] for m in moe), default=0),
                   moe_intermediate_size=max((m["expert"]["ff"] for m in moe), default=0), **fields)
@@ -619,7 +675,80 @@ class ModelConfig:
                 "logit_scale": self.logit_scale, "max_positions": self.max_position_embeddings,
                 "norm": {"eps": self.rms_norm_eps}, "vocab": self.vocab_size, "width": self.hidden_size}
 
+    @classmethod
+    def _from_dikopel(cls, cfg: dict, overrides: dict) -> "ModelConfig":
+        """``config.json`` of a Dikopel checkpoint: layers of mLSTM (``mlstm``) or of sigmoid attention beside a gated delta
+        rule (``parallel``: mixers ``left`` and ``right``), a dense feed-forward or a mixture of experts in groups with a
+        gated shared expert on the same norm, a short convolution ahead of every mixer (``canon``), and layers that run with
+        an earlier layer's weights (``weights_of``)."""
+        specs = []
+        for i, layer in enumerate(cfg["layers"]):
+            t, m, mlp, src = layer["type"], layer["mixer"], layer.get("mlp"), layer.get("weights_of")
+            if t == "mlstm":
+                spec = {k: m[k] for k in ("heads", "dim", "vdim", "gate_cap")}
+            elif t == "parallel":
+                left = {k: m["left"][k] for k in ("heads", "kv_heads", "dim", "vdim", "scale")}
+                right = {k: m["right"][k] for k in ("heads", "kv_heads", "dim", "vdim", "conv")}
+                for part in (left, right):
+                    if part["heads"] % part["kv_heads"]:
+                        raise ValueError(f"layer {i}: {part['heads']} heads do not divide into {part['kv_heads']} groups")
+                if right["conv"] < 1:
+                    raise ValueError(f"layer {i}: a convolution of {right['conv']} taps")
+                spec = {"left": dict(left, weights="sigmoid"), "right": right}
+            else:
+                raise NotImplementedError(f"layer {i}: mixer {t!r}; supported are 'mlstm' and 'parallel'")
+            ff = None
+            if mlp is not None and mlp.get("kind", "dense") == "dense":
+                ff = {"kind": "dense", "ff": mlp["ff"], "act": "swiglu"}
+            elif mlp is not None:
+                if mlp["kind"] != "moe":
+                    raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']!r}; supported are 'dense' and 'moe'")
+                r = mlp["router"]
+                groups = {k: int((r.get("groups") or {"count": 1, "keep": 1})[k]) for k in ("count", "keep")}
+                size, rest = divmod(r["experts"], groups["count"])
+                if rest or not 1 <= groups["keep"] <= groups["count"] or not 1 <= r["top"] <= groups["keep"] * size:
+                    raise ValueError(f"layer {i}: {r['top']} of {r['experts']} experts from {groups['keep']} of "
+                                     f"{groups['count']} groups")
+                ff = {"kind": "moe", "act": "swiglu", "expert": {"ff": mlp["expert"]["ff"]},
+                      "router": {"experts": r["experts"], "top": r["top"], "score": "sigmoid", "renorm": True,
+                                 "scale": float(r.get("scale", 1.0)), "groups": groups}}
+                if mlp.get("shared"):
+                    ff["shared"] = {"ff": mlp["shared"]["ff"], "gate": True}
+            out = {"type": "mixer_pair" if t == "parallel" else t, "mixer": spec, "mlp": ff}
+            if src is not None:
+                if not 0 <= src < i or {k: specs[src][k] for k in out} != out:
+                    raise ValueError(f"layer {i}: it cannot run with the weights of layer {src}")
+                out["weights_of"] = src
+            specs.append(out)
+        taps = int(cfg["canon"]["taps"])
+        if taps < 1:
+            raise ValueError(f"a convolution of {taps} taps")
+        emb = cfg.get("embedding") or {}
+        return cls._layered("dikopel", cfg, specs, overrides, layer_norms="parallel", input_conv=taps, sinusoid_positions=True,
+                            embedding_scale=float(emb.get("scale", 1.0)), residual_mult=float(cfg["residual_mult"]))
+
+    def _to_dikopel(self) -> dict:
+        layers = []
+        for s in self.layer_specs:
+            m, mlp = s["mixer"], s["mlp"]
+            if s["type"] == "mixer_pair":
+                m = {"left": {k: v for k, v in m["left"].items() if k != "weights"}, "right": m["right"]}
+            if mlp is not None and mlp["kind"] == "moe":
+                r = {k: mlp["router"][k] for k in ("experts", "groups", "scale", "top")}
+                mlp = dict({"kind": "moe", "expert": mlp["expert"], "router": r},
+                           **({"shared": {"ff": mlp["shared"]["ff"]}} if mlp.get("shared") else {}))
+            elif mlp is not None:
+                mlp = {"kind": "dense", "ff": mlp["ff"]}
+            layers.append({"type": "parallel" if s["type"] == "mixer_pair" else s["type"], "mixer": m, "mlp": mlp})
+            if s.get("weights_of") is not None:
+                layers[-1]["weights_of"] = s["weights_of"]
+        return {"architecture": "Dikopel", "canon": {"taps": self.input_conv}, "embedding": {"scale": self.embedding_scale},
+                "layers": layers, "norm": {"eps": self.rms_norm_eps}, "residual_mult": self.residual_mult,
+                "vocab": self.vocab_size, "width": self.hidden_size}
+
     def to_hf_config(self) -> dict:
+        if self.model_type == "dikopel":
+            return self._to_dikopel()
         if self.model_type == "felosun":
             return self._to_felosun()
         if self.model_type == "gatolix":
@@ -768,6 +897,8 @@ def _rotation(rot: dict, width: int, layer: int) -> dict:
 _TINY_LATENT = {"heads": 4, "dim": 32, "rot_dim": 16, "vdim": 24, "kv_rank": 80, "scale": 0.15, "mask": {"size": 50},
                 "rot": {"base": 1e4, "dims": 16, "scaling": {"factor": 4.0, "original": 512, "fast": 16.0, "slow": 1.0}}}
 
+_TINY_PAIR = {"left": {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 32, "scale": 0.18},
+              "right": {"heads": 4, "kv_heads": 2, "dim": 32, "vdim": 48, "conv": 3}}
 _TINY_WINDOWED = {"heads": 6, "kv_heads": 2, "dim": 32, "vdim": 40, "scale": 0.25, "mask": {"size": 24, "keep_first": 5},
                   "rot": {"base": 1e4, "dims": 16}}
 _TINY_MIXTURE = {"kind": "moe", "router": {"experts": 6, "top": 2}, "expert": {"ff": 96, "limit": 3.0},
@@ -904,6 +1035,17 @@ PRESETS: dict[str, ModelConfig] = {
             {"type": "attention_2", "mixer": {"heads": 4, "kv_heads": 4, "dim": 48, "vdim": 32, "scale": 0.2, "softcap": 20.0,
                                               "rot": {"base": 5e3, "dims": 24, "scaling": {"factor": 2.0}}}, "mlp": None},
             {"type": "attention", "mixer": _TINY_WINDOWED, "mlp": _TINY_MIXTURE, "weights_of": 0}]}, {}),
+    # Dikopel at test size: both kinds of mixer, both kinds of feed-forward and none, a repeated layer
+    "tiny-dikopel": ModelConfig._from_dikopel({
+        "vocab": 1024, "width": 160, "norm": {"eps": 1e-6}, "embedding": {"scale": 6.0}, "residual_mult": 0.4,
+        "canon": {"taps": 3}, "layers": [
+            {"type": "mlstm", "mixer": {"heads": 3, "dim": 32, "vdim": 48, "gate_cap": 12.0}, "mlp": {"kind": "dense", "ff": 224}},
+            {"type": "parallel", "mixer": _TINY_PAIR, "mlp": {
+                "kind": "moe", "router": {"experts": 9, "top": 2, "scale": 2.0, "groups": {"count": 3, "keep": 2}},
+                "expert": {"ff": 64}, "shared": {"ff": 96}}},
+            {"type": "parallel", "mixer": _TINY_PAIR, "mlp": None},
+            {"type": "mlstm", "mixer": {"heads": 3, "dim": 32, "vdim": 48, "gate_cap": 12.0}, "mlp": {"kind": "dense", "ff": 224},
+             "weights_of": 0}]}, {}),
     # DeepSeek-V2-Lite: latent attention without the query bottleneck, softmax routing, two shared experts
     "deepseek-v2-lite": ModelConfig(model_type="deepseek_v2", vocab_size=102400, hidden_size=2048,
                                     intermediate_size=10944, num_hidden_layers=27, num_attention_heads=16,

@@ -5,22 +5,27 @@ optional feed-forward, on an fp32 residual stream:
     x = x + wrap1(mixer(norm1(x)));   x = x + wrap2(ff(norm2(x)))     per layer; a layer may have no feed-forward
     logits = head norm(x) * scale
 
+or, where ``layer_norms`` is "parallel", with one norm that both sublayers read, the mixer through a short convolution:
+
+    h = norm1(x);   x = x + residual_mult * (mixer(h + conv(h)) + ff(h))
+
 Norms (``ModelConfig.layer_norms``): Dynamic Tanh, ``tanh(alpha x) * w + b`` (Zhu, Chen, He, LeCun, Liu, "Transformers
 without Normalization") with a learned per-column scale as ``wrap``; layer norm with a second layer norm as ``wrap``; no
-norm in front and an RMS norm as ``wrap`` (the sublayers then read the stream itself).
+norm in front and an RMS norm as ``wrap`` (the sublayers then read the stream itself); layer norm in front of both.
 Every sublayer hands the activations in front of its output projection to the next norm's ``join``, which projects,
 wraps, adds to the residual and normalises in as few kernels as the shapes allow (``ops/dyt.py``, ``ops/layer_norm.py``),
 so the model is a flat list of sublayers between the embedding and the head.
 
 Mixers (``MIXERS``): HGRN2 (``models/hgrn2.py``), lightning attention with configured decays
 (``models/lightning.py``), latent attention over a compressed cache (``models/mla.py``), grouped-query attention
-(``models/gqa.py``). Feed-forwards (``make_mlp``): dense with PolyNorm or squared ReLU, mixture of gated experts, with or
-without a shared expert. A layer may run with an earlier layer's weights (``ModelConfig.weights_layer``) and a cache of
+(``models/gqa.py``), mLSTM (``models/mlstm.py``), attention and a gated delta rule side by side (``models/delta.py``).
+Feed-forwards (``make_mlp``): dense with PolyNorm, squared ReLU or SwiGLU, mixture of gated experts, with or without a shared
+expert. A layer may run with an earlier layer's weights (``ModelConfig.weights_layer``) and a cache of
 its own. A sublayer has ``hidden(y, ctx, cache, rec)``, an output
 projection ``o`` (None: ``hidden`` is the sublayer's result) and ``tensors(prefix)``; what a mixer keeps per sequence is
-declared by ``ModelConfig.cache_shapes`` / ``recurrent_shape``, allocated by the rollout engine and passed in.
+declared by ``ModelConfig.cache_shapes`` / ``state_shapes``, allocated by the rollout engine and passed in.
 
-The Fofosun, Gatolix and Felosun families are built this way. The class shares loading, the head and the engine interface
+The Fofosun, Gatolix, Felosun and Dikopel families are built this way. The class shares loading, the head and the engine interface
 (``prefill`` / ``decode``) with ``QwenModel``. It is served by the rollout engine and runs forward and backward for
 training on one process per replica (data parallelism).
 """
@@ -33,21 +38,24 @@ from typing import Any, Iterator
 import torch
 import torch.nn as nn
 
-from ..ops import dyt, layer_norm as ln, residual_rms as rms
+from ..ops import dyt, layer_norm as ln, residual_rms as rms, residual_sum as rs
 from ..ops.attention import VarlenMeta
 from ..ops.gemm import linear, linear_relu2, linear_slices
 from ..ops.latent_attn import rotary_tables
 from ..ops.lm_head import soft_cap_
 from ..ops.moe import ExpertRows, GatedAct, gated_experts, gated_linear, route_tokens
+from ..ops.short_conv import ConvTail, conv_prefill
 from .config import ModelConfig
+from .delta import MixerPair
 from .gqa import GroupedAttention
 from .hgrn2 import HGRN2
 from .lightning import ConstantDecayLightning
 from .mla import LatentAttention
+from .mlstm import MLSTM
 from .qwen import QwenModel
 
 MIXERS = {"hgrn2": HGRN2, "lightning": ConstantDecayLightning, "latent_attention": LatentAttention,
-          "grouped_attention": GroupedAttention}
+          "grouped_attention": GroupedAttention, "mlstm": MLSTM, "mixer_pair": MixerPair}
 
 
 class ColumnScale(nn.Module):
@@ -150,10 +158,23 @@ class RMSNorm(Stream):
         yield name, self.weight
 
 
+class SharedLayerNorm(LayerNorm):
+    """The layer norm that both sublayers of a layer read. ``conv``: the input convolution behind it (decode steps), see
+    :class:`ops.short_conv.ConvTail`; the norm then hands over a pair."""
+
+    def embed(self, ids, table, conv=None, scale: float = 1.0, pos=None, pos_table=None):
+        return rs.embed_sum(ids, table, scale, pos, self.args, self.eps, conv)
+
+    def join(self, a: rs.ParallelSum, o, wrap: float, res, conv=None):
+        """``(norm(res), res)`` of ``res + wrap * (what both sublayers of the layer in front add)``."""
+        return rs.residual_sum(a, wrap, res, self.args, self.eps, conv)
+
+
 # norm, what is wrapped around a sublayer's result, the latter's checkpoint names, and the norm in front of the head
 NORMS = {"dynamic_tanh": (DynamicTanh, lambda n, eps, dtype, device: ColumnScale(n, dtype, device), ("ls1", "ls2"), DynamicTanh),
          "layer_norm": (LayerNorm, LayerNorm, ("norm1b", "norm2b"), LayerNorm),
-         "post_rms": (Stream, RMSNorm, ("norm1", "norm2"), RMSNorm)}
+         "post_rms": (Stream, RMSNorm, ("norm1", "norm2"), RMSNorm),
+         "parallel": (SharedLayerNorm, None, (), SharedLayerNorm)}
 
 
 class Relu2MLP(nn.Module):
@@ -175,9 +196,10 @@ class Relu2MLP(nn.Module):
 class ExpertsMLP(nn.Module):
     """Mixture of gated experts. Scores ``s`` are the softmax of the router's logits (32-bit) over all experts, or each
     expert's sigmoid (``router["score"]``); the ``top`` largest of ``s``, plus a learned correction unless
-    ``router["correction"]`` is false, are chosen and weighted by ``s``, not renormalised. The weight multiplies an expert's
-    result, or what goes into it (``spec["weight"]`` "input"). Every token also passes through the ``shared`` expert, when
-    there is one. An expert is ``W_down act(W_gate y, W_up y)`` with the activation of ``ops/moe.py::GatedAct``. Gate and
+    ``router["correction"]`` is false, are chosen, with ``router["groups"]`` from the best groups only, and weighted by ``s``,
+    renormalised with ``router["renorm"]``, times ``router["scale"]``. The weight multiplies an expert's result, or what goes
+    into it (``spec["weight"]`` "input"). Every token also passes through the ``shared`` expert, when there is one; with its
+    ``gate`` that result is multiplied by the sigmoid of one more row of the router. An expert is ``W_down act(W_gate y, W_up y)`` with the activation of ``ops/moe.py::GatedAct``. Gate and
     up rows alternate in ``gate_up`` so that the activation runs in the product's epilogue."""
 
     o = None
@@ -189,34 +211,44 @@ class ExpertsMLP(nn.Module):
         E, ff = router["experts"], spec["expert"]["ff"]
         mk = lambda *shape: nn.Parameter(torch.empty(*shape, dtype=dtype, device=device))
         self.top, self.score = router["top"], router.get("score", "softmax")
-        self.act, self.scale_input = act(spec["expert"]["limit"]), spec.get("weight") == "input"
-        self.router = mk(E, hidden)
+        self.renorm, self.scale = bool(router.get("renorm")), float(router.get("scale", 1.0))
+        groups = router.get("groups") or {"count": 1, "keep": 1}
+        self.groups = (groups["count"], groups["keep"])
+        self.act, self.scale_input = act(spec["expert"].get("limit", INF)), spec.get("weight") == "input"
+        self.gates = int(bool(spec.get("shared") and spec["shared"].get("gate")))
+        self.router = mk(E + self.gates, hidden)
         self.correction = nn.Parameter(torch.zeros(E, dtype=dtype, device=device)) if router.get("correction", True) else None
         self.gate_up = mk(E, 2 * ff, hidden)
         self.down = mk(E, hidden, ff)
-        self.shared = GatedMLP(hidden, spec["shared"]["ff"], act(spec["shared"]["limit"]), dtype, device) \
+        self.shared = GatedMLP(hidden, spec["shared"]["ff"], act(spec["shared"].get("limit", INF)), dtype, device) \
             if spec.get("shared") else None
 
     def hidden(self, y, ctx=None, cache=None, rec=None):
-        idx, w = route_tokens(y, self.router, self.top, False, self.correction, self.score)
+        idx, w, *gate = route_tokens(y, self.router, self.top, self.renorm, self.correction, self.score, self.groups, self.scale,
+                                     self.gates)
         e = gated_experts(y, idx, w, self.gate_up, self.down, self.act, self.scale_input)
         if self.shared is None:
             return e
         if not isinstance(e, ExpertRows):
-            return e + linear(self.shared.hidden(y), self.shared.o).float()
+            s = linear(self.shared.hidden(y), self.shared.o).float()
+            return e + (s * torch.sigmoid(gate[0]) if gate else s)
+        e.add_gate = gate[0] if gate else None
         e.add = linear_slices(self.shared.hidden(y), self.shared.o)
         return e
 
     def tensors(self, p: str):
-        for e in range(self.router.shape[0]):
+        E = self.down.shape[0]
+        for e in range(E):
             yield f"{p}e{e}.gate", self.gate_up[e, 0::2]
             yield f"{p}e{e}.up", self.gate_up[e, 1::2]
             yield f"{p}e{e}.down", self.down[e]
-        yield p + "router", self.router
+        yield p + "router", self.router[:E]
         if self.correction is not None:
             yield p + "correction", self.correction
         if self.shared is not None:
             yield from self.shared.tensors(p + "shared.")
+        if self.gates:
+            yield p + "shared.sg", self.router[E:]
 
 
 class GatedMLP(nn.Module):
@@ -237,7 +269,14 @@ class GatedMLP(nn.Module):
         yield p + "down", self.o
 
 
+INF = float("inf")
+
+
 def make_mlp(hidden: int, spec: dict, eps: float, dtype, device):
+    if spec.get("act") == "swiglu":
+        if spec["kind"] == "moe":
+            return ExpertsMLP(hidden, spec, lambda limit: GatedAct(limit=float(limit)), dtype, device)
+        return GatedMLP(hidden, spec["ff"], GatedAct(), dtype, device)
     if spec["kind"] == "moe":
         # x * sigmoid(1.702 x) approximates GELU (Hendrycks and Gimpel, "Gaussian Error Linear Units")
         return ExpertsMLP(hidden, spec, lambda limit: GatedAct(alpha=1.702, beta=1.0, limit=float(limit)), dtype, device)
@@ -264,6 +303,55 @@ class PolyNormMLP(nn.Module):
         yield p + "down", self.o
 
 
+class ParallelBlock(nn.Module):
+    """A layer whose mixer and feed-forward read the same norm, the mixer through ``h + conv(h)``. To the decoder it is one
+    sublayer: ``hidden`` returns an :class:`ops.residual_sum.ParallelSum`."""
+
+    o = None
+
+    def __init__(self, cfg: ModelConfig, i: int, dtype, device):
+        super().__init__()
+        h, spec, eps = cfg.hidden_size, cfg.layer_specs[i], cfg.rms_norm_eps
+        self.norm1 = NORMS[cfg.layer_norms][0](h, eps, dtype, device)
+        self.attn = MIXERS[spec["type"]](h, spec["mixer"], eps, dtype, device)
+        self.attn.index = i
+        self.mlp = make_mlp(h, spec["mlp"], eps, dtype, device) if spec["mlp"] is not None else None
+        self.conv = nn.Parameter(torch.empty(h, cfg.input_conv, dtype=dtype, device=device))
+        self.mult = cfg.residual_mult
+
+    def sublayers(self, cache, rec):
+        return [(self, self.mult, self.norm1, cache, rec)]
+
+    def tail(self, ctx, rec):
+        """What the norm in front goes on to in a decode step."""
+        return ConvTail(self.conv, rec["conv"], ctx.state_slots, ctx.pos) if ctx.decode else None
+
+    def hidden(self, y, ctx, cache=None, rec=None):
+        if ctx.decode:
+            h, hc = y
+        else:
+            h = y
+            hc = conv_prefill(h, self.conv, ctx.meta, ctx.pos, add=True, ring=rec["conv"] if rec is not None else None,
+                              slots=ctx.state_slots)
+        if self.attn.o is None:
+            mixer = self.attn.results(hc, ctx, cache, rec)
+        else:
+            mixer = [(linear_slices(self.attn.hidden(hc, ctx, cache, rec), self.attn.o), None)]
+        ff = None
+        if self.mlp is not None:
+            ff = self.mlp.hidden(h, ctx)
+            if self.mlp.o is not None:
+                ff = linear_slices(ff, self.mlp.o)
+        return rs.ParallelSum(mixer, ff)
+
+    def tensors(self, p: str):
+        yield from self.norm1.tensors(p + "norm1")
+        yield from self.attn.tensors(p + "mix.")
+        if self.mlp is not None:
+            yield from self.mlp.tensors(p + "mlp.")
+        yield p + "canon1", self.conv
+
+
 class LayeredBlock(nn.Module):
     def __init__(self, cfg: ModelConfig, i: int, dtype, device):
         super().__init__()
@@ -278,6 +366,11 @@ class LayeredBlock(nn.Module):
             self.norm2 = norm(h, eps, dtype, device)
             self.mlp = make_mlp(h, spec["mlp"], eps, dtype, device)
             self.wrap2 = wrap(h, eps, dtype, device)
+
+    def sublayers(self, cache, rec):
+        """``(sublayer, its wrap, its norm, its cache, its state)`` in order."""
+        out = [(self.attn, self.wrap1, self.norm1, cache, rec)]
+        return out if self.mlp is None else out + [(self.mlp, self.wrap2, self.norm2, None, None)]
 
     def tensors(self, p: str):
         yield from self.norm1.tensors(p + "norm1")
@@ -329,9 +422,10 @@ class LayeredModel(QwenModel):
         self.embed = mk(cfg.vocab_size, cfg.hidden_size)
         self.pos = mk(cfg.max_position_embeddings, cfg.hidden_size) if cfg.learned_positions else None
         self.layers = nn.ModuleList()
+        block = ParallelBlock if cfg.layer_norms == "parallel" else LayeredBlock
         for i in self.layer_ids:  # a layer that runs with another's weights is the same module once more
             j = cfg.weights_layer(i)
-            self.layers.append(LayeredBlock(cfg, i, dtype, device) if j == i else self.layers[j])
+            self.layers.append(block(cfg, i, dtype, device) if j == i else self.layers[j])
         # the head is linear: the logits' scale is the last norm's
         scaled = dict(scale=cfg.logit_scale) if cfg.logit_scale != 1.0 else {}
         self.norm = NORMS[cfg.layer_norms][3](cfg.hidden_size, cfg.rms_norm_eps, dtype, device, **scaled)
@@ -375,21 +469,21 @@ class LayeredModel(QwenModel):
     def _run(self, input_ids, ctx: StepContext, kv_caches=None, state=None):
         """Embedding, every sublayer, final norm: ``[T, hidden]`` in the model's dtype."""
         ctx.shared = self._shared
-        subs = []  # (sublayer, its wrap, its norm, its cache, its state)
+        subs = []
         for i, layer in enumerate(self.layers):
             cache = kv_caches[self.cfg.cache_layer(i)] if kv_caches is not None else None
             if cache is not None and len(cache) == 1:
                 cache = cache[0]
-            subs.append((layer.attn, layer.wrap1, layer.norm1, cache, state.rec[i] if state is not None else None))
-            if layer.mlp is not None:
-                subs.append((layer.mlp, layer.wrap2, layer.norm2, None, None))
+            subs += layer.sublayers(cache, state.rec[i] if state is not None else None)
         norms = [s[2] for s in subs] + [self.norm]
+        # what a norm goes on to for the sublayer behind it
+        tails = [(s[0].tail(ctx, s[4]),) if hasattr(s[0], "tail") else () for s in subs] + [()]
         extra = {}
-        if self.pos is not None or self.cfg.embedding_scale != 1.0:
+        if self.pos is not None or self.cfg.embedding_scale != 1.0 or self.cfg.sinusoid_positions:
             extra = dict(scale=self.cfg.embedding_scale, pos=ctx.pos, pos_table=self.pos)
-        y, res = norms[0].embed(input_ids, self.embed, **extra)
+        y, res = norms[0].embed(input_ids, self.embed, *tails[0], **extra)
         for k, (sub, wrap, _, cache, rec) in enumerate(subs):
-            y, res = norms[k + 1].join(sub.hidden(y, ctx, cache, rec), sub.o, wrap, res)
+            y, res = norms[k + 1].join(sub.hidden(y, ctx, cache, rec), sub.o, wrap, res, *tails[k + 1])
         return y
 
     def forward(self, input_ids, position_ids, meta: VarlenMeta, attn_fn=None, **unsupported):

@@ -76,13 +76,16 @@ def _rope_partial(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, rot: in
 
 
 class RecurrentState:
-    """``rec[i] [slots, heads, key width, value width]`` fp32 for every layer with a matrix state per head
-    (``ModelConfig.recurrent_shape``), ``None`` for the others."""
+    """``rec[i] [slots, heads, key width, value width]`` fp32 for every layer that keeps a matrix state per head and nothing
+    else, a dictionary ``name -> [slots, ...]`` for layers that keep more (``ModelConfig.state_shapes``), ``None`` for those
+    without a state."""
 
     def __init__(self, cfg: ModelConfig, max_slots: int, dtype, device):
-        shapes = [cfg.recurrent_shape(i) for i in range(cfg.num_hidden_layers)]
-        self.rec = [None if s is None else torch.zeros(max_slots, *s, dtype=torch.float32, device=device)
-                    for s in shapes]
+        self.rec = []
+        for i in range(cfg.num_hidden_layers):
+            rec = {name: torch.zeros(max_slots, *s, dtype=torch.float32 if wide else dtype, device=device)
+                   for name, (s, wide) in cfg.state_shapes(i).items()}
+            self.rec.append(rec["S"] if set(rec) == {"S"} else rec or None)
 
 
 class LightningAttention(nn.Module):

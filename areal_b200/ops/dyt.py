@@ -111,26 +111,27 @@ def polynorm(z: torch.Tensor, coef: torch.Tensor, eps: float):
     return y
 
 
-def group_rms_ref(o, w, groups: int, eps: float, gate=None, dtype=None):
+def group_rms_ref(o, w, groups: int, eps: float, gate=None, dtype=None, act: str = "sigmoid"):
     T, n = o.shape[0], o.shape[1] // groups
     of = o.float().view(T, groups, n)
     y = of * torch.rsqrt(of.pow(2).mean(-1, keepdim=True) + eps)
     y = (y * w.float().view(-1, n)).reshape(T, groups * n)
     if gate is not None:
-        y = y * torch.sigmoid(gate.float())
+        y = y * (torch.sigmoid(gate.float()) if act == "sigmoid" else torch.nn.functional.silu(gate.float()))
     return y.to(dtype or w.dtype)
 
 
-def group_rms(o: torch.Tensor, w: torch.Tensor, groups: int, eps: float, gate: torch.Tensor | None = None):
+def group_rms(o: torch.Tensor, w: torch.Tensor, groups: int, eps: float, gate: torch.Tensor | None = None,
+              act: str = "sigmoid"):
     """RMS norm of fp32 ``o [T, groups * n]`` over each group of columns; ``w`` is ``[n]`` (shared by the groups) or
-    ``[groups * n]``; times ``sigmoid(gate)`` when given. The result has the weight's dtype."""
+    ``[groups * n]``; times ``sigmoid(gate)`` (or ``silu(gate)``) when given. The result has the weight's dtype."""
     if not kernel_ok(o, w, gate):
-        return group_rms_ref(o, w, groups, eps, gate)
+        return group_rms_ref(o, w, groups, eps, gate, act=act)
     T, n = o.shape[0], o.shape[1] // groups
     assert o.is_contiguous() and o.dtype == torch.float32 and w.numel() in (n, groups * n)
     y = torch.empty(o.shape, dtype=w.dtype, device=o.device)
     rc = _lib.kernels().b200_group_rms(_lib.ptr(o), _lib.ptr(w), ctypes.c_int(int(w.numel() != n)), _lib.ptr(gate),
-                                       ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _lib.ptr(y),
+                                       ctypes.c_longlong(gate.stride(0) if gate is not None else 0), ctypes.c_int(int(act == "silu")), _lib.ptr(y),
                                        ctypes.c_longlong(T), ctypes.c_int(groups), ctypes.c_int(n), ctypes.c_float(eps),
                                        fp32_flag(w), _lib.stream_ptr())
     _lib.check(rc, "b200_group_rms")

@@ -1,5 +1,6 @@
-"""Grouped-query softmax attention over packed prompts and paged caches, with a window that keeps the first tokens, a
-soft cap on the scores, a sink in the softmax and a gate per head (``csrc/gqa_prep.cu``, ``csrc/gqa_prefill.cu``,
+"""Grouped-query attention over packed prompts and paged caches, with a window that keeps the first tokens, a soft cap on the
+scores, a sink in the softmax, a gate per head, or sigmoids of the scores as weights (Ramapuram et al., "Theory, Analysis, and
+Best Practices for Sigmoid Self-Attention") in place of the softmax (``csrc/gqa_prep.cu``, ``csrc/gqa_prefill.cu``,
 ``csrc/gqa_decode.cu``; ``csrc/latent_attn.cu`` for 32-bit models and odd widths), with their PyTorch statements (the CPU
 path, and the path under autograd).
 
@@ -33,6 +34,7 @@ class GroupedSpec:
     rot_dims: int = 0
     rot_halves: bool = False        # pair i is (i, i + rot_dims / 2); else (2i, 2i + 1)
     unit_eps: float | None = None   # q and k divided by sqrt(mean of squares + eps) after the rotation; None: not
+    sigmoid: bool = False           # weights are sigmoid(score + bias[h]), each by itself; no softmax, no sink
 
     @property
     def group(self) -> int:
@@ -100,11 +102,18 @@ def _softmax_ref(s, sink):
     return torch.cat((s, col), -1).softmax(-1)[..., :-1]
 
 
+def _weights_ref(s, a, sink, bias):
+    """Weights of the scores ``s [H, ..., keys]``; -inf: not visible."""
+    if not a.sigmoid:
+        return _softmax_ref(s, sink)
+    return torch.sigmoid(s + bias.float().view(-1, *([1] * (s.dim() - 1))))
+
+
 def _cap_ref(s, cap):
     return cap * torch.tanh(s / cap) if cap else s
 
 
-def prefill_ref(q, k, v, cu, a: GroupedSpec, sink=None, gate=None):
+def prefill_ref(q, k, v, cu, a: GroupedSpec, sink=None, gate=None, bias=None):
     outs = []
     cu = [int(c) for c in cu]
     for s, e in zip(cu[:-1], cu[1:]):
@@ -115,14 +124,14 @@ def prefill_ref(q, k, v, cu, a: GroupedSpec, sink=None, gate=None):
         seen = j <= i
         if a.window:
             seen &= (i - j < a.window) | (j < a.keep_first)
-        outs.append(torch.einsum("hij,jhd->ihd", _softmax_ref(att.masked_fill(~seen, float("-inf")), sink), vv))
+        outs.append(torch.einsum("hij,jhd->ihd", _weights_ref(att.masked_fill(~seen, float("-inf")), a, sink, bias), vv))
     o = torch.cat(outs) if outs else q.new_zeros(0, a.heads, a.vdim).float()
     if gate is not None:
         o = o * torch.sigmoid(gate.float())[..., None]
     return o.reshape(q.shape[0], a.heads * a.vdim).to(q.dtype)
 
 
-def decode_ref(q, kc, vc, block_table, seq_lens, a: GroupedSpec, sink=None, gate=None):
+def decode_ref(q, kc, vc, block_table, seq_lens, a: GroupedSpec, sink=None, gate=None, bias=None):
     B, bs = q.shape[0], kc.shape[2]
     out = torch.zeros(B, a.heads, a.vdim, dtype=torch.float32, device=q.device)
     for b in range(B):
@@ -136,7 +145,7 @@ def decode_ref(q, kc, vc, block_table, seq_lens, a: GroupedSpec, sink=None, gate
         if lo > a.keep_first:
             k, v = (torch.cat((t[:a.keep_first], t[lo:])) for t in (k, v))
         s = _cap_ref(torch.einsum("hd,jhd->hj", q[b].float(), k) * a.scale, a.softcap)
-        out[b] = torch.einsum("hj,jhd->hd", _softmax_ref(s, sink), v)
+        out[b] = torch.einsum("hj,jhd->hd", _weights_ref(s, a, sink, bias), v)
     if gate is not None:
         out = out * torch.sigmoid(gate.float())[..., None]
     return out.reshape(B, a.heads * a.vdim).to(q.dtype)
@@ -201,15 +210,16 @@ def _tile(t, width: int):
     return torch.nn.functional.pad(t, (0, width - n)).contiguous()
 
 
-def _extras(a: GroupedSpec, sink, gate):
-    """``window, keep_first, softcap, sink, gate, gate pitch`` of the attention launchers."""
+def _extras(a: GroupedSpec, sink, gate, bias):
+    """``window, keep_first, softcap, sink, gate, gate pitch, sigmoid bias`` of the attention launchers."""
     assert gate is None or gate.stride(1) == 1
     assert sink is None or sink.is_contiguous()
+    assert (bias is not None) == a.sigmoid and (bias is None or (sink is None and bias.is_contiguous()))
     return (ctypes.c_int(a.window or 0), ctypes.c_int(a.keep_first if a.window else 0), ctypes.c_float(a.softcap),
-            _lib.ptr(sink), _lib.ptr(gate), ctypes.c_longlong(gate.stride(0) if gate is not None else 0))
+            _lib.ptr(sink), _lib.ptr(gate), ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _lib.ptr(bias))
 
 
-def _attend(q, k, ldk, hk, v, ldv, hv, a, sink, gate, seq_start, kv_len, bt, bs, page_rows, nsplit):
+def _attend(q, k, ldk, hk, v, ldv, hv, a, sink, gate, bias, seq_start, kv_len, bt, bs, page_rows, nsplit):
     n, c, ll = q.shape[0], ctypes.c_int, ctypes.c_longlong
     out = torch.empty((n, a.heads * a.vdim), dtype=q.dtype, device=q.device)
     o_part = ml = None
@@ -220,17 +230,17 @@ def _attend(q, k, ldk, hk, v, ldv, hv, a, sink, gate, seq_start, kv_len, bt, bs,
         _lib.ptr(q), ll(q.stride(0)), c(q.stride(1)), _lib.ptr(k), ll(ldk), c(hk), _lib.ptr(v), ll(ldv), c(hv), c(a.dim),
         c(a.vdim), _lib.ptr(seq_start), _lib.ptr(kv_len), _lib.ptr(bt), c(bt.shape[1] if bt is not None else 0), c(bs),
         c(page_rows), _lib.ptr(o_part), _lib.ptr(ml), _lib.ptr(out), ll(out.stride(0)), c(n), c(a.heads), c(a.kv_heads),
-        c(nsplit), ctypes.c_float(a.scale), *_extras(a, sink, gate), fp32_flag(q), _lib.stream_ptr())
+        c(nsplit), ctypes.c_float(a.scale), *_extras(a, sink, gate, bias), fp32_flag(q), _lib.stream_ptr())
     _lib.check(rc, "b200_attend_grouped")
     _lib.count_launch(2 if nsplit > 1 else 1)
     return out
 
 
-def prefill(q, k, v, meta, a: GroupedSpec, sink=None, gate=None):
+def prefill(q, k, v, meta, a: GroupedSpec, sink=None, gate=None, bias=None):
     """Causal attention of a packed batch: ``q [T, heads, dim]``, ``k [T, kv_heads, dim]``, ``v [T, kv_heads, vdim]`` as
     :func:`qkv_prep` returns them. Returns ``[T, heads * vdim]``."""
-    if not kernel_ok(q, k, v, sink):
-        return prefill_ref(q, k, v, meta.cu_cpu, a, sink, gate)
+    if not kernel_ok(q, k, v, sink, bias):
+        return prefill_ref(q, k, v, meta.cu_cpu, a, sink, gate, bias)
     T, H, Dv = q.shape[0], a.heads, a.vdim
     if q.dtype == torch.bfloat16 and a.dim <= 256 and Dv <= 256:
         Dp, Vp = pad16(a.dim), pad16(Dv)
@@ -241,19 +251,20 @@ def prefill(q, k, v, meta, a: GroupedSpec, sink=None, gate=None):
         rc = _lib.kernels().b200_gqa_prefill(
             _lib.ptr(q), ll(q.stride(0)), c(q.stride(1)), _lib.ptr(k), ll(k.stride(0)), c(k.stride(1)), _lib.ptr(v),
             ll(v.stride(0)), c(v.stride(1)), _lib.ptr(out), _lib.ptr(meta.fwd_tiles), c(meta.n_fwd), c(T), c(H),
-            c(a.kv_heads), c(Dp), c(Dv), ctypes.c_float(a.scale), ctypes.c_float(a.score_bound), *_extras(a, sink, gate),
+            c(a.kv_heads), c(Dp), c(Dv), ctypes.c_float(a.scale), ctypes.c_float(a.score_bound), *_extras(a, sink, gate, bias),
             _lib.stream_ptr())
         _lib.check(rc, "b200_gqa_prefill")
         _lib.count_launch()
         return out
     start, length = _query_rows(meta)
-    return _attend(q, k, k.stride(0), k.stride(1), v, v.stride(0), v.stride(1), a, sink, gate, start, length, None, 1, 1, 1)
+    return _attend(q, k, k.stride(0), k.stride(1), v, v.stride(0), v.stride(1), a, sink, gate, bias, start, length, None, 1, 1, 1)
 
 
-def decode(q, kc, vc, block_table, seq_lens, a: GroupedSpec, sink=None, gate=None, max_seq_len: int | None = None):
+def decode(q, kc, vc, block_table, seq_lens, a: GroupedSpec, sink=None, gate=None, max_seq_len: int | None = None,
+           bias=None):
     """One query token per sequence, ``q [B, heads, dim]``, against its pages. Returns ``[B, heads * vdim]``."""
     if not kernel_ok(q, sink):
-        return decode_ref(q, kc, vc, block_table, seq_lens, a, sink, gate)
+        return decode_ref(q, kc, vc, block_table, seq_lens, a, sink, gate, bias)
     B, bs, H, G = q.shape[0], kc.shape[2], a.heads, a.kv_heads
     Dp, Vp = kc.shape[3], vc.shape[3]
     max_seq_len = max_seq_len or block_table.shape[1] * bs
@@ -278,7 +289,7 @@ def decode(q, kc, vc, block_table, seq_lens, a: GroupedSpec, sink=None, gate=Non
         rc = _lib.kernels().b200_gqa_decode(
             _lib.ptr(q), ll(q.stride(0)), c(q.stride(1)), _lib.ptr(kc), _lib.ptr(vc), _lib.ptr(block_table),
             c(block_table.shape[1]), c(bs), c(kc.shape[0]), _lib.ptr(seq_lens), _lib.ptr(out), _lib.ptr(o_part), _lib.ptr(ml),
-            c(B), c(H), c(G), c(Dp), c(Vp), c(a.vdim), c(nsplit), ctypes.c_float(a.scale), *_extras(a, sink, gate),
+            c(B), c(H), c(G), c(Dp), c(Vp), c(a.vdim), c(nsplit), ctypes.c_float(a.scale), *_extras(a, sink, gate, bias),
             _lib.stream_ptr())
         _lib.check(rc, "b200_gqa_decode")
         _lib.count_launch(2 if nsplit > 1 else 1)
@@ -286,4 +297,4 @@ def decode(q, kc, vc, block_table, seq_lens, a: GroupedSpec, sink=None, gate=Non
     nsplit = 1
     while B * -(-H // 4) * nsplit < 1184 and nsplit < 64 and span // (nsplit * 2) >= 64:
         nsplit *= 2
-    return _attend(q, kc, Dp, bs * Dp, vc, Vp, bs * Vp, a, sink, gate, None, seq_lens, block_table, bs, G * bs, nsplit)
+    return _attend(q, kc, Dp, bs * Dp, vc, Vp, bs * Vp, a, sink, gate, bias, None, seq_lens, block_table, bs, G * bs, nsplit)

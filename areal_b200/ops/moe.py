@@ -35,16 +35,27 @@ from .gemm import Slices, _splitk_plan, _tma_rows, gemm, linear
 _SCORES = {"softmax": 0, "sigmoid": 1}
 
 
-def route_ref(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None, score: str = "softmax"):
+def _open_groups(pick: torch.Tensor, groups: tuple[int, int]):
+    """``pick [T, E]`` with -inf outside the best ``groups[1]`` of ``groups[0]`` equal groups of neighbours, a group's score
+    being the sum of its two best."""
+    count, keep = groups
+    if keep >= count:
+        return pick
+    g = pick.view(pick.shape[0], count, -1)
+    best = g.topk(min(2, g.shape[-1]), dim=-1).values.sum(-1).topk(keep, dim=-1).indices
+    open_ = torch.zeros(g.shape[:2], dtype=torch.bool, device=pick.device).scatter_(1, best, True)
+    return g.masked_fill(~open_[..., None], float("-inf")).view_as(pick)
+
+
+def route_ref(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None, score: str = "softmax",
+              groups: tuple[int, int] = (1, 1), scale: float = 1.0):
     probs = logits.float().softmax(-1) if score == "softmax" else torch.sigmoid(logits.float())
-    if correction is None:
-        w, idx = probs.topk(k, dim=-1)
-    else:
-        idx = (probs + correction.float()).topk(k, dim=-1).indices
-        w = probs.gather(-1, idx)
+    pick = probs if correction is None else probs + correction.float()
+    idx = _open_groups(pick, groups).topk(k, dim=-1).indices
+    w = probs.gather(-1, idx)
     if renorm:
-        w = w / w.sum(-1, keepdim=True)
-    return idx.to(torch.int32), w
+        w = w / (w.sum(-1, keepdim=True) + 1e-20)
+    return idx.to(torch.int32), w * scale if scale != 1.0 else w
 
 
 def permute_by_expert(idx: torch.Tensor, num_experts: int):
@@ -80,48 +91,60 @@ def moe_experts_ref(x, idx, w, gate_up, down):
 # --------------------------------------------------------------------------- CUDA pieces
 
 
-def route(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None, score: str = "softmax"):
+def _groups_args(groups: tuple[int, int], scale: float):
+    return ctypes.c_int(groups[0]), ctypes.c_int(groups[1]), ctypes.c_float(scale)
+
+
+def route(logits: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None, score: str = "softmax",
+          groups: tuple[int, int] = (1, 1), scale: float = 1.0):
     """``logits [T, E]`` fp32 → ``(idx [T,k] int32, w [T,k] fp32)``. Scores are the softmax over all experts or each
     expert's sigmoid. ``correction [E]`` is added to the scores when the experts are chosen; their weights are the scores
-    without it."""
+    without it, with ``renorm`` over their sum, times ``scale``. ``groups = (count, keep)``: only experts of the best ``keep``
+    groups of neighbours can be chosen, by the sum of a group's two largest (corrected) scores."""
     T, E = logits.shape
     if not (_lib.use_cuda_kernels(logits) and logits.dtype == torch.float32 and E <= 256 and k <= 32
             and (correction is None or correction.dtype in (torch.float32, torch.bfloat16))):
-        return route_ref(logits, k, renorm, correction, score)
-    logits = logits if logits.is_contiguous() else logits.contiguous()
+        return route_ref(logits, k, renorm, correction, score, groups, scale)
+    logits = logits if logits.stride(1) == 1 else logits.contiguous()
     idx = torch.empty((T, k), dtype=torch.int32, device=logits.device)
     w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
-    rc = _lib.kernels().b200_moe_route(_lib.ptr(logits), _lib.ptr(correction),
+    rc = _lib.kernels().b200_moe_route(_lib.ptr(logits), ctypes.c_longlong(logits.stride(0)), _lib.ptr(correction),
                                        ctypes.c_int(int(correction is not None and correction.dtype == torch.float32)),
                                        _lib.ptr(idx), _lib.ptr(w), ctypes.c_int(T), ctypes.c_int(E),
                                        ctypes.c_int(k), ctypes.c_int(int(renorm)), ctypes.c_int(_SCORES[score]),
-                                       _lib.stream_ptr())
+                                       *_groups_args(groups, scale), _lib.stream_ptr())
     _lib.check(rc, "b200_moe_route")
     _lib.count_launch()
     return idx, w
 
 
 def route_tokens(x: torch.Tensor, router: torch.Tensor, k: int, renorm: bool, correction: torch.Tensor | None = None,
-                 score: str = "softmax"):
+                 score: str = "softmax", groups: tuple[int, int] = (1, 1), scale: float = 1.0, gates: int = 0):
     """Router projection (fp32 products and sums) and choice: ``x [T, H]``, ``router [E, H]``. A decode step's few tokens
-    take one kernel."""
+    take one kernel. ``gates``: the router's last rows are no experts; their projections ``[T, gates]`` (fp32) come third."""
     T, H = x.shape
-    E = router.shape[0]
-    if kernel_ok(x, router) and T <= 256 and E <= 256 and k <= 32 and (H + E) * 4 <= 200 * 1024:
+    R = router.shape[0]
+    E = R - gates
+    if kernel_ok(x, router) and T <= 256 and E <= 256 and k <= 32 and (H + R) * 4 <= 200 * 1024:
         x = x if x.stride(1) == 1 and x.data_ptr() % 16 == 0 and x.stride(0) % 4 == 0 else x.contiguous()
         idx = torch.empty((T, k), dtype=torch.int32, device=x.device)
         w = torch.empty((T, k), dtype=torch.float32, device=x.device)
+        z = torch.empty((T, gates), dtype=torch.float32, device=x.device) if gates else None
         rc = _lib.kernels().b200_moe_router(
             _lib.ptr(x), ctypes.c_longlong(x.stride(0)), _lib.ptr(router), _lib.ptr(correction), _lib.ptr(idx), _lib.ptr(w),
-            ctypes.c_int(T), ctypes.c_int(H), ctypes.c_int(E), ctypes.c_int(k), ctypes.c_int(int(renorm)),
-            ctypes.c_int(_SCORES[score]), fp32_flag(x), _lib.stream_ptr())
+            _lib.ptr(z), ctypes.c_int(T), ctypes.c_int(H), ctypes.c_int(E), ctypes.c_int(gates), ctypes.c_int(k),
+            ctypes.c_int(int(renorm)), ctypes.c_int(_SCORES[score]), *_groups_args(groups, scale), fp32_flag(x),
+            _lib.stream_ptr())
         _lib.check(rc, "b200_moe_router")
         _lib.count_launch()
-        return idx, w
+        return (idx, w, z) if gates else (idx, w)
     if kernel_ok(x, router):
         logits = gemm(x, router, out_dtype=torch.float32) if x.dtype == torch.bfloat16 else torch.nn.functional.linear(x, router)
-        return route(logits, k, renorm, correction, score)
-    return route_ref(torch.nn.functional.linear(x.float(), router.float()), k, renorm, correction, score)
+        out = route(logits[:, :E], k, renorm, correction, score, groups, scale)
+    else:
+        logits = torch.nn.functional.linear(x.float(), router.float())
+        out = route_ref(logits[:, :E], k, renorm, correction, score, groups, scale)
+    return (*out, logits[:, E:].contiguous()) if gates else out
 
 
 @dataclass
@@ -323,24 +346,26 @@ class GatedAct:
 @dataclass
 class ExpertRows:
     """Results of the chosen experts, not yet combined: row ``dest[t * k + j]`` of ``rows`` belongs to choice ``j`` of
-    token ``t`` and counts ``w[t, j]`` (None: 1). ``add``: what every token adds to the sum of its ``k`` choices."""
+    token ``t`` and counts ``w[t, j]`` (None: 1). ``add``: what every token adds to the sum of its ``k`` choices; ``add_gate``: times the
+    sigmoid of the token's number there (fp32)."""
 
     rows: torch.Tensor
     dest: torch.Tensor
     k: int
     w: torch.Tensor | None
     add: "torch.Tensor | Slices | None" = None
+    add_gate: torch.Tensor | None = None
 
     def args(self):
-        """``rows, dest, w, k`` and the addend's ``rows, pitch, slices, slice stride, number of slices`` for the kernels
-        that combine."""
+        """``rows, dest, w, k`` and the addend's ``rows, pitch, slices, slice stride, number of slices, gate`` for the
+        kernels that combine."""
         ll, c, p = ctypes.c_longlong, ctypes.c_int, _lib.ptr
         sl = self.add if isinstance(self.add, Slices) else None
         add = self.add if sl is None else None
         if add is not None and not (add.stride(1) == 1 and add.stride(0) % 4 == 0 and add.data_ptr() % 16 == 0):
             add = self.add = add.contiguous()
         return (p(self.rows), p(self.dest), p(self.w), c(self.k), p(add), ll(add.stride(0) if add is not None else 0),
-                p(sl.ws if sl else None), ll(sl.stride if sl else 0), c(sl.n if sl else 0))
+                p(sl.ws if sl else None), ll(sl.stride if sl else 0), c(sl.n if sl else 0), p(self.add_gate))
 
 
 def gated_experts_ref(x, idx, w, gate_up, down, act: GatedAct, scale_input: bool = False):
