@@ -92,10 +92,15 @@ struct ExpertSrc {
   const T* add;      // null, or [rows][ld_add]: added to the sum of the choices
   long long ld_add;
   SliceSrc slices;   // S > 0: the same as the slices of a split product
+  const float* add_gate;  // null, or [rows]: what is added is multiplied by the sigmoid of the row's number
   template <int V>
   __device__ __forceinline__ float4 load(long long row, int c) const {
     float4 a = slices.template load<V>(row, c);
     if (add) a = ldv(add + row * ld_add + c, V);
+    if (add_gate) {
+      const float s = 1.f / (1.f + expf(-__ldg(add_gate + row)));
+      a = make_float4(a.x * s, a.y * s, a.z * s, a.w * s);
+    }
 #pragma unroll 4
     for (int j = 0; j < k; ++j) {
       const float s = w ? __ldg(w + row * k + j) : 1.f;

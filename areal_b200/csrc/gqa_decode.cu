@@ -1,5 +1,6 @@
 // Decode attention over a paged cache for grouped-query heads of up to 256 with the options of ops/gqa.py: a window that
-// keeps the first tokens, a soft cap on the scores, a sink, a gate per head. One query token per sequence.
+// keeps the first tokens, a soft cap on the scores, a sink, a gate per head, sigmoids as weights. One query token per
+// sequence.
 //
 //   k_cache [blocks, G, block_size, D], v_cache [blocks, G, block_size, Dv]   bf16, D and Dv in steps of 16
 //
@@ -8,7 +9,8 @@
 // the rows of an m16n8k16 tile (groups past 16 take several CTAs). What differs:
 //   * the walk over slabs has two parts: those of the first tokens that a window keeps, then those inside the window;
 //   * softmax weights enter the second product as two bf16 terms (hi + lo), so they keep fp32-like precision;
-//   * the sink joins the denominator once, and the gate scales a head's result, where the splits meet.
+//   * the sink joins the denominator once, and the gate scales a head's result, where the splits meet;
+//   * sigmoid weights count as they are: neither maxima nor sums are kept (the reference stays 0).
 #include "common/host_utils.h"
 #include "common/io.cuh"
 #include "common/mma16.cuh"
@@ -30,13 +32,15 @@ struct GqaDecodeArgs {
   int window, keep;
   const __nv_bfloat16 *sink, *gate;
   long long ldg;
+  const __nv_bfloat16* sig_bias;  // null: softmax; else [H], added to the scores
 };
 
 // Result of a head from its accumulated sum `l` (against the reference m, in units of log 2): the factor on the
 // accumulators, with the sink's term and the gate.
 __device__ __forceinline__ float gqa_final(float m, float l, int h, long long row, const __nv_bfloat16* sink,
-                                           const __nv_bfloat16* gate, long long ldg) {
+                                           const __nv_bfloat16* gate, long long ldg, bool sigmoid) {
   float f = 1.f;
+  if (sigmoid) return gate ? sigmoid_as(__bfloat162float(gate[row * ldg + h]), gate) : 1.f;
   if (sink) {
     const float sv = __bfloat162float(sink[h]) * 1.4426950408889634f, mn = fmaxf(m, sv);
     f = m == -INFINITY ? 0.f : ex2_fast(m - mn);
@@ -120,6 +124,14 @@ gqa_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     for (int c = 0; c < 4; ++c) o[i][c] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   constexpr float kLog2e = 1.4426950408889634f;
+  float sig[2] = {0.f, 0.f};
+  if (a.sig_bias) {
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      m[e] = 0.f;
+      if (row + e * 8 < nh) sig[e] = __bfloat162float(a.sig_bias[h0 + row + e * 8]) * kLog2e;
+    }
+  }
   const float scale_log2 = a.scale * kLog2e, cap_log2 = a.cap * kLog2e, to_cap = a.cap > 0.f ? a.scale / a.cap : 0.f;
 
   const int lm = lane >> 3, lr = lane & 7;  // ldmatrix: matrix and row in it
@@ -156,6 +168,14 @@ gqa_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
         v[c] = a.cap > 0.f ? cap_log2 * tanh_as(v[c] * to_cap, a.q) : v[c] * scale_log2;
         if (tok >= L || (tok < lo && tok >= a.keep)) v[c] = -INFINITY;
       }
+      float p[4];
+      if (a.sig_bias) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c) p[c] = rcp_fast(1.f + ex2_fast(-(v[c] + sig[e])));  // -inf: 0
+        hi[e] = split2(p[0], p[1], low[e]);
+        hi[2 + e] = split2(p[2], p[3], low[2 + e]);
+        continue;
+      }
       float mx = fmaxf(fmaxf(v[0], v[1]), fmaxf(v[2], v[3]));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
@@ -170,7 +190,6 @@ gqa_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
         m[e] = mn;
       }
       const float mref = m[e] == -INFINITY ? 0.f : m[e];
-      float p[4];
 #pragma unroll
       for (int c = 0; c < 4; ++c) p[c] = ex2_fast(v[c] - mref);
       l[e] += (p[0] + p[1]) + (p[2] + p[3]);
@@ -238,7 +257,7 @@ gqa_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant
     }
     const long long bh = static_cast<long long>(b) * a.H + h0 + g;
     if (a.nsplit == 1) {
-      if (d < a.dv) a.out[bh * a.dv + d] = __float2bfloat16(at * gqa_final(mn, lt, h0 + g, b, a.sink, a.gate, a.ldg));
+      if (d < a.dv) a.out[bh * a.dv + d] = __float2bfloat16(at * gqa_final(mn, lt, h0 + g, b, a.sink, a.gate, a.ldg, a.sig_bias));
     } else {
       const long long u = bh * a.nsplit + split;
       a.o_part[u * a.Dv + d] = at;
@@ -264,7 +283,7 @@ __global__ void gqa_merge_kernel(const GqaDecodeArgs a) {
     if (threadIdx.x == 0) w[s] = e;
   }
   __syncthreads();
-  const float f = gqa_final(m, l, h, u / a.H, a.sink, a.gate, a.ldg);
+  const float f = gqa_final(m, l, h, u / a.H, a.sink, a.gate, a.ldg, a.sig_bias);
   for (int d = threadIdx.x; d < a.dv; d += blockDim.x) {
     float t = 0.f;
     for (int s = 0; s < a.nsplit; ++s)
@@ -305,15 +324,17 @@ extern "C" {
 
 // q [B][ldq] + h * hq (multiples of 8, zeros between a head's width and D); caches as above, 16-byte aligned; out [B, H *
 // dv], dv <= Dv. o_part fp32 [B, H, nsplit, Dv] and ml_part [B, H, nsplit, 2] when nsplit > 1 (at most 64). window 0: none;
-// keep counts only with a window. softcap 0: none. sink: null or [H]; gate: null or [B][ldg].
+// keep counts only with a window. softcap 0: none. sink: null or [H]; gate: null or [B][ldg]; sig_bias: null, or [H] for
+// sigmoid weights (without a sink).
 int b200_gqa_decode(const void* q, long long ldq, int hq, const void* k_cache, const void* v_cache, const int* block_table,
                     int max_blocks, int block_size, int num_blocks, const int* seq_lens, void* out, float* o_part,
                     float* ml_part, int B, int H, int G, int D, int Dv, int dv, int nsplit, float scale, int window,
-                    int keep, float softcap, const void* sink, const void* gate, long long ldg, cudaStream_t stream) {
+                    int keep, float softcap, const void* sink, const void* gate, long long ldg, const void* sig_bias,
+                    cudaStream_t stream) {
   using namespace b200;
   if (B <= 0) return 0;
   if (G < 1 || H % G || D < 16 || Dv < 16 || D % 16 || Dv % 16 || D > 256 || Dv > 256 || dv > Dv || block_size % kGdSlab ||
-      ((ldq | hq) & 7) || nsplit < 1 || nsplit > 64)
+      ((ldq | hq) & 7) || nsplit < 1 || nsplit > 64 || (sink && sig_bias))
     return -100;
   using bf = __nv_bfloat16;
   const auto dt = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
@@ -324,7 +345,8 @@ int b200_gqa_decode(const void* q, long long ldq, int hq, const void* k_cache, c
   rc = make_tmap_2d(&tmV, v_cache, dt, 2, rows, Dv, static_cast<uint64_t>(Dv) * 2, kGdSlab, 64);
   if (rc) return rc;
   const GqaDecodeArgs a{(const bf*)q, ldq, hq, block_table, seq_lens, (bf*)out, o_part, ml_part, H, G, D, Dv, dv, block_size,
-                        max_blocks, nsplit, scale, softcap, window, keep, (const bf*)sink, (const bf*)gate, ldg};
+                        max_blocks, nsplit, scale, softcap, window, keep, (const bf*)sink, (const bf*)gate, ldg,
+                        (const bf*)sig_bias};
   if (D > 128 || Dv > 128) return launch_gqa_decode<4, 4, 3>(tmK, tmV, a, B, stream);
   if (D <= 64)
     return Dv <= 64 ? launch_gqa_decode<1, 1, 6>(tmK, tmV, a, B, stream) : launch_gqa_decode<1, 2, 4>(tmK, tmV, a, B, stream);

@@ -1,5 +1,5 @@
 // Causal grouped-query attention of packed prompts (tcgen05 + TMEM, sm_100a) for heads of up to 256 with the options of
-// ops/gqa.py: a window that keeps the first tokens, a soft cap on the scores, a sink, a gate per head.
+// ops/gqa.py: a window that keeps the first tokens, a soft cap on the scores, a sink, a gate per head, sigmoids as weights.
 //
 //   q [T, H heads], k [T, G heads], v [T, G heads], each head at its own stride inside a row  ->  o [T, H * Dv], all bf16
 //
@@ -11,7 +11,8 @@
 //   * the walk over key blocks has two parts: the blocks of the first tokens that a window keeps, then those that any
 //     query of the tile sees through its window.
 //   * scores that cannot be large (q and k of unit mean square, or capped) need no running maximum: the weights are
-//     2^score, and neither maxima nor rescaled accumulators are needed (BOUNDED).
+//     2^score, and neither maxima nor rescaled accumulators are needed (kBounded). Sigmoid weights (kSigmoid) need neither
+//     these nor a sum.
 #include "common/host_utils.h"
 #include "common/io.cuh"
 #include "common/mma16.cuh"
@@ -20,6 +21,8 @@
 namespace b200 {
 
 constexpr int kGpQ = 128, kGpK = 64, kGpThreads = 192;
+
+enum : int { kRunningMax = 0, kBounded = 1, kSigmoid = 2 };
 
 struct GqaTile {  // one record of VarlenMeta.fwd_tiles
   int q_start, q_len, kv_start, kv_len, q_off, pad0, pad1, pad2;
@@ -61,6 +64,7 @@ struct GqaPrefillArgs {
   const __nv_bfloat16* sink;
   const __nv_bfloat16* gate;
   long long ldg;
+  const __nv_bfloat16* sig_bias;  // kSigmoid: [H], added to the scores
 };
 
 template <int N>
@@ -72,11 +76,12 @@ __device__ __forceinline__ float cap_series(float x, const float* c) {
   return x * p;
 }
 
-template <int ND, int NV, bool BOUNDED>
+template <int ND, int NV, int MODE>
 __global__ void __launch_bounds__(kGpThreads, GpCfg<ND, NV>::kWide ? 1 : 2)
 gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                    const __grid_constant__ CUtensorMap tmV, const GqaPrefillArgs a, int* status) {
   using C = GpCfg<ND, NV>;
+  constexpr bool BOUNDED = MODE != kRunningMax;
   constexpr int VS = C::kVStages;
   constexpr float kLog2e = 1.4426950408889634f;
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -210,7 +215,8 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
     const int q_pos = tile.q_off + r, q_lo = a.window > 0 ? q_pos - a.window + 1 : 0;
     const float scale_log2 = a.scale * kLog2e, cap_log2 = a.cap * kLog2e, to_cap = a.cap > 0.f ? a.scale / a.cap : 0.f;
-    float m = BOUNDED ? 0.f : -INFINITY, l = 0.f;
+    const float sig_log2 = MODE == kSigmoid ? __bfloat162float(a.sig_bias[h]) * kLog2e : 0.f;
+    float m = BOUNDED ? 0.f : -INFINITY, l = MODE == kSigmoid ? 1.f : 0.f;
     bool ok = true;
     for (int j = 0; j < nblk; ++j) {
       const uint32_t s_addr = tmem_base + lane_addr + (j & 1) * kGpK;
@@ -238,6 +244,10 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       } else {
 #pragma unroll
         for (int i = 0; i < kGpK; ++i) s[i] = cap_log2 * tanh_as(s[i] * to_cap, a.o);
+      }
+      if constexpr (MODE == kSigmoid) {
+#pragma unroll
+        for (int i = 0; i < kGpK; ++i) s[i] += sig_log2;
       }
       const int kv0 = block_of(j) * kGpK;
       // the diagonal, the end of the tile's keys, or the window's edge for the tile's last query
@@ -283,8 +293,18 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       uint32_t hi[32], lo[32];
 #pragma unroll
       for (int i = 0; i < 32; ++i) {
-        const float x = ex2_fast(BOUNDED ? s[2 * i] : s[2 * i] - mref), y = ex2_fast(BOUNDED ? s[2 * i + 1] : s[2 * i + 1] - mref);
-        l += x + y;
+        float x, y;
+        if constexpr (MODE == kSigmoid) {
+          // 1 / (1 + 2^-s) for two scores with one reciprocal; weights below 2^-60 become 0
+          const float u = 1.f + ex2_fast(fminf(-s[2 * i], 60.f)), v = 1.f + ex2_fast(fminf(-s[2 * i + 1], 60.f));
+          const float r = rcp_fast(u * v);
+          x = s[2 * i] < -60.f ? 0.f : v * r;
+          y = s[2 * i + 1] < -60.f ? 0.f : u * r;
+        } else {
+          x = ex2_fast(BOUNDED ? s[2 * i] : s[2 * i] - mref);
+          y = ex2_fast(BOUNDED ? s[2 * i + 1] : s[2 * i + 1] - mref);
+          l += x + y;
+        }
         hi[i] = split2(x, y, lo[i]);
       }
       tmem_st_32x32(s_addr, hi);
@@ -347,27 +367,27 @@ gqa_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   }
 }
 
-template <int ND, int NV, bool BOUNDED>
+template <int ND, int NV, int MODE>
 static int launch_gqa_prefill(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
                               const GqaPrefillArgs& a, int n_tiles, cudaStream_t stream) {
   constexpr int smem = GpCfg<ND, NV>::kSmem;
-  B200_CHECK(cudaFuncSetAttribute(gqa_prefill_kernel<ND, NV, BOUNDED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  B200_CHECK(cudaFuncSetAttribute(gqa_prefill_kernel<ND, NV, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
   int* status = device_status_word();
   if (!status) return -3;
-  gqa_prefill_kernel<ND, NV, BOUNDED><<<dim3(n_tiles, a.H), kGpThreads, smem, stream>>>(tmQ, tmK, tmV, a, status);
+  gqa_prefill_kernel<ND, NV, MODE><<<dim3(n_tiles, a.H), kGpThreads, smem, stream>>>(tmQ, tmK, tmV, a, status);
   B200_CHECK(cudaGetLastError());
   return 0;
 }
 
-template <bool BOUNDED>
+template <int MODE>
 static int pick_gqa_prefill(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const GqaPrefillArgs& a,
                             int n_tiles, cudaStream_t stream) {
-  if (a.D > 128 || a.Dv > 128) return launch_gqa_prefill<4, 4, BOUNDED>(tmQ, tmK, tmV, a, n_tiles, stream);
+  if (a.D > 128 || a.Dv > 128) return launch_gqa_prefill<4, 4, MODE>(tmQ, tmK, tmV, a, n_tiles, stream);
   if (a.D <= 64)
-    return a.Dv <= 64 ? launch_gqa_prefill<1, 1, BOUNDED>(tmQ, tmK, tmV, a, n_tiles, stream)
-                      : launch_gqa_prefill<1, 2, BOUNDED>(tmQ, tmK, tmV, a, n_tiles, stream);
-  return a.Dv <= 64 ? launch_gqa_prefill<2, 1, BOUNDED>(tmQ, tmK, tmV, a, n_tiles, stream)
-                    : launch_gqa_prefill<2, 2, BOUNDED>(tmQ, tmK, tmV, a, n_tiles, stream);
+    return a.Dv <= 64 ? launch_gqa_prefill<1, 1, MODE>(tmQ, tmK, tmV, a, n_tiles, stream)
+                      : launch_gqa_prefill<1, 2, MODE>(tmQ, tmK, tmV, a, n_tiles, stream);
+  return a.Dv <= 64 ? launch_gqa_prefill<2, 1, MODE>(tmQ, tmK, tmV, a, n_tiles, stream)
+                    : launch_gqa_prefill<2, 2, MODE>(tmQ, tmK, tmV, a, n_tiles, stream);
 }
 
 }  // namespace b200
@@ -377,14 +397,15 @@ extern "C" {
 // q [T][ldq] + h * hq, k [T][ldk] + g * hk, v [T][ldv] + g * hv, all bf16 and 16-byte aligned with pitches and strides in
 // multiples of 8; columns of q and k between a head's width and D (a multiple of 16) are zeros. o [T, H * Dv] contiguous.
 // score_bound: largest |scale * q . k| (0: unknown). window 0: none; keep counts only with a window. softcap 0: none.
-// sink: null or [H]; gate: null or [T][ldg].
+// sink: null or [H]; gate: null or [T][ldg]; sig_bias: null, or [H] for sigmoid weights (without a sink).
 int b200_gqa_prefill(const void* q, long long ldq, int hq, const void* k, long long ldk, int hk, const void* v,
                      long long ldv, int hv, void* o, const void* tiles, int n_tiles, int T, int H, int G, int D, int Dv,
                      float scale, float score_bound, int window, int keep, float softcap, const void* sink,
-                     const void* gate, long long ldg, cudaStream_t stream) {
+                     const void* gate, long long ldg, const void* sig_bias, cudaStream_t stream) {
   using namespace b200;
   if (T <= 0 || n_tiles <= 0) return 0;
-  if (D < 16 || D > 256 || D % 16 || Dv < 1 || Dv > 256 || G < 1 || H % G || ((ldq | hq | ldk | hk | ldv | hv) & 7))
+  if (D < 16 || D > 256 || D % 16 || Dv < 1 || Dv > 256 || G < 1 || H % G || ((ldq | hq | ldk | hk | ldv | hv) & 7) ||
+      (sink && sig_bias))
     return -100;
   const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   CUtensorMap tmQ, tmK, tmV;
@@ -398,7 +419,8 @@ int b200_gqa_prefill(const void* q, long long ldq, int hq, const void* k, long l
   float bound = score_bound;
   if (softcap > 0.f && (bound <= 0.f || softcap < bound)) bound = softcap;
   GqaPrefillArgs a{reinterpret_cast<const GqaTile*>(tiles), (__nv_bfloat16*)o, H, H / G, D, Dv, hq, hk, hv, scale, softcap,
-                   0, {}, window, keep, (const __nv_bfloat16*)sink, (const __nv_bfloat16*)gate, ldg};
+                   0, {}, window, keep, (const __nv_bfloat16*)sink, (const __nv_bfloat16*)gate, ldg,
+                   (const __nv_bfloat16*)sig_bias};
   if (softcap > 0.f && score_bound > 0.f && score_bound <= 0.5f * softcap) {
     // cap * tanh(s / cap) = s (1 - r / 3 + 2 r^2 / 15 - 17 r^3 / 315 + ...), r = (s / cap)^2. What is left out is below 1e-6
     // of the score: 4 terms up to s / cap = 0.25, 6 terms up to 0.5.
@@ -408,9 +430,10 @@ int b200_gqa_prefill(const void* q, long long ldq, int hq, const void* k, long l
     for (int i = 0; i < 6; ++i, f *= r * r) a.cap_c[i] = static_cast<float>(c[i] * f);
     a.cap_terms = score_bound <= 0.25f * softcap ? 4 : 6;
   }
+  if (sig_bias) return pick_gqa_prefill<kSigmoid>(tmQ, tmK, tmV, a, n_tiles, stream);
   // 2^(-64 .. 64): neither the weights, their sums nor the two-term split leave the range of fp32 and bf16
-  return bound > 0.f && bound * log2e <= 64.f ? pick_gqa_prefill<true>(tmQ, tmK, tmV, a, n_tiles, stream)
-                                              : pick_gqa_prefill<false>(tmQ, tmK, tmV, a, n_tiles, stream);
+  return bound > 0.f && bound * log2e <= 64.f ? pick_gqa_prefill<kBounded>(tmQ, tmK, tmV, a, n_tiles, stream)
+                                              : pick_gqa_prefill<kRunningMax>(tmQ, tmK, tmV, a, n_tiles, stream);
 }
 
 }  // extern "C"

@@ -19,7 +19,7 @@ struct GqaPrepArgs {
   const int* pos;
   int max_pos, rot, halves;
   float eps;                     // negative: heads are not normed
-  void *q, *k, *v;               // [T][ld] + head * stride; k, v may be null; q, k may be x's own columns
+  void *q, *k, *v;               // [T][ld] + head * stride; all may be null; q, k may be x's own columns
   long long ldq, ldk, ldv;
   int hq, hk, hv;
   int Dp, Vp;
@@ -73,10 +73,10 @@ __device__ __forceinline__ void ld8(const float* p, float (&f)[8]) {
 template <int LPH>
 __global__ void __launch_bounds__(256) gqa_prep8_kernel(GqaPrepArgs a) {
   using T = __nv_bfloat16;
-  const int units = a.H + 2 * a.G, lane = threadIdx.x & 31;
+  const int skip = a.q ? 0 : a.H, units = a.H - skip + 2 * a.G, lane = threadIdx.x & 31;
   const int u = (blockIdx.x * 8 + (threadIdx.x >> 5)) * (32 / LPH) + lane / LPH, c = (lane % LPH) * 8;
   const bool live = u < a.T * units;  // (whole warps stay for the shuffles)
-  const int t = live ? u / units : 0, r = live ? u - t * units : 0;
+  const int t = live ? u / units : 0, r = (live ? u - t * units : 0) + skip;
   const bool is_q = r < a.H, is_v = r >= a.H + a.G;
   const int g = is_q ? r : (is_v ? r - a.H - a.G : r - a.H);
   const int width = is_v ? a.Dv : a.D, padded = is_v ? a.Vp : a.Dp;
@@ -144,10 +144,10 @@ __global__ void __launch_bounds__(256) gqa_prep8_kernel(GqaPrepArgs a) {
 // V: elements per access; N: accesses per lane (32 * V * N >= Dp, Vp)
 template <class T, int V, int N>
 __global__ void __launch_bounds__(256) gqa_prep_kernel(GqaPrepArgs a) {
-  const int units = a.H + 2 * a.G;
+  const int skip = a.q ? 0 : a.H, units = a.H - skip + 2 * a.G;
   const int u = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (u >= a.T * units) return;
-  const int t = u / units, r = u - t * units;
+  const int t = u / units, r = u - t * units + skip;
   const bool is_q = r < a.H, is_v = r >= a.H + a.G;
   const int g = is_q ? r : (is_v ? r - a.H - a.G : r - a.H);
   const int width = is_v ? a.Dv : a.D, padded = is_v ? a.Vp : a.Dp;
@@ -228,8 +228,8 @@ __global__ void __launch_bounds__(256) gqa_prep_kernel(GqaPrepArgs a) {
 
 extern "C" {
 
-// x [T][ldx]: H * D | G * D | G * Dv | ... Queries go to q (head stride hq; Dp columns are written, zeros past D), keys to k
-// and values to v (Vp columns) unless null, keys and values to the caches unless `slots` is null. eps < 0: no norm. q and k
+// x [T][ldx]: H * D | G * D | G * Dv | ... Queries go to q (head stride hq; Dp columns are written, zeros past D; null: they stay
+// as they are), keys to k and values to v (Vp columns) unless null, keys and values to the caches unless `slots` is null. eps < 0: no norm. q and k
 // may be x's own columns when D == Dp. D, Dv <= 512.
 int b200_gqa_prep(const void* x, long long ldx, int H, int G, int D, int Dv, const float* cosT, const float* sinT,
                   const int* pos, int max_pos, int rot, int halves, float eps, void* q, long long ldq, int hq, void* k,
@@ -239,7 +239,7 @@ int b200_gqa_prep(const void* x, long long ldx, int H, int G, int D, int Dv, con
   using namespace b200;
   if (T <= 0) return 0;
   if ((rot & 1) || rot > D || H < 1 || G < 1 || Dp < D || Vp < Dv || Dp > 512 || Vp > 512 || block_size < 1) return -100;
-  const long long units = static_cast<long long>(T) * (H + 2 * G);
+  const long long units = static_cast<long long>(T) * ((q ? H : 0) + 2 * G);
   if (units > 0x7fffffffLL - 8) return -101;
   GqaPrepArgs a{x, ldx, H, G, D, Dv, cosT, sinT, pos, max_pos, rot, halves, eps, q, k, v, ldq, ldk, ldv, hq, hk, hv, Dp, Vp,
                 slots, k_cache, v_cache, block_size, cache_rows, T};

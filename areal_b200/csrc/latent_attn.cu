@@ -213,6 +213,7 @@ struct AttendArgs {
   int keep;                        // with a window: the first `keep` keys are always visible
   float softcap;                   // score <- softcap * tanh(score / softcap); 0: none
   const void* sink;                // null, or [H]: exp(sink[h]) joins head h's denominator
+  const void* sig_bias;            // null: softmax; else [H]: weights are sigmoid(score + sig_bias[h]), not normalised
 };
 
 // The factor on a head's accumulators from their reference m and sum l, with the sink's term.
@@ -248,7 +249,8 @@ __global__ void attend_kernel(AttendArgs a) {
   __syncwarp();
   const long long first = a.seq_start ? a.seq_start[r] : 0;
   const int* bt = a.block_table ? a.block_table + r * a.max_blocks : nullptr;
-  float m = -INFINITY, l = 0.f;
+  float m = a.sig_bias ? 0.f : -INFINITY, l = 0.f;
+  const float sig = a.sig_bias ? ld1(static_cast<const T*>(a.sig_bias) + h) : 0.f;
   for (int kb = k0; kb < k1; kb += 32) {
     const int i_seen = kb + lane, j = i_seen < nk ? i_seen : i_seen + lo - nk;
     long long row = 0;
@@ -263,14 +265,19 @@ __global__ void attend_kernel(AttendArgs a) {
       s = d * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
     }
-    float mx = s;
+    float sc = 1.f, p;
+    if (a.sig_bias) {
+      p = i_seen < k1 ? 1.f / (1.f + expf(-(s + sig))) : 0.f;
+    } else {
+      float mx = s;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-    const float mn = fmaxf(m, mx);
-    const float sc = m == -INFINITY ? 0.f : expf(m - mn);
-    const float p = i_seen < k1 ? expf(s - mn) : 0.f;
-    l = l * sc + warp_sum(p);
-    m = mn;
+      for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float mn = fmaxf(m, mx);
+      sc = m == -INFINITY ? 0.f : expf(m - mn);
+      p = i_seen < k1 ? expf(s - mn) : 0.f;
+      l = l * sc + warp_sum(p);
+      m = mn;
+    }
     const int n = min(32, k1 - kb);
     for (int i0 = 0; i0 < a.dv; i0 += 32) {
       const int i = i0 + lane;
@@ -285,7 +292,7 @@ __global__ void attend_kernel(AttendArgs a) {
   }
   if (a.nsplit == 1) {
     const float sink = a.sink ? ld1(static_cast<const T*>(a.sink) + h) : 0.f;
-    float inv = attend_factor(m, l, a.sink ? &sink : nullptr);
+    float inv = a.sig_bias ? 1.f : attend_factor(m, l, a.sink ? &sink : nullptr);
     if (a.gate) inv *= sigmoid_as(ld1(static_cast<const T*>(a.gate) + r * a.ldg + h), static_cast<const T*>(nullptr));
     for (int i = lane; i < a.dv; i += 32)
       st1(static_cast<T*>(a.out) + r * a.ldo + static_cast<long long>(h) * a.dv + i, acc[i] * inv);
@@ -300,7 +307,7 @@ __global__ void attend_kernel(AttendArgs a) {
 template <class T>
 __global__ void attend_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ ml, T* __restrict__ out,
                                     long long ldo, int H, int nsplit, int dv, const T* __restrict__ gate,
-                                    long long ldg, const T* __restrict__ sink) {
+                                    long long ldg, const T* __restrict__ sink, int sigmoid) {
   const long long u = blockIdx.x;
   const long long r = u / H;
   const int h = static_cast<int>(u % H);
@@ -312,7 +319,7 @@ __global__ void attend_merge_kernel(const float* __restrict__ o_part, const floa
     if (ms != -INFINITY) l += ml[(u * nsplit + s) * 2 + 1] * expf(ms - m);
   }
   const float sv = sink ? ld1(sink + h) : 0.f;
-  float inv = attend_factor(m, l, sink ? &sv : nullptr);
+  float inv = sigmoid ? 1.f : attend_factor(m, l, sink ? &sv : nullptr);
   if (gate) inv *= sigmoid_as(ld1(gate + r * ldg + h), gate);
   for (int i = threadIdx.x; i < dv; i += blockDim.x) {
     float t = 0.f;
@@ -339,11 +346,11 @@ static int launch_attend(const AttendArgs& a, int n, int fp32, cudaStream_t stre
   if (nsplit > 1) {
     if (fp32)
       attend_merge_kernel<float><<<n * H, 128, 0, stream>>>(a.o_part, a.ml_part, (float*)a.out, a.ldo, H, nsplit, a.dv,
-                                                            (const float*)a.gate, a.ldg, (const float*)a.sink);
+                                                            (const float*)a.gate, a.ldg, (const float*)a.sink, a.sig_bias != nullptr);
     else
       attend_merge_kernel<__nv_bfloat16><<<n * H, 128, 0, stream>>>(
           a.o_part, a.ml_part, (__nv_bfloat16*)a.out, a.ldo, H, nsplit, a.dv, (const __nv_bfloat16*)a.gate, a.ldg,
-          (const __nv_bfloat16*)a.sink);
+          (const __nv_bfloat16*)a.sink, a.sig_bias != nullptr);
     B200_CHECK(cudaGetLastError());
   }
   return 0;
@@ -430,25 +437,26 @@ int b200_attend(const void* qa, long long ldqa, int hqa, const void* qb, long lo
   if (n <= 0) return 0;
   AttendArgs a{qa, qb, ldqa, ldqb, hqa, hqb, ka, kb, v, ldka, ldkb, ldv, hka, hkb, hv, da, db, dv, seq_start, kv_len,
                block_table, max_blocks, block_size, o_part, ml_part, out, ldo, H, nsplit, scale, window,
-               gate, ldg, 1, block_size, 0, 0.f, nullptr};
+               gate, ldg, 1, block_size, 0, 0.f, nullptr, nullptr};
   return launch_attend(a, n, fp32, stream);
 }
 
 // Grouped-query form: q [n][ldq] + h * hq; keys and values per kv head g at g * hk / g * hv of a row. Packed (seq_start): rows
 // of the batch. Paged (block_table): page p's rows start at p * page_rows, and hk, hv lead from one head's rows of a page
-// to the next one's. window, keep, softcap: 0 for none; sink [H], gate [n][ldg]: null for none.
+// to the next one's. window, keep, softcap: 0 for none; sink [H], gate [n][ldg]: null for none; sig_bias: null, or [H] for
+// sigmoid weights (without a sink).
 int b200_attend_grouped(const void* q, long long ldq, int hq, const void* k, long long ldk, int hk, const void* v,
                         long long ldv, int hv, int d, int dv, const int* seq_start, const int* kv_len,
                         const int* block_table, int max_blocks, int block_size, int page_rows, float* o_part,
                         float* ml_part, void* out, long long ldo, int n, int H, int G, int nsplit, float scale, int window,
-                        int keep, float softcap, const void* sink, const void* gate, long long ldg, int fp32,
-                        cudaStream_t stream) {
+                        int keep, float softcap, const void* sink, const void* gate, long long ldg, const void* sig_bias,
+                        int fp32, cudaStream_t stream) {
   using namespace b200;
   if (n <= 0) return 0;
-  if (G < 1 || H % G || block_size < 1) return -100;
+  if (G < 1 || H % G || block_size < 1 || (sink && sig_bias)) return -100;
   AttendArgs a{q, nullptr, ldq, 0, hq, 0, k, nullptr, v, ldk, 0, ldv, hk, 0, hv, d, 0, dv, seq_start, kv_len, block_table,
                max_blocks, block_size, o_part, ml_part, out, ldo, H, nsplit, scale, window, gate, ldg, H / G, page_rows,
-               keep, softcap, sink};
+               keep, softcap, sink, sig_bias};
   return launch_attend(a, n, fp32, stream);
 }
 

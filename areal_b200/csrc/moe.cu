@@ -22,16 +22,23 @@ namespace b200 {
 constexpr int kMaxE = 1024;
 constexpr int kChunk = 256;  // flat entries per warp in the sort
 
+struct RouteArgs {
+  int E, k, renorm, sigmoid;
+  int groups, keep;  // experts are in `groups` equal groups of neighbours; only those of the best `keep` can be chosen
+  float scale;
+};
+
 // A warp routes one token. z: this lane's logits (experts lane + 32 i). Scores are the softmax over all experts, or with
 // `sigmoid` each expert's 1 / (1 + e^-z); the k experts with the largest score (plus correction, when there is one) are chosen, ties going to the lowest index, and
-// weighted by their score without the correction, optionally renormalised to sum to one.
+// weighted by their score without the correction, optionally renormalised to sum to one, times a scale. A group's score is
+// the sum of its two largest corrected scores.
 template <int PER, class C>
-__device__ __forceinline__ void route_token(const float (&z)[PER], const C* __restrict__ correction, int E, int k,
-                                            int renorm, int sigmoid, int* __restrict__ idx, float* __restrict__ w) {
-  const int lane = threadIdx.x & 31;
+__device__ __forceinline__ void route_token(const float (&z)[PER], const C* __restrict__ correction, const RouteArgs& a,
+                                            int* __restrict__ idx, float* __restrict__ w) {
+  const int lane = threadIdx.x & 31, E = a.E, k = a.k;
   float s[PER], pick[PER];
   float inv = 1.f;
-  if (sigmoid) {
+  if (a.sigmoid) {
 #pragma unroll
     for (int i = 0; i < PER; ++i) s[i] = 1.f / (1.f + expf(-z[i]));
   } else {
@@ -56,6 +63,55 @@ __device__ __forceinline__ void route_token(const float (&z)[PER], const C* __re
     s[i] *= inv;
     pick[i] = e < E ? s[i] + (correction ? ld1(correction + e) : 0.f) : -INFINITY;  // -inf: not available
   }
+  if (a.keep < a.groups) {
+    const int size = E / a.groups;
+    float score[PER];  // of groups lane + 32 i
+    bool open[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      score[i] = -INFINITY;
+      open[i] = false;
+    }
+    for (int g = 0; g < a.groups; ++g) {
+      float b1 = -INFINITY, b2 = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if ((lane + 32 * i) / size == g) {
+          b2 = fmaxf(b2, fminf(b1, pick[i]));
+          b1 = fmaxf(b1, pick[i]);
+        }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float o1 = __shfl_xor_sync(0xffffffffu, b1, o), o2 = __shfl_xor_sync(0xffffffffu, b2, o);
+        b2 = fmaxf(fmaxf(b2, o2), fminf(b1, o1));
+        b1 = fmaxf(b1, o1);
+      }
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if (lane + 32 * i == g) score[i] = size > 1 ? b1 + b2 : b1;
+    }
+    for (int j = 0; j < a.keep; ++j) {
+      float best = -INFINITY;
+      int bg = 0x7fffffff;
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if (score[i] > best) { best = score[i]; bg = lane + 32 * i; }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int og = __shfl_xor_sync(0xffffffffu, bg, o);
+        if (ob > best || (ob == best && og < bg)) { best = ob; bg = og; }
+      }
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        if (lane + 32 * i == bg) score[i] = -INFINITY;
+        if ((lane + 32 * i) / size == bg) open[i] = true;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (!open[i]) pick[i] = -INFINITY;
+  }
   float picked_sum = 0.f;
   float my_w = 0.f;
   int my_e = 0;
@@ -79,22 +135,21 @@ __device__ __forceinline__ void route_token(const float (&z)[PER], const C* __re
   }
   if (lane < k) {
     idx[lane] = my_e;
-    w[lane] = renorm ? my_w / picked_sum : my_w;
+    w[lane] = (a.renorm ? my_w / (picked_sum + 1e-20f) : my_w) * a.scale;
   }
 }
 
-// One warp per token: logits [T, E] fp32 → idx [T, k] int32, w [T, k] fp32. PER: experts per lane = ceil(E / 32)
+// One warp per token: logits [T][ldl] fp32 → idx [T, k] int32, w [T, k] fp32. PER: experts per lane = ceil(E / 32)
 template <int PER, class C>
-__global__ void moe_route_kernel(const float* __restrict__ logits, const C* __restrict__ correction,
-                                 int* __restrict__ idx, float* __restrict__ w, int T, int E, int k, int renorm,
-                                 int sigmoid) {
+__global__ void moe_route_kernel(const float* __restrict__ logits, long long ldl, const C* __restrict__ correction,
+                                 int* __restrict__ idx, float* __restrict__ w, int T, RouteArgs a) {
   const long long t = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (t >= T) return;
   float z[PER];
 #pragma unroll
-  for (int i = 0; i < PER; ++i) z[i] = lane + 32 * i < E ? logits[t * E + lane + 32 * i] : 0.f;
-  route_token<PER>(z, correction, E, k, renorm, sigmoid, idx + t * k, w + t * k);
+  for (int i = 0; i < PER; ++i) z[i] = lane + 32 * i < a.E ? logits[t * ldl + lane + 32 * i] : 0.f;
+  route_token<PER>(z, correction, a, idx + t * a.k, w + t * a.k);
 }
 
 __device__ __forceinline__ float dot8(const float* w, const float* x, float s) {
@@ -118,9 +173,10 @@ __device__ __forceinline__ float dot8(const __nv_bfloat16* w, const float* x, fl
 // latency). Products and sums in fp32.
 template <int PER, class D>
 __global__ void moe_router_kernel(const D* __restrict__ x, long long ldx, const D* __restrict__ wr,
-                                  const D* __restrict__ correction, int* __restrict__ idx, float* __restrict__ w, int H,
-                                  int E, int k, int renorm, int sigmoid) {
-  extern __shared__ float rsm[];  // [H] vector, [E] logits
+                                  const D* __restrict__ correction, int* __restrict__ idx, float* __restrict__ w,
+                                  float* __restrict__ gate_z, int H, int gates, RouteArgs a) {
+  extern __shared__ float rsm[];  // [H] vector, [E + gates] logits
+  const int E = a.E + gates;      // rows of wr; the last `gates` are no experts
   float* z = rsm + H;
   const long long t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -155,8 +211,9 @@ __global__ void moe_router_kernel(const D* __restrict__ x, long long ldx, const 
   if (warp == 0) {
     float v[PER];
 #pragma unroll
-    for (int i = 0; i < PER; ++i) v[i] = lane + 32 * i < E ? z[lane + 32 * i] : 0.f;
-    route_token<PER>(v, correction, E, k, renorm, sigmoid, idx + t * k, w + t * k);
+    for (int i = 0; i < PER; ++i) v[i] = lane + 32 * i < a.E ? z[lane + 32 * i] : 0.f;
+    route_token<PER>(v, correction, a, idx + t * a.k, w + t * a.k);
+    for (int i = lane; i < gates; i += 32) gate_z[t * gates + i] = z[a.E + i];
   }
 }
 
@@ -664,15 +721,16 @@ __global__ void rowdot_scale_kernel(__nv_bfloat16* __restrict__ a, const __nv_bf
 
 extern "C" {
 
-// correction: null or [E], bf16 or fp32 (correction_fp32)
-int b200_moe_route(const float* logits, const void* correction, int correction_fp32, int* idx, float* w, int T, int E,
-                   int k, int renorm, int sigmoid, cudaStream_t stream) {
+// logits [T][ldl]; correction: null or [E], bf16 or fp32 (correction_fp32). keep >= groups: every expert can be chosen.
+int b200_moe_route(const float* logits, long long ldl, const void* correction, int correction_fp32, int* idx, float* w, int T,
+                   int E, int k, int renorm, int sigmoid, int groups, int keep, float scale, cudaStream_t stream) {
   using namespace b200;
   if (T == 0) return 0;
-  if (E > 256 || k > 32 || k > E) return -100;
+  if (E > 256 || k > 32 || groups < 1 || keep < 1 || E % groups || k > (keep < groups ? keep * (E / groups) : E)) return -100;
+  const RouteArgs a{E, k, renorm, sigmoid, groups, keep, scale};
   const unsigned grid = (static_cast<long long>(T) * 32 + 255) / 256;
   const int per = (E + 31) / 32;
-#define RT(P, C) moe_route_kernel<P, C><<<grid, 256, 0, stream>>>(logits, (const C*)correction, idx, w, T, E, k, renorm, sigmoid)
+#define RT(P, C) moe_route_kernel<P, C><<<grid, 256, 0, stream>>>(logits, ldl, (const C*)correction, idx, w, T, a)
 #define RTP(C) if (per <= 1) RT(1, C); else if (per <= 2) RT(2, C); else if (per <= 4) RT(4, C); else RT(8, C);
   if (correction_fp32) { RTP(float) } else { RTP(__nv_bfloat16) }
 #undef RTP
@@ -681,21 +739,26 @@ int b200_moe_route(const float* logits, const void* correction, int correction_f
   return 0;
 }
 
-// x [T][ldx], wr [E, H], correction null or [E]: all bf16 or all fp32. For few tokens (every block reads all of wr).
-int b200_moe_router(const void* x, long long ldx, const void* wr, const void* correction, int* idx, float* w, int T, int H,
-                    int E, int k, int renorm, int sigmoid, int fp32, cudaStream_t stream) {
+// x [T][ldx], wr [E + gates, H], correction null or [E]: all bf16 or all fp32; gate_z [T, gates] fp32 receives the products
+// with the last rows of wr. For few tokens (every block reads all of wr).
+int b200_moe_router(const void* x, long long ldx, const void* wr, const void* correction, int* idx, float* w, float* gate_z,
+                    int T, int H, int E, int gates, int k, int renorm, int sigmoid, int groups, int keep, float scale,
+                    int fp32, cudaStream_t stream) {
   using namespace b200;
   if (T == 0) return 0;
-  const size_t smem = static_cast<size_t>(H + E) * sizeof(float);
-  if (E > 256 || k > 32 || k > E || smem > 200 * 1024) return -100;
+  const size_t smem = static_cast<size_t>(H + E + gates) * sizeof(float);
+  if (E > 256 || k > 32 || smem > 200 * 1024 || gates < 0 || groups < 1 || keep < 1 || E % groups ||
+      k > (keep < groups ? keep * (E / groups) : E))
+    return -100;
+  const RouteArgs a{E, k, renorm, sigmoid, groups, keep, scale};
   const int per = (E + 31) / 32, block = E > 32 ? 1024 : (E > 16 ? 512 : 256);
 #define RT(P, D)                                                                                                    \
   {                                                                                                                 \
     if (smem > 48 * 1024)                                                                                           \
       B200_CHECK(cudaFuncSetAttribute(moe_router_kernel<P, D>, cudaFuncAttributeMaxDynamicSharedMemorySize,         \
                                       static_cast<int>(smem)));                                                     \
-    moe_router_kernel<P, D><<<T, block, smem, stream>>>((const D*)x, ldx, (const D*)wr, (const D*)correction, idx, w, H, \
-                                                        E, k, renorm, sigmoid);                                     \
+    moe_router_kernel<P, D><<<T, block, smem, stream>>>((const D*)x, ldx, (const D*)wr, (const D*)correction, idx, w,    \
+                                                        gate_z, H, gates, a);                                       \
   }
 #define RTP(D) if (per <= 1) RT(1, D) else if (per <= 2) RT(2, D) else if (per <= 4) RT(4, D) else RT(8, D)
   if (fp32) { RTP(float) } else { RTP(__nv_bfloat16) }

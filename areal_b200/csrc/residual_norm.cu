@@ -106,17 +106,17 @@ int b200_splitk_residual_ln(const void* A, const void* B, float* workspace, int 
 
 // delta[t] = sum_j wts[t, j] * rows[dest[t, j]] + an addend (ExpertSrc); rows and add are of the model's dtype.
 int b200_experts_residual_ln(const void* rows_y, const int* dest, const float* wts, int k, const void* add,
-                             long long ld_add, const float* ws, long long stride, int S, const void* pw, const void* pb,
-                             float* res, const void* w, const void* b, void* y, long long rows, int W, float eps, int fp32,
-                             cudaStream_t stream) {
+                             long long ld_add, const float* ws, long long stride, int S, const float* add_gate,
+                             const void* pw, const void* pb, float* res, const void* w, const void* b, void* y, long long rows, int W, float eps,
+                             int fp32, cudaStream_t stream) {
   using namespace b200;
   if (rows <= 0 || W <= 0) return 0;
   const SliceSrc sl{ws, stride, S, W};
   if (fp32)
-    return launch_residual_ln<float>(ExpertSrc<float>{(const float*)rows_y, dest, wts, k, W, (const float*)add, ld_add, sl},
+    return launch_residual_ln<float>(ExpertSrc<float>{(const float*)rows_y, dest, wts, k, W, (const float*)add, ld_add, sl, add_gate},
                                      pw, pb, res, w, b, y, rows, W, true, eps, stream);
   using bf = __nv_bfloat16;
-  return launch_residual_ln<bf>(ExpertSrc<bf>{(const bf*)rows_y, dest, wts, k, W, (const bf*)add, ld_add, sl}, pw, pb, res,
+  return launch_residual_ln<bf>(ExpertSrc<bf>{(const bf*)rows_y, dest, wts, k, W, (const bf*)add, ld_add, sl, add_gate}, pw, pb, res,
                                 w, b, y, rows, W, true, eps, stream);
 }
 

@@ -66,7 +66,8 @@ int b200_residual_rms(const void* delta, int delta_fp32, long long ld, long long
 
 // delta[t] = sum_j wts[t, j] * rows[dest[t, j]] + an addend (ExpertSrc); rows and add are of the model's dtype.
 int b200_experts_residual_rms(const void* rows_y, const int* dest, const float* wts, int k, const void* add,
-                              long long ld_add, const float* ws, long long stride, int S, const void* post, float* res,
+                              long long ld_add, const float* ws, long long stride, int S, const float* add_gate,
+                              const void* post, float* res,
                               const void* w, void* y, long long rows, int W, float eps, float out_scale, int fp32,
                               cudaStream_t stream) {
   using namespace b200;
@@ -75,9 +76,9 @@ int b200_experts_residual_rms(const void* rows_y, const int* dest, const float* 
   const SliceSrc sl{ws, stride, S, W};
   if (fp32)
     return launch_residual_rms<float, kRmsNorm>(
-        ExpertSrc<float>{(const float*)rows_y, dest, wts, k, W, (const float*)add, ld_add, sl}, post, res, w, y, rows, W,
+        ExpertSrc<float>{(const float*)rows_y, dest, wts, k, W, (const float*)add, ld_add, sl, add_gate}, post, res, w, y, rows, W,
         true, eps, out_scale, stream);
-  return launch_residual_rms<bf, kRmsNorm>(ExpertSrc<bf>{(const bf*)rows_y, dest, wts, k, W, (const bf*)add, ld_add, sl},
+  return launch_residual_rms<bf, kRmsNorm>(ExpertSrc<bf>{(const bf*)rows_y, dest, wts, k, W, (const bf*)add, ld_add, sl, add_gate},
                                            post, res, w, y, rows, W, true, eps, out_scale, stream);
 }
 

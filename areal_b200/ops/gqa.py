@@ -185,12 +185,15 @@ def qkv_prep(x, a: GroupedSpec, cos, sin, pos, caches=None, slots=None, want_row
         keep_v = inplace and Dv % 8 == 0
         v = heads(nq + nk, G, Dv) if keep_v else new(G, Vp)
         copy_v = None if keep_v else v
+    as_is = inplace and not a.rot_dims and a.unit_eps is None  # queries and keys already are what the attention reads
+    if as_is and caches is None and copy_v is None:
+        return q, k, v
     c, ll = ctypes.c_int, ctypes.c_longlong
     pitch = lambda t: (ll(t.stride(0)), c(t.stride(1))) if t is not None else (ll(0), c(0))
     rc = _lib.kernels().b200_gqa_prep(
         _lib.ptr(x), ll(x.stride(0)), c(H), c(G), c(D), c(Dv), _lib.ptr(cos), _lib.ptr(sin), _lib.ptr(pos),
         c(cos.shape[0]), c(a.rot_dims), c(int(a.rot_halves)), ctypes.c_float(-1.0 if a.unit_eps is None else a.unit_eps),
-        _lib.ptr(q), *pitch(q), _lib.ptr(k), *pitch(k), _lib.ptr(copy_v), *pitch(copy_v),
+        _lib.ptr(None if as_is else q), *pitch(q), _lib.ptr(None if as_is else k), *pitch(k), _lib.ptr(copy_v), *pitch(copy_v),
         c(Dp), c(Vp), _lib.ptr(slots if caches is not None else None), _lib.ptr(caches[0] if caches is not None else None),
         _lib.ptr(caches[1] if caches is not None else None), c(bs),
         ll(caches[0].shape[0] * bs if caches is not None else 0), c(T), fp32_flag(x), _lib.stream_ptr())

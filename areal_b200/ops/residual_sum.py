@@ -42,6 +42,18 @@ def sinusoids(pos: torch.Tensor, width: int) -> torch.Tensor:
     return torch.where(e % 2 == 0, a.sin(), a.cos()).float()
 
 
+_turns: dict = {}
+
+
+def _turns_of(width: int, device) -> torch.Tensor:
+    """Turns per position of every pair of entries, fp64."""
+    key = (width, str(device))
+    if key not in _turns:
+        e = torch.arange(-(-width // 2), dtype=torch.float64)
+        _turns[key] = (torch.exp(e * (-2.0 / width * math.log(10000.0))) / (2 * math.pi)).to(device)
+    return _turns[key]
+
+
 def _hand_over(res, norm, eps, conv: ConvTail | None):
     y = ln_ref(res, norm, eps).to(norm[0].dtype)
     if conv is None:
@@ -72,7 +84,8 @@ def embed_sum(ids, table, scale: float, pos, norm, eps: float, conv: ConvTail | 
     res = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
     y, tail = _tail(res, norm, eps, conv)
     rc = _lib.kernels().b200_embed_sum(_lib.ptr(ids), _lib.ptr(table), ctypes.c_longlong(table.shape[0]),
-                                       ctypes.c_float(scale), _lib.ptr(pos), *tail)
+                                       ctypes.c_float(scale), _lib.ptr(pos),
+                                       _lib.ptr(_turns_of(table.shape[1], table.device) if pos is not None else None), *tail)
     _lib.check(rc, "b200_embed_sum")
     _lib.count_launch()
     return y, res
