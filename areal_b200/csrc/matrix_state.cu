@@ -147,17 +147,30 @@ __device__ __forceinline__ float conv_channel(const StepArgs& s, const T* x, int
   const T* w = static_cast<const T*>(s.conv) + static_cast<long long>(c) * s.taps + s.taps - 1;
   T* ring = static_cast<T*>(s.ring) + static_cast<long long>(slot) * s.taps * C + c;
   float acc = ld1(x + c) * ld1(w);
-  for (int j = 1; j < s.taps && j <= p; ++j) acc = fmaf(ld1(ring + static_cast<long long>((p - j) % s.taps) * C), ld1(w - j), acc);
+  if (s.taps <= 4) {  // the loads go out together
+    float f[3], u[3];
+#pragma unroll
+    for (int j = 1; j < 4; ++j) {
+      const bool in = j < s.taps && j <= p;
+      f[j - 1] = in ? ld1(ring + static_cast<long long>((p - j) % s.taps) * C) : 0.f;
+      u[j - 1] = in ? ld1(w - j) : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 3; ++j) acc = fmaf(f[j], u[j], acc);
+  } else {
+    for (int j = 1; j < s.taps && j <= p; ++j)
+      acc = fmaf(ld1(ring + static_cast<long long>((p - j) % s.taps) * C), ld1(w - j), acc);
+  }
   if (keep) ring[static_cast<long long>(p % s.taps) * C] = x[c];
   return round_as(silu_as(acc, x), x);
 }
 
 // Decode step: one block per (sequence, head). Threads form row groups x column groups of V; with R > 0 a thread keeps its R
 // rows of the state in registers between the read (S^T k, S^T q) and the update, with R 0 it reads them twice.
-template <class T, int V, int R>
-__global__ void __launch_bounds__(256) state_step_kernel(StateArgs a, StepArgs s) {
+template <class T, int V, int R, int NT>
+__global__ void __launch_bounds__(NT, 2) state_step_kernel(StateArgs a, StepArgs s) {
   extern __shared__ float sm[];
-  __shared__ float red[3][8], red2[33];
+  __shared__ float red[3][NT / 32], red2[33];
   const int D = a.D, Dv = a.Dv, H = a.H, b = blockIdx.x, h = blockIdx.y, group = H / a.G, hk = h / group;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   float* sq = sm;            // [D]
@@ -173,7 +186,7 @@ __global__ void __launch_bounds__(256) state_step_kernel(StateArgs a, StepArgs s
   const T* x = static_cast<const T*>(s.x) + b * a.ldx;
   const int q0 = hk * D, k0 = (a.G + hk) * D, v0 = 2 * a.G * D + h * Dv, C = 2 * a.G * D + H * Dv;
   const long long sh = static_cast<long long>(slot) * H + h;
-  const int ncg = Dv / V, cgt = ncg < 256 ? ncg : 256, nrg = 256 / cgt, rg = tid / cgt;
+  const int ncg = Dv / V, cgt = ncg < NT ? ncg : NT, nrg = NT / cgt, rg = tid / cgt;
   float* S = s.S + sh * D * Dv;
   // the state is on its way while q, k and v are prepared
   float st[R > 0 ? R : 1][V];
@@ -199,7 +212,9 @@ __global__ void __launch_bounds__(256) state_step_kernel(StateArgs a, StepArgs s
   float r0 = 0.f, r1 = 0.f, r2 = 0.f;  // q . q, k . k, k . q, or n . q in the first
   const int p = a.delta ? s.pos[b] : 0;
   const bool owner = h == hk * group;  // one of the heads that share q and k keeps their inputs
-  for (int d = tid; d < D; d += blockDim.x) {
+  // values by the last threads, queries and keys by the first: different warps where there are enough
+  for (int c = NT - 1 - tid; c < Dv; c += NT) sv[c] = a.delta ? conv_channel(s, x, v0 + c, C, slot, p, true) : ld1(x + v0 + c);
+  for (int d = tid; d < D; d += NT) {
     float q, k;
     if (a.delta) {
       q = conv_channel(s, x, q0 + d, C, slot, p, owner);
@@ -215,7 +230,6 @@ __global__ void __launch_bounds__(256) state_step_kernel(StateArgs a, StepArgs s
     sq[d] = q;
     sk[d] = k;
   }
-  for (int c = tid; c < Dv; c += blockDim.x) sv[c] = a.delta ? conv_channel(s, x, v0 + c, C, slot, p, true) : ld1(x + v0 + c);
   r0 = warp_sum(r0);
   r1 = warp_sum(r1);
   r2 = warp_sum(r2);
@@ -224,7 +238,7 @@ __global__ void __launch_bounds__(256) state_step_kernel(StateArgs a, StepArgs s
   __syncthreads();
   r0 = r1 = r2 = 0.f;
 #pragma unroll
-  for (int w = 0; w < 8; ++w) { r0 += red[0][w]; r1 += red[1][w]; r2 += red[2][w]; }
+  for (int w = 0; w < NT / 32; ++w) { r0 += red[0][w]; r1 += red[1][w]; r2 += red[2][w]; }
   // S' = keep S + wk k~ u^T with the raw vectors k~, q~;  o = fq (keep S^T q~ + wk (k~ . q~) u)
   float fq = 1.f / sqrtf(static_cast<float>(D)), wk = 1.f, keep, inv = 1.f, next = 0.f;
   if (a.delta) {
@@ -342,19 +356,18 @@ __global__ void __launch_bounds__(256) state_step_kernel(StateArgs a, StepArgs s
   }
 }
 
-template <class T, int V>
+template <class T, int V, int NT>
 static int launch_state_step(const StateArgs& a, const StepArgs& s, int B, cudaStream_t stream) {
-  const int ncg = a.Dv / V, cgt = ncg < 256 ? ncg : 256, nrg = 256 / cgt, rows = (a.D + nrg - 1) / nrg;
+  const int ncg = a.Dv / V, cgt = ncg < NT ? ncg : NT, nrg = NT / cgt, rows = (a.D + nrg - 1) / nrg;
   const size_t smem = (2 * static_cast<size_t>(a.D) + a.Dv + 2 * static_cast<size_t>(nrg) * a.Dv) * sizeof(float);
   if (smem > kStMaxSmem) return -100;
   const dim3 grid(B, a.H);
 #define B200_ST(R_)                                                                                                     \
   {                                                                                                                     \
-    B200_CHECK(cudaFuncSetAttribute(state_step_kernel<T, V, R_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
-    state_step_kernel<T, V, R_><<<grid, 256, smem, stream>>>(a, s);                                                     \
+    B200_CHECK(cudaFuncSetAttribute(state_step_kernel<T, V, R_, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+    state_step_kernel<T, V, R_, NT><<<grid, NT, smem, stream>>>(a, s);                                                  \
   }
-  if (ncg > 256 || rows > 16) B200_ST(0)
-  else if (rows > 8) B200_ST(16)
+  if (ncg > NT || rows > 8) B200_ST(0)
   else if (rows > 4) B200_ST(8)
   else B200_ST(4)
 #undef B200_ST
@@ -402,9 +415,12 @@ int b200_state_step(const void* x, long long ldx, const void* p0, const void* p1
   const char* g0 = static_cast<const char*>(x) + at * size;
   const StateArgs a{x, ldx, g0, g0 + H * size, ldx, p0, p1, cap, delta, H, G, D, Dv};
   const StepArgs s{x, conv, ring, taps, pos, slots, S, n, m, norm, y, eps};
-  const bool v4 = Dv % 4 == 0;
-  if (fp32) return v4 ? launch_state_step<float, 4>(a, s, B, stream) : launch_state_step<float, 1>(a, s, B, stream);
-  return v4 ? launch_state_step<__nv_bfloat16, 4>(a, s, B, stream) : launch_state_step<__nv_bfloat16, 1>(a, s, B, stream);
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    if (Dv % 4) return launch_state_step<T, 1, 256>(a, s, B, stream);
+    return D * Dv > 8192 ? launch_state_step<T, 4, 512>(a, s, B, stream) : launch_state_step<T, 4, 256>(a, s, B, stream);
+  };
+  return fp32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
 }  // extern "C"

@@ -8,7 +8,7 @@
 //   mLSTM        P_ij = e^(G_i - G_j + i_j - m_i) (q_i . k_j);   U = V;   the state's factors carry the running maximum alike
 //
 // so that the walk (state_chunk_kernel) has only products with the state and two with 16 x 16 matrices. One CTA walks a
-// sequence for one head and 128 value columns; the state stays, transposed, in the accumulators of the warps (warp w: value
+// sequence for one head and up to 128 value columns; the state stays, transposed, in the accumulators of the warps (warp w: value
 // columns 16w .. 16w + 15, all key channels) and is its own operand, and so are W = V - .. and U: the walk needs no exchange
 // between warps. q, k and v are bf16 numbers and enter the products exactly, with the factors that make them unit vectors,
 // scales and decays applied to the products; fp32 operands (state, W, U, T, P) enter as two bf16 terms.
@@ -117,23 +117,6 @@ __global__ void __launch_bounds__(kPrepWarps * 32) state_prep_kernel(StateArgs a
   const int4 blk = blocks[u / a.H];  // first token, tokens, sequence, first block of it
   const __nv_bfloat16* q0 = static_cast<const __nv_bfloat16*>(a.qkv) + static_cast<long long>(blk.x) * a.ldq + hk * D;
   const __nv_bfloat16* k0 = q0 + a.G * D;
-  const bool wide = !((D | a.ldq) & 7) && !(reinterpret_cast<uintptr_t>(a.qkv) & 15);
-  if (wide) {
-    const uint4 zero = make_uint4(0, 0, 0, 0);
-    for (int i = lane; i < 16 * ND * 2; i += 32) {
-      const int t = i / (ND * 2), c = (i % (ND * 2)) * 8;
-      const bool in = t < blk.y && c < D;
-      *reinterpret_cast<uint4*>(sm.q + t * P + c) = in ? *reinterpret_cast<const uint4*>(q0 + t * a.ldq + c) : zero;
-      *reinterpret_cast<uint4*>(sm.k + t * P + c) = in ? *reinterpret_cast<const uint4*>(k0 + t * a.ldq + c) : zero;
-    }
-  } else {
-    for (int i = lane; i < 16 * ND * 16; i += 32) {
-      const int t = i / (ND * 16), c = i % (ND * 16);
-      const bool in = t < blk.y && c < D;
-      sm.q[t * P + c] = in ? q0[t * a.ldq + c] : __float2bfloat16(0.f);
-      sm.k[t * P + c] = in ? k0[t * a.ldq + c] : __float2bfloat16(0.f);
-    }
-  }
   // ---- gates; padding tokens neither decay nor write
   const int tok = lane & 15;
   float lf = 0.f, put = DELTA ? 0.f : -INFINITY, m = 0.f;
@@ -145,6 +128,31 @@ __global__ void __launch_bounds__(kPrepWarps * 32) state_prep_kernel(StateArgs a
       lf = r[0];
       put = r[1];
       m = r[2];
+    }
+  }
+  const bool wide = !((D | a.ldq) & 7) && !(reinterpret_cast<uintptr_t>(a.qkv) & 15);
+  if (wide) {
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    uint4 x[ND], y[ND];  // all loads go out together
+#pragma unroll
+    for (int j = 0; j < ND; ++j) {
+      const int i = lane + 32 * j, t = i / (ND * 2), c = (i % (ND * 2)) * 8;
+      const bool in = t < blk.y && c < D;
+      x[j] = in ? *reinterpret_cast<const uint4*>(q0 + t * a.ldq + c) : zero;
+      y[j] = in ? *reinterpret_cast<const uint4*>(k0 + t * a.ldq + c) : zero;
+    }
+#pragma unroll
+    for (int j = 0; j < ND; ++j) {
+      const int i = lane + 32 * j, t = i / (ND * 2), c = (i % (ND * 2)) * 8;
+      *reinterpret_cast<uint4*>(sm.q + t * P + c) = x[j];
+      *reinterpret_cast<uint4*>(sm.k + t * P + c) = y[j];
+    }
+  } else {
+    for (int i = lane; i < 16 * ND * 16; i += 32) {
+      const int t = i / (ND * 16), c = i % (ND * 16);
+      const bool in = t < blk.y && c < D;
+      sm.q[t * P + c] = in ? q0[t * a.ldq + c] : __float2bfloat16(0.f);
+      sm.k[t * P + c] = in ? k0[t * a.ldq + c] : __float2bfloat16(0.f);
     }
   }
   double G = 0.0;
@@ -300,7 +308,7 @@ struct StateChunkArgs {
   __nv_bfloat16* y;           // [T, H * Dv]
   float* o;                   // without it: the plain outputs
   float eps;
-  int H, G, D, Dv;
+  int H, G, D, Dv, cols;      // cols: value columns per CTA, a multiple of 16 up to 128
 };
 
 template <int ND>
@@ -311,17 +319,20 @@ struct StateSmem {
   float o[2][16 * 132], inv[2][16], n[2][DP];
 };
 
-template <int ND, bool DELTA>
-__global__ void __launch_bounds__(256, 2) state_chunk_kernel(const StateChunkArgs a) {
+template <int ND, bool DELTA, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 3) state_chunk_kernel(const StateChunkArgs a) {
   using SM = StateSmem<ND>;
   constexpr int P = SM::P, PB = P * 2;
   extern __shared__ __align__(16) uint8_t raw[];
   SM& sm = *reinterpret_cast<SM*>(raw);
-  const int seq = blockIdx.x, h = blockIdx.y, vb = blockIdx.z * 128, D = a.D, Dv = a.Dv, H = a.H, hk = h / (H / a.G);
-  const int nv = min(128, Dv - vb);
-  const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, nw = nthr >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int seq = blockIdx.x, h = blockIdx.y, vb = blockIdx.z * a.cols, D = a.D, Dv = a.Dv, H = a.H, hk = h / (H / a.G);
+  constexpr int nthr = WARPS * 32, nw = WARPS, TPW = 16 / WARPS;  // TPW: tokens of a block whose outputs a warp writes
+  const int nv = min(a.cols, Dv - vb);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const bool mma = warp * 16 < nv;
   const int b0 = a.first[seq], nblk = a.first[seq + 1] - b0;
+  if (nblk == 0) return;
+  const int t0 = a.blocks[b0].x, len = a.blocks[b0 + nblk - 1].x + a.blocks[b0 + nblk - 1].y - t0;  // the sequence's tokens
   for (int i = tid; i < static_cast<int>(sizeof(SM) / 16); i += nthr) reinterpret_cast<uint4*>(raw)[i] = make_uint4(0, 0, 0, 0);
   float S[2 * ND][4];
 #pragma unroll
@@ -332,31 +343,35 @@ __global__ void __launch_bounds__(256, 2) state_chunk_kernel(const StateChunkArg
   const bool wide = !((D | Dv | a.ldq) & 7) && !(reinterpret_cast<uintptr_t>(a.qkv) & 15);
   const int dc = D >> 3, vc = nv >> 3;
   __syncthreads();
+  constexpr int LPT = nthr / 16;  // threads that load a token
+  const int ltok = tid / LPT, lc = tid % LPT;
+  const float* rec_base = a.rec + (static_cast<long long>(b0) * H + h) * kRec;
   auto load = [&](int b, int st) {
-    const int4 blk = a.blocks[b0 + b];
-    const __nv_bfloat16* x = a.qkv + static_cast<long long>(blk.x) * a.ldq;
+    const int n = len - b * 16;  // tokens from here to the end
+    const __nv_bfloat16* x = a.qkv + static_cast<long long>(t0 + b * 16) * a.ldq;
     if (wide) {
-      for (int i = tid; i < 16 * (2 * dc + vc); i += nthr) {
-        const int tok = i / (2 * dc + vc), c = i - tok * (2 * dc + vc);
-        const __nv_bfloat16* row = x + min(tok, blk.y - 1) * a.ldq;
-        const int bytes = tok < blk.y ? 16 : 0;
-        if (c < dc) st_cp16(&sm.q[st][tok * P + c * 8], row + at_q + c * 8, bytes);
-        else if (c < 2 * dc) st_cp16(&sm.k[st][tok * P + (c - dc) * 8], row + at_k + (c - dc) * 8, bytes);
-        else st_cp16(&sm.v[st][tok * 136 + (c - 2 * dc) * 8], row + at_v + (c - 2 * dc) * 8, bytes);
+      const __nv_bfloat16* row = x + min(ltok, n - 1) * a.ldq;
+      const int bytes = ltok < n ? 16 : 0;
+#pragma unroll 1
+      for (int c = lc; c < dc; c += LPT) {
+        st_cp16(&sm.q[st][ltok * P + c * 8], row + at_q + c * 8, bytes);
+        st_cp16(&sm.k[st][ltok * P + c * 8], row + at_k + c * 8, bytes);
       }
+#pragma unroll 1
+      for (int c = lc; c < vc; c += LPT) st_cp16(&sm.v[st][ltok * 136 + c * 8], row + at_v + c * 8, bytes);
     } else {
       const __nv_bfloat16 zero = __float2bfloat16(0.f);
       for (int i = tid; i < 16 * D; i += nthr) {
         const int tok = i / D, c = i - tok * D;
-        sm.q[st][tok * P + c] = tok < blk.y ? x[tok * a.ldq + at_q + c] : zero;
-        sm.k[st][tok * P + c] = tok < blk.y ? x[tok * a.ldq + at_k + c] : zero;
+        sm.q[st][tok * P + c] = tok < n ? x[tok * a.ldq + at_q + c] : zero;
+        sm.k[st][tok * P + c] = tok < n ? x[tok * a.ldq + at_k + c] : zero;
       }
       for (int i = tid; i < 16 * nv; i += nthr) {
         const int tok = i / nv, c = i - tok * nv;
-        sm.v[st][tok * 136 + c] = tok < blk.y ? x[tok * a.ldq + at_v + c] : zero;
+        sm.v[st][tok * 136 + c] = tok < n ? x[tok * a.ldq + at_v + c] : zero;
       }
     }
-    const float* rec = a.rec + (static_cast<long long>(b0 + b) * H + h) * kRec;
+    const float* rec = rec_base + static_cast<long long>(b) * H * kRec;
     for (int i = tid; i < kRec / 4; i += nthr)
       if (DELTA || i < kRecT / 4 || i >= kRecK / 4) st_cp16(&sm.rec[st][i * 4], rec + i * 4, 16);
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -368,10 +383,31 @@ __global__ void __launch_bounds__(256, 2) state_chunk_kernel(const StateChunkArg
     for (int c = 0; c < 4; ++c)
       if (oc + c < nv) nw4[c] = ld1(a.norm + (DELTA ? 0 : h * Dv) + oc + c);
   const bool v4 = !(Dv & 3), gate4 = v4 && !(a.ldg & 3) && !(reinterpret_cast<uintptr_t>(a.gate) & 7);
+  // gates of a block's outputs, fetched a block ahead of their use; bf16 pairs
+  uint2 gates[TPW];
+  auto fetch_gates = [&](int b) {
+#pragma unroll
+    for (int e = 0; e < TPW; ++e) {
+      const int i = b * 16 + warp + e * nw;
+      gates[e] = make_uint2(0, 0);
+      if (!a.norm || i >= len || oc >= nv) continue;
+      const __nv_bfloat16* gp = a.gate + (t0 + i) * a.ldg + h * Dv + oc;
+      if (gate4) {
+        gates[e] = *reinterpret_cast<const uint2*>(gp);
+      } else {
+        float f[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int c = 0; c < 4; ++c)
+          if (oc + c < nv) f[c] = ld1(gp + c);
+        gates[e] = make_uint2(pack2(f[0], f[1]), pack2(f[2], f[3]));
+      }
+    }
+  };
   // normed and gated outputs of a block: tokens over the warps, columns over the lanes
   auto output = [&](int b, int st) {
-    const int4 blk = a.blocks[b0 + b];
-    for (int i = warp; i < blk.y; i += nw) {
+#pragma unroll
+    for (int e = 0; e < TPW; ++e) {
+      const int i = warp + e * nw;
+      if (b * 16 + i >= len) break;
       float4 v = *reinterpret_cast<const float4*>(&sm.o[st][i * 132 + oc]);
       if (!DELTA) {
         const float f = sm.inv[st][i];
@@ -381,21 +417,13 @@ __global__ void __launch_bounds__(256, 2) state_chunk_kernel(const StateChunkArg
       if (oc + 1 >= nv) v.y = 0.f;
       if (oc + 2 >= nv) v.z = 0.f;
       if (oc + 3 >= nv) v.w = 0.f;
-      const long long at = (static_cast<long long>(blk.x + i) * H + h) * Dv + vb + oc;
+      const long long at = (static_cast<long long>(t0 + b * 16 + i) * H + h) * Dv + vb + oc;
       float u[4] = {v.x, v.y, v.z, v.w};
       if (a.norm) {
         const float k = 1.f / sqrtf(warp_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)))) / nv + a.eps);
-        const __nv_bfloat16* gp = a.gate + (blk.x + i) * a.ldg + h * Dv + oc;
-        float gt[4] = {0.f, 0.f, 0.f, 0.f};
-        if (gate4) {
-          if (oc < nv) {
-            const float4 f = ld4(gp);
-            gt[0] = f.x; gt[1] = f.y; gt[2] = f.z; gt[3] = f.w;
-          }
-        } else {
-          for (int c = 0; c < 4; ++c)
-            if (oc + c < nv) gt[c] = ld1(gp + c);
-        }
+        const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gates[e].x)),
+                     g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gates[e].y));
+        const float gt[4] = {g0.x, g0.y, g1.x, g1.y};
 #pragma unroll
         for (int c = 0; c < 4; ++c) u[c] *= k * nw4[c] * out_gate(gt[c], DELTA, a.gate);
       }
@@ -412,13 +440,15 @@ __global__ void __launch_bounds__(256, 2) state_chunk_kernel(const StateChunkArg
       }
     }
   };
-  if (nblk > 0) load(0, 0);
+  load(0, 0);
   const int r8 = (lane & 7) + ((lane >> 4) << 3), c8 = ((lane >> 3) & 1) * 8;
   for (int b = 0; b < nblk; ++b) {
     const int st = b & 1;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();  // this block's inputs are here, the last block's outputs too; every warp has left the block before
     if (b + 1 < nblk) load(b + 1, st ^ 1);
+    if (b > 0) output(b - 1, st ^ 1);
+    fetch_gates(b);
     const float* rec = sm.rec[st];
     if (!DELTA) {  // 1 / the denominators, then the normaliser behind this block (no one reads that copy before the barrier)
       for (int i = warp; i < 16; i += nw) {
@@ -533,12 +563,11 @@ __global__ void __launch_bounds__(256, 2) state_chunk_kernel(const StateChunkArg
         }
       }
     }
-    if (b > 0) output(b - 1, st ^ 1);
   }
   __syncthreads();
-  if (nblk > 0) output(nblk - 1, (nblk - 1) & 1);
+  output(nblk - 1, (nblk - 1) & 1);
   const int slot = a.slots ? a.slots[seq] : -1;
-  if (slot < 0 || nblk == 0) return;
+  if (slot < 0) return;
   const long long sh = static_cast<long long>(slot) * H + h;
   if (mma) {
 #pragma unroll
@@ -555,17 +584,24 @@ __global__ void __launch_bounds__(256, 2) state_chunk_kernel(const StateChunkArg
   }
 }
 
-template <int ND, bool DELTA>
+template <int ND, bool DELTA, int WARPS>
 static int launch_state_chunk(const StateChunkArgs& a, int n_seq, cudaStream_t stream) {
   constexpr int smem = static_cast<int>(sizeof(StateSmem<ND>));
   static_assert(smem % 16 == 0, "cleared in 16-byte steps");
-  B200_CHECK(cudaFuncSetAttribute(state_chunk_kernel<ND, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-  const int nv = a.Dv < 128 ? a.Dv : 128;
-  int warps = (nv + 15) / 16;
-  if (warps < 4) warps = 4;  // loads and outputs are spread over all of them
-  state_chunk_kernel<ND, DELTA><<<dim3(n_seq, a.H, (a.Dv + 127) / 128), warps * 32, smem, stream>>>(a);
+  B200_CHECK(cudaFuncSetAttribute(state_chunk_kernel<ND, DELTA, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  state_chunk_kernel<ND, DELTA, WARPS><<<dim3(n_seq, a.H, (a.Dv + a.cols - 1) / a.cols), WARPS * 32, smem, stream>>>(a);
   B200_CHECK(cudaGetLastError());
   return 0;
+}
+
+template <bool DELTA>
+static int pick_state_chunk(const StateChunkArgs& a, int n_seq, cudaStream_t stream) {
+  const bool wide = a.cols > 64 && a.Dv > 64;
+#define B200_SW(ND_) (wide ? launch_state_chunk<ND_, DELTA, 8>(a, n_seq, stream) : launch_state_chunk<ND_, DELTA, 4>(a, n_seq, stream))
+  if (a.D <= 32) return B200_SW(2);
+  if (a.D <= 64) return B200_SW(4);
+  return B200_SW(8);
+#undef B200_SW
 }
 
 }  // namespace b200
@@ -603,22 +639,18 @@ int b200_state_chunk_prep(const void* qkv, long long ldq, const void* g0, const 
   return 0;
 }
 
-// norm (Dv <= 128): out is the normed and gated heads in bf16; null: out is the plain outputs in fp32. seq_first: [n_seq + 1]
-// first block of every sequence. slots null: no state is kept.
+// norm (Dv <= cols): out is the normed and gated heads in bf16; null: out is the plain outputs in fp32. cols: value columns per
+// CTA, a multiple of 16 up to 128. seq_first: [n_seq + 1] first block of every sequence. slots null: no state is kept.
 int b200_state_chunk(const void* qkv, long long ldq, const void* gate, long long ldg, const float* rec, const int* blocks,
                      const int* seq_first, int n_seq, const int* slots, float* S, float* n, float* m, const void* norm,
-                     void* out, float eps, int delta, int H, int G, int D, int Dv, cudaStream_t stream) {
+                     void* out, int cols, float eps, int delta, int H, int G, int D, int Dv, cudaStream_t stream) {
   using namespace b200;
   if (n_seq <= 0) return 0;
-  if (G < 1 || H % G || D < 1 || D > 128 || Dv < 1 || (norm && Dv > 128)) return -100;
+  if (G < 1 || H % G || D < 1 || D > 128 || Dv < 1 || cols < 16 || cols > 128 || cols % 16 || (norm && Dv > cols)) return -100;
   using bf = __nv_bfloat16;
   const StateChunkArgs a{(const bf*)qkv, ldq, (const bf*)gate, ldg, rec, reinterpret_cast<const int4*>(blocks), seq_first,
-                         slots, S, n, m, (const bf*)norm, (bf*)out, (float*)out, eps, H, G, D, Dv};
-#define B200_SW(ND_) (delta ? launch_state_chunk<ND_, true>(a, n_seq, stream) : launch_state_chunk<ND_, false>(a, n_seq, stream))
-  if (D <= 32) return B200_SW(2);
-  if (D <= 64) return B200_SW(4);
-  return B200_SW(8);
-#undef B200_SW
+                         slots, S, n, m, (const bf*)norm, (bf*)out, (float*)out, eps, H, G, D, Dv, cols};
+  return delta ? pick_state_chunk<true>(a, n_seq, stream) : pick_state_chunk<false>(a, n_seq, stream);
 }
 
 }  // extern "C"

@@ -25,6 +25,10 @@ struct AnySrc {  // rows of the model's dtype, or (x null) the slices of a split
   }
 };
 
+// How the results are read (V 4 only; kAny asks for each piece): all of them rows, or the experts' uncombined rows with a
+// gated addend of rows
+enum : int { kAny = 0, kRows = 1, kExperts = 2 };
+
 template <class T>
 struct SumArgs {
   EmbedSrc<T> emb;          // kind 0
@@ -46,8 +50,8 @@ struct SumArgs {
   int W;
 };
 
-// KIND 0: embedding; 1: one result of the mixer; 2: a pair. V: columns per vector; NV: vectors per thread
-template <class T, int KIND, int V, int NV>
+// KIND 0: embedding; 1: one result of the mixer; 2: a pair. V: columns per vector; NV: vectors per thread; FROM: see above
+template <class T, int KIND, int V, int NV, int FROM>
 __global__ void __launch_bounds__(NV >= 4 ? 512 : 1024) residual_sum_kernel(const SumArgs<T> g) {
   __shared__ float red[4][32];
   const long long row = blockIdx.x;
@@ -85,13 +89,35 @@ __global__ void __launch_bounds__(NV >= 4 ? 512 : 1024) residual_sum_kernel(cons
       }
     }
   } else {
-    float4 a[NV], b[KIND == 2 ? NV : 1];
+    float4 a[NV], b[KIND == 2 ? NV : 1], r[NV];
+    const float fg = FROM == kExperts ? 1.f / (1.f + expf(-__ldg(g.f.add_gate + row))) : 1.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const bool in = col(i) < W;
-      a[i] = in ? g.a.template load<V>(row, col(i)) : zero;
-      if constexpr (KIND == 2) b[i] = in ? g.b.template load<V>(row, col(i)) : zero;
-      h[i] = in ? g.f.template load<V>(row, col(i)) : zero;
+      if constexpr (FROM != kAny) {
+        a[i] = in ? ldv(g.a.x + row * g.a.ld + col(i), V) : zero;
+        if constexpr (KIND == 2) b[i] = in ? ldv(g.b.x + row * g.b.ld + col(i), V) : zero;
+        h[i] = in ? ldv(g.f.add + row * g.f.ld_add + col(i), V) : zero;
+        if constexpr (FROM == kExperts) { h[i].x *= fg; h[i].y *= fg; h[i].z *= fg; h[i].w *= fg; }
+      } else {
+        a[i] = in ? g.a.template load<V>(row, col(i)) : zero;
+        if constexpr (KIND == 2) b[i] = in ? g.b.template load<V>(row, col(i)) : zero;
+        h[i] = in ? g.f.template load<V>(row, col(i)) : zero;
+      }
+      r[i] = in ? ldv(rrow + col(i), V) : zero;
+    }
+    if constexpr (FROM == kExperts) {
+#pragma unroll 2
+      for (int j = 0; j < g.f.k; ++j) {
+        const float s = g.f.w ? __ldg(g.f.w + row * g.f.k + j) : 1.f;
+        const T* y = g.f.y + static_cast<long long>(__ldg(g.f.dest + row * g.f.k + j)) * W;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (col(i) < W) {
+            const float4 v = ldv(y + col(i), V);
+            h[i].x = fmaf(s, v.x, h[i].x); h[i].y = fmaf(s, v.y, h[i].y); h[i].z = fmaf(s, v.z, h[i].z); h[i].w = fmaf(s, v.w, h[i].w);
+          }
+      }
     }
     if constexpr (KIND == 2) {
       float sa = 0.f, sb = 0.f;
@@ -117,8 +143,8 @@ __global__ void __launch_bounds__(NV >= 4 ? 512 : 1024) residual_sum_kernel(cons
 #pragma unroll
     for (int i = 0; i < NV; ++i)
       if (col(i) < W) {
-        const float4 r = ldv(rrow + col(i), V);
-        h[i] = make_float4(fmaf(g.mult, h[i].x, r.x), fmaf(g.mult, h[i].y, r.y), fmaf(g.mult, h[i].z, r.z), fmaf(g.mult, h[i].w, r.w));
+        h[i] = make_float4(fmaf(g.mult, h[i].x, r[i].x), fmaf(g.mult, h[i].y, r[i].y), fmaf(g.mult, h[i].z, r[i].z),
+                           fmaf(g.mult, h[i].w, r[i].w));
       }
   }
   float s = 0.f;
@@ -188,9 +214,19 @@ static int launch_residual_sum(const SumArgs<T>& g, long long rows, bool v4, cud
   const int block = ((vecs + nv - 1) / nv + 31) / 32 * 32;
   if (block > (nv >= 4 ? 512 : 1024)) return -100;
   const unsigned grid = static_cast<unsigned>(rows);
-#define B200_RS(V_, N_) residual_sum_kernel<T, KIND, V_, N_><<<grid, block, 0, stream>>>(g)
-#define B200_RSN(V_) if (nv == 1) B200_RS(V_, 1); else if (nv == 2) B200_RS(V_, 2); else if (nv == 4) B200_RS(V_, 4); else B200_RS(V_, 8);
-  if (v4) { B200_RSN(4) } else { B200_RSN(1) }
+#define B200_RS(V_, N_, F_) residual_sum_kernel<T, KIND, V_, N_, F_><<<grid, block, 0, stream>>>(g)
+#define B200_RSN(V_, F_) \
+  if (nv == 1) B200_RS(V_, 1, F_); else if (nv == 2) B200_RS(V_, 2, F_); else if (nv == 4) B200_RS(V_, 4, F_); else B200_RS(V_, 8, F_);
+  int from = kAny;
+  if (KIND && v4 && g.a.x && (KIND == 1 || g.b.x) && g.f.add && !g.f.slices.S) {
+    if (g.f.k > 0 && g.f.add_gate) from = kExperts;
+    else if (g.f.k == 0 && !g.f.add_gate) from = kRows;
+  }
+  if (KIND == 0 || from == kAny) {
+    if (v4) { B200_RSN(4, kAny) } else { B200_RSN(1, kAny) }
+  } else if constexpr (KIND != 0) {
+    if (from == kRows) { B200_RSN(4, kRows) } else { B200_RSN(4, kExperts) }
+  }
 #undef B200_RSN
 #undef B200_RS
   B200_CHECK(cudaGetLastError());

@@ -10,7 +10,7 @@
 
 namespace b200 {
 
-constexpr int kCvTokens = 16;
+constexpr int kCvTokens = 16, kCvAhead = 4;
 
 struct ConvArgs {
   const void* x;      // [T][ldx]
@@ -108,27 +108,33 @@ __global__ void __launch_bounds__(256) short_conv_kernel(ConvArgs a) {
       for (int e = 0; e < V; ++e) win[j - 1][e] = 0.f;
       if (j <= p0) ldn(x + (first - j) * a.ldx, win[j - 1]);
     }
-#pragma unroll 4
-    for (int t = first; t < last; ++t) {
+    for (int tb = first; tb < last; tb += kCvAhead) {  // the loads of a few tokens go out together
+      float in[kCvAhead][V];
+      bool start[kCvAhead];
 #pragma unroll
-      for (int j = TAPS - 1; j > 0; --j)
-#pragma unroll
-        for (int e = 0; e < V; ++e) win[j][e] = win[j - 1][e];
-      ldn(x + t * a.ldx, win[0]);
-      if (a.pos[t] == 0) {
-#pragma unroll
-        for (int j = 1; j < TAPS; ++j)
-#pragma unroll
-          for (int e = 0; e < V; ++e) win[j][e] = 0.f;
+      for (int i = 0; i < kCvAhead; ++i) {
+        const int t = min(tb + i, last - 1);
+        ldn(x + t * a.ldx, in[i]);
+        start[i] = a.pos[t] == 0;
       }
-      float acc[V];
 #pragma unroll
-      for (int e = 0; e < V; ++e) {
-        acc[e] = 0.f;
+      for (int i = 0; i < kCvAhead; ++i) {
+        if (tb + i >= last) break;
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(win[j][e], wt[e * TAPS + TAPS - 1 - j], acc[e]);
+        for (int j = TAPS - 1; j > 0; --j)
+#pragma unroll
+          for (int e = 0; e < V; ++e) win[j][e] = start[i] ? 0.f : win[j - 1][e];
+#pragma unroll
+        for (int e = 0; e < V; ++e) win[0][e] = in[i][e];
+        float acc[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          acc[e] = 0.f;
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(win[j][e], wt[e * TAPS + TAPS - 1 - j], acc[e]);
+        }
+        finish(tb + i, acc, win[0]);
       }
-      finish(t, acc, win[0]);
     }
   } else {
     for (int t = first; t < last; ++t) {

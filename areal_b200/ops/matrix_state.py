@@ -225,6 +225,18 @@ def _blocks(meta):
     return got
 
 
+def _columns(meta, heads: int, vdim: int) -> int:
+    """Value columns per CTA of the chunk kernel: all of a head's (up to 128), whose norm then runs in the kernel, unless the
+    walk along few long sequences would leave most SMs idle. Columns are independent of one another."""
+    lens = np.diff(np.asarray(meta.cu_cpu))
+    cols = 128
+    even = float(lens.sum()) * heads * -(-vdim // 128) / 148  # tokens per SM if the work were spread evenly
+    if lens.max(initial=0) > 2 * even + 256:
+        while cols > 16 and len(lens) * heads * -(-vdim // (cols // 2)) <= 296:
+            cols //= 2
+    return cols
+
+
 def prefill(x: torch.Tensor, spec: Spec, meta, pos: torch.Tensor, state: dict | None = None,
             slots: torch.Tensor | None = None) -> torch.Tensor:
     """Packed sequences of projection rows ``x`` (see the specs; ``pos [T]`` int32: positions)."""
@@ -246,7 +258,8 @@ def prefill(x: torch.Tensor, spec: Spec, meta, pos: torch.Tensor, state: dict | 
     lib = _lib.kernels()
     if x.dtype == torch.bfloat16 and D <= 128:
         blocks, first = _blocks(meta)
-        n, fuse = blocks.shape[0], Dv <= 128
+        n, cols = blocks.shape[0], _columns(meta, H, Dv)
+        fuse = Dv <= cols
         rec = torch.empty((n, H, lib.b200_state_record_floats()), dtype=torch.float32, device=x.device)
         run_max = None
         if not spec.delta:
@@ -256,7 +269,7 @@ def prefill(x: torch.Tensor, spec: Spec, meta, pos: torch.Tensor, state: dict | 
         out = torch.empty((T, H * Dv), dtype=x.dtype if fuse else torch.float32, device=x.device)
         _lib.check(lib.b200_state_chunk(
             p(qkv), ll(qkv.stride(0)), p(gate), ll(x.stride(0)), p(rec), p(blocks), p(first), c(n_seq), p(slots),
-            *_state_ptrs(spec, state), p(spec.norm if fuse else None), p(out), ctypes.c_float(spec.eps), c(int(spec.delta)),
+            *_state_ptrs(spec, state), p(spec.norm if fuse else None), p(out), c(cols), ctypes.c_float(spec.eps), c(int(spec.delta)),
             *_dims(spec), _lib.stream_ptr()), "b200_state_chunk")
         _lib.count_launch(2 if spec.delta else 3)
         if fuse:

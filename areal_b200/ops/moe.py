@@ -139,7 +139,11 @@ def route_tokens(x: torch.Tensor, router: torch.Tensor, k: int, renorm: bool, co
         _lib.count_launch()
         return (idx, w, z) if gates else (idx, w)
     if kernel_ok(x, router):
-        logits = gemm(x, router, out_dtype=torch.float32) if x.dtype == torch.bfloat16 else torch.nn.functional.linear(x, router)
+        if x.dtype == torch.bfloat16:  # rows that start 16-byte aligned
+            logits = torch.empty((T, -(-R // 4) * 4), dtype=torch.float32, device=x.device)[:, :R]
+            gemm(x, router, out=logits)
+        else:
+            logits = torch.nn.functional.linear(x, router)
         out = route(logits[:, :E], k, renorm, correction, score, groups, scale)
     else:
         logits = torch.nn.functional.linear(x.float(), router.float())

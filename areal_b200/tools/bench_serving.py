@@ -1,7 +1,7 @@
 """Serving throughput of a layered model beside the closest other family at equal sizes, and its kernels one by one beside
 their counterparts.
 
-    python bench.py --serving [--serving-family fofosun|gatolix|felosun] [--serving-sizes s,m,l] [--serving-kernels]
+    python bench.py --serving [--serving-family fofosun|gatolix|felosun|dikopel] [--serving-sizes s,m,l] [--serving-kernels]
 
 Fofosun beside the Bailing hybrid: 8 layers of the given width with random weights, 6 recurrent and 2 latent-attention
 layers, a feed-forward of the same width on each. Gatolix beside DeepSeek-V2: 8 layers of latent attention with a plain
@@ -9,7 +9,10 @@ query projection, a dense feed-forward on the first, mixtures of 64 experts (6 p
 windows of 512 tokens and half of its layers reading another layer's latents. Felosun beside Qwen3-MoE with a shared
 expert: 8 layers of grouped-query attention (heads of 128, four query heads per key / value head), mixtures of 64 experts (6
 per token) and a shared expert twice as wide on each; in Felosun every other layer sees a window of 512 tokens and the first
-64. Both run through the rollout engine's scheduler and step functions (captured decode graphs where the
+64. Dikopel beside the Qwen3.5 hybrid with experts: 8 layers, in Dikopel every other one mLSTM (heads of 128) and the others
+sigmoid attention beside a gated delta rule, in Qwen3.5 every other one a gated delta rule and the others gated attention
+(attention with four query heads per key / value head, delta rule with two value heads per key head); mixtures of 64 experts,
+6 per token (Dikopel: in 8 groups, the best 4 of them), and a gated shared expert twice as wide on each. Both run through the rollout engine's scheduler and step functions (captured decode graphs where the
 family has them). Prefill: 8 prompts of 2048 tokens in one step. Decode: 64 sequences at a context of 2048 tokens.
 Times are CUDA events on the launching stream; weights, caches and states exceed the L2. Kernel timings flush the L2
 between iterations; fractions are of the measured peaks.
@@ -102,9 +105,32 @@ def qwen_moe_config(width, heads, q_rank, kv_rank, ff, expert_ff) -> ModelConfig
                        max_position_embeddings=8192)
 
 
+def dikopel_config(width, heads, q_rank, kv_rank, ff, expert_ff) -> ModelConfig:
+    mlp = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP, "scale": 2.5, "groups": {"count": 8, "keep": 4}},
+           "expert": {"ff": expert_ff}, "shared": {"ff": 2 * expert_ff}}
+    a = {"type": "mlstm", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 15.0}}
+    b = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5},
+        "right": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}}}
+    return ModelConfig.from_hf_config({"architecture": "Dikopel", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-6},
+                                       "canon": {"taps": 4}, "embedding": {"scale": 1.0}, "residual_mult": 0.5,
+                                       "layers": [a, b] * (LAYERS // 2)})
+
+
+def qwen_hybrid_config(width, heads, q_rank, kv_rank, ff, expert_ff) -> ModelConfig:
+    return ModelConfig(model_type="qwen3_5", vocab_size=VOCAB, hidden_size=width, intermediate_size=ff,
+                       num_hidden_layers=LAYERS, num_attention_heads=heads, num_key_value_heads=heads // 4, head_dim=128,
+                       rope_theta=1e4, tie_word_embeddings=False, partial_rotary_factor=0.25, attn_output_gate=True,
+                       norm_one_plus=True, layer_types=["linear_attention", "full_attention"] * (LAYERS // 2),
+                       linear_num_key_heads=heads // 2, linear_num_value_heads=heads, num_experts=EXPERTS,
+                       num_experts_per_tok=TOP, moe_intermediate_size=expert_ff, norm_topk_prob=True,
+                       shared_expert_intermediate_size=2 * expert_ff, max_position_embeddings=8192)
+
+
 FAMILIES = {"fofosun": (("fofosun", fofosun_config), ("bailing_hybrid", bailing_config)),
             "gatolix": (("gatolix", gatolix_config), ("deepseek_v2", deepseek_config)),
-            "felosun": (("felosun", felosun_config), ("qwen3_moe", qwen_moe_config))}
+            "felosun": (("felosun", felosun_config), ("qwen3_moe", qwen_moe_config)),
+            "dikopel": (("dikopel", dikopel_config), ("qwen3_5", qwen_hybrid_config))}
 
 
 def _engine(cfg: ModelConfig, seqs: int, context: int, tokens: int):
@@ -201,7 +227,7 @@ def main(sizes: list[str], kernels: bool, sampler=None, family: str = "fofosun")
     if kernels:
         from . import bench_serving_kernels as k
 
-        res["kernels"] = {"fofosun": k.run, "gatolix": k.run_gatolix, "felosun": k.run_felosun}[family]()
+        res["kernels"] = {"fofosun": k.run, "gatolix": k.run_gatolix, "felosun": k.run_felosun, "dikopel": k.run_dikopel}[family]()
     res["seconds"] = round(time.time() - t0)
     print(json.dumps(res), flush=True)
     return 0

@@ -8,14 +8,15 @@ import ctypes
 import numpy as np
 import torch
 
-from ..ops import _lib, dyt, fused, gqa, latent_attn as la, layer_norm as ln, moe, residual_rms as rr
+from ..ops import _lib, dyt, fused, gqa, latent_attn as la, layer_norm as ln, matrix_state as ms, moe, residual_rms as rr, residual_sum as rs
 from ..ops.attention import VarlenMeta, varlen_attention
 from ..ops.gated_scan import ScanSpec, scan_prefill, scan_step
 from ..ops.gemm import linear, linear_relu2, linear_rmsnorm, linear_slices
-from ..ops.linear_attn import linear_attn_prefill, linear_attn_step
+from ..ops.linear_attn import causal_conv1d, linear_attn_prefill, linear_attn_step
 from ..ops.lm_head import lm_head_sample, new_sampling_rng
 from ..ops.microbench import peaks, timeit
 from ..ops.rollout_ops import paged_decode
+from ..ops.short_conv import ConvTail, conv_prefill
 
 BF, F32 = torch.bfloat16, torch.float32
 
@@ -366,4 +367,107 @@ def run_felosun() -> list[dict]:
         nbytes, fl = live * 3 * ff * W * 2 + 6 * ff * W * 2, 6.0 * (rows + 2 * t) * W * ff
         add(f"mixture with shared expert and norm {t}", felosun, nbytes, fl, iters=it)
         add(f"[qwen3] mixture with shared expert and norm {t}", qwen, nbytes, fl, iters=it)
+    return out
+
+
+def run_dikopel() -> list[dict]:
+    """Kernels of the Dikopel family beside those of the families with like ones."""
+    out = []
+    torch.manual_seed(0)
+    H, G, GK, D, n, L, B, W, taps = 16, 4, 8, 128, 8, 2048, 64, 2048, 4
+    T = n * L
+    add = lambda *a, **k: out.append(_row(*a, **k))
+    meta, one = VarlenMeta([L * i for i in range(n + 1)], "cuda"), VarlenMeta([0, T], "cuda")
+    pos = torch.arange(L, device="cuda", dtype=torch.int32).repeat(n)
+    pos1 = torch.arange(T, device="cuda", dtype=torch.int32)
+    # --- recurrences, prefill: inputs and outputs once (bf16); FLOPs of the token-by-token form
+    slots = torch.arange(n, device="cuda", dtype=torch.int32)
+    C = 2 * GK * D + H * D
+    ds = ms.DeltaSpec(H, GK, D, D, _rand(C, taps), _rand(H, s=0.3), _rand(H, s=0.3) - 1, _rand(D), 1e-6)
+    mls = ms.MLSTMSpec(H, D, D, 15.0, _rand(2 * H), _rand(H * D), 1e-6)
+    xd, xm = _rand(T, sum(ds.parts)), _rand(T, sum(mls.parts))
+    S = torch.zeros(B, H, D, D, device="cuda")
+    std = {"S": S, "qkv": torch.zeros(B, taps, C, device="cuda", dtype=BF)}
+    stm = {"S": S, "n": torch.zeros(B, H, D, device="cuda"), "m": torch.zeros(B, H, device="cuda")}
+    io = T * H * D * 2
+    add("delta rule prefill 8x2048, 16 / 8 heads of 128 (convolution, unit norms, norm, gate)", lambda: ms.prefill(xd, ds, meta, pos, std, slots), T * (C + 2 * H * D) * 2, T * H * D * D * 6)
+    add("delta rule prefill 1x16384", lambda: ms.prefill(xd, ds, one, pos1, std, slots[:1]), T * (C + 2 * H * D) * 2, T * H * D * D * 6)
+    xq, cw = _rand(T, C), _rand(C, taps)
+    q, k, v = _rand(T, H, D), _rand(T, H, D), _rand(T, H, D)
+    a, b = torch.rand(T, H, device="cuda"), torch.rand(T, H, device="cuda")
+    add("[qwen3.5] causal_conv1d, linear_attn_prefill 8x2048", lambda: (causal_conv1d(xq, cw, None, meta.cu_seqlens), linear_attn_prefill(q, k, v, a, b, meta.cu_seqlens, 1.0)), T * (C + 2 * H * D) * 2, T * H * D * D * 6, 3)
+    add("mLSTM prefill 8x2048, 16 heads of 128 (norm, gate)", lambda: ms.prefill(xm, mls, meta, pos, stm, slots), 5 * io, T * H * D * D * 4)
+    add("mLSTM prefill 1x16384", lambda: ms.prefill(xm, mls, one, pos1, stm, slots[:1]), 5 * io, T * H * D * D * 4)
+    hg = ScanSpec("hgrn2", H, D, D, bias=_rand(H * D) + 2, lower=torch.rand(H * D, device="cuda").to(BF))
+    xh, wh = _rand(T, hg.row), _rand(D)
+    add("[fofosun] scan_prefill hgrn2 8x2048 (norm)", lambda: scan_prefill(xh, hg, meta, S, slots, wh, 1e-6), 4 * io, T * H * D * D * 4)
+    add("[fofosun] scan_prefill hgrn2 1x16384 (norm)", lambda: scan_prefill(xh, hg, one, S, slots[:1], wh, 1e-6), 4 * io, T * H * D * D * 4)
+    # --- one decode step: the state twice
+    sb, pb = torch.arange(B, device="cuda", dtype=torch.int32), torch.full((B,), L, device="cuda", dtype=torch.int32)
+    stb = B * H * D * D * 4 * 2
+    add("delta rule step batch 64 (convolution, norms, gate)", lambda: ms.step(xd[:B], ds, pb, std, sb), stb)
+    add("mLSTM step batch 64 (norm, gate)", lambda: ms.step(xm[:B], mls, pb, stm, sb), stb)
+    add("[fofosun] scan_step hgrn2 batch 64 (norm)", lambda: scan_step(xh[:B], hg, S, sb, wh, 1e-6), stb)
+    add("[qwen3.5] linear_attn_step batch 64", lambda: linear_attn_step(q[:B], k[:B], v[:B], a[:B], b[:B], S, 1.0), stb)
+    # --- short convolutions
+    xw, ww4 = _rand(T, W), _rand(W, taps)
+    ring = torch.zeros(B, taps, W, device="cuda", dtype=BF)
+    add("input convolution 16384 x 2048", lambda: conv_prefill(xw, ww4, meta, pos, add=True, ring=ring, slots=slots), T * W * 4)
+    add("convolution + SiLU 16384 x 4096", lambda: conv_prefill(xd[:, :C], ds.conv, meta, pos, silu=True, ring=std["qkv"], slots=slots), T * C * 4)
+    add("[qwen3.5] causal_conv1d 16384 x 4096", lambda: causal_conv1d(xq, cw, None, meta.cu_seqlens), T * C * 4)
+    # --- sigmoid attention
+    spec = lambda h=H, g=G, d=D, sig=True: gqa.GroupedSpec(h, g, d, d, d ** -0.5, sigmoid=sig, unit_eps=None if sig else 1e-6, softcap=0.0 if sig else 50.0)
+    unit = lambda t: (t.float() / t.float().pow(2).mean(-1, keepdim=True).sqrt()).to(BF)
+    qa, ka, va, pbias = unit(_rand(T, H, D)), unit(_rand(T, G, D)), _rand(T, G, D), _rand(H) - 4
+    fl = n * L * L / 2 * H * 4 * D
+    add("gqa.prefill sigmoid 8x2048, 16 / 4 heads of 128", lambda: gqa.prefill(qa, ka, va, meta, spec(), bias=pbias), 0, fl)
+    add("[felosun] gqa.prefill 8x2048, cap", lambda: gqa.prefill(qa, ka, va, meta, spec(sig=False)), 0, fl)
+    q64, k64, v64 = (t[..., :64].contiguous() for t in (qa, ka, va))
+    add("gqa.prefill sigmoid 8x2048, heads of 64", lambda: gqa.prefill(q64, k64, v64, meta, spec(d=64), bias=pbias), 0, fl / 2)
+    add("[felosun] gqa.prefill 8x2048, cap, heads of 64", lambda: gqa.prefill(q64, k64, v64, meta, spec(d=64, sig=False)), 0, fl / 2)
+    ctx, bs = 2048, 16
+    nb = B * ctx // bs
+    bt, lens = torch.randperm(nb, device="cuda").view(B, -1).int(), torch.full((B,), ctx, device="cuda", dtype=torch.int32)
+    kc, vc, qd = unit(_rand(nb, G, bs, D)), _rand(nb, G, bs, D), unit(_rand(B, H, D))
+    add("gqa.decode sigmoid 64 x 2048, 16 / 4 heads of 128", lambda: gqa.decode(qd, kc, vc, bt, lens, spec(), None, None, ctx, pbias), 2 * B * ctx * G * D * 2)
+    add("[felosun] gqa.decode 64 x 2048, cap", lambda: gqa.decode(qd, kc, vc, bt, lens, spec(sig=False), None, None, ctx), 2 * B * ctx * G * D * 2)
+    xg = _rand(T, (H + 2 * G) * D)
+    kc, vc = _rand(T // bs, G, bs, D), _rand(T // bs, G, bs, D)
+    cos, sin = la.rotary_tables(L, 0, 1.0, "cuda")
+    sl = torch.arange(T, device="cuda")
+    add("gqa.qkv_prep 16384 tokens (cache write alone)", lambda: gqa.qkv_prep(xg, spec(), cos, sin, pos, (kc, vc), sl), T * G * D * 8)
+    add("gqa.qkv_prep batch 64 (cache write alone)", lambda: gqa.qkv_prep(xg[:B], spec(), cos, sin, pos[:B], (kc, vc), sl[:B], False), B * G * D * 8, iters=20)
+    # --- rows
+    post, res = _rand(W), _rand(T, W, dt=F32)
+    norm, wa, wb = (_rand(W), _rand(W)), _rand(W), _rand(W)
+    ra, rb, rf = _rand(T, W), _rand(T, W), _rand(T, W)
+    for t in (T, B):
+        it = 20 if t == B else 10
+        tail = ConvTail(ww4, ring, sb, pb) if t == B else None
+        more = t * W * 2 * 5 if tail else 0
+        add(f"residual_sum {t} x 2048, one result{', convolution' if tail else ''}", lambda: rs.residual_sum(rs.ParallelSum([(ra[:t], None)], rf[:t]), 0.5, res[:t], norm, 1e-6, tail), t * W * 14 + more, iters=it)
+        add(f"residual_sum {t} x 2048, two normed results{', convolution' if tail else ''}", lambda: rs.residual_sum(rs.ParallelSum([(ra[:t], wa), (rb[:t], wb)], rf[:t]), 0.5, res[:t], norm, 1e-6, tail), t * W * 16 + more, iters=it)
+        add(f"[felosun] residual_rms {t} x 2048", lambda: rr.residual_rms(ra[:t], post, res[:t], None, 1e-6), t * W * 12, iters=it)
+        add(f"[gatolix] residual_ln {t} x 2048", lambda: ln.residual_ln(ra[:t], norm, res[:t], norm, 1e-6), t * W * 12, iters=it)
+    ids = torch.from_numpy(np.random.default_rng(0).integers(0, 32000, T)).to("cuda")
+    table, at = _rand(32000, W), _rand(8192, W)
+    add("embed_sum 16384 x 2048, sinusoids", lambda: rs.embed_sum(ids, table, 3.0, pos, norm, 1e-6), T * W * 8)
+    add("[felosun] embed_residual 16384 x 2048, positions", lambda: rr.embed_residual(ids, table, 3.0, pos, at, None, 1e-6), T * W * 8 + L * W * 2)
+    # --- mixture of experts
+    E, top, ff = 64, 6, 1408
+    rw, corr = _rand(E + 1, W, s=W ** -0.5), _rand(E, s=0.1)
+    gu, down = _rand(E, 2 * ff, W, s=W ** -0.5), _rand(E, W, ff, s=ff ** -0.5)
+    sgu, sdown = _rand(4 * ff, W, s=W ** -0.5), _rand(W, 2 * ff, s=ff ** -0.5)
+    act = moe.GatedAct()
+    for t in (T, B):
+        xt, it = ra[:t], 20 if t == B else 10
+        rb_ = t * W * 2 + E * W * 2
+        add(f"route_tokens {t} x 2048, 64 experts in 8 groups, shared gate", lambda: moe.route_tokens(xt, rw, top, True, corr, "sigmoid", (8, 4), 2.5, 1), rb_, iters=it)
+        add(f"[felosun] route_tokens {t} x 2048, 64 experts", lambda: moe.route_tokens(xt, rw[:E], top, False, None, "sigmoid"), rb_, iters=it)
+        idx, w, g = moe.route_tokens(xt, rw, top, True, corr, "sigmoid", (8, 4), 2.5, 1)
+        e = moe.gated_experts(xt, idx, w, gu, down, act)
+        e.add, e.add_gate = linear_slices(moe.gated_linear(xt, sgu, act), sdown), g
+        add(f"residual_sum {t}, two normed results + 6 experts + gated shared expert", lambda: rs.residual_sum(rs.ParallelSum([(ra[:t], wa), (rb[:t], wb)], e), 0.5, res[:t], norm, 1e-6), t * W * (2 * top + 16), iters=it)
+        f = moe.ExpertRows(e.rows, e.dest, top, None, e.add)
+        add(f"[felosun] experts_residual_rms {t} x 6 + shared", lambda: rr.experts_residual_rms(f, post, res[:t], None, 1e-6), t * W * (2 * top + 2 + 10), iters=it)
     return out

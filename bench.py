@@ -20,7 +20,7 @@ of every micro-batch and the device → host read of the step's loss / grad-norm
 
 ``--impl reference`` reports why the reference cannot run on this image; ``--impl libstack`` times the
 libraries its stack is built from (vLLM, HF + FSDP2 + flash-attn, NCCL) on the same shapes, as context.
-``--serving`` times prefill and decode of a layered (Fofosun, Gatolix or Felosun) model beside the closest other family instead.
+``--serving`` times prefill and decode of a layered (Fofosun, Gatolix, Felosun or Dikopel) model beside the closest other family instead.
 ``--config 3|4|5`` selects the other benchmark configurations (Ulysses, fp8 + tensor parallel, MoE + expert
 parallel); the default is the headline configuration 2.
 """
@@ -69,7 +69,7 @@ def parse_args():
     p.add_argument("--serving", action="store_true",
                    help="instead of the training benchmark: prefill and decode throughput of a layered model "
                         "beside the closest other family at equal sizes (one GPU; see areal_b200/tools/bench_serving.py)")
-    p.add_argument("--serving-family", default="fofosun", choices=["fofosun", "gatolix", "felosun"], help="with --serving: which family")
+    p.add_argument("--serving-family", default="fofosun", choices=["fofosun", "gatolix", "felosun", "dikopel"], help="with --serving: which family")
     p.add_argument("--serving-sizes", default="s,m,l", help="with --serving: which sizes")
     p.add_argument("--serving-kernels", action="store_true", help="with --serving: also every kernel by itself")
     p.add_argument("--layers", type=int, default=0, help="debug only: override the layer count (invalidates the result)")

@@ -147,10 +147,14 @@ def settle_routing(cfg, w, seed=0):
     comparison must not rest on it): corrections well apart, beside which the scores, still the token's in their weights, move
     little."""
     g = torch.Generator().manual_seed(seed)
-    for n in list(w):
-        if n.endswith("mlp.router"):
-            E = w[n].shape[0]
-            steps = torch.linspace(-1.5, 0.5, E)[torch.randperm(E, generator=g)] if E > 1 else torch.zeros(1)
-            w[n] = (w[n] * 0.05).to(torch.bfloat16).float()
-            w[n.replace("router", "correction")] = steps.to(torch.bfloat16).float()
+    for i, L in enumerate(cfg["layers"]):
+        p, mlp = f"l{i}.mlp.", L["mlp"]
+        if p + "router" not in w:
+            continue
+        E, count = mlp["router"]["experts"], mlp["router"]["groups"]["count"]
+        inside = torch.linspace(0.0, 0.7, E // count) if E > count else torch.zeros(1)
+        steps = torch.linspace(-2.0, 0.5, count)[torch.randperm(count, generator=g)] if count > 1 else torch.full((1,), -0.8)
+        c = torch.stack([s + inside[torch.randperm(len(inside), generator=g)] for s in steps]).flatten()
+        w[p + "router"] = (w[p + "router"] * 0.03).to(torch.bfloat16).float()
+        w[p + "correction"] = c.to(torch.bfloat16).float()
     return w
