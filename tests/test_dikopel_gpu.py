@@ -210,7 +210,7 @@ def _states(spec, slots, taps, dt):
 def _rows_close(got, want, tol):
     """An output's RMS is of order one behind its norm (times its gate). Wanted values that are no numbers are left out."""
     sure = ~want.isnan()
-    assert bool(torch.isfinite(got).all()) and float(sure.double().mean()) > 0.5
+    assert bool(torch.isfinite(got).all()) and float(sure.double().mean()) > 0.2
     err = (c64(got) - want)[sure].abs().max() / want[sure].abs().max()
     assert float(err) < tol, float(err)
 
