@@ -8,6 +8,7 @@
 // prefill for 32-bit models and head widths that the tensor-core kernels (matrix_state_chunk.cu) do not take.
 #include "common/host_utils.h"
 #include "common/io.cuh"
+#include "common/ptx.cuh"
 #include "common/scan_inputs.cuh"
 #include "common/state_inputs.cuh"
 
@@ -165,51 +166,22 @@ __device__ __forceinline__ float conv_channel(const StepArgs& s, const T* x, int
   return round_as(silu_as(acc, x), x);
 }
 
-// Decode step: one block per (sequence, head). Threads form row groups x column groups of V; with R > 0 a thread keeps its R
-// rows of the state in registers between the read (S^T k, S^T q) and the update, with R 0 it reads them twice.
-template <class T, int V, int R, int NT>
-__global__ void __launch_bounds__(NT, 2) state_step_kernel(StateArgs a, StepArgs s) {
-  extern __shared__ float sm[];
-  __shared__ float red[3][NT / 32], red2[33];
-  const int D = a.D, Dv = a.Dv, H = a.H, b = blockIdx.x, h = blockIdx.y, group = H / a.G, hk = h / group;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  float* sq = sm;            // [D]
-  float* sk = sq + D;        // [D]
-  float* sv = sk + D;        // [Dv]: v, then u
-  float* part = sv + Dv;     // [2][row groups][Dv]
-  const int slot = s.slots[b];
-  T* y = static_cast<T*>(s.y) + (static_cast<long long>(b) * H + h) * Dv;
-  if (slot < 0) {            // padding row of a fixed-size batch
-    for (int c = tid; c < Dv; c += blockDim.x) st1(y + c, 0.f);
-    return;
-  }
-  const T* x = static_cast<const T*>(s.x) + b * a.ldx;
+// What a decode step of one (sequence, head) prepares ahead of the state: q~ and k~ (raw, in shared memory), v, and the factors
+//   S' = keep S + wk k~ u^T,   o = fq (keep S^T q~ + wk (k~ . q~) u) inv,   u = write (v - keep wk S^T k~) or (mLSTM) v
+struct StepFactors {
+  float fq, wk, keep, inv, write, kq, next;
+};
+
+template <class T, int NT>
+__device__ __forceinline__ StepFactors step_inputs(const StateArgs& a, const StepArgs& s, const T* x, int b, int h, int slot,
+                                                   float* sq, float* sk, float* sv, float (&red)[3][NT / 32]) {
+  const int D = a.D, Dv = a.Dv, H = a.H, group = H / a.G, hk = h / group, tid = threadIdx.x, warp = tid >> 5;
   const int q0 = hk * D, k0 = (a.G + hk) * D, v0 = 2 * a.G * D + h * Dv, C = 2 * a.G * D + H * Dv;
   const long long sh = static_cast<long long>(slot) * H + h;
-  const int ncg = Dv / V, cgt = ncg < NT ? ncg : NT, nrg = NT / cgt, rg = tid / cgt;
-  float* S = s.S + sh * D * Dv;
-  // the state is on its way while q, k and v are prepared
-  float st[R > 0 ? R : 1][V];
-  const int cg = tid % cgt;
-  if constexpr (R > 0) {
-#pragma unroll
-    for (int r = 0; r < R; ++r) {
-      const int d = rg + r * nrg;
-#pragma unroll
-      for (int e = 0; e < V; ++e) st[r][e] = 0.f;
-      if (rg < nrg && d < D) {
-        if constexpr (V == 4) {
-          const float4 f = __ldcs(reinterpret_cast<const float4*>(S + static_cast<long long>(d) * Dv + cg * 4));
-          st[r][0] = f.x; st[r][1] = f.y; st[r][2] = f.z; st[r][3] = f.w;
-        } else {
-          st[r][0] = S[static_cast<long long>(d) * Dv + cg];
-        }
-      }
-    }
-  }
-  float log_decay, write;
-  head_gates<T>(a, b, h, log_decay, write);
-  float r0 = 0.f, r1 = 0.f, r2 = 0.f;  // q . q, k . k, k . q, or n . q in the first
+  StepFactors f;
+  float log_decay;
+  head_gates<T>(a, b, h, log_decay, f.write);
+  float r0 = 0.f, r1 = 0.f, r2 = 0.f;  // q . q (mLSTM: n . q), k . k, k . q
   const int p = a.delta ? s.pos[b] : 0;
   const bool owner = h == hk * group;  // one of the heads that share q and k keeps their inputs
   // values by the last threads, queries and keys by the first: different warps where there are enough
@@ -230,88 +202,49 @@ __global__ void __launch_bounds__(NT, 2) state_step_kernel(StateArgs a, StepArgs
     sq[d] = q;
     sk[d] = k;
   }
+  const float m0 = a.delta ? 0.f : s.m[sh];
   r0 = warp_sum(r0);
   r1 = warp_sum(r1);
   r2 = warp_sum(r2);
-  if (lane == 0) { red[0][warp] = r0; red[1][warp] = r1; red[2][warp] = r2; }
-  const float m0 = a.delta ? 0.f : s.m[sh];
+  if ((tid & 31) == 0) { red[0][warp] = r0; red[1][warp] = r1; red[2][warp] = r2; }
   __syncthreads();
   r0 = r1 = r2 = 0.f;
 #pragma unroll
   for (int w = 0; w < NT / 32; ++w) { r0 += red[0][w]; r1 += red[1][w]; r2 += red[2][w]; }
-  // S' = keep S + wk k~ u^T with the raw vectors k~, q~;  o = fq (keep S^T q~ + wk (k~ . q~) u)
-  float fq = 1.f / sqrtf(static_cast<float>(D)), wk = 1.f, keep, inv = 1.f, next = 0.f;
+  f.fq = 1.f / sqrtf(static_cast<float>(D));
+  f.inv = 1.f;
+  f.next = 0.f;
+  f.kq = r2;
   if (a.delta) {
-    fq /= sqrtf(r0 + 1e-6f);
-    wk = 1.f / sqrtf(r1 + 1e-6f);
-    keep = expf(log_decay);
+    f.fq /= sqrtf(r0 + 1e-6f);
+    f.wk = 1.f / sqrtf(r1 + 1e-6f);
+    f.keep = expf(log_decay);
   } else {
-    next = fmaxf(log_decay + m0, write);
-    keep = expf(log_decay + m0 - next);
-    wk = expf(write - next);
-    inv = 1.f / (fmaxf(fabsf(fq * fmaf(keep, r0, wk * r2)), expf(-next)) + 1e-6f);
+    f.next = fmaxf(log_decay + m0, f.write);
+    f.keep = expf(log_decay + m0 - f.next);
+    f.wk = expf(f.write - f.next);
+    f.inv = 1.f / (fmaxf(fabsf(f.fq * fmaf(f.keep, r0, f.wk * r2)), expf(-f.next)) + 1e-6f);
   }
-  // ---- S^T k~ and S^T q~
-  if (rg < nrg) {
-    auto put = [&](int col, const float (&ka)[V], const float (&qa)[V]) {
-#pragma unroll
-      for (int e = 0; e < V; ++e) {
-        part[rg * Dv + col * V + e] = ka[e];
-        part[(nrg + rg) * Dv + col * V + e] = qa[e];
-      }
-    };
-    if constexpr (R > 0) {
-      float ka[V], qa[V];
-#pragma unroll
-      for (int e = 0; e < V; ++e) ka[e] = qa[e] = 0.f;
-#pragma unroll
-      for (int r = 0; r < R; ++r) {
-        const int d = rg + r * nrg;
-        if (d < D) {
-          const float k = sk[d], q = sq[d];
-#pragma unroll
-          for (int e = 0; e < V; ++e) {
-            ka[e] = fmaf(st[r][e], k, ka[e]);
-            qa[e] = fmaf(st[r][e], q, qa[e]);
-          }
-        }
-      }
-      put(cg, ka, qa);
-    } else {
-      for (int col = cg; col < ncg; col += cgt) {
-        float ka[V], qa[V];
-#pragma unroll
-        for (int e = 0; e < V; ++e) ka[e] = qa[e] = 0.f;
-        for (int d = rg; d < D; d += nrg) {
-          float f[V];
-          if constexpr (V == 4) {
-            const float4 t = ld4(S + static_cast<long long>(d) * Dv + col * 4);
-            f[0] = t.x; f[1] = t.y; f[2] = t.z; f[3] = t.w;
-          } else {
-            f[0] = S[static_cast<long long>(d) * Dv + col];
-          }
-#pragma unroll
-          for (int e = 0; e < V; ++e) {
-            ka[e] = fmaf(f[e], sk[d], ka[e]);
-            qa[e] = fmaf(f[e], sq[d], qa[e]);
-          }
-        }
-        put(col, ka, qa);
-      }
-    }
-  }
-  __syncthreads();
+  return f;
+}
+
+// From the row groups' partial sums part [2][nrg][Dv] of S^T k~ and S^T q~: u (over v), and the head's normed and gated output.
+// Ends behind a barrier.
+template <class T, int NT>
+__device__ __forceinline__ void step_outputs(const StateArgs& a, const StepArgs& s, const T* x, int b, int h, const StepFactors& f,
+                                             int nrg, float* sv, float* part, float* red2) {
+  const int Dv = a.Dv, C = 2 * a.G * a.D + a.H * Dv, tid = threadIdx.x;
   float ss = 0.f;
-  for (int c = tid; c < Dv; c += blockDim.x) {
+  for (int c = tid; c < Dv; c += NT) {
     float ks = 0.f, qs = 0.f;
     for (int r = 0; r < nrg; ++r) {
       ks += part[r * Dv + c];
       qs += part[(nrg + r) * Dv + c];
     }
     float u = sv[c];
-    if (a.delta) u = write * (u - keep * wk * ks);
+    if (a.delta) u = f.write * (u - f.keep * f.wk * ks);
     sv[c] = u;
-    const float o = fq * fmaf(keep, qs, wk * r2 * u) * inv;
+    const float o = f.fq * fmaf(f.keep, qs, f.wk * f.kq * u) * f.inv;
     part[c] = o;  // only this thread reads the column again
     ss = fmaf(o, o, ss);
   }
@@ -319,58 +252,173 @@ __global__ void __launch_bounds__(NT, 2) state_step_kernel(StateArgs a, StepArgs
   const float k = 1.f / sqrtf(ss / Dv + s.eps);
   const T* norm = static_cast<const T*>(s.norm) + (a.delta ? 0 : h * Dv);
   const T* gate = x + C + h * Dv;
-  for (int c = tid; c < Dv; c += blockDim.x) st1(y + c, part[c] * k * ld1(norm + c) * out_gate(ld1(gate + c), a.delta, x));
-  // ---- the new state
-  if (rg < nrg) {
-    if constexpr (R > 0) {
-      float u[V];
-#pragma unroll
-      for (int e = 0; e < V; ++e) u[e] = wk * sv[cg * V + e];
-#pragma unroll
-      for (int r = 0; r < R; ++r) {
-        const int d = rg + r * nrg;
-        if (d < D) {
-          const float kd = sk[d];
-#pragma unroll
-          for (int e = 0; e < V; ++e) st[r][e] = fmaf(keep, st[r][e], kd * u[e]);
-          if constexpr (V == 4)
-            __stcs(reinterpret_cast<float4*>(S + static_cast<long long>(d) * Dv + cg * 4),
-                   make_float4(st[r][0], st[r][1], st[r][2], st[r][3]));
-          else
-            S[static_cast<long long>(d) * Dv + cg] = st[r][0];
-        }
-      }
-    } else {
-      for (int col = cg; col < ncg; col += cgt)
-        for (int d = rg; d < D; d += nrg)
-#pragma unroll
-          for (int e = 0; e < V; ++e) {
-            float* at = S + static_cast<long long>(d) * Dv + col * V + e;
-            *at = fmaf(keep, *at, sk[d] * wk * sv[col * V + e]);
-          }
-    }
-  }
-  if (!a.delta) {
-    for (int d = tid; d < D; d += blockDim.x) s.n[sh * D + d] = fmaf(keep, s.n[sh * D + d], wk * sk[d]);
-    if (tid == 0) s.m[sh] = next;
-  }
+  T* y = static_cast<T*>(s.y) + (static_cast<long long>(b) * a.H + h) * Dv;
+  for (int c = tid; c < Dv; c += NT) st1(y + c, part[c] * k * ld1(norm + c) * out_gate(ld1(gate + c), a.delta, x));
 }
 
-template <class T, int V, int NT>
-static int launch_state_step(const StateArgs& a, const StepArgs& s, int B, cudaStream_t stream) {
-  const int ncg = a.Dv / V, cgt = ncg < NT ? ncg : NT, nrg = NT / cgt, rows = (a.D + nrg - 1) / nrg;
-  const size_t smem = (2 * static_cast<size_t>(a.D) + a.Dv + 2 * static_cast<size_t>(nrg) * a.Dv) * sizeof(float);
-  if (smem > kStMaxSmem) return -100;
-  const dim3 grid(B, a.H);
-#define B200_ST(R_)                                                                                                     \
-  {                                                                                                                     \
-    B200_CHECK(cudaFuncSetAttribute(state_step_kernel<T, V, R_, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
-    state_step_kernel<T, V, R_, NT><<<grid, NT, smem, stream>>>(a, s);                                                  \
+template <class T, int NT>
+__device__ __forceinline__ void step_normaliser(const StateArgs& a, const StepArgs& s, long long sh, const StepFactors& f,
+                                                const float* sk) {
+  if (a.delta) return;
+  for (int d = threadIdx.x; d < a.D; d += NT) s.n[sh * a.D + d] = fmaf(f.keep, s.n[sh * a.D + d], f.wk * sk[d]);
+  if (threadIdx.x == 0) s.m[sh] = f.next;
+}
+
+// Decode step, one block per (sequence, head), for states that fit shared memory: one bulk copy brings the state in while q, k
+// and v are prepared, it is read and updated there, and one bulk copy takes it back. Dv in steps of 4. Threads form row groups
+// x groups of four columns.
+template <class T, int NT>
+__global__ void __launch_bounds__(NT) state_step_kernel(StateArgs a, StepArgs s, int* status) {
+  extern __shared__ __align__(128) float sm[];
+  __shared__ float red[3][NT / 32], red2[33];
+  __shared__ uint64_t bar;
+  __shared__ int abort_word;
+  const int D = a.D, Dv = a.Dv, b = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  float* S = sm;             // [D][Dv]
+  float* sq = S + D * Dv;    // [D]
+  float* sk = sq + D;        // [D]
+  float* sv = sk + D;        // [Dv]: v, then u
+  float* part = sv + Dv;     // [2][row groups][Dv]
+  const int slot = s.slots[b];
+  if (slot < 0) {            // padding row of a fixed-size batch
+    T* y = static_cast<T*>(s.y) + (static_cast<long long>(b) * a.H + h) * Dv;
+    for (int c = tid; c < Dv; c += NT) st1(y + c, 0.f);
+    return;
   }
-  if (ncg > NT || rows > 8) B200_ST(0)
-  else if (rows > 4) B200_ST(8)
-  else B200_ST(4)
-#undef B200_ST
+  const long long sh = static_cast<long long>(slot) * a.H + h;
+  float* home = s.S + sh * D * Dv;
+  const uint32_t bytes = static_cast<uint32_t>(D) * Dv * 4;
+  if (tid == 0) {
+    abort_word = 0;
+    mbar_init(&bar, 1);
+    fence_mbar_init();
+    mbar_arrive_expect_tx(&bar, bytes);
+    bulk_load(S, home, bytes, &bar);
+  }
+  const T* x = static_cast<const T*>(s.x) + b * a.ldx;
+  const StepFactors f = step_inputs<T, NT>(a, s, x, b, h, slot, sq, sk, sv, red);
+  if (!mbar_wait(&bar, 0, &abort_word)) {
+    abort_word = 1;
+    if (tid == 0) {
+      atomicCAS(status, 0, kErrMbarTimeoutProducer);
+      const unsigned long long t0 = globaltimer_ns();  // the copy in flight lands before the CTA retires
+      while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(1000);
+    }
+    __syncthreads();
+    return;
+  }
+  const int ncg = Dv / 4, cgt = ncg < NT ? ncg : NT, nrg = NT / cgt, rg = tid / cgt;
+  if (rg < nrg) {
+    for (int col = tid % cgt; col < ncg; col += cgt) {
+      float4 ka = make_float4(0.f, 0.f, 0.f, 0.f), qa = ka;
+#pragma unroll 4
+      for (int d = rg; d < D; d += nrg) {
+        const float4 t = *reinterpret_cast<const float4*>(S + d * Dv + col * 4);
+        const float k = sk[d], q = sq[d];
+        ka.x = fmaf(t.x, k, ka.x); ka.y = fmaf(t.y, k, ka.y); ka.z = fmaf(t.z, k, ka.z); ka.w = fmaf(t.w, k, ka.w);
+        qa.x = fmaf(t.x, q, qa.x); qa.y = fmaf(t.y, q, qa.y); qa.z = fmaf(t.z, q, qa.z); qa.w = fmaf(t.w, q, qa.w);
+      }
+      *reinterpret_cast<float4*>(part + rg * Dv + col * 4) = ka;
+      *reinterpret_cast<float4*>(part + (nrg + rg) * Dv + col * 4) = qa;
+    }
+  }
+  __syncthreads();
+  step_outputs<T, NT>(a, s, x, b, h, f, nrg, sv, part, red2);
+  if (rg < nrg) {
+    for (int col = tid % cgt; col < ncg; col += cgt) {
+      const float4 v = *reinterpret_cast<const float4*>(sv + col * 4);
+      const float4 u = make_float4(f.wk * v.x, f.wk * v.y, f.wk * v.z, f.wk * v.w);
+#pragma unroll 4
+      for (int d = rg; d < D; d += nrg) {
+        float4* at = reinterpret_cast<float4*>(S + d * Dv + col * 4);
+        const float k = sk[d];
+        const float4 t = *at;
+        *at = make_float4(fmaf(f.keep, t.x, k * u.x), fmaf(f.keep, t.y, k * u.y), fmaf(f.keep, t.z, k * u.z),
+                          fmaf(f.keep, t.w, k * u.w));
+      }
+    }
+  }
+  fence_proxy_async_smem();
+  __syncthreads();
+  if (tid == 0) {
+    bulk_store(home, S, bytes);
+    tma_store_commit();
+  }
+  step_normaliser<T, NT>(a, s, sh, f, sk);
+  if (tid == 0) tma_store_wait_read<0>();
+}
+
+// The same for any width: the state is read where it lies, twice.
+template <class T, int NT>
+__global__ void __launch_bounds__(NT) state_step_wide_kernel(StateArgs a, StepArgs s) {
+  extern __shared__ float sm[];
+  __shared__ float red[3][NT / 32], red2[33];
+  const int D = a.D, Dv = a.Dv, b = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  float* sq = sm;            // [D]
+  float* sk = sq + D;        // [D]
+  float* sv = sk + D;        // [Dv]: v, then u
+  float* part = sv + Dv;     // [2][row groups][Dv]
+  const int slot = s.slots[b];
+  if (slot < 0) {
+    T* y = static_cast<T*>(s.y) + (static_cast<long long>(b) * a.H + h) * Dv;
+    for (int c = tid; c < Dv; c += NT) st1(y + c, 0.f);
+    return;
+  }
+  const long long sh = static_cast<long long>(slot) * a.H + h;
+  float* S = s.S + sh * D * Dv;
+  const T* x = static_cast<const T*>(s.x) + b * a.ldx;
+  const StepFactors f = step_inputs<T, NT>(a, s, x, b, h, slot, sq, sk, sv, red);
+  const int cgt = Dv < NT ? Dv : NT, nrg = NT / cgt, rg = tid / cgt;
+  if (rg < nrg) {
+    for (int c = tid % cgt; c < Dv; c += cgt) {
+      float ka = 0.f, qa = 0.f;
+#pragma unroll 4
+      for (int d = rg; d < D; d += nrg) {
+        const float t = S[static_cast<long long>(d) * Dv + c];
+        ka = fmaf(t, sk[d], ka);
+        qa = fmaf(t, sq[d], qa);
+      }
+      part[rg * Dv + c] = ka;
+      part[(nrg + rg) * Dv + c] = qa;
+    }
+  }
+  __syncthreads();
+  step_outputs<T, NT>(a, s, x, b, h, f, nrg, sv, part, red2);
+  if (rg < nrg) {
+    for (int c = tid % cgt; c < Dv; c += cgt) {
+      const float u = f.wk * sv[c];
+#pragma unroll 4
+      for (int d = rg; d < D; d += nrg) {
+        float* at = S + static_cast<long long>(d) * Dv + c;
+        *at = fmaf(f.keep, *at, sk[d] * u);
+      }
+    }
+  }
+  step_normaliser<T, NT>(a, s, sh, f, sk);
+}
+
+template <class T>
+static int launch_state_step(const StateArgs& a, const StepArgs& s, int B, cudaStream_t stream) {
+  constexpr int NT = 256;
+  const dim3 grid(B, a.H);
+  const bool v4 = a.Dv % 4 == 0;
+  const int ncg = v4 ? a.Dv / 4 : a.Dv, nrg = NT / (ncg < NT ? ncg : NT);
+  const size_t vecs = (2 * static_cast<size_t>(a.D) + a.Dv + 2 * static_cast<size_t>(nrg) * a.Dv) * sizeof(float);
+  const size_t whole = static_cast<size_t>(a.D) * a.Dv * sizeof(float) + vecs;
+  // (shared memory is carved up in floats: 16-byte accesses behind q and k want D in steps of 2 as well)
+  if (v4 && a.D % 2 == 0 && whole <= 200 * 1024 && !(reinterpret_cast<uintptr_t>(s.S) & 15)) {
+    int* status = device_status_word();
+    if (!status) return -3;
+    B200_CHECK(cudaFuncSetAttribute(state_step_kernel<T, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)whole));
+    state_step_kernel<T, NT><<<grid, NT, whole, stream>>>(a, s, status);
+    B200_CHECK(cudaGetLastError());
+    return 0;
+  }
+  const int wide_nrg = NT / (a.Dv < NT ? a.Dv : NT);
+  const size_t smem = (2 * static_cast<size_t>(a.D) + a.Dv + 2 * static_cast<size_t>(wide_nrg) * a.Dv) * sizeof(float);
+  if (smem > kStMaxSmem) return -100;
+  B200_CHECK(cudaFuncSetAttribute(state_step_wide_kernel<T, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  state_step_wide_kernel<T, NT><<<grid, NT, smem, stream>>>(a, s);
   B200_CHECK(cudaGetLastError());
   return 0;
 }
@@ -415,12 +463,7 @@ int b200_state_step(const void* x, long long ldx, const void* p0, const void* p1
   const char* g0 = static_cast<const char*>(x) + at * size;
   const StateArgs a{x, ldx, g0, g0 + H * size, ldx, p0, p1, cap, delta, H, G, D, Dv};
   const StepArgs s{x, conv, ring, taps, pos, slots, S, n, m, norm, y, eps};
-  auto run = [&](auto tag) {
-    using T = decltype(tag);
-    if (Dv % 4) return launch_state_step<T, 1, 256>(a, s, B, stream);
-    return D * Dv > 8192 ? launch_state_step<T, 4, 512>(a, s, B, stream) : launch_state_step<T, 4, 256>(a, s, B, stream);
-  };
-  return fp32 ? run(float{}) : run(__nv_bfloat16{});
+  return fp32 ? launch_state_step<float>(a, s, B, stream) : launch_state_step<__nv_bfloat16>(a, s, B, stream);
 }
 
 }  // extern "C"

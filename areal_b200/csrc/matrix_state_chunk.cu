@@ -13,6 +13,12 @@
 // between warps. q, k and v are bf16 numbers and enter the products exactly, with the factors that make them unit vectors,
 // scales and decays applied to the products; fp32 operands (state, W, U, T, P) enter as two bf16 terms.
 //
+// Few long sequences would leave most SMs idle. The columns of a state are independent, so a head's may be spread over several
+// CTAs (its norm is then another kernel's). An mLSTM's state only decays by a number from token to token, so its sequences are
+// instead cut into segments: a first pass computes every segment's end state from zero and its decay (the running maximum is
+// that of the whole sequence in both passes), a scan over a sequence's segments turns them into the states that the segments
+// start from, and the second pass computes the outputs.
+//
 // The output of a block is normed and gated one block later, behind the barrier that the next block needs anyway.
 #include "common/host_utils.h"
 #include "common/mma16.cuh"
@@ -302,7 +308,10 @@ struct StateChunkArgs {
   long long ldg;
   const float* rec;           // [blocks, H, kRec]
   const int4* blocks;
-  const int *first, *slots;   // first block of every sequence [n_seq + 1]; slots may be null
+  const int4* segs;           // first block, blocks, sequence, 1 for the last segment of its sequence
+  const int* slots;           // may be null
+  float *seg_S, *seg_n, *seg_f;  // per segment: [H, D, Dv], [H, D], [H]; the first pass writes, the second reads S and n (null:
+                                 // segments are whole sequences)
   float *S, *n, *m;
   const __nv_bfloat16* norm;  // with it y gets the normed and gated heads
   __nv_bfloat16* y;           // [T, H * Dv]
@@ -319,20 +328,23 @@ struct StateSmem {
   float o[2][16 * 132], inv[2][16], n[2][DP];
 };
 
-template <int ND, bool DELTA, int WARPS>
+// STATE_ONLY: the first pass over segments
+template <int ND, bool DELTA, int WARPS, bool STATE_ONLY>
 __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 3) state_chunk_kernel(const StateChunkArgs a) {
   using SM = StateSmem<ND>;
   constexpr int P = SM::P, PB = P * 2;
   extern __shared__ __align__(16) uint8_t raw[];
   SM& sm = *reinterpret_cast<SM*>(raw);
-  const int seq = blockIdx.x, h = blockIdx.y, vb = blockIdx.z * a.cols, D = a.D, Dv = a.Dv, H = a.H, hk = h / (H / a.G);
+  const int4 seg = a.segs[blockIdx.x];
+  const int seq = seg.z, h = blockIdx.y, vb = blockIdx.z * a.cols, D = a.D, Dv = a.Dv, H = a.H, hk = h / (H / a.G);
   constexpr int nthr = WARPS * 32, nw = WARPS, TPW = 16 / WARPS;  // TPW: tokens of a block whose outputs a warp writes
   const int nv = min(a.cols, Dv - vb);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const bool mma = warp * 16 < nv;
-  const int b0 = a.first[seq], nblk = a.first[seq + 1] - b0;
-  if (nblk == 0) return;
-  const int t0 = a.blocks[b0].x, len = a.blocks[b0 + nblk - 1].x + a.blocks[b0 + nblk - 1].y - t0;  // the sequence's tokens
+  const int b0 = seg.x, nblk = seg.y;
+  if (nblk == 0 || (STATE_ONLY && seg.w)) return;  // (nothing starts from the last segment's end state)
+  const int t0 = a.blocks[b0].x, len = a.blocks[b0 + nblk - 1].x + a.blocks[b0 + nblk - 1].y - t0;  // the segment's tokens
+  const long long sgh = static_cast<long long>(blockIdx.x) * H + h;
   for (int i = tid; i < static_cast<int>(sizeof(SM) / 16); i += nthr) reinterpret_cast<uint4*>(raw)[i] = make_uint4(0, 0, 0, 0);
   float S[2 * ND][4];
 #pragma unroll
@@ -343,6 +355,19 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 3) state_chunk_ke
   const bool wide = !((D | Dv | a.ldq) & 7) && !(reinterpret_cast<uintptr_t>(a.qkv) & 15);
   const int dc = D >> 3, vc = nv >> 3;
   __syncthreads();
+  if (!STATE_ONLY && !DELTA && a.seg_S) {
+    if (mma) {
+#pragma unroll
+      for (int i = 0; i < 2 * ND; ++i)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const int d = i * 8 + 2 * t + (c & 1), col = vb + warp * 16 + g + (c >> 1) * 8;
+          if (d < D && col < Dv) S[i][c] = a.seg_S[(sgh * D + d) * Dv + col];
+        }
+    }
+    for (int d = tid; d < D; d += nthr) sm.n[0][d] = a.seg_n[sgh * D + d];
+  }
+  float seg_f = 1.f;
   constexpr int LPT = nthr / 16;  // threads that load a token
   const int ltok = tid / LPT, lc = tid % LPT;
   const float* rec_base = a.rec + (static_cast<long long>(b0) * H + h) * kRec;
@@ -447,11 +472,14 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 3) state_chunk_ke
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();  // this block's inputs are here, the last block's outputs too; every warp has left the block before
     if (b + 1 < nblk) load(b + 1, st ^ 1);
-    if (b > 0) output(b - 1, st ^ 1);
-    fetch_gates(b);
+    if (!STATE_ONLY) {
+      if (b > 0) output(b - 1, st ^ 1);
+      fetch_gates(b);
+    }
     const float* rec = sm.rec[st];
+    if (STATE_ONLY) seg_f *= rec[kRecS];
     if (!DELTA) {  // 1 / the denominators, then the normaliser behind this block (no one reads that copy before the barrier)
-      for (int i = warp; i < 16; i += nw) {
+      for (int i = STATE_ONLY ? 16 : warp; i < 16; i += nw) {
         float x = 0.f;
         for (int d = lane; d < D; d += 32) x = fmaf(sm.n[st][d], __bfloat162float(sm.q[st][i * P + d]), x);
         x = fmaf(warp_sum(x), rec[kRecQ + i], rec[kRecSum + i]);
@@ -473,7 +501,7 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 3) state_chunk_ke
         for (int c = 0; c < 4; ++c) ks[n][c] = o[n][c] = 0.f;
       // ---- K S and Q S, transposed: [value column, token]
 #pragma unroll
-      for (int kt = 0; kt < ND; ++kt) {
+      for (int kt = 0; kt < (STATE_ONLY ? 0 : ND); ++kt) {
         uint32_t hi[4], lo[4], bq[4], bk[4];
         hi[0] = split2(S[2 * kt][0], S[2 * kt][1], lo[0]);
         hi[1] = split2(S[2 * kt][2], S[2 * kt][3], lo[1]);
@@ -536,16 +564,18 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 3) state_chunk_ke
         }
       }
       // ---- outputs of the block itself
-      uint32_t ph[4], pl[4];
-      *reinterpret_cast<uint4*>(ph) = *reinterpret_cast<const uint4*>(rec + kRecP + lane * 8);
-      *reinterpret_cast<uint4*>(pl) = *reinterpret_cast<const uint4*>(rec + kRecP + lane * 8 + 4);
+      if constexpr (!STATE_ONLY) {
+        uint32_t ph[4], pl[4];
+        *reinterpret_cast<uint4*>(ph) = *reinterpret_cast<const uint4*>(rec + kRecP + lane * 8);
+        *reinterpret_cast<uint4*>(pl) = *reinterpret_cast<const uint4*>(rec + kRecP + lane * 8 + 4);
 #pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        mma_bf16(o[n], uh, ph[2 * n], ph[2 * n + 1]);
-        if (DELTA) mma_bf16(o[n], ul, ph[2 * n], ph[2 * n + 1]);
-        mma_bf16(o[n], uh, pl[2 * n], pl[2 * n + 1]);
+        for (int n = 0; n < 2; ++n) {
+          mma_bf16(o[n], uh, ph[2 * n], ph[2 * n + 1]);
+          if (DELTA) mma_bf16(o[n], ul, ph[2 * n], ph[2 * n + 1]);
+          mma_bf16(o[n], uh, pl[2 * n], pl[2 * n + 1]);
 #pragma unroll
-        for (int c = 0; c < 4; ++c) sm.o[st][(n * 8 + 2 * t + (c & 1)) * 132 + warp * 16 + g + (c >> 1) * 8] = o[n][c];
+          for (int c = 0; c < 4; ++c) sm.o[st][(n * 8 + 2 * t + (c & 1)) * 132 + warp * 16 + g + (c >> 1) * 8] = o[n][c];
+        }
       }
       // ---- the state behind the block
       const float fs = rec[kRecS];
@@ -565,39 +595,63 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 3) state_chunk_ke
     }
   }
   __syncthreads();
-  output(nblk - 1, (nblk - 1) & 1);
-  const int slot = a.slots ? a.slots[seq] : -1;
-  if (slot < 0) return;
-  const long long sh = static_cast<long long>(slot) * H + h;
+  if (!STATE_ONLY) output(nblk - 1, (nblk - 1) & 1);
+  const int slot = !STATE_ONLY && a.slots && seg.w ? a.slots[seq] : -1;
+  if (!STATE_ONLY && slot < 0) return;
+  const long long sh = STATE_ONLY ? sgh : static_cast<long long>(slot) * H + h;
+  float *dS = STATE_ONLY ? a.seg_S : a.S, *dn = STATE_ONLY ? a.seg_n : a.n;
   if (mma) {
 #pragma unroll
     for (int i = 0; i < 2 * ND; ++i)
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int d = i * 8 + 2 * t + (c & 1), col = vb + warp * 16 + g + (c >> 1) * 8;
-        if (d < D && col < Dv) a.S[(sh * D + d) * Dv + col] = S[i][c];
+        if (d < D && col < Dv) dS[(sh * D + d) * Dv + col] = S[i][c];
       }
   }
   if (!DELTA && blockIdx.z == 0) {
-    for (int d = tid; d < D; d += nthr) a.n[sh * D + d] = sm.n[nblk & 1][d];
-    if (tid == 0) a.m[sh] = sm.rec[(nblk - 1) & 1][kRecM];
+    for (int d = tid; d < D; d += nthr) dn[sh * D + d] = sm.n[nblk & 1][d];
+    if (tid == 0) {
+      if (STATE_ONLY) a.seg_f[sgh] = seg_f;
+      else a.m[sh] = sm.rec[(nblk - 1) & 1][kRecM];
+    }
   }
 }
 
-template <int ND, bool DELTA, int WARPS>
-static int launch_state_chunk(const StateChunkArgs& a, int n_seq, cudaStream_t stream) {
+// End states of segments from zero -> the states that the segments start from. grid (elements of S and n / 256, sequences)
+__global__ void state_segments_kernel(float* __restrict__ S, float* __restrict__ n, const float* __restrict__ f,
+                                      const int* __restrict__ first, int H, int D, int Dv) {
+  const long long ns = static_cast<long long>(H) * D * Dv, nn = static_cast<long long>(H) * D;
+  const long long e = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (e >= ns + nn) return;
+  const bool is_s = e < ns;
+  const long long at = is_s ? e : e - ns, size = is_s ? ns : nn;
+  const int h = static_cast<int>(at / (size / H)), s1 = first[blockIdx.y + 1];
+  float* x = (is_s ? S : n) + at;
+  float run = 0.f;
+  for (int s = first[blockIdx.y]; s < s1; ++s) {
+    const float add = s + 1 < s1 ? x[s * size] : 0.f;
+    x[s * size] = run;
+    if (s + 1 < s1) run = fmaf(f[static_cast<long long>(s) * H + h], run, add);
+  }
+}
+
+template <int ND, bool DELTA, int WARPS, bool STATE_ONLY>
+static int launch_state_chunk(const StateChunkArgs& a, int n_seg, cudaStream_t stream) {
   constexpr int smem = static_cast<int>(sizeof(StateSmem<ND>));
   static_assert(smem % 16 == 0, "cleared in 16-byte steps");
-  B200_CHECK(cudaFuncSetAttribute(state_chunk_kernel<ND, DELTA, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-  state_chunk_kernel<ND, DELTA, WARPS><<<dim3(n_seq, a.H, (a.Dv + a.cols - 1) / a.cols), WARPS * 32, smem, stream>>>(a);
+  B200_CHECK(cudaFuncSetAttribute(state_chunk_kernel<ND, DELTA, WARPS, STATE_ONLY>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+  state_chunk_kernel<ND, DELTA, WARPS, STATE_ONLY><<<dim3(n_seg, a.H, (a.Dv + a.cols - 1) / a.cols), WARPS * 32, smem, stream>>>(a);
   B200_CHECK(cudaGetLastError());
   return 0;
 }
 
-template <bool DELTA>
-static int pick_state_chunk(const StateChunkArgs& a, int n_seq, cudaStream_t stream) {
+template <bool DELTA, bool STATE_ONLY>
+static int pick_state_chunk(const StateChunkArgs& a, int n_seg, cudaStream_t stream) {
   const bool wide = a.cols > 64 && a.Dv > 64;
-#define B200_SW(ND_) (wide ? launch_state_chunk<ND_, DELTA, 8>(a, n_seq, stream) : launch_state_chunk<ND_, DELTA, 4>(a, n_seq, stream))
+#define B200_SW(ND_)                                                               \
+  (wide ? launch_state_chunk<ND_, DELTA, 8, STATE_ONLY>(a, n_seg, stream)          \
+        : launch_state_chunk<ND_, DELTA, 4, STATE_ONLY>(a, n_seg, stream))
   if (a.D <= 32) return B200_SW(2);
   if (a.D <= 64) return B200_SW(4);
   return B200_SW(8);
@@ -640,17 +694,30 @@ int b200_state_chunk_prep(const void* qkv, long long ldq, const void* g0, const 
 }
 
 // norm (Dv <= cols): out is the normed and gated heads in bf16; null: out is the plain outputs in fp32. cols: value columns per
-// CTA, a multiple of 16 up to 128. seq_first: [n_seq + 1] first block of every sequence. slots null: no state is kept.
+// CTA, a multiple of 16 up to 128. segs: int32 [n_seg, 4] as in StateChunkArgs. seg_first: [n_seq + 1] first segment of every
+// sequence; seg_S, seg_n, seg_f: scratch, all null when every segment is a whole sequence (mLSTM only). slots null: no state is
+// kept.
 int b200_state_chunk(const void* qkv, long long ldq, const void* gate, long long ldg, const float* rec, const int* blocks,
-                     const int* seq_first, int n_seq, const int* slots, float* S, float* n, float* m, const void* norm,
-                     void* out, int cols, float eps, int delta, int H, int G, int D, int Dv, cudaStream_t stream) {
+                     const int* segs, int n_seg, const int* seg_first, int n_seq, float* seg_S, float* seg_n, float* seg_f,
+                     const int* slots, float* S, float* n, float* m, const void* norm, void* out, int cols, float eps,
+                     int delta, int H, int G, int D, int Dv, cudaStream_t stream) {
   using namespace b200;
-  if (n_seq <= 0) return 0;
+  if (n_seg <= 0 || n_seq <= 0) return 0;
+  if (delta && seg_S) return -100;
   if (G < 1 || H % G || D < 1 || D > 128 || Dv < 1 || cols < 16 || cols > 128 || cols % 16 || (norm && Dv > cols)) return -100;
   using bf = __nv_bfloat16;
-  const StateChunkArgs a{(const bf*)qkv, ldq, (const bf*)gate, ldg, rec, reinterpret_cast<const int4*>(blocks), seq_first,
-                         slots, S, n, m, (const bf*)norm, (bf*)out, (float*)out, eps, H, G, D, Dv, cols};
-  return delta ? pick_state_chunk<true>(a, n_seq, stream) : pick_state_chunk<false>(a, n_seq, stream);
+  const StateChunkArgs a{(const bf*)qkv, ldq, (const bf*)gate, ldg, rec, reinterpret_cast<const int4*>(blocks),
+                         reinterpret_cast<const int4*>(segs), slots, seg_S, seg_n, seg_f, S, n, m, (const bf*)norm, (bf*)out, (float*)out, eps, H, G, D, Dv, cols};
+  if (delta) return pick_state_chunk<true, false>(a, n_seg, stream);
+  if (seg_S) {
+    const int rc = pick_state_chunk<false, true>(a, n_seg, stream);
+    if (rc) return rc;
+    const long long e = static_cast<long long>(H) * D * (Dv + 1);
+    state_segments_kernel<<<dim3(static_cast<unsigned>((e + 255) / 256), n_seq), 256, 0, stream>>>(seg_S, seg_n, seg_f, seg_first,
+                                                                                                  H, D, Dv);
+    B200_CHECK(cudaGetLastError());
+  }
+  return pick_state_chunk<false, false>(a, n_seg, stream);
 }
 
 }  // extern "C"

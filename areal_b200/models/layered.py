@@ -32,6 +32,7 @@ training on one process per replica (data parallelism).
 
 from __future__ import annotations
 
+import contextlib
 from dataclasses import dataclass, field
 from typing import Any, Iterator
 
@@ -333,16 +334,20 @@ class ParallelBlock(nn.Module):
             h = y
             hc = conv_prefill(h, self.conv, ctx.meta, ctx.pos, add=True, ring=rec["conv"] if rec is not None else None,
                               slots=ctx.state_slots)
+        with ctx.beside(h):  # the two do not depend on each other
+            ff = self._feed_forward(h, ctx)
         if self.attn.o is None:
             mixer = self.attn.results(hc, ctx, cache, rec)
         else:
             mixer = [(linear_slices(self.attn.hidden(hc, ctx, cache, rec), self.attn.o), None)]
-        ff = None
-        if self.mlp is not None:
-            ff = self.mlp.hidden(h, ctx)
-            if self.mlp.o is not None:
-                ff = linear_slices(ff, self.mlp.o)
+        ctx.join(h)
         return rs.ParallelSum(mixer, ff)
+
+    def _feed_forward(self, h, ctx):
+        if self.mlp is None:
+            return None
+        ff = self.mlp.hidden(h, ctx)
+        return ff if self.mlp.o is None else linear_slices(ff, self.mlp.o)
 
     def tensors(self, p: str):
         yield from self.norm1.tensors(p + "norm1")
@@ -400,6 +405,21 @@ class StepContext:
     shared: frozenset = frozenset()
     latents: dict = field(default_factory=dict)
 
+    def beside(self, x: torch.Tensor):
+        """What is launched inside may run beside what follows up to :meth:`join`: in a decode step, whose kernels leave much
+        of the device idle, on a second stream (a branch of a captured graph). Memory that either side frees is used again
+        only behind the join: the second stream waits for the first whenever it starts."""
+        side = self.model.side_stream(x) if self.decode else None
+        if side is None:
+            return contextlib.nullcontext()
+        side.wait_stream(torch.cuda.current_stream(x.device))
+        return torch.cuda.stream(side)
+
+    def join(self, x: torch.Tensor):
+        side = self.model.side_stream(x) if self.decode else None
+        if side is not None:
+            torch.cuda.current_stream(x.device).wait_stream(side)
+
     def rotary(self, rot: dict):
         n = self.max_seq_len if self.decode else self.meta.max_seqlen
         return self.model.rotary(rot, n or 1, self.pos.device)
@@ -434,6 +454,7 @@ class LayeredModel(QwenModel):
         self.checkpoint_every = 0
         self._tables: dict[tuple, tuple[torch.Tensor, torch.Tensor]] = {}
         self._positions = 1
+        self._side = None
         self._shared = frozenset(j for i in self.layer_ids if (j := cfg.cache_layer(i)) != i)
 
     @torch.no_grad()
@@ -453,6 +474,14 @@ class LayeredModel(QwenModel):
         """Positions up to ``n`` will be used: rotary tables are built that long from the start (a captured decode step
         keeps their addresses)."""
         self._positions = max(self._positions, int(n))
+
+    def side_stream(self, x: torch.Tensor):
+        """A second stream on ``x``'s device (None on the CPU)."""
+        if not x.is_cuda:
+            return None
+        if self._side is None:
+            self._side = torch.cuda.Stream(x.device, priority=-1)
+        return self._side
 
     def rotary(self, rot: dict, n: int, device):
         dims, base, scaling = rot["dims"], rot["base"], rot.get("scaling")

@@ -26,6 +26,7 @@ import torch.nn.functional as F
 
 from . import _lib
 from .dyt import fp32_flag, group_rms, group_rms_ref, kernel_ok
+from .gated_scan import segment_length
 from .linear_attn import linear_attn_chunked
 from .short_conv import conv_prefill, conv_prefill_ref, conv_step_ref, ring_write_ref
 
@@ -208,8 +209,7 @@ def _state_ptrs(spec: Spec, state):
 
 
 def _blocks(meta):
-    """Device table of the 16-token blocks of a packed batch ``(first token, tokens, sequence, first of its sequence)`` and
-    every sequence's first block."""
+    """Device table of the 16-token blocks of a packed batch: ``(first token, tokens, sequence, first of its sequence)``."""
     got = meta.__dict__.get("_state_blocks")
     if got is None:
         cu = np.asarray(meta.cu_cpu, dtype=np.int64)
@@ -219,15 +219,35 @@ def _blocks(meta):
         seq = np.repeat(np.arange(len(lens)), per)
         at = (np.arange(int(first[-1])) - first[seq]) * _BLOCK
         tab = np.stack([cu[seq] + at, np.minimum(_BLOCK, lens[seq] - at), seq, at == 0], 1).astype(np.int32)
-        dev = meta.cu_seqlens.device
-        got = meta.__dict__["_state_blocks"] = (torch.from_numpy(tab.reshape(-1, 4)).to(dev),
-                                                torch.from_numpy(first.astype(np.int32)).to(dev))
+        got = meta.__dict__["_state_blocks"] = torch.from_numpy(tab.reshape(-1, 4)).to(meta.cu_seqlens.device)
     return got
 
 
+def _segments(meta, units: int):
+    """Device tables of the walks along a packed batch, ``(first block, blocks, sequence, last of its sequence)``, and every
+    sequence's first; whether any sequence is cut. ``units``: CTAs that walk one sequence side by side (0: nothing is cut)."""
+    cu = [int(c) for c in meta.cu_cpu]
+    lens = [b - a for a, b in zip(cu[:-1], cu[1:])]
+    L = segment_length(lens, units) // _BLOCK if units else 0
+    cache = meta.__dict__.setdefault("_state_segments", {})
+    if L not in cache:
+        segs, first, b0 = [], [0], 0
+        for n, tokens in enumerate(lens):
+            total = -(-tokens // _BLOCK)
+            for b in range(0, total, L or max(total, 1)):
+                size = min(L or total, total - b)
+                segs.append((b0 + b, size, n, int(b + size >= total)))
+            b0 += total
+            first.append(len(segs))
+        dev = meta.cu_seqlens.device
+        cache[L] = (torch.tensor(segs, dtype=torch.int32).reshape(-1, 4).to(dev), torch.tensor(first, dtype=torch.int32).to(dev),
+                    len(segs) > len(lens))
+    return cache[L]
+
+
 def _columns(meta, heads: int, vdim: int) -> int:
-    """Value columns per CTA of the chunk kernel: all of a head's (up to 128), whose norm then runs in the kernel, unless the
-    walk along few long sequences would leave most SMs idle. Columns are independent of one another."""
+    """Value columns per CTA of the delta rule's chunk kernel: all of a head's (up to 128), whose norm then runs in the kernel,
+    unless the walk along few long sequences would leave most SMs idle. Columns are independent of one another."""
     lens = np.diff(np.asarray(meta.cu_cpu))
     cols = 128
     even = float(lens.sum()) * heads * -(-vdim // 128) / 148  # tokens per SM if the work were spread evenly
@@ -257,8 +277,9 @@ def prefill(x: torch.Tensor, spec: Spec, meta, pos: torch.Tensor, state: dict | 
     n_seq = meta.cu_seqlens.numel() - 1
     lib = _lib.kernels()
     if x.dtype == torch.bfloat16 and D <= 128:
-        blocks, first = _blocks(meta)
-        n, cols = blocks.shape[0], _columns(meta, H, Dv)
+        blocks = _blocks(meta)
+        n, cols = blocks.shape[0], _columns(meta, H, Dv) if spec.delta else 128
+        segs, seg_first, cut = _segments(meta, 0 if spec.delta else H * -(-Dv // 128))
         fuse = Dv <= cols
         rec = torch.empty((n, H, lib.b200_state_record_floats()), dtype=torch.float32, device=x.device)
         run_max = None
@@ -267,11 +288,13 @@ def prefill(x: torch.Tensor, spec: Spec, meta, pos: torch.Tensor, state: dict | 
         _lib.check(lib.b200_state_chunk_prep(*srcs, *_params(spec), p(blocks), c(n), p(meta.cu_seqlens), c(n_seq), p(run_max),
                                              p(rec), *_dims(spec), _lib.stream_ptr()), "b200_state_chunk_prep")
         out = torch.empty((T, H * Dv), dtype=x.dtype if fuse else torch.float32, device=x.device)
+        new = lambda *shape: torch.empty((segs.shape[0], *shape), dtype=torch.float32, device=x.device)
+        seg = (new(H, D, Dv), new(H, D), new(H)) if cut else (None, None, None)
         _lib.check(lib.b200_state_chunk(
-            p(qkv), ll(qkv.stride(0)), p(gate), ll(x.stride(0)), p(rec), p(blocks), p(first), c(n_seq), p(slots),
-            *_state_ptrs(spec, state), p(spec.norm if fuse else None), p(out), c(cols), ctypes.c_float(spec.eps), c(int(spec.delta)),
+            p(qkv), ll(qkv.stride(0)), p(gate), ll(x.stride(0)), p(rec), p(blocks), p(segs), c(segs.shape[0]), p(seg_first),
+            c(n_seq), *(p(t) for t in seg), p(slots), *_state_ptrs(spec, state), p(spec.norm if fuse else None), p(out), c(cols), ctypes.c_float(spec.eps), c(int(spec.delta)),
             *_dims(spec), _lib.stream_ptr()), "b200_state_chunk")
-        _lib.count_launch(2 if spec.delta else 3)
+        _lib.count_launch(2 if spec.delta else 5 if cut else 3)
         if fuse:
             return out
     else:

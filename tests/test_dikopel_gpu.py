@@ -262,15 +262,15 @@ def test_mlstm_prefill(dt, H, G, D, Dv, i_shift, f_shift, cap, extra):
 @pytest.mark.parametrize("kind", ["delta", "mlstm"])
 @pytest.mark.parametrize("lens", [[3000], [2500, 40, 1], [1025, 1024, 1023]])
 def test_long_sequences(kind, lens):
-    """Few long sequences: the value columns of a head are spread over several CTAs. Also more tokens than a chunk of the
-    running maximum's scan."""
-    from areal_b200.ops.matrix_state import _columns, prefill
+    """Few long sequences: the value columns of a delta rule's head are spread over several CTAs, an mLSTM's sequences are cut
+    into segments. Also more tokens than a chunk of the running maximum's scan."""
+    from areal_b200.ops.matrix_state import _columns, _segments, prefill
     from areal_b200.ops.short_conv import conv_prefill
 
     H, G, D, Dv, dt = 2, 1, 32, 72, torch.bfloat16
     cu, meta, pos = _packed(lens)
     if max(lens) > 2000:
-        assert _columns(meta, H, Dv) < Dv
+        assert _columns(meta, H, Dv) < Dv and _segments(meta, H)[2]
     spec, x = _delta(H, G, D, Dv, dt, cu[-1], decay=-3.0) if kind == "delta" else _mlstm(H, D, Dv, dt, cu[-1], -2.0, 5.0, 8.0)
     state, slots = _states(spec, 3, 4, dt), torch.arange(len(lens), dtype=torch.int32, device="cuda")
     got = prefill(x, spec, meta, pos, state, slots)
