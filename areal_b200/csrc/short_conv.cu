@@ -1,6 +1,6 @@
 // Short causal convolutions over time, one filter per channel, of packed sequences:
 //
-//   y_t = act(sum_j w[c][j] x_(t - taps + 1 + j)) (+ x_t),  zeros before a sequence's start
+//   y_t = act(sum_j w[c][j] x_(t - taps + 1 + j)) (+ x_t),  x_s = 0 for s < 0
 //
 // and the rings that later steps go on from: ring [slots][taps][C] holds the input of position p in row p % taps. A
 // thread walks 16 tokens of a few channels with the last inputs in registers.

@@ -158,7 +158,7 @@ def parse_args(argv=None) -> argparse.Namespace:
     ap.add_argument("--max-num-batched-tokens", type=int, default=16384)
     ap.add_argument("--num-kv-blocks", type=int, default=None)
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
-                    help="float32: true 32-bit serving (families whose kernels have a 32-bit form, e.g. fofosun, gatolix, felosun)")
+                    help="float32: true 32-bit serving (families whose kernels have a 32-bit form, e.g. fofosun, gatolix, felosun, dikopel)")
     ap.add_argument("--seed", type=int, default=1)
     ap.add_argument("--device", default=None)
     ap.add_argument("--disable-cuda-graph", action="store_true")

@@ -6,7 +6,8 @@
 
 A mixer's result is one set of rows, or the mean of two that are RMS normed each (``rms(a; wa) / 2 + rms(b; wb) / 2``). In a
 decode step the kernels go on to what the next mixer reads, ``h + conv(h)`` (:class:`ops.short_conv.ConvTail`). The
-sinusoids of position ``p``: entry ``2i`` is ``sin(p * 10000^(-2i / width))``, entry ``2i + 1`` the cosine."""
+sinusoids of a position ``p`` are the sine and the cosine of ``p / 10000^(2i / W)`` side by side, ``i < W / 2`` (Vaswani et al.,
+"Attention Is All You Need")."""
 
 from __future__ import annotations
 

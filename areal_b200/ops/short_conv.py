@@ -1,7 +1,7 @@
 """Short causal convolutions over time, one filter per channel (``csrc/short_conv.cu``), with their PyTorch statement (the CPU
 path, and the path under autograd):
 
-    y_t = act(sum_j w[:, j] x_(t - taps + 1 + j))  (+ x_t),   zeros before the sequence's start
+    y_t = act(sum_j w[:, j] x_(t - taps + 1 + j))  (+ x_t),   x_s = 0 for s < 0
 
 What a sequence needs to go on is kept in a ring ``[slots, taps, channels]``: the input of position ``p`` lies in row ``p %
 taps``. A row counts only if its position exists, so rings need no clearing when a slot changes hands, and a step writes its

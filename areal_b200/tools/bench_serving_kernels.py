@@ -396,6 +396,7 @@ def run_dikopel() -> list[dict]:
     q, k, v = _rand(T, H, D), _rand(T, H, D), _rand(T, H, D)
     a, b = torch.rand(T, H, device="cuda"), torch.rand(T, H, device="cuda")
     add("[qwen3.5] causal_conv1d, linear_attn_prefill 8x2048", lambda: (causal_conv1d(xq, cw, None, meta.cu_seqlens), linear_attn_prefill(q, k, v, a, b, meta.cu_seqlens, 1.0)), T * (C + 2 * H * D) * 2, T * H * D * D * 6, 3)
+    add("[qwen3.5] linear_attn_prefill 1x16384", lambda: linear_attn_prefill(q, k, v, a, b, one.cu_seqlens, 1.0), T * (C + 2 * H * D) * 2, T * H * D * D * 6, 1)
     add("mLSTM prefill 8x2048, 16 heads of 128 (norm, gate)", lambda: ms.prefill(xm, mls, meta, pos, stm, slots), 5 * io, T * H * D * D * 4)
     add("mLSTM prefill 1x16384", lambda: ms.prefill(xm, mls, one, pos1, stm, slots[:1]), 5 * io, T * H * D * D * 4)
     hg = ScanSpec("hgrn2", H, D, D, bias=_rand(H * D) + 2, lower=torch.rand(H * D, device="cuda").to(BF))

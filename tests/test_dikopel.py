@@ -200,7 +200,7 @@ def test_gated_delta_rule_in_prompts_and_steps(H, G, D, Dv, taps, decay):
         assert not y[3].any()
 
 
-def test_the_read_out_sees_the_current_write():
+def test_a_token_reads_what_it_has_just_written():
     q = k = torch.tensor([[[1.0, 0.0]], [[1.0, 0.0]]]).double()
     v = torch.tensor([[[3.0]], [[5.0]]]).double()
     o = oracle.delta_rule(q, k, v, torch.tensor([[0.5], [0.5]]).double(), torch.tensor([[1.0], [0.25]]).double())
