@@ -25,7 +25,7 @@ import torch
 import torch.nn.functional as F
 
 from . import _lib
-from .dyt import fp32_flag, group_rms, group_rms_ref, kernel_ok
+from .dyt import fp32_flag, group_rms, kernel_ok
 from .gated_scan import segment_length
 from .linear_attn import linear_attn_chunked
 from .short_conv import conv_prefill, conv_prefill_ref, conv_step_ref, ring_write_ref
